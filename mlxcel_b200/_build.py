@@ -12,6 +12,7 @@ Objects are rebuilt only when their source (or a shared header) is newer.
 """
 from __future__ import annotations
 
+import hashlib
 import os
 import shutil
 import subprocess
@@ -31,6 +32,16 @@ NVCC_FLAGS = [
     "-gencode", "arch=compute_100a,code=sm_100a", "-lineinfo", "-O3", "-std=c++17",
     "-Xcompiler", "-fPIC", "-Xptxas", "-v",
 ]
+
+# Sources a model family needs, for processes that serve one model from a tree without a built library:
+# they compile these alone, into a library of their own (the full one is used where it exists).
+MODEL_UNITS = {
+    "pamasun": ("attention", "attention_tc", "delta_rule", "gemm", "misc", "sampling", "simt", "stream_norm"),
+}
+
+
+def partial_lib(units) -> Path:
+    return LIB / f"libmlxcel_b200_{hashlib.sha1(','.join(sorted(units)).encode()).hexdigest()[:10]}.so"
 
 
 def _nvcc() -> str | None:
@@ -53,13 +64,19 @@ def host_ext_path() -> Path:
     return LIB / f"_mlxcel_host{suffix}"
 
 
-def build_cuda(verbose: bool = False, force: bool = False) -> Path:
+def build_cuda(verbose: bool = False, force: bool = False, units=None) -> Path:
+    """Compiles the kernel library: every source, or only the named ``units`` (file stems) into
+    :func:`partial_lib`. Returns the library's path."""
     nvcc = _nvcc()
     if nvcc is None:
         raise RuntimeError("nvcc not found: cannot build the sm_100a kernel library")
     OBJ.mkdir(parents=True, exist_ok=True)
     headers = sorted(CSRC.glob("*.cuh")) + sorted(CSRC.glob("*.h"))
     sources = sorted(CSRC.glob("*.cu"))
+    target = CUDA_LIB
+    if units is not None:
+        sources = [s for s in sources if s.stem in units]
+        target = partial_lib(units)
     logs: dict[str, str] = {}
 
     def compile_one(src: Path) -> Path:
@@ -74,18 +91,20 @@ def build_cuda(verbose: bool = False, force: bool = False) -> Path:
 
     with ThreadPoolExecutor(max_workers=min(8, len(sources) or 1)) as ex:
         objs = list(ex.map(compile_one, sources))
-    if force or not CUDA_LIB.exists() or any(o.stat().st_mtime > CUDA_LIB.stat().st_mtime for o in objs):
-        cmd = [nvcc, "-shared", "-o", str(CUDA_LIB), *map(str, objs), "-lcudart"]
+    if force or not target.exists() or any(o.stat().st_mtime > target.stat().st_mtime for o in objs):
+        part = target.with_suffix(f".{os.getpid()}.tmp")           # (an interrupted link leaves no library behind)
+        cmd = [nvcc, "-shared", "-o", str(part), *map(str, objs), "-lcudart"]
         r = subprocess.run(cmd, capture_output=True, text=True)
         if r.returncode != 0:
             raise RuntimeError(f"link failed:\n{r.stderr[-4000:]}")
-    if logs:
+        os.replace(part, target)
+    if logs and units is None:
         (LIB / "ptxas_info.txt").write_text(
             "\n".join(f"==== {k}\n{v}" for k, v in sorted(logs.items())))
     if verbose:
         for k, v in sorted(logs.items()):
             print(f"==== {k}\n{v}")
-    return CUDA_LIB
+    return target
 
 
 def build_host(force: bool = False) -> Path:

@@ -11,6 +11,9 @@ Multi-head latent attention with ``cfg.extra["mla_latent"]`` keeps ONE entry per
 ``[normalised latent (kv_lora_rank) | rotary key (qk_rope_head_dim)]`` (576 values for DeepSeek-V3
 instead of 2 * heads * head_dim), in the K slab with a single head; the V slab is empty
 (the reference's MLA cache, src/lib/mlxcel-core/src/mla/cache.rs:253).
+
+Models with ``cfg.kv_geometry()`` (attention layers of different head counts, keys and values of
+different widths) get one slab pair per attention run with exactly those sizes.
 """
 from __future__ import annotations
 
@@ -31,6 +34,19 @@ class KVPool:
         L = cfg.num_hidden_layers if num_layers is None else num_layers
         shape = (num_blocks, self.Hkv, block_size, self.D)
         self.layers: list[KVLayer] = []
+        geo = cfg.kv_geometry()
+        if geo is not None:
+            # one slab pair per attention run, each with its own head count and key / value widths
+            if kv_bits != 16:
+                raise ValueError("models with per-layer attention geometry keep 16-bit (or fp32) KV: kv_bits must be 16")
+            if tp_size != 1:
+                raise ValueError("per-layer attention geometry is not sharded across tensor-parallel ranks")
+            self.latent = False
+            for h, dk, dv in geo:
+                k = torch.zeros((num_blocks, h, block_size, dk), dtype=dtype, device=device)
+                v = torch.zeros((num_blocks, h, block_size, dv), dtype=dtype, device=device)
+                self.layers.append(KVLayer(k, v, None, None, block_size, kv_bits))
+            return
         self.latent = bool(cfg.extra.get("mla_latent"))
         if self.latent:
             if kv_bits != 16:
@@ -66,6 +82,8 @@ class KVPool:
                         num_layers: int | None = None) -> int:
         Hkv = max(1, cfg.num_key_value_heads // tp_size)
         L = cfg.num_hidden_layers if num_layers is None else num_layers
+        if cfg.kv_geometry() is not None:
+            return cfg.kv_bytes_per_token(kv_bits) * block_size
         if cfg.extra.get("mla_latent"):
             return KVPool.latent_width(cfg) * 2 * block_size * L
         per_tok = Hkv * cfg.head_dim * kv_bits // 8

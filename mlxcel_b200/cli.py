@@ -38,6 +38,8 @@ def _add_model_args(p):
     p.add_argument("--keep", type=int, default=0, help="tokens at the start of a sequence that context shifting never drops")
     p.add_argument("--no-prompt-cache", action="store_true")
     p.add_argument("--no-cuda-graphs", action="store_true")
+    p.add_argument("--dtype", choices=["bfloat16", "float32"], default="bfloat16",
+                   help="precision of weights, activations and cache (float32: designs with fp32 kernels)")
     p.add_argument("--no-warmup", action="store_true", help="serve: skip the one-token request made before listening")
     p.add_argument("--dequantize", action="store_true", help="dequantize quantized checkpoints at load")
     p.add_argument("--tp", type=int, default=1, help="tensor-parallel ranks (launch with torch.distributed.run)")
@@ -233,7 +235,8 @@ def load_llm(a):
         llm.tokenizer = ByteTokenizer(llm.cfg.vocab_size)
     else:
         llm = LLM.from_pretrained(a.model, device=dev, engine_config=ecfg, comm=comm, dequantize=a.dequantize,
-                                  surgery=getattr(a, "surgery", None), config_overrides=config_overrides(a))
+                                  surgery=getattr(a, "surgery", None), config_overrides=config_overrides(a),
+                                  dtype=getattr(torch, getattr(a, "dtype", None) or "bfloat16"))
     attach_drafter(llm, a, dev)
     if llm.engine.drafter is not None:
         from .speculative import SpecPolicy
@@ -1091,7 +1094,7 @@ def cmd_inspect(a):
 
 
 _HYBRID = {"nemotron_h", "granitemoehybrid", "jamba", "qwen3_next", "qwen3_5", "qwen3_5_text", "qwen3_5_moe",
-           "qwen3_5_moe_text", "falcon_h1", "lfm2", "lfm2_moe", "recurrent_gemma"}
+           "qwen3_5_moe_text", "falcon_h1", "lfm2", "lfm2_moe", "recurrent_gemma", "pamasun"}
 _STATE_SPACE = {"mamba", "mamba2"}
 _CHECKED_BY_READING = {"internlm3", "minicpm", "mimo", "yi", "kimi_k2", "deepseek"}       # no independent implementation at hand
 _CHECKED_BY_LAYOUT = {"internlm2", "baichuan", "exaone", "telechat3"}                                 # round trip against the Llama form
@@ -1113,6 +1116,8 @@ def arch_catalog() -> dict:
             how = f"transformers logits (as {name}_text)"
         if name == "deepseek_v32":
             how = "transformers logits (as glm_moe_dsa)"
+        if name == "pamasun":
+            how = "a plain PyTorch statement of the model (no library has it)"
         if name == "dbrx":
             how = "a plain PyTorch statement of the model (the transformers implementation is not usable)"
         fams.append(dict(name=name, executor=ex, checked_against=how))
@@ -1159,6 +1164,11 @@ def cmd_random_init(a):
     if cfg.model_type == "nemotron_h":
         from .models.hybrid import hybrid_config_dict, random_hybrid_weights, save_hybrid_checkpoint
         save_hybrid_checkpoint(a.out, hybrid_config_dict(cfg), random_hybrid_weights(cfg, seed=a.seed), cfg)
+        print("wrote", a.out)
+        return
+    if cfg.model_type == "pamasun":
+        from .models.pamasun import random_pamasun_tensors, save_pamasun_checkpoint
+        save_pamasun_checkpoint(a.out, cfg, random_pamasun_tensors(cfg, seed=a.seed))
         print("wrote", a.out)
         return
     w = random_weights(cfg, seed=a.seed, dtype=torch.bfloat16)
@@ -1363,6 +1373,10 @@ def main(argv=None):
     p.add_argument("-m", "--model", required=True)
     p.add_argument("text")
     p.set_defaults(fn=cmd_tokenize)
+    p = sub.add_parser("trace", help="replay given token ids step by step and write logits (also bin/trace_run)")
+    from . import trace
+    trace.add_arguments(p)
+    p.set_defaults(fn=lambda a: sys.exit(trace.run(a)))
     p = sub.add_parser("random-init", help="write a random checkpoint of a preset architecture")
     p.add_argument("preset")
     p.add_argument("out")

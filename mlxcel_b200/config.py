@@ -141,7 +141,15 @@ class ModelConfig:
             return []
         return [int(x) for x in e] if isinstance(e, (list, tuple)) else [int(e)]
 
+    def kv_geometry(self) -> list[tuple[int, int, int]] | None:
+        """(key / value heads, key width, value width) of every KV-pool layer for models whose attention
+        layers differ or whose keys and values have different widths; None = uniform."""
+        return self.extra.get("kv_geometry")
+
     def kv_bytes_per_token(self, kv_bits: int = 16) -> int:
+        geo = self.kv_geometry()
+        if geo is not None:
+            return sum(h * (dk + dv) for h, dk, dv in geo) * kv_bits // 8
         per = self.num_key_value_heads * self.head_dim
         if kv_bits == 16:
             b = per * 2
@@ -181,7 +189,8 @@ class ModelConfig:
                 # the wrapper owns the LM head: its flag says whether the head is the embedding table
                 inner["tie_word_embeddings"] = raw["tie_word_embeddings"]
             raw = inner
-        mt = raw.get("model_type", "llama")
+        # designs without a published ``model_type`` name themselves in ``architecture``
+        mt = raw.get("model_type") or str(raw.get("architecture", "llama")).lower()
         fam = FAMILIES.get(mt)
         if fam is None:
             raise ValueError(f"unsupported model_type {mt!r}; supported: {sorted(FAMILIES)}")
@@ -1283,6 +1292,52 @@ def _lfm2(c: ModelConfig, raw: dict) -> None:
     c.layer_types = None
 
 
+def _pamasun(c: ModelConfig, raw: dict) -> None:
+    """Pamasun: an explicit layer list (attention or generalized-delta mixer, dense MLP or none), every
+    sub-layer normalised on both sides with a layer scale, and optionally a run of layers repeated with
+    the same weights (``loop``). ``extra["layer_specs"]`` keeps the list, ``extra["layer_runs"]`` the layer
+    index of every run in order; each attention run owns a KV-pool layer, each delta run a state slab."""
+    c.vocab_size, c.hidden_size = int(raw["vocab"]), int(raw["width"])
+    c.embed_scale = float((raw.get("embedding") or {}).get("scale", 1.0))
+    c.rms_norm_eps = float(raw["norm"]["eps"])
+    c.norm_weight_bias = 1.0
+    specs = []
+    for i, spec in enumerate(raw["layers"]):
+        kind, m, mlp = spec["type"], dict(spec["mixer"]), spec.get("mlp")
+        if kind == "attention":
+            m = dict(heads=int(m["heads"]), kv_heads=int(m["kv_heads"]), dim=int(m["dim"]), vdim=int(m["vdim"]),
+                     scale=float(m["scale"]))
+            if m["heads"] % m["kv_heads"]:
+                raise ValueError(f"layer {i}: heads must be a multiple of kv_heads")
+        elif kind == "general_delta":
+            m = dict(heads=int(m["heads"]), dim=int(m["dim"]))
+        else:
+            raise ValueError(f"layer {i}: unknown mixer type {kind!r}")
+        if mlp is not None:
+            if mlp.get("kind", "dense") != "dense":
+                raise ValueError(f"layer {i}: unknown feed-forward kind {mlp.get('kind')!r}")
+            mlp = dict(kind="dense", ff=int(mlp["ff"]))
+        specs.append(dict(type=kind, mixer=m, mlp=mlp))
+    n = len(specs)
+    runs = list(range(n))
+    loop = raw.get("loop")
+    if loop:
+        a, b, times = int(loop["start"]), int(loop["stop"]), int(loop["times"])
+        if not (0 <= a <= b <= n) or times < 0:
+            raise ValueError(f"loop {loop} does not fit {n} layers")
+        runs = runs[:a] + runs[a:b] * times + runs[b:]
+        c.extra["loop"] = dict(start=a, stop=b, times=times)
+    c.extra["layer_specs"], c.extra["layer_runs"] = specs, runs
+    c.num_hidden_layers = n
+    att = [specs[i]["mixer"] for i in runs if specs[i]["type"] == "attention"]
+    c.extra["kv_geometry"] = [(m["kv_heads"], m["dim"], m["vdim"]) for m in att]
+    # (uniform fields other parts read: the first attention layer's, or the minimum a pool accepts)
+    m0 = att[0] if att else dict(heads=1, kv_heads=1, dim=16)
+    c.num_attention_heads, c.num_key_value_heads, c.head_dim = m0["heads"], m0["kv_heads"], m0["dim"]
+    c.partial_rotary_factor = 0.0
+    c.intermediate_size = max([s["mlp"]["ff"] for s in specs if s["mlp"]] or [1])
+
+
 def _baichuan(c: ModelConfig, raw: dict) -> None:
     """Baichuan (7B layout): Llama block with q, k, v fused in ``W_pack`` (reference src/models/baichuan.rs).
     The 13B models replace RoPE by ALiBi, which no attention kernel here implements."""
@@ -1306,6 +1361,7 @@ FAMILIES = {
     "gpt_neox": _gpt_neox, "gpt2": _gpt2, "gpt_bigcode": _gpt2, "phi": _phi, "olmo": _olmo1, "granitemoe": _granitemoe, "granitemoehybrid": _granitemoehybrid, "jamba": _jamba, "bitnet": _bitnet, "lfm2_moe": _lfm2, "exaone": _exaone, "telechat3": _telechat3, "deepseek": _deepseek_v1, "recurrent_gemma": _recurrent_gemma, "glm_moe_dsa": _glm_moe_dsa, "deepseek_v32": _glm_moe_dsa, "mistral4": _mistral4, "afmoe": _afmoe, "dbrx": _dbrx, "llama4": _llama4, "llama4_text": _llama4, "qwen3_next": _qwen3_next, "qwen3_5": _qwen3_next, "qwen3_5_text": _qwen3_next, "qwen3_5_moe": _qwen3_next, "qwen3_5_moe_text": _qwen3_next, "falcon_h1": _falcon_h1, "cohere2": _cohere2, "arcee": _arcee, "glm": _glm, "glm4": _glm4, "glm4v": _glm4v, "glm4v_text": _glm4v, "glm4v_moe": _glm4v_moe, "glm4v_moe_text": _glm4v_moe, "cohere2_vision": _cohere2, "paddleocr_vl": _paddleocr_vl, "glm_ocr": _glm_ocr, "glm_ocr_text": _glm_ocr, "paddleocr_vl_text": _paddleocr_vl, "nemotron": _nemotron,
     "ministral3": _ministral3, "granitemoeshared": _granitemoeshared, "nanochat": _nanochat, "code_llama": _plain, "cwm": _plain, "glm4_moe_lite": _deepseek_v3,
     "vaultgemma": _vaultgemma, "solar_open": _solar_open, "minimax_m2": _minimax_m2, "exaone_moe": _exaone_moe, "lfm2": _lfm2, "internlm2": _plain, "baichuan": _baichuan,
+    "pamasun": _pamasun,
 }
 
 
@@ -1367,6 +1423,12 @@ def preset(name: str) -> ModelConfig:
             model_type="nemotron_h", hidden_size=128, hybrid_override_pattern="M-M*-M-", mamba_num_heads=8,
             mamba_head_dim=32, ssm_state_size=32, conv_kernel=4, n_groups=2, intermediate_size=256,
             num_attention_heads=4, num_key_value_heads=2, head_dim=64, vocab_size=1024, layer_norm_epsilon=1e-5))
+    if name == "tiny-pamasun":
+        attn = dict(type="attention", mixer=dict(heads=6, kv_heads=2, dim=32, vdim=48, scale=0.2), mlp=dict(kind="dense", ff=224))
+        delta = dict(type="general_delta", mixer=dict(heads=3, dim=40), mlp=dict(kind="dense", ff=160))
+        return ModelConfig.from_dict(dict(
+            architecture="Pamasun", vocab=512, width=144, layers=[delta, attn, dict(delta, mlp=None), attn],
+            loop=dict(start=1, stop=3, times=2), embedding=dict(scale=12.0), norm=dict(eps=1e-5)))
     if name == "mamba2-2.7b":
         return ModelConfig.from_dict(dict(
             model_type="mamba2", num_hidden_layers=64, hidden_size=2560, num_heads=80, head_dim=64,

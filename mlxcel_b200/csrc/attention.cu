@@ -44,6 +44,15 @@ struct DecodeParams {
   int* counters;       // [B * Hkv]
   int B, Hq, Hkv, block_size, max_blocks, window, num_splits;
   float scale_log2, softcap;
+  // Extended form (template parameter EXT of the tensor-core kernel): key and value rows of dk / dv
+  // elements (multiples of 8 up to the padded tile widths), a logarithmic distance bias per query head
+  // (r1[h] ln(1 + r2[h] d) is taken off the score of a key d tokens back) and an output gate
+  // (result *= sigmoid(gate)). bias and gate may be NULL.
+  int dk, dv;
+  const float* bias_r1;
+  const float* bias_r2;
+  const __nv_bfloat16* gate;
+  long long gate_stride;
 };
 
 // Loads 8 consecutive elements of a K/V row as floats.
@@ -631,12 +640,19 @@ constexpr int kDmThreads = kDmWarps * 32;
 constexpr int kDmStages = 3;
 constexpr int kDmKeys = 16;  // keys per group (one MMA k-step of P V)
 
-template <int D, int KV_BITS, bool BS16>
+template <int DK, int DV, int KV_BITS, bool BS16, bool EXT>
 __global__ void __launch_bounds__(kDmThreads)
 paged_decode_mma_kernel(const DecodeParams p, const int G) {
-  constexpr int CH = D / 8;
-  constexpr int TILE_BYTES = kDmKeys * D * 2;            // one K (or V) group in bf16
-  constexpr int STAGE_BYTES = 2 * TILE_BYTES;            // K + V
+  // DK / DV: tile widths of keys and values; the plain form has rows of exactly D = DK = DV elements,
+  // the extended one rows of p.dk / p.dv whose missing columns are zero-filled on load.
+  constexpr int D = DK;
+  static_assert(EXT || DK == DV, "plain form: one head width");
+  static_assert(!EXT || KV_BITS == 16, "the extended form reads bf16 pools");
+  constexpr int CH = DK / 8, CHV = DV / 8;
+  constexpr int TILE_BYTES = kDmKeys * DK * 2;           // one K group in bf16
+  constexpr int VTILE_BYTES = kDmKeys * DV * 2;          // one V group
+  constexpr int STAGE_BYTES = TILE_BYTES + VTILE_BYTES;
+  const int dk = EXT ? p.dk : DK, dv = EXT ? p.dv : DV;
   constexpr int WARP_BYTES = kDmStages * STAGE_BYTES;
   // Quantized pools: a ring stage holds the RAW group (K codes, V codes, K and V scale/offset
   // pairs), fetched with cp.async like the bf16 tiles so that the ring keeps several groups in
@@ -681,8 +697,8 @@ paged_decode_mma_kernel(const DecodeParams p, const int G) {
     const int grp = s_begin + static_cast<int>(threadIdx.x);
     if (threadIdx.x < kPrefetchGroups && grp < s_end) {
       const size_t row16 = (static_cast<size_t>(table[grp]) * p.Hkv + h) * kDmKeys;
-      bulk_prefetch_l2(static_cast<const __nv_bfloat16*>(p.k_pool) + row16 * D, TILE_BYTES);
-      bulk_prefetch_l2(static_cast<const __nv_bfloat16*>(p.v_pool) + row16 * D, TILE_BYTES);
+      bulk_prefetch_l2(static_cast<const __nv_bfloat16*>(p.k_pool) + row16 * dk, kDmKeys * dk * 2);
+      bulk_prefetch_l2(static_cast<const __nv_bfloat16*>(p.v_pool) + row16 * dv, kDmKeys * dv * 2);
     }
   }
   pdl_wait();
@@ -691,9 +707,9 @@ paged_decode_mma_kernel(const DecodeParams p, const int G) {
   for (int i = threadIdx.x; i < 16 * CH; i += kDmThreads) {
     const int r = i / CH, c = i - r * CH;
     uint4 v = make_uint4(0, 0, 0, 0);
-    if (r < G)
+    if (r < G && (!EXT || c * 8 < dk))
       v = *reinterpret_cast<const uint4*>(p.q + static_cast<size_t>(b) * p.q_stride +
-                                          static_cast<size_t>(h * G + r) * D + c * 8);
+                                          static_cast<size_t>(h * G + r) * dk + c * 8);
     *reinterpret_cast<uint4*>(q_sm + swz<D>(r, c)) = v;
   }
   __syncthreads();
@@ -716,10 +732,11 @@ paged_decode_mma_kernel(const DecodeParams p, const int G) {
       const size_t row16 = (static_cast<size_t>(blk16) * p.Hkv + h) * kDmKeys;
       const int rows_ok = len - grp * kDmKeys;  // rows below this index hold real keys
       if constexpr (!kQuant) {
+        constexpr int CM = CH > CHV ? CH : CHV;
 #pragma unroll
-        for (int it = 0; it < (kDmKeys * CH) / 32; ++it) {
+        for (int it = 0; it < (kDmKeys * CM) / 32; ++it) {
           const int i = lane + it * 32;
-          const int r = i / CH, c = i - r * CH;
+          const int r = i / CM, c = i - r * CM;
           const bool ok = r < rows_ok;
           size_t row;
           if (BS16) {
@@ -729,10 +746,21 @@ paged_decode_mma_kernel(const DecodeParams p, const int G) {
             const int blk = ok ? table[key / p.block_size] : 0;
             row = (static_cast<size_t>(blk) * p.Hkv + h) * p.block_size + (ok ? key % p.block_size : 0);
           }
-          cp_async16(smem_u32(ks) + swz<D>(r, c),
-                     static_cast<const __nv_bfloat16*>(p.k_pool) + row * D + c * 8, ok);
-          cp_async16(smem_u32(vs) + swz<D>(r, c),
-                     static_cast<const __nv_bfloat16*>(p.v_pool) + row * D + c * 8, ok);
+          if constexpr (!EXT) {
+            cp_async16(smem_u32(ks) + swz<DK>(r, c),
+                       static_cast<const __nv_bfloat16*>(p.k_pool) + row * DK + c * 8, ok);
+            cp_async16(smem_u32(vs) + swz<DV>(r, c),
+                       static_cast<const __nv_bfloat16*>(p.v_pool) + row * DV + c * 8, ok);
+          } else {
+            // columns past the row's width are zero-filled from a valid address
+            const bool kok = ok && c * 8 < dk, vok = ok && c * 8 < dv;
+            if (c < CH)
+              cp_async16(smem_u32(ks) + swz<DK>(r, c),
+                         static_cast<const __nv_bfloat16*>(p.k_pool) + row * dk + (kok ? c * 8 : 0), kok);
+            if (c < CHV)
+              cp_async16(smem_u32(vs) + swz<DV>(r, c),
+                         static_cast<const __nv_bfloat16*>(p.v_pool) + row * dv + (vok ? c * 8 : 0), vok);
+          }
         }
       }
       if constexpr (kQuant) {
@@ -782,9 +810,17 @@ paged_decode_mma_kernel(const DecodeParams p, const int G) {
   auto table_at = [&](int grp) -> int { return (BS16 && grp < s_end) ? table[grp] : 0; };
 
   float m_lo = -INFINITY, m_hi = -INFINITY, l_lo = 0.f, l_hi = 0.f;
-  float o_acc[D / 8][4];
+  float o_acc[DV / 8][4];
 #pragma unroll
-  for (int i = 0; i < D / 8; ++i) o_acc[i][0] = o_acc[i][1] = o_acc[i][2] = o_acc[i][3] = 0.f;
+  for (int i = 0; i < DV / 8; ++i) o_acc[i][0] = o_acc[i][1] = o_acc[i][2] = o_acc[i][3] = 0.f;
+  float b1_lo = 0.f, b1_hi = 0.f, b2_lo = 0.f, b2_hi = 0.f;   // distance bias of this lane's two rows
+  if constexpr (EXT) {
+    if (p.bias_r1 != nullptr) {
+      const int g_lo = lane >> 2, g_hi = g_lo + 8;
+      if (g_lo < G) b1_lo = p.bias_r1[h * G + g_lo], b2_lo = p.bias_r2[h * G + g_lo];
+      if (g_hi < G) b1_hi = p.bias_r1[h * G + g_hi], b2_hi = p.bias_r2[h * G + g_hi];
+    }
+  }
 
   const int first = s_begin + warp;
 #pragma unroll
@@ -860,6 +896,11 @@ paged_decode_mma_kernel(const DecodeParams p, const int G) {
         const int key = key0 + nt * 8 + (lane & 3) * 2 + (e & 1);
         float v = sacc[nt][e] * p.scale_log2;
         if (p.softcap > 0.f) v = p.softcap * tanhf(v / (kLog2e * p.softcap)) * kLog2e;
+        if constexpr (EXT) {
+          // in the log2 domain the bias is r1 log2(1 + r2 d): the natural logarithm's factor cancels
+          const float dist = static_cast<float>(max(len - 1 - key, 0));
+          v -= (e < 2 ? b1_lo : b1_hi) * log2f(fmaf(e < 2 ? b2_lo : b2_hi, dist, 1.f));
+        }
         v = (key >= begin && key < len) ? v : -INFINITY;
         sacc[nt][e] = v;
         if (e < 2) tmax_lo = fmaxf(tmax_lo, v);
@@ -893,7 +934,7 @@ paged_decode_mma_kernel(const DecodeParams p, const int G) {
     // whenever no row of the warp moved its maximum.
     if (__any_sync(0xffffffffu, sc_lo != 1.0f || sc_hi != 1.0f)) {
 #pragma unroll
-      for (int i = 0; i < D / 8; ++i) {
+      for (int i = 0; i < DV / 8; ++i) {
         o_acc[i][0] *= sc_lo;
         o_acc[i][1] *= sc_lo;
         o_acc[i][2] *= sc_hi;
@@ -906,11 +947,11 @@ paged_decode_mma_kernel(const DecodeParams p, const int G) {
     a[2] = pack_bf16(sacc[1][0], sacc[1][1]);
     a[3] = pack_bf16(sacc[1][2], sacc[1][3]);
 #pragma unroll
-    for (int nt = 0; nt < D / 16; ++nt) {
+    for (int nt = 0; nt < DV / 16; ++nt) {
       uint32_t bfr[4];
       const int row = (lane & 7) + ((lane >> 3) & 1) * 8;
       const int chunk = nt * 2 + (lane >> 4);
-      ldmatrix_x4_trans(bfr, vs + swz<D>(row, chunk));
+      ldmatrix_x4_trans(bfr, vs + swz<DV>(row, chunk));
       mma_bf16_16816(o_acc[nt * 2], a, bfr[0], bfr[1]);
       mma_bf16_16816(o_acc[nt * 2 + 1], a, bfr[2], bfr[3]);
     }
@@ -934,10 +975,10 @@ paged_decode_mma_kernel(const DecodeParams p, const int G) {
       l_s[warp][r_hi] = l_hi;
     }
 #pragma unroll
-    for (int i = 0; i < D / 8; ++i) {
+    for (int i = 0; i < DV / 8; ++i) {
       const int col = i * 8 + (lane & 3) * 2;
-      float* dlo = o_s + (warp * 16 + r_lo) * D + col;
-      float* dhi = o_s + (warp * 16 + r_hi) * D + col;
+      float* dlo = o_s + (warp * 16 + r_lo) * DV + col;
+      float* dhi = o_s + (warp * 16 + r_hi) * DV + col;
       dlo[0] = o_acc[i][0];
       dlo[1] = o_acc[i][1];
       dhi[0] = o_acc[i][2];
@@ -946,10 +987,18 @@ paged_decode_mma_kernel(const DecodeParams p, const int G) {
   }
   __syncthreads();
   const size_t part_idx = (static_cast<size_t>(b) * p.Hkv + h) * p.num_splits + split;
-  float* part_o = p.scratch_o + part_idx * (static_cast<size_t>(G) * D);
+  float* part_o = p.scratch_o + part_idx * (static_cast<size_t>(G) * dv);
+  const auto finish = [&](int g, int d, float r) {
+    const size_t col = static_cast<size_t>(h * G + g) * dv + d;
+    if constexpr (EXT) {
+      if (p.gate != nullptr)
+        r *= 1.f / (1.f + __expf(-__bfloat162float(p.gate[static_cast<size_t>(b) * p.gate_stride + col])));
+    }
+    p.out[static_cast<size_t>(b) * p.Hq * dv + col] = __float2bfloat16(r);
+  };
   float* part_ml = p.scratch_ml + part_idx * (static_cast<size_t>(G) * 2);
-  for (int i = threadIdx.x; i < G * D; i += kDmThreads) {
-    const int g = i / D, d = i - g * D;
+  for (int i = threadIdx.x; i < G * dv; i += kDmThreads) {
+    const int g = i / dv, d = i - g * dv;
     float m = -INFINITY;
 #pragma unroll
     for (int w = 0; w < kDmWarps; ++w) m = fmaxf(m, m_s[w][g]);
@@ -958,7 +1007,7 @@ paged_decode_mma_kernel(const DecodeParams p, const int G) {
     for (int w = 0; w < kDmWarps; ++w) {
       const float sc = (m_s[w][g] > -INFINITY) ? exp2f(m_s[w][g] - m) : 0.f;
       l += l_s[w][g] * sc;
-      o += o_s[(w * 16 + g) * D + d] * sc;
+      o += o_s[(w * 16 + g) * DV + d] * sc;
     }
     if (p.num_splits == 1) {
       if (p.sinks != nullptr) {
@@ -968,8 +1017,7 @@ paged_decode_mma_kernel(const DecodeParams p, const int G) {
         l = l * sc + exp2f(sk - m2);
         o *= sc;
       }
-      const float r = l > 0.f ? o / l : 0.f;
-      p.out[static_cast<size_t>(b) * p.Hq * D + (h * G + g) * D + d] = __float2bfloat16(r);
+      finish(g, d, l > 0.f ? o / l : 0.f);
     } else {
       part_o[i] = o;
       if (d == 0) {
@@ -991,8 +1039,8 @@ paged_decode_mma_kernel(const DecodeParams p, const int G) {
   if (!last_s) return;
   __threadfence();
   const size_t base_idx = (static_cast<size_t>(b) * p.Hkv + h) * p.num_splits;
-  for (int i = threadIdx.x; i < G * D; i += kDmThreads) {
-    const int g = i / D, d = i - g * D;
+  for (int i = threadIdx.x; i < G * dv; i += kDmThreads) {
+    const int g = i / dv, d = i - g * dv;
     float m = -INFINITY;
     for (int s2 = 0; s2 < p.num_splits; ++s2)
       m = fmaxf(m, __ldcg(&p.scratch_ml[(base_idx + s2) * (G * 2) + g * 2]));
@@ -1007,19 +1055,19 @@ paged_decode_mma_kernel(const DecodeParams p, const int G) {
       const float ls = __ldcg(&p.scratch_ml[(base_idx + s2) * (G * 2) + g * 2 + 1]);
       const float sc = (ms > -INFINITY) ? exp2f(ms - m) : 0.f;
       l += ls * sc;
-      o += __ldcg(&p.scratch_o[(base_idx + s2) * (static_cast<size_t>(G) * D) + i]) * sc;
+      o += __ldcg(&p.scratch_o[(base_idx + s2) * (static_cast<size_t>(G) * dv) + i]) * sc;
     }
     if (p.sinks != nullptr) l += exp2f(sk - m);
-    const float r = l > 0.f ? o / l : 0.f;
-    p.out[static_cast<size_t>(b) * p.Hq * D + (h * G + g) * D + d] = __float2bfloat16(r);
+    finish(g, d, l > 0.f ? o / l : 0.f);
   }
 }
 
-template <int D, int KV_BITS, bool BS16>
+template <int DK, int DV, int KV_BITS, bool BS16, bool EXT>
 static int launch_decode_mma_bs(const DecodeParams& p, int G, int grid, cudaStream_t st) {
-  constexpr int smem = 16 * D * 2 + kDmWarps * kDmStages * 2 * kDmKeys * D * 2;
-  static_assert(kDmWarps * kDmStages * 2 * kDmKeys * D * 2 >= kDmWarps * 16 * D * 4, "merge buffer");
-  auto kern = paged_decode_mma_kernel<D, KV_BITS, BS16>;
+  constexpr int ring = kDmWarps * kDmStages * kDmKeys * (DK + DV) * 2;
+  constexpr int smem = 16 * DK * 2 + ring;
+  static_assert(ring >= kDmWarps * 16 * DV * 4, "merge buffer");
+  auto kern = paged_decode_mma_kernel<DK, DV, KV_BITS, BS16, EXT>;
   static bool configured = false;
   if (!configured) {
     cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
@@ -1033,8 +1081,14 @@ static int launch_decode_mma_bs(const DecodeParams& p, int G, int grid, cudaStre
 
 template <int D, int KV_BITS>
 static int launch_decode_mma(const DecodeParams& p, int G, int grid, cudaStream_t st) {
-  if (p.block_size == kDmKeys) return launch_decode_mma_bs<D, KV_BITS, true>(p, G, grid, st);
-  return launch_decode_mma_bs<D, KV_BITS, false>(p, G, grid, st);
+  if (p.block_size == kDmKeys) return launch_decode_mma_bs<D, D, KV_BITS, true, false>(p, G, grid, st);
+  return launch_decode_mma_bs<D, D, KV_BITS, false, false>(p, G, grid, st);
+}
+
+template <int DK, int DV>
+static int launch_decode_ext(const DecodeParams& p, int G, int grid, cudaStream_t st) {
+  if (p.block_size == kDmKeys) return launch_decode_mma_bs<DK, DV, 16, true, true>(p, G, grid, st);
+  return launch_decode_mma_bs<DK, DV, 16, false, true>(p, G, grid, st);
 }
 
 // ----------------------------------------------------------------------------- dispatch
@@ -1082,9 +1136,14 @@ static int launch_prefill(const PrefillParams& p, int D, int G, int grid, cudaSt
 
 using namespace mx;
 
+// Split-arrival counters sit at the start of the scratch buffer and must read zero at every call. Their
+// region has one size for all calls, so that the partials of a call with few (sequence, kv head) pairs
+// never land where a later call with more pairs keeps counters.
+constexpr int kDecodeCounters = 65536;
+
 extern "C" long long mx_paged_decode_scratch_floats(int B, int Hq, int D, int num_splits) {
-  // o partials + (m, l) pairs + one counter per (sequence, kv head) (<= B * Hq ints)
-  return static_cast<long long>(B) * Hq * num_splits * (D + 2) + static_cast<long long>(B) * Hq + 64;
+  // o partials + (m, l) pairs behind the counters of the (sequence, kv head) pairs
+  return static_cast<long long>(B) * Hq * num_splits * (D + 2) + kDecodeCounters;
 }
 
 extern "C" int mx_paged_decode(const void* q, long long q_stride, const void* k_pool,
@@ -1111,8 +1170,8 @@ extern "C" int mx_paged_decode(const void* q, long long q_stride, const void* k_
   p.out = static_cast<__nv_bfloat16*>(out);
   // scratch layout: counters first (they must stay zero between calls), then (m,l), then o.
   p.counters = reinterpret_cast<int*>(scratch);
-  const size_t n_cnt = ((static_cast<size_t>(B) * Hkv + 63) / 64) * 64;
-  p.scratch_ml = scratch + n_cnt;
+  if (num_splits > 1 && static_cast<long long>(B) * Hkv > kDecodeCounters) return -1;
+  p.scratch_ml = scratch + kDecodeCounters;
   p.scratch_o = p.scratch_ml + static_cast<size_t>(B) * Hkv * num_splits * G * 2;
   p.B = B;
   p.Hq = Hq;
@@ -1140,6 +1199,54 @@ extern "C" int mx_paged_decode(const void* q, long long q_stride, const void* k_
   if (kv_bits == 16) return launch_decode<16>(p, D, G, grid, stream);
   if (kv_bits == 8) return launch_decode<8>(p, D, G, grid, stream);
   return -1;
+}
+
+// Extended decode form over bf16 pools: key / value rows of Dk / Dv elements (multiples of 8, at most
+// 128), distance bias and output gate optional. -10 = not covered (use mx_paged_attention_any).
+extern "C" int mx_paged_decode_ext(const void* q, long long q_stride, const void* k_pool, const void* v_pool,
+                                   const int* block_tables, const int* context_lens, const float* sinks,
+                                   const float* bias_r1, const float* bias_r2, const void* gate, long long gate_stride,
+                                   void* out, float* scratch, int B, int Hq, int Hkv, int Dk, int Dv, int block_size,
+                                   int max_blocks, int window, float scale, int num_splits, void* stream_) {
+  if (B <= 0) return 0;
+  if (Hkv <= 0 || Hq % Hkv || (bias_r1 == nullptr) != (bias_r2 == nullptr)) return -1;
+  const int G = Hq / Hkv;
+  const auto al16 = [](const void* a) { return (reinterpret_cast<uintptr_t>(a) & 15) == 0; };
+  if (G > 16 || Dk % 8 || Dv % 8 || Dk > 128 || Dv > 128 || block_size % 16 || q_stride % 8 || !al16(q) || !al16(k_pool) ||
+      !al16(v_pool))
+    return -10;
+  if (num_splits < 1) num_splits = 1;
+  DecodeParams p{};
+  p.q = static_cast<const __nv_bfloat16*>(q);
+  p.q_stride = q_stride;
+  p.k_pool = k_pool;
+  p.v_pool = v_pool;
+  p.block_tables = block_tables;
+  p.context_lens = context_lens;
+  p.sinks = sinks;
+  p.out = static_cast<__nv_bfloat16*>(out);
+  p.counters = reinterpret_cast<int*>(scratch);
+  if (num_splits > 1 && static_cast<long long>(B) * Hkv > kDecodeCounters) return -1;
+  p.scratch_ml = scratch + kDecodeCounters;
+  p.scratch_o = p.scratch_ml + static_cast<size_t>(B) * Hkv * num_splits * G * 2;
+  p.B = B;
+  p.Hq = Hq;
+  p.Hkv = Hkv;
+  p.block_size = block_size;
+  p.max_blocks = max_blocks;
+  p.window = window;
+  p.num_splits = num_splits;
+  p.scale_log2 = scale * kLog2e;
+  p.dk = Dk;
+  p.dv = Dv;
+  p.bias_r1 = bias_r1;
+  p.bias_r2 = bias_r2;
+  p.gate = static_cast<const __nv_bfloat16*>(gate);
+  p.gate_stride = gate_stride;
+  const int grid = B * Hkv * num_splits;
+  cudaStream_t st = static_cast<cudaStream_t>(stream_);
+  if (Dk <= 64) return Dv <= 64 ? launch_decode_ext<64, 64>(p, G, grid, st) : launch_decode_ext<64, 128>(p, G, grid, st);
+  return Dv <= 64 ? launch_decode_ext<128, 64>(p, G, grid, st) : launch_decode_ext<128, 128>(p, G, grid, st);
 }
 
 extern "C" int mx_paged_prefill(const void* q, long long q_stride, const void* k_pool,

@@ -45,22 +45,37 @@ struct TcPrefillParams {
   int* status;
   int num_seqs, Hq, Hkv, max_blocks, window, tiles_per_seq;
   float scale_log2;
+  // Extended form (EXT): rows of dk / dv elements inside tiles of DK / DV columns (the tensor maps end at
+  // the row's width, so the missing columns arrive as zeros), a logarithmic distance bias
+  // r1[h] ln(1 + r2[h] d) taken off the scores, an output gate (result *= sigmoid(gate)); bias and gate
+  // may be NULL.
+  int dk, dv;
+  const float* bias_r1;
+  const float* bias_r2;
+  const __nv_bfloat16* gate;
+  long long gate_stride;
 };
 
-template <int D>
+// Distances inside a (query tile, key tile) pair span 255 values; a softmax warp (32 rows) meets 159 of
+// them, so it tabulates its biases once per tile instead of taking a logarithm per score.
+constexpr int kBiasTab = 160;
+
+template <int DK, int DV, bool EXT>
 __global__ void __launch_bounds__(kTcThreads, 1)
 paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
                         const __grid_constant__ CUtensorMap map_v, const TcPrefillParams p) {
-  constexpr int DC = D / 64;                          // 64-column (128-byte) sub-tiles per row
+  constexpr int DC = DK / 64, DCV = DV / 64;          // 64-column (128-byte) sub-tiles per row
   constexpr int SUB_BYTES = 128 * 128;                // one [128 rows][64 cols] sub-tile
   constexpr int Q_BYTES = DC * SUB_BYTES;
-  constexpr int K_BYTES = DC * SUB_BYTES;             // [128 keys][D]
-  constexpr int V_BYTES = DC * SUB_BYTES;
+  constexpr int K_BYTES = DC * SUB_BYTES;             // [128 keys][DK]
+  constexpr int V_BYTES = DCV * SUB_BYTES;
   constexpr int P_BYTES = 2 * SUB_BYTES;              // [128 rows][128 keys]
   constexpr int S_COLS = kTcKeys;                     // fp32 columns of one score buffer
   constexpr int O_COL = 2 * S_COLS;                   // first TMEM column of O
   constexpr uint32_t TMEM_COLS = 512;
-  static_assert(D == 64 || D == 128, "head dim");
+  static_assert((DK == 64 || DK == 128) && (DV == 64 || DV == 128), "head dims");
+  static_assert(EXT || DK == DV, "plain form: one head width");
+  const int dk = EXT ? p.dk : DK, dv = EXT ? p.dv : DV;
 
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) &
@@ -80,6 +95,7 @@ paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
   uint64_t* pv_done = p_full + 1;            // 1
   uint64_t* k_empty = pv_done + 1;           // [stages] K tile consumed (after the score MMA)
   uint32_t* tmem_ptr = reinterpret_cast<uint32_t*>(k_empty + kTcStages);
+  float* bias_tab = reinterpret_cast<float*>(p_sm + P_BYTES + 256);   // EXT: 4 warps x kBiasTab
 
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
 
@@ -139,7 +155,7 @@ paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
     if (lane == 0) {
       mbar_expect_tx(q_full, Q_BYTES);
       for (int c = 0; c < DC; ++c)
-        tma_load_2d(q_sm + c * SUB_BYTES, &map_q, q_full, hq * D + c * 64, q0 + tok0, pol_q);
+        tma_load_2d(q_sm + c * SUB_BYTES, &map_q, q_full, hq * dk + c * 64, q0 + tok0, pol_q);
     }
     int stage = 0;
     uint32_t phase = 0;
@@ -172,7 +188,7 @@ paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
       if (!ok) break;
       if (lane < kTcKeys / kTcBlock) {
         uint8_t* vd = v_sm + stage * V_BYTES + lane * (kTcBlock * 128);
-        for (int c = 0; c < DC; ++c) tma_load_2d(vd + c * SUB_BYTES, &map_v, &v_full[stage], c * 64, row0, pol_kv);
+        for (int c = 0; c < DCV; ++c) tma_load_2d(vd + c * SUB_BYTES, &map_v, &v_full[stage], c * 64, row0, pol_kv);
       }
       __syncwarp();
       if (++stage == kTcStages) {
@@ -184,7 +200,7 @@ paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
     // ------------------------------------------------------------------ MMA issuer
     if (lane == 0) {
       constexpr uint32_t idesc_qk = umma_idesc_bf16(kTcKeys, false, false);   // N = keys
-      constexpr uint32_t idesc_pv = umma_idesc_bf16(D, false, true);          // N = D, V is MN-major
+      constexpr uint32_t idesc_pv = umma_idesc_bf16(DV, false, true);         // N = DV, V is MN-major
       bool ok = mbar_wait(q_full, 0, p.status, kErrAttnMma);
       auto issue_qk = [&](int j) -> bool {
         const int stage = j % kTcStages;
@@ -196,7 +212,7 @@ paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
         tc_fence_after_sync();
         const uint32_t qa = smem_u32(q_sm), kb = smem_u32(k_sm + stage * K_BYTES);
 #pragma unroll
-        for (int kk = 0; kk < D / 16; ++kk) {
+        for (int kk = 0; kk < DK / 16; ++kk) {
           const uint32_t off = (kk >> 2) * SUB_BYTES + (kk & 3) * 32;
           umma_bf16(tmem_base + sb * S_COLS, umma_desc_k_sw128(qa + off), umma_desc_k_sw128(kb + off),
                     idesc_qk, kk > 0 ? 1u : 0u);
@@ -234,6 +250,11 @@ paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
     const int qpos = pos_base + tok0 + row;         // absolute position of this row's token
     float m_used = -INFINITY;   // the maximum the stored exponentials refer to (scaled, log2 units)
     float l = 0.f;
+    float* tab = bias_tab + q4 * kBiasTab;
+    float r1 = 0.f, r2 = 0.f;
+    if constexpr (EXT) {
+      if (p.bias_r1 != nullptr) r1 = p.bias_r1[hq], r2 = p.bias_r2[hq];
+    }
     bool ok = true;
     for (int j = 0; j < n_tiles && ok; ++j) {
       const int sb = j & 1;
@@ -250,6 +271,18 @@ paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
         hi = min(kTcKeys, qpos - key0 + 1);
         if (p.window > 0) lo = max(0, qpos - p.window + 1 - key0);
       }
+      if constexpr (EXT) {
+        // tab[i] = bias of distance base + i, where row r of this warp and key column c are at
+        // i = r - c + 127 (log2 domain: the natural logarithm's factor cancels against log2 e)
+        const int base = pos_base + tok0 + q4 * 32 - key0 - (kTcKeys - 1);
+        __syncwarp();
+#pragma unroll
+        for (int i = 0; i < kBiasTab / 32; ++i) {
+          const float d = static_cast<float>(max(base + lane + i * 32, 0));
+          tab[lane + i * 32] = r1 * log2f(fmaf(r2, d, 1.f));
+        }
+        __syncwarp();
+      }
       float sv[kTcKeys];
 #pragma unroll
       for (int c = 0; c < kTcKeys / 32; ++c) {
@@ -257,7 +290,10 @@ paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
         tmem_ld_32x32(lane_addr + sb * S_COLS + c * 32, r);
         tmem_ld_wait();
 #pragma unroll
-        for (int i = 0; i < 32; ++i) sv[c * 32 + i] = __uint_as_float(r[i]) * p.scale_log2;
+        for (int i = 0; i < 32; ++i) {
+          sv[c * 32 + i] = __uint_as_float(r[i]) * p.scale_log2;
+          if constexpr (EXT) sv[c * 32 + i] -= tab[lane + (kTcKeys - 1) - (c * 32 + i)];
+        }
       }
       tc_fence_before_sync();
       __syncwarp();
@@ -291,7 +327,7 @@ paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
       }
       if (__any_sync(0xffffffffu, rescale)) {
 #pragma unroll
-        for (int c = 0; c < D / 32; ++c) {
+        for (int c = 0; c < DV / 32; ++c) {
           uint32_t r[32];
           tmem_ld_32x32(lane_addr + O_COL + c * 32, r);
           tmem_ld_wait();
@@ -342,15 +378,31 @@ paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
         l = l * osc + exp2f(sk - m2);
       }
       const float inv = l > 0.f ? osc / l : 0.f;
-      __nv_bfloat16* dst = p.out + static_cast<size_t>(q0 + tok0 + row) * p.Hq * D + hq * D;
+      __nv_bfloat16* dst = p.out + static_cast<size_t>(q0 + tok0 + row) * p.Hq * dv + hq * dv;
+      const __nv_bfloat16* gate = nullptr;
+      if constexpr (EXT) {
+        if (p.gate != nullptr) gate = p.gate + static_cast<size_t>(q0 + tok0 + row) * p.gate_stride + hq * dv;
+      }
 #pragma unroll
-      for (int c = 0; c < D / 32; ++c) {
+      for (int c = 0; c < DV / 32; ++c) {
         uint32_t r[32];
         tmem_ld_32x32(lane_addr + O_COL + c * 32, r);
         tmem_ld_wait();
         if (row < rows_valid) {
 #pragma unroll
           for (int i = 0; i < 32; i += 8) {
+            if constexpr (EXT) {
+              if (c * 32 + i >= dv) break;
+              if (gate != nullptr) {
+                const uint4 gv = *reinterpret_cast<const uint4*>(gate + c * 32 + i);
+                const uint32_t gw[4] = {gv.x, gv.y, gv.z, gv.w};
+#pragma unroll
+                for (int e = 0; e < 4; ++e) {
+                  r[i + 2 * e] = __float_as_uint(__uint_as_float(r[i + 2 * e]) / (1.f + __expf(-bf16_lo(gw[e]))));
+                  r[i + 2 * e + 1] = __float_as_uint(__uint_as_float(r[i + 2 * e + 1]) / (1.f + __expf(-bf16_hi(gw[e]))));
+                }
+              }
+            }
             uint4 pk;
             pk.x = pack_bf16(__uint_as_float(r[i]) * inv, __uint_as_float(r[i + 1]) * inv);
             pk.y = pack_bf16(__uint_as_float(r[i + 2]) * inv, __uint_as_float(r[i + 3]) * inv);
@@ -372,13 +424,13 @@ paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
   }
 }
 
-template <int D>
+template <int DK, int DV, bool EXT>
 static int launch_prefill_tc(const CUtensorMap& mq, const CUtensorMap& mk, const CUtensorMap& mv,
                              const TcPrefillParams& p, int grid, cudaStream_t stream) {
-  constexpr int DC = D / 64;
   constexpr int SUB = 128 * 128;
-  const int smem = DC * SUB * (1 + 2 * kTcStages) + 2 * SUB + 1024 + 256;
-  auto kern = paged_prefill_tc_kernel<D>;
+  const int smem = (DK / 64) * SUB * (1 + kTcStages) + (DV / 64) * SUB * kTcStages + 2 * SUB + 1024 + 256 +
+                   (EXT ? 4 * kBiasTab * 4 : 0);
+  auto kern = paged_prefill_tc_kernel<DK, DV, EXT>;
   static bool configured = false;
   if (!configured) {
     cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
@@ -432,6 +484,60 @@ extern "C" int mx_paged_prefill_tc(const void* q, long long q_stride, const void
   const uint64_t pool_rows = static_cast<uint64_t>(pool_blocks) * Hkv * kTcBlock;
   if (!make_tensor_map_bf16(&mk, k_pool, pool_rows, D, D, kTcBlock, 64)) return -4;
   if (!make_tensor_map_bf16(&mv, v_pool, pool_rows, D, D, kTcBlock, 64)) return -4;
-  if (D == 64) return launch_prefill_tc<64>(mq, mk, mv, p, static_cast<int>(grid), stream);
-  return launch_prefill_tc<128>(mq, mk, mv, p, static_cast<int>(grid), stream);
+  if (D == 64) return launch_prefill_tc<64, 64, false>(mq, mk, mv, p, static_cast<int>(grid), stream);
+  return launch_prefill_tc<128, 128, false>(mq, mk, mv, p, static_cast<int>(grid), stream);
+}
+
+// Extended form: key / value rows of Dk / Dv elements (multiples of 8, at most 128), distance bias and
+// output gate optional. Returns -10 when not covered (use mx_paged_attention_any).
+extern "C" int mx_paged_prefill_ext(const void* q, long long q_stride, const void* k_pool, const void* v_pool,
+                                    long long pool_blocks, const int* block_tables, const int* cu_q,
+                                    const int* context_lens, const float* sinks, const float* bias_r1,
+                                    const float* bias_r2, const void* gate, long long gate_stride, void* out,
+                                    int num_seqs, int total_q, int max_q_len, int Hq, int Hkv, int Dk, int Dv,
+                                    int block_size, int max_blocks, int window, float scale, void* status,
+                                    void* stream_) {
+  cudaStream_t stream = static_cast<cudaStream_t>(stream_);
+  if (num_seqs <= 0 || total_q <= 0) return 0;
+  if (Hkv <= 0 || Hq % Hkv || (bias_r1 == nullptr) != (bias_r2 == nullptr)) return -1;
+  const auto al16 = [](const void* a) { return (reinterpret_cast<uintptr_t>(a) & 15) == 0; };
+  if (block_size != kTcBlock || Dk % 8 || Dv % 8 || Dk > 128 || Dv > 128 || q_stride % 8 || gate_stride % 8 || !al16(q) ||
+      !al16(out) || !al16(gate) || !al16(k_pool) || !al16(v_pool))
+    return -10;
+  TcPrefillParams p{};
+  p.block_tables = block_tables;
+  p.cu_q = cu_q;
+  p.context_lens = context_lens;
+  p.sinks = sinks;
+  p.out = static_cast<__nv_bfloat16*>(out);
+  p.status = static_cast<int*>(status);
+  p.num_seqs = num_seqs;
+  p.Hq = Hq;
+  p.Hkv = Hkv;
+  p.max_blocks = max_blocks;
+  p.window = window;
+  p.tiles_per_seq = (max_q_len + kTcRows - 1) / kTcRows;
+  p.scale_log2 = scale * 1.4426950408889634f;
+  p.dk = Dk;
+  p.dv = Dv;
+  p.bias_r1 = bias_r1;
+  p.bias_r2 = bias_r2;
+  p.gate = static_cast<const __nv_bfloat16*>(gate);
+  p.gate_stride = gate_stride;
+  const long long grid = static_cast<long long>(num_seqs) * Hq * p.tiles_per_seq;
+  if (grid > 0x7fffffffll) return -1;
+  CUtensorMap mq, mk, mv;
+  // a query box may run into the next head's columns: the keys' columns there are zero
+  if (!make_tensor_map_bf16(&mq, q, static_cast<uint64_t>(total_q), static_cast<uint64_t>(Hq) * Dk,
+                            static_cast<uint64_t>(q_stride), kTcRows, 64))
+    return -4;
+  const uint64_t pool_rows = static_cast<uint64_t>(pool_blocks) * Hkv * kTcBlock;
+  if (!make_tensor_map_bf16(&mk, k_pool, pool_rows, Dk, Dk, kTcBlock, 64)) return -4;
+  if (!make_tensor_map_bf16(&mv, v_pool, pool_rows, Dv, Dv, kTcBlock, 64)) return -4;
+  const int g = static_cast<int>(grid);
+  if (Dk <= 64)
+    return Dv <= 64 ? launch_prefill_tc<64, 64, true>(mq, mk, mv, p, g, stream)
+                    : launch_prefill_tc<64, 128, true>(mq, mk, mv, p, g, stream);
+  return Dv <= 64 ? launch_prefill_tc<128, 64, true>(mq, mk, mv, p, g, stream)
+                  : launch_prefill_tc<128, 128, true>(mq, mk, mv, p, g, stream);
 }

@@ -1,0 +1,367 @@
+// Row kernels of layers that keep the residual stream in fp32 and normalise on both sides of a
+// sub-layer, each for bf16 and fp32 activations:
+//   embed_stream   h = scale * table[id];  x = norm(h)
+//   stream_norm    h += norm(y) * layer scale;  x = norm(h)     (either half optional)
+//   polynorm       a N(z) + b N(z^2) + c N(z^3) + e, N = division by the row's root mean square
+//   qk_norm_append per-head RMS norm of q and k, k and v rows into the paged pool (key and value heads
+//                  may differ in width; no rotation)
+// A norm weight w acts as (w_bias + w); all norm weights and layer scales are fp32 vectors, all
+// arithmetic is fp32 and only the results are narrowed to the activation type.
+#include "api.h"
+#include "typed.cuh"
+
+namespace mx {
+
+// One CTA per row, V elements per access, up to VPT accesses per thread kept in registers: every
+// input is read once and every output written once.
+template <typename T, int V, int VPT>
+__global__ void __launch_bounds__(1024)
+stream_norm_kernel(const T* __restrict__ y, float* __restrict__ h, const int* __restrict__ rows,
+                   const float* __restrict__ post_w, const float* __restrict__ ls,
+                   const float* __restrict__ pre_w, T* __restrict__ x, int dim, float eps, float w_bias) {
+  __shared__ float red[33];
+  pdl_trigger();
+  pdl_wait();
+  const size_t row = blockIdx.x;
+  float* hr = h + static_cast<size_t>(rows != nullptr ? rows[row] : row) * dim;
+  float hv[VPT][V];
+  float s[1] = {0.f};
+#pragma unroll
+  for (int i = 0; i < VPT; ++i) {
+    const int c = (threadIdx.x + i * blockDim.x) * V;
+    if (c < dim) load_v<V>(hr + c, hv[i]);
+  }
+  if (y != nullptr) {
+    float yv[VPT][V];
+#pragma unroll
+    for (int i = 0; i < VPT; ++i) {
+      const int c = (threadIdx.x + i * blockDim.x) * V;
+      if (c < dim) {
+        load_v<V>(y + row * dim + c, yv[i]);
+#pragma unroll
+        for (int e = 0; e < V; ++e) s[0] += yv[i][e] * yv[i][e];
+      }
+    }
+    block_sums<1>(s, red);
+    const float r = 1.f / sqrtf(s[0] / dim + eps);
+    s[0] = 0.f;
+#pragma unroll
+    for (int i = 0; i < VPT; ++i) {
+      const int c = (threadIdx.x + i * blockDim.x) * V;
+      if (c < dim) {
+        float w[V], l[V];
+        load_v<V>(post_w + c, w);
+        if (ls != nullptr) load_v<V>(ls + c, l);
+#pragma unroll
+        for (int e = 0; e < V; ++e) {
+          const float b = yv[i][e] * r * (w_bias + w[e]);
+          hv[i][e] += ls != nullptr ? b * l[e] : b;
+        }
+        store_v<V>(hr + c, hv[i]);
+      }
+    }
+  }
+  if (x == nullptr) return;
+#pragma unroll
+  for (int i = 0; i < VPT; ++i) {
+    const int c = (threadIdx.x + i * blockDim.x) * V;
+    if (c < dim) {
+#pragma unroll
+      for (int e = 0; e < V; ++e) s[0] += hv[i][e] * hv[i][e];
+    }
+  }
+  block_sums<1>(s, red);
+  const float r = 1.f / sqrtf(s[0] / dim + eps);
+#pragma unroll
+  for (int i = 0; i < VPT; ++i) {
+    const int c = (threadIdx.x + i * blockDim.x) * V;
+    if (c < dim) {
+      float w[V], o[V];
+      load_v<V>(pre_w + c, w);
+#pragma unroll
+      for (int e = 0; e < V; ++e) o[e] = hv[i][e] * r * (w_bias + w[e]);
+      store_v<V>(x + row * dim + c, o);
+    }
+  }
+}
+
+template <typename T, int V, int VPT>
+__global__ void __launch_bounds__(1024)
+embed_stream_kernel(const int* __restrict__ ids, const T* __restrict__ table, float* __restrict__ h,
+                    const float* __restrict__ pre_w, T* __restrict__ x, int dim, int vocab, float scale, float eps,
+                    float w_bias) {
+  __shared__ float red[33];
+  pdl_trigger();
+  pdl_wait();
+  const size_t row = blockIdx.x;
+  const int id = ids[row];
+  const bool ok = id >= 0 && id < vocab;
+  const T* tr = table + static_cast<size_t>(ok ? id : 0) * dim;
+  float hv[VPT][V];
+  float s[1] = {0.f};
+#pragma unroll
+  for (int i = 0; i < VPT; ++i) {
+    const int c = (threadIdx.x + i * blockDim.x) * V;
+    if (c < dim) {
+      load_v<V>(tr + c, hv[i]);
+#pragma unroll
+      for (int e = 0; e < V; ++e) {
+        hv[i][e] = ok ? hv[i][e] * scale : 0.f;
+        s[0] += hv[i][e] * hv[i][e];
+      }
+      store_v<V>(h + row * dim + c, hv[i]);
+    }
+  }
+  block_sums<1>(s, red);
+  const float r = 1.f / sqrtf(s[0] / dim + eps);
+#pragma unroll
+  for (int i = 0; i < VPT; ++i) {
+    const int c = (threadIdx.x + i * blockDim.x) * V;
+    if (c < dim) {
+      float w[V], o[V];
+      load_v<V>(pre_w + c, w);
+#pragma unroll
+      for (int e = 0; e < V; ++e) o[e] = hv[i][e] * r * (w_bias + w[e]);
+      store_v<V>(x + row * dim + c, o);
+    }
+  }
+}
+
+template <typename T, int V, int VPT>
+__global__ void __launch_bounds__(1024)
+polynorm_kernel(const T* __restrict__ z, const float* __restrict__ coef, T* __restrict__ out, int dim, float eps) {
+  __shared__ float red[3 * 33];
+  pdl_trigger();
+  pdl_wait();
+  const size_t row = blockIdx.x;
+  float zv[VPT][V];
+  float s[3] = {0.f, 0.f, 0.f};
+#pragma unroll
+  for (int i = 0; i < VPT; ++i) {
+    const int c = (threadIdx.x + i * blockDim.x) * V;
+    if (c < dim) {
+      load_v<V>(z + row * dim + c, zv[i]);
+#pragma unroll
+      for (int e = 0; e < V; ++e) {
+        const float q = zv[i][e] * zv[i][e];
+        s[0] += q;
+        s[1] += q * q;
+        s[2] += q * q * q;
+      }
+    }
+  }
+  block_sums<3>(s, red);
+  const float a = coef[0] / sqrtf(s[0] / dim + eps), b = coef[1] / sqrtf(s[1] / dim + eps),
+              g = coef[2] / sqrtf(s[2] / dim + eps), e0 = coef[3];
+#pragma unroll
+  for (int i = 0; i < VPT; ++i) {
+    const int c = (threadIdx.x + i * blockDim.x) * V;
+    if (c < dim) {
+      float o[V];
+#pragma unroll
+      for (int e = 0; e < V; ++e) o[e] = ((g * zv[i][e] + b) * zv[i][e] + a) * zv[i][e] + e0;
+      store_v<V>(out + row * dim + c, o);
+    }
+  }
+}
+
+// Rows of q | k | v (| more), `ld` elements apart. A warp handles one (token, head) of the Hq query,
+// Hkv key and Hkv value heads: queries are normalised in place, keys normalised into the pool
+// [blocks, Hkv, block_size, Dk], values copied into [blocks, Hkv, block_size, Dv]. Tokens with a
+// negative slot append nothing. A lane keeps up to 4 groups of V elements (Dk <= 128 V) in registers;
+// wider heads are read twice.
+template <typename T, int V>
+__global__ void __launch_bounds__(256)
+qk_norm_append_kernel(T* __restrict__ qkv, long long ld, const int* __restrict__ slots, T* __restrict__ k_pool,
+                      T* __restrict__ v_pool, const float* __restrict__ qw, const float* __restrict__ kw, int T_,
+                      int Hq, int Hkv, int Dk, int Dv, int block_size, float eps) {
+  pdl_trigger();
+  pdl_wait();
+  const int lane = threadIdx.x & 31, per = Hq + 2 * Hkv;
+  const long long gw = (static_cast<long long>(blockIdx.x) * blockDim.x + threadIdx.x) >> 5;
+  if (gw >= static_cast<long long>(T_) * per) return;
+  const int t = static_cast<int>(gw / per), hd = static_cast<int>(gw - static_cast<long long>(t) * per);
+  T* row = qkv + static_cast<size_t>(t) * ld;
+  const int slot = slots[t];
+  T *src, *dst;
+  const float* w;
+  int D;
+  if (hd < Hq) {
+    src = dst = row + static_cast<size_t>(hd) * Dk, w = qw, D = Dk;
+    if (w == nullptr) return;
+  } else {
+    if (slot < 0) return;
+    const int blk = slot / block_size, off = slot - blk * block_size;
+    const bool key = hd < Hq + Hkv;
+    const int g = key ? hd - Hq : hd - Hq - Hkv;
+    D = key ? Dk : Dv;
+    src = row + static_cast<size_t>(Hq) * Dk + (key ? static_cast<size_t>(g) * Dk : static_cast<size_t>(Hkv) * Dk + static_cast<size_t>(g) * Dv);
+    dst = (key ? k_pool : v_pool) + ((static_cast<size_t>(blk) * Hkv + g) * block_size + off) * D;
+    w = key ? kw : nullptr;
+  }
+  constexpr int R = 4;
+  float f[R][V];
+  float s = 0.f;
+#pragma unroll
+  for (int i = 0; i < R; ++i) {
+    const int c = (lane + 32 * i) * V;
+    if (c < D) {
+      load_v<V>(src + c, f[i]);
+#pragma unroll
+      for (int e = 0; e < V; ++e) s += f[i][e] * f[i][e];
+    }
+  }
+  for (int c = (lane + 32 * R) * V; c < D; c += 32 * V) {
+    float g[V];
+    load_v<V>(src + c, g);
+#pragma unroll
+    for (int e = 0; e < V; ++e) s += g[e] * g[e];
+  }
+  float r = 1.f;
+  if (w != nullptr) r = 1.f / sqrtf(warp_sum(s) / D + eps);
+  const auto emit = [&](int c, const float(&g)[V]) {
+    float o[V], wv[V];
+    if (w != nullptr) load_v<V>(w + c, wv);
+#pragma unroll
+    for (int e = 0; e < V; ++e) o[e] = w != nullptr ? g[e] * r * wv[e] : g[e];
+    store_v<V>(dst + c, o);
+  };
+#pragma unroll
+  for (int i = 0; i < R; ++i) {
+    const int c = (lane + 32 * i) * V;
+    if (c < D) emit(c, f[i]);
+  }
+  for (int c = (lane + 32 * R) * V; c < D; c += 32 * V) {
+    float g[V];
+    load_v<V>(src + c, g);
+    emit(c, g);
+  }
+}
+
+// Launch shape of a row kernel: groups of V elements per row -> threads and accesses per thread.
+struct RowShape {
+  int threads, vpt;
+};
+static RowShape row_shape(int dim, int v) {
+  const int groups = (dim + v - 1) / v;
+  int threads = (groups + 31) / 32 * 32;
+  if (threads > 256) threads = groups > 8 * 256 ? 1024 : 256;
+  if (threads < 64) threads = 64;
+  const int need = (groups + threads - 1) / threads;
+  return {threads, need <= 1 ? 1 : need <= 2 ? 2 : need <= 4 ? 4 : need <= 8 ? 8 : 0};
+}
+
+#define MX_ROW_DISPATCH(KERN, T, V, SHAPE, ROWS, STREAM, ...)                                                        \
+  switch ((SHAPE).vpt) {                                                                                             \
+    case 1: return static_cast<int>(launch_kernel(KERN<T, V, 1>, dim3(ROWS), dim3((SHAPE).threads), 0, STREAM, __VA_ARGS__)); \
+    case 2: return static_cast<int>(launch_kernel(KERN<T, V, 2>, dim3(ROWS), dim3((SHAPE).threads), 0, STREAM, __VA_ARGS__)); \
+    case 4: return static_cast<int>(launch_kernel(KERN<T, V, 4>, dim3(ROWS), dim3((SHAPE).threads), 0, STREAM, __VA_ARGS__)); \
+    case 8: return static_cast<int>(launch_kernel(KERN<T, V, 8>, dim3(ROWS), dim3((SHAPE).threads), 0, STREAM, __VA_ARGS__)); \
+    default: return -1;                                                                                              \
+  }
+
+template <typename T>
+static int stream_norm_typed(const void* y, void* h, const void* rows, const float* post_w, const float* ls, const float* pre_w,
+                             void* x, int n, int dim, float eps, float w_bias, bool vec, cudaStream_t st) {
+  const T* yp = static_cast<const T*>(y);
+  const int* rp = static_cast<const int*>(rows);
+  if (vec) {
+    const RowShape sh = row_shape(dim, 4);
+    MX_ROW_DISPATCH(stream_norm_kernel, T, 4, sh, n, st, yp, static_cast<float*>(h), rp, post_w, ls, pre_w, static_cast<T*>(x), dim, eps, w_bias)
+  }
+  const RowShape sh = row_shape(dim, 1);
+  MX_ROW_DISPATCH(stream_norm_kernel, T, 1, sh, n, st, yp, static_cast<float*>(h), rp, post_w, ls, pre_w, static_cast<T*>(x), dim, eps, w_bias)
+}
+
+template <typename T>
+static int embed_stream_typed(const int* ids, const void* table, void* h, const float* pre_w, void* x, int n, int dim, int vocab,
+                              float scale, float eps, float w_bias, bool vec, cudaStream_t st) {
+  const T* tp = static_cast<const T*>(table);
+  if (vec) {
+    const RowShape sh = row_shape(dim, 4);
+    MX_ROW_DISPATCH(embed_stream_kernel, T, 4, sh, n, st, ids, tp, static_cast<float*>(h), pre_w, static_cast<T*>(x), dim, vocab, scale, eps, w_bias)
+  }
+  const RowShape sh = row_shape(dim, 1);
+  MX_ROW_DISPATCH(embed_stream_kernel, T, 1, sh, n, st, ids, tp, static_cast<float*>(h), pre_w, static_cast<T*>(x), dim, vocab, scale, eps, w_bias)
+}
+
+template <typename T>
+static int polynorm_typed(const void* z, const float* coef, void* out, int n, int dim, float eps, bool vec, cudaStream_t st) {
+  const T* zp = static_cast<const T*>(z);
+  if (vec) {
+    const RowShape sh = row_shape(dim, 4);
+    MX_ROW_DISPATCH(polynorm_kernel, T, 4, sh, n, st, zp, coef, static_cast<T*>(out), dim, eps)
+  }
+  const RowShape sh = row_shape(dim, 1);
+  MX_ROW_DISPATCH(polynorm_kernel, T, 1, sh, n, st, zp, coef, static_cast<T*>(out), dim, eps)
+}
+
+template <typename T>
+static int qk_norm_append_typed(void* qkv, long long ld, const int* slots, void* k_pool, void* v_pool, const float* qw,
+                                const float* kw, int n, int Hq, int Hkv, int Dk, int Dv, int bs, float eps, bool vec,
+                                cudaStream_t st) {
+  const long long warps = static_cast<long long>(n) * (Hq + 2 * Hkv);
+  const long long blocks = (warps + 7) / 8;
+  if (blocks > 0x7fffffffLL) return -1;
+  const dim3 grid(static_cast<unsigned>(blocks)), block(256);
+  T *qp = static_cast<T*>(qkv), *kp = static_cast<T*>(k_pool), *vp = static_cast<T*>(v_pool);
+  if (vec) return static_cast<int>(launch_kernel(qk_norm_append_kernel<T, 4>, grid, block, 0, st, qp, ld, slots, kp, vp, qw, kw, n, Hq, Hkv, Dk, Dv, bs, eps));
+  return static_cast<int>(launch_kernel(qk_norm_append_kernel<T, 1>, grid, block, 0, st, qp, ld, slots, kp, vp, qw, kw, n, Hq, Hkv, Dk, Dv, bs, eps));
+}
+
+}  // namespace mx
+
+using namespace mx;
+
+// fp32: 1 = fp32 activations, 0 = bf16. y / rows / ls / x may be NULL (no branch to add, identity
+// row map, no layer scale, no output norm).
+extern "C" int mx_stream_norm(const void* y, void* h, const void* rows, const void* post_w, const void* ls,
+                              const void* pre_w, void* x, int n, int dim, float eps, float w_bias, int fp32,
+                              void* stream) {
+  if (n <= 0 || dim <= 0) return 0;
+  if (h == nullptr || (y != nullptr && (post_w == nullptr || rows != nullptr)) || (x != nullptr && pre_w == nullptr)) return -1;
+  const size_t ab = fp32 ? 16 : 8;
+  const bool vec = dim % 4 == 0 && aligned_to(y, ab) && aligned_to(x, ab) && aligned_to(h, 16) && aligned_to(post_w, 16) &&
+                   aligned_to(ls, 16) && aligned_to(pre_w, 16);
+  auto st = static_cast<cudaStream_t>(stream);
+  const float *pw = static_cast<const float*>(post_w), *lp = static_cast<const float*>(ls), *nw = static_cast<const float*>(pre_w);
+  return fp32 ? stream_norm_typed<float>(y, h, rows, pw, lp, nw, x, n, dim, eps, w_bias, vec, st)
+              : stream_norm_typed<__nv_bfloat16>(y, h, rows, pw, lp, nw, x, n, dim, eps, w_bias, vec, st);
+}
+
+extern "C" int mx_embed_stream(const void* ids, const void* table, void* h, const void* pre_w, void* x, int n, int dim,
+                               int vocab, float scale, float eps, float w_bias, int fp32, void* stream) {
+  if (n <= 0 || dim <= 0) return 0;
+  const size_t ab = fp32 ? 16 : 8;
+  const bool vec = dim % 4 == 0 && aligned_to(table, ab) && aligned_to(x, ab) && aligned_to(h, 16) && aligned_to(pre_w, 16);
+  auto st = static_cast<cudaStream_t>(stream);
+  const float* nw = static_cast<const float*>(pre_w);
+  const int* ip = static_cast<const int*>(ids);
+  return fp32 ? embed_stream_typed<float>(ip, table, h, nw, x, n, dim, vocab, scale, eps, w_bias, vec, st)
+              : embed_stream_typed<__nv_bfloat16>(ip, table, h, nw, x, n, dim, vocab, scale, eps, w_bias, vec, st);
+}
+
+extern "C" int mx_polynorm(const void* z, const void* coef, void* out, int n, int dim, float eps, int fp32, void* stream) {
+  if (n <= 0 || dim <= 0) return 0;
+  const size_t ab = fp32 ? 16 : 8;
+  const bool vec = dim % 4 == 0 && aligned_to(z, ab) && aligned_to(out, ab);
+  auto st = static_cast<cudaStream_t>(stream);
+  const float* cp = static_cast<const float*>(coef);
+  return fp32 ? polynorm_typed<float>(z, cp, out, n, dim, eps, vec, st)
+              : polynorm_typed<__nv_bfloat16>(z, cp, out, n, dim, eps, vec, st);
+}
+
+extern "C" int mx_qk_norm_append(void* qkv, long long ld, const void* slots, void* k_pool, void* v_pool, const void* qw,
+                                 const void* kw, int n, int Hq, int Hkv, int Dk, int Dv, int block_size, float eps,
+                                 int fp32, void* stream) {
+  if (n <= 0) return 0;
+  if (Hq <= 0 || Hkv <= 0 || Dk <= 0 || Dv <= 0 || block_size <= 0) return -1;
+  const size_t ab = fp32 ? 16 : 8;
+  const bool vec = Dk % 4 == 0 && Dv % 4 == 0 && ld % 4 == 0 && aligned_to(qkv, ab) && aligned_to(k_pool, ab) &&
+                   aligned_to(v_pool, ab) && aligned_to(qw, 16) && aligned_to(kw, 16);
+  auto st = static_cast<cudaStream_t>(stream);
+  const int* sp = static_cast<const int*>(slots);
+  const float *q = static_cast<const float*>(qw), *k = static_cast<const float*>(kw);
+  return fp32 ? qk_norm_append_typed<float>(qkv, ld, sp, k_pool, v_pool, q, k, n, Hq, Hkv, Dk, Dv, block_size, eps, vec, st)
+              : qk_norm_append_typed<__nv_bfloat16>(qkv, ld, sp, k_pool, v_pool, q, k, n, Hq, Hkv, Dk, Dv, block_size, eps, vec, st);
+}

@@ -103,6 +103,7 @@ class EngineConfig:
     window_release: bool = True          # sliding-window layers get their own block pool and give back
     #                                      the blocks that fell out of the window (RotatingKVCache role)
     status_check_interval: int = 64      # steps between reads of the device status word (0 = never)
+    state_slots: int = 0                 # recurrent-state slots (0 = 2 * max_batch)
 
 
 class Engine:
@@ -117,8 +118,11 @@ class Engine:
         self.recurrent = bool(getattr(model, "recurrent", False))
         if self.recurrent:
             # per-sequence recurrent state lives in the model, not in the block pool: a cached prefix has
-            # no state to resume from, and the state slot indices change from step to step
-            e.prefix_cache = e.cuda_graphs = e.lookahead = False
+            # no state to resume from. Executors whose decode kernels read the slot indices from a device
+            # buffer (and skip padding rows) replay CUDA graphs; for the others the indices are baked in
+            e.prefix_cache = False
+            if not getattr(model, "state_slots_on_device", False):
+                e.cuda_graphs = e.lookahead = False
         self.pipeline = getattr(model, "ctx", None) is not None
         # token-sharded expert parallelism (parallel/dp_ep.py): ticks are taken in lockstep with the
         # other ranks; the lookahead pipeline (two forwards in flight) does not fit that
@@ -139,7 +143,7 @@ class Engine:
         if e.num_blocks <= 0:
             e.num_blocks = self._auto_num_blocks(tp, nl)
         # fp32 models (CPU oracles) keep fp32 keys / values; everything else stores bf16 (or 8-bit)
-        wdt = getattr(getattr(model.w, "final_norm", None), "dtype", torch.bfloat16)
+        wdt = getattr(model, "dtype", None) or getattr(getattr(model.w, "final_norm", None), "dtype", torch.bfloat16)
         kv_dtype = torch.float32 if wdt == torch.float32 else torch.bfloat16
         # Sliding-window layers (gpt-oss alternates 128-token windows with full layers, Mistral / Gemma
         # have them too) never attend beyond their window: they get a pool of their own whose blocks
@@ -262,7 +266,7 @@ class Engine:
         if self.is_cuda:
             free, total = torch.cuda.mem_get_info(self.device)
             budget = free - (1.0 - e.gpu_memory_utilization) * total - (6 << 30)
-            n = int(max(budget, 1 << 30) // per_block)
+            n = int(max(budget, 1 << 30) // max(per_block, 1))
         else:
             n = 2048
         need = (e.max_model_len // e.block_size + 2) * e.max_batch * 2
@@ -302,10 +306,14 @@ class Engine:
         self.h_cu, self.d_cu = host(S + 1, torch.int32), dev(S + 1, torch.int32)
         self.h_rows, self.d_rows = host(B * 9 + S, torch.int64), dev(B * 9 + S, torch.int64)
         self.h_out, self.d_out = host(B + S, torch.int32), dev(B + S, torch.int32)
+        # state slots of the decode rows, for executors that read them on the device
+        self.state_on_device = bool(getattr(self.model, "state_slots_on_device", False))
+        self.h_state, self.d_state = host(B, torch.int32), dev(B, torch.int32)
         # second staging set + token read-back buffers for the lookahead pipeline
         self.la_host = [dict(pos=host(B, torch.int32), slots=host(B, torch.int32), lens=host(B, torch.int32),
                              tables=host((B, MB), torch.int32), out=host(B, torch.int32),
-                             slots_w=host(B, torch.int32), tables_w=host((B, MB), torch.int32)) for _ in range(2)]
+                             slots_w=host(B, torch.int32), tables_w=host((B, MB), torch.int32),
+                             state=host(B, torch.int32)) for _ in range(2)]
         self._inflight = None
         self._la_parity = 0
         self.np_dec_tables = self.h_dec_tables.numpy()
@@ -597,6 +605,11 @@ class Engine:
         if nd:
             self.d_dec_tables[:nd].copy_(self.h_dec_tables[:nd], non_blocking=nb)
             self.d_dec_lens[:nd].copy_(self.h_dec_lens[:nd], non_blocking=nb)
+            if self.state_on_device:
+                for i, s in enumerate(decode):
+                    self.h_state[i] = self.model.state_slot(s.seq_id)
+                self.d_state[:nd].copy_(self.h_state[:nd], non_blocking=nb)
+                self.stats["h2d_bytes"] += 4 * nd
         if sp:
             self.d_pf_tables[:sp].copy_(self.h_pf_tables[:sp], non_blocking=nb)
             self.d_pf_lens[:sp].copy_(self.h_pf_lens[:sp], non_blocking=nb)
@@ -631,6 +644,8 @@ class Engine:
             b.positions3 = torch.from_numpy(pos3[:, :t].copy()).to(self.device)
         b.seq_ids = [s.seq_id for s in decode] + [p[0].seq_id for p in pieces]
         b.pf_starts = [p[1] for p in pieces]
+        if self.state_on_device and nd and not pieces:
+            b.state_slots = self.d_state[:nd]
         return b, R
 
     def _media_embeds(self, b: StepBatch, nd: int, pieces) -> torch.Tensor:
@@ -670,8 +685,8 @@ class Engine:
         bp = min(bp, e.max_batch) if e.max_batch >= nd else nd
         if bp < nd:
             return None
-        splits = ops.decode_splits(bp, self.model.Hkv, max(max_len, 1))
-        key = (bp, splits)
+        split_key = getattr(self.model, "decode_split_key", None)
+        key = (bp, split_key(bp, max(max_len, 1)) if split_key else ops.decode_splits(bp, self.model.Hkv, max(max_len, 1)))
         # padding rows: no KV append, zero context
         if bp > nd:
             self.d_tokens[nd:bp].zero_()
@@ -682,6 +697,8 @@ class Engine:
             if self.bm_win is not None:
                 self.d_slots_w[nd:bp].fill_(-1)
                 self.d_dec_tables_w[nd:bp].zero_()
+            if self.state_on_device:
+                self.d_state[nd:bp].fill_(-1)
         ent = self._graphs.get(key)
         if ent is None:
             b = StepBatch(token_ids=self.d_tokens[:bp], positions=self.d_pos[:bp],
@@ -690,6 +707,12 @@ class Engine:
                           dec_max_len=max_len, logits_rows=None,
                           slot_mapping_win=self.d_slots_w[:bp] if self.bm_win is not None else None,
                           dec_block_tables_win=self.d_dec_tables_w[:bp] if self.bm_win is not None else None)
+            live_state = None
+            if self.state_on_device:
+                # the warm-up below runs for real: it must not advance any sequence's state
+                b.state_slots = self.d_state[:bp]
+                live_state = b.state_slots.clone()
+                b.state_slots.fill_(-1)
             fwd = lambda: self.model.forward(b, self.kv_layers)  # noqa: E731
             # warm-up outside capture (sets function attributes, fills descriptor caches). With
             # token-sharded experts this pass is this rank's alone, so it runs "dry": no exchange
@@ -707,6 +730,8 @@ class Engine:
                     if a2a is not None:
                         a2a.dry = False
             torch.cuda.current_stream().wait_stream(s)
+            if live_state is not None:
+                b.state_slots.copy_(live_state)
             from ..ops import _lib
             n0 = _lib.launches()
             g = torch.cuda.CUDAGraph()
@@ -778,6 +803,11 @@ class Engine:
             if self.bm_win is not None:
                 self.bm_win.fill_slots(s.seq_id, L - 1, 1, hb["slots_w"].numpy(), i)
             max_len = max(max_len, L)
+            if self.state_on_device:
+                hb["state"][i] = self.model.state_slot(s.seq_id)
+        if self.state_on_device:
+            self.d_state[:nd].copy_(hb["state"][:nd], non_blocking=True)
+            self.stats["h2d_bytes"] += 4 * nd
         self.bm.fill_tables([s.seq_id for s in seqs], hb["tables"].numpy())
         if self.bm_win is not None:
             self.bm_win.fill_tables([s.seq_id for s in seqs], hb["tables_w"].numpy())
@@ -890,6 +920,102 @@ class Engine:
             return ended + self._run_scheduled(decode, pieces)
         return self._run_scheduled(decode, pieces)
 
+    def _forward_batch(self, b: StepBatch, decode, pieces) -> torch.Tensor | None:
+        """The step's forward pass: logits of the batch's rows (decode rows first). Pure decode batches replay
+        a CUDA graph where graphs are on."""
+        nd = len(decode)
+        # a decode graph holds the expert kernels chosen for decode-sized groups; in a tick in which
+        # another data-parallel rank prefills, this rank's experts get that rank's rows too
+        if not pieces and nd and not (self.dp_lockstep and getattr(self.model.comm, "heavy", False)):
+            gl = self._decode_graph(nd, b.dec_max_len)
+            if gl is not None:
+                self.stats["decode_steps"] += 1
+                return gl[:nd]
+        if self.drafter is not None and getattr(self.drafter, "needs_hidden", False):
+            if self.pipeline:
+                # the residual stream exists on the last stage only, and so does the drafter
+                h = self.model.pipeline_hidden(b, self.kv_layers)
+                logits = self.model.logits(h, b.logits_rows) if h is not None else None
+            else:
+                h = self.model.forward_hidden(b, self.kv_layers)
+                logits = self.model.logits(h, b.logits_rows)
+            if h is not None:
+                self.drafter.on_forward(self, decode, pieces, h)
+            return logits
+        return self.model.forward(b, self.kv_layers)
+
+    # ------------------------------------------------------------------ replay of given tokens
+    # Teacher-forced steps: the caller brings every token, nothing is sampled. Batches are built, run and
+    # accounted for by the same code as scheduled steps (block manager, state slots, decode graphs).
+    def open_sequence(self) -> int:
+        """A sequence that :meth:`feed` extends; holds nothing until its first tokens."""
+        sid = self._next_id
+        self._next_id += 1
+        self.seqs[sid] = Sequence(sid, [], SamplingParams(), arrival=time.perf_counter())
+        self._kv_create(sid)
+        return sid
+
+    def close_sequence(self, seq_id: int) -> None:
+        """Gives the sequence's cache blocks and state slot back."""
+        self._kv_free(seq_id)
+        if self.recurrent:
+            self.model.release_seq(seq_id)
+        del self.seqs[seq_id]
+
+    @torch.inference_mode()
+    def feed(self, entries: list[tuple[int, list[int], list[int]]]) -> torch.Tensor | None:
+        """One forward pass over the next tokens of several open sequences. ``entries``: (sequence id, tokens,
+        places among these tokens whose logits are wanted). Single tokens behind a sequence's first portion
+        run as decode rows, everything else as prompt portions, all in one batch. Returns the logits in the
+        order of the entries and places, or None when none are wanted."""
+        e = self.ecfg
+        if self._inflight is not None or self.pipeline or self.dp_lockstep:
+            raise RuntimeError("feed() runs between scheduled steps of a single executor")
+        if sum(len(t) for _, t, _ in entries) > e.max_num_batched_tokens:
+            raise ValueError("more tokens than one step takes (max_num_batched_tokens)")
+        if len({sid for sid, _, _ in entries}) != len(entries) or any(not t for _, t, _ in entries):
+            raise ValueError("one non-empty entry per sequence and step")
+        decode, pieces = [], []
+        for sid, toks, _ in entries:
+            s = self.seqs[sid]
+            if s.total_len + len(toks) > e.max_model_len:
+                raise ValueError(f"sequence {sid} exceeds max_model_len {e.max_model_len}")
+            if not self._kv_reserve(sid, s.total_len + len(toks)):
+                raise RuntimeError("the KV pool cannot hold these tokens")
+            start = s.total_len
+            s.prompt.extend(int(t) for t in toks)
+            if start > 0 and len(toks) == 1:
+                decode.append(s)
+            else:
+                pieces.append((s, start, len(toks)))
+        if len(decode) > e.max_batch or len(pieces) > e.max_prefill_seqs:
+            raise ValueError("more sequences than one step takes (max_batch, max_prefill_seqs)")
+        self._check_device_status()
+        b, _ = self._build_batch(decode, pieces)
+        first, row = {}, 0
+        for s, n in [(s, 1) for s in decode] + [(p[0], p[2]) for p in pieces]:
+            first[s.seq_id] = row
+            row += n
+        rows = [first[sid] + w for sid, _, want in entries for w in want]
+        idx = torch.tensor(rows, dtype=torch.int64).to(self.device)
+        logits = None
+        if pieces:
+            b.logits_rows, b.logits_rows_host = idx, rows
+            if rows:
+                logits = self._forward_batch(b, decode, pieces)
+            else:
+                self.model.forward_hidden(b, self.kv_layers)
+        else:
+            logits = self._forward_batch(b, decode, pieces)
+            logits = logits.index_select(0, idx) if rows else None
+        for sid, _, _ in entries:
+            self.seqs[sid].num_computed = self.seqs[sid].total_len
+        self._release_window([self.seqs[sid] for sid, _, _ in entries])
+        self.stats["steps"] += 1
+        self.stats["decode_tokens"] += len(decode)
+        self.stats["prefill_tokens"] += sum(p[2] for p in pieces)
+        return logits
+
     def _run_scheduled(self, decode, pieces) -> list[Sequence]:
         if not decode and not pieces:
             return []
@@ -903,31 +1029,11 @@ class Engine:
         t_step = time.perf_counter()
         b, R = self._build_batch(decode, pieces)
         nd = len(decode)
-        logits = None
         timing = self._step_timing
         if timing:
             ev0, ev1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
             ev0.record()
-        # a decode graph holds the expert kernels chosen for decode-sized groups; in a tick in which
-        # another data-parallel rank prefills, this rank's experts get that rank's rows too
-        if not pieces and nd and not (self.dp_lockstep and getattr(self.model.comm, "heavy", False)):
-            gl = self._decode_graph(nd, b.dec_max_len)
-            if gl is not None:
-                logits = gl[:nd]
-                self.stats["decode_steps"] += 1
-        if logits is None:
-            if self.drafter is not None and getattr(self.drafter, "needs_hidden", False):
-                if self.pipeline:
-                    # the residual stream exists on the last stage only, and so does the drafter
-                    h = self.model.pipeline_hidden(b, self.kv_layers)
-                    logits = self.model.logits(h, b.logits_rows) if h is not None else None
-                else:
-                    h = self.model.forward_hidden(b, self.kv_layers)
-                    logits = self.model.logits(h, b.logits_rows)
-                if h is not None:
-                    self.drafter.on_forward(self, decode, pieces, h)
-            else:
-                logits = self.model.forward(b, self.kv_layers)
+        logits = self._forward_batch(b, decode, pieces)
         # rows: decode rows first, then prefill rows that completed their prompt
         sample_seqs = list(decode) + [s for (s, start, cnt) in pieces if start + cnt >= s.total_len]
         if self.pipeline:

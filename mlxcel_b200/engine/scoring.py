@@ -29,7 +29,7 @@ def prefill_hidden(model, cfg, ids: list[int], block_size: int = 16) -> torch.Te
     if layers is None:
         layers = len(model.w.layers)
     pool = KVPool(cfg, max(nb, 1), block_size, device=dev, tp_size=comm.tp_size if comm is not None else 1,
-                  num_layers=max(layers, 1), dtype=model.w.final_norm.dtype)
+                  num_layers=max(layers, 1), dtype=getattr(model, "dtype", None) or model.w.final_norm.dtype)
     i32 = dict(dtype=torch.int32, device=dev)
     b = StepBatch(token_ids=torch.tensor(ids, **i32), positions=torch.arange(T, **i32), slot_mapping=torch.arange(T, **i32),
                   num_prefill_seqs=1, pf_block_tables=torch.arange(nb, **i32)[None], pf_cu_q=torch.tensor([0, T], **i32),

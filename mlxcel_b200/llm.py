@@ -28,13 +28,14 @@ class LLM:
         if model is not None:
             self.model = model
         elif cfg.model_type in ("mamba", "mamba2", "nemotron_h", "granitemoehybrid", "jamba", "qwen3_next", "qwen3_5", "qwen3_5_text",
-                                "qwen3_5_moe", "qwen3_5_moe_text", "falcon_h1", "lfm2", "lfm2_moe", "recurrent_gemma"):
+                                "qwen3_5_moe", "qwen3_5_moe_text", "falcon_h1", "lfm2", "lfm2_moe", "recurrent_gemma", "pamasun"):
             from .models.hybrid import HybridModel
             from .models.mamba1 import Mamba1Model
             from .models.mamba2 import Mamba2Model
             cls = {"mamba": Mamba1Model, "mamba2": Mamba2Model}.get(cfg.model_type, HybridModel)
-            self.model = cls(cfg, weights, comm=comm,
-                             max_seqs=2 * (engine_config.max_batch if engine_config else EngineConfig().max_batch))
+            ec = engine_config or EngineConfig()
+            kw = dict(kv_bits=ec.kv_bits) if cfg.model_type == "pamasun" else {}
+            self.model = cls(cfg, weights, comm=comm, max_seqs=ec.state_slots or 2 * ec.max_batch, **kw)
         else:
             self.model = DecoderModel(cfg, weights, comm=comm,
                                       kv_bits=(engine_config.kv_bits if engine_config else 16),
@@ -58,6 +59,9 @@ class LLM:
         if cfg.model_type == "nemotron_h":
             from .models.hybrid import random_hybrid_weights
             return LLM(cfg, random_hybrid_weights(cfg, seed=seed, dtype=dtype, device=device), engine_config, comm=comm)
+        if cfg.model_type == "pamasun":
+            from .models.pamasun import random_pamasun_weights
+            return LLM(cfg, random_pamasun_weights(cfg, seed=seed, dtype=dtype, device=device), engine_config, comm=comm)
         tp = comm.tp_size if comm is not None else 1
         rank = comm.tp_rank if comm is not None else 0
         hook = None
@@ -80,11 +84,19 @@ class LLM:
     @staticmethod
     def from_pretrained(path: str | Path, *, device="cuda", engine_config: EngineConfig | None = None,
                         comm=None, dequantize: bool = False, surgery: str | None = None,
-                        config_overrides: dict | None = None) -> "LLM":
+                        config_overrides: dict | None = None, dtype: torch.dtype | None = None) -> "LLM":
+        """``dtype``: precision of weights, activations and cache (default bf16). fp32 is for the designs whose
+        kernels exist in both precisions."""
         from .loading.checkpoint import load_model_weights
         from .tokenizer import load_tokenizer
 
         cfg = ModelConfig.from_path(path, config_overrides)
+        if cfg.model_type == "pamasun":
+            from .models.pamasun import load_pamasun_weights
+            return LLM(cfg, load_pamasun_weights(path, cfg, dtype=dtype or torch.bfloat16, device=device), engine_config,
+                       comm=comm, tokenizer=load_tokenizer(path))
+        if dtype not in (None, torch.bfloat16):
+            raise ValueError(f"{cfg.model_type} models are served in bf16")
         if cfg.model_type == "mamba2":
             from .models.mamba2 import load_mamba2_weights
             return LLM(cfg, load_mamba2_weights(path, cfg, device=device), engine_config, comm=comm,

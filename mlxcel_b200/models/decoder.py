@@ -59,6 +59,8 @@ class StepBatch:
     # Multimodal rotary positions [3, T] (temporal, height, width) when a row's three components
     # differ (image tokens of the Qwen2-VL family); ``positions`` then holds the temporal one.
     positions3: torch.Tensor | None = None
+    # Recurrent executors that read slot indices on the device: [num_decode] int32 (-1 = padding row)
+    state_slots: torch.Tensor | None = None
 
     @property
     def num_tokens(self) -> int:

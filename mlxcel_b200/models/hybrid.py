@@ -14,6 +14,12 @@ A model is a flat list of pre-norm residual blocks; the family decides the list 
 ``E``  mixture of experts (``models/moe.py``)                    Jamba, Qwen3-Next
 =====  ===============================================================================================
 
+A second layout ("stream") serves designs that keep the residual in fp32 and normalise every sub-layer on
+both sides: ``h <- h + layer_scale * norm(branch(norm(h)))``. Its blocks carry ``post_norm`` / ``layer_scale``, its
+mixers are ``attention_mixer`` (``models/attention_mixer.py``) and ``general_delta`` (``models/general_delta.py``),
+and ``HybridWeights.runs`` lists the layers in execution order: a layer may run several times with the same
+weights, each run with a KV-pool layer or state slab of its own (Pamasun).
+
 Nemotron-H gives one block per layer through ``hybrid_override_pattern`` (``"M-M-M*-..."``); the other
 families have a mixer block and an MLP / MoE block per layer. Reference: src/models/nemotron_h.rs,
 granitemoehybrid.rs, jamba.rs, falcon_h1.rs, qwen3_next.rs.
@@ -52,6 +58,10 @@ class HybridBlock:
     out_gate: torch.Tensor | None = None        # gated attention (Qwen3-Next): [Hq * D, H] sigmoid gate projection
     latent_in: torch.Tensor | None = None       # Nemotron-H MoE: optional projections around the routed experts
     latent_out: torch.Tensor | None = None      #   ([latent, H] and [H, latent]); up / down hold the shared expert
+    # stream layout: fp32 vectors (norm weights are offsets from ``cfg.norm_weight_bias``)
+    post_norm: torch.Tensor | None = None       # norm of the branch's result
+    layer_scale: torch.Tensor | None = None     # element-wise factor behind it
+    act_coef: torch.Tensor | None = None        # polynomial-norm activation (a, b, c, e)
 
 
 @dataclass
@@ -61,6 +71,7 @@ class HybridWeights:
     final_norm: torch.Tensor
     lm_head: torch.Tensor
     layers: list = field(default_factory=list)  # the attention blocks' LayerWeights (= KV-pool layers)
+    runs: list | None = None                    # stream layout: the layers (lists of blocks) in execution order
 
 
 _KINDS = {"M": "mamba2", "m": "mamba1", "L": "gdn", "C": "shortconv", "R": "rglru", "P": "parallel", "*": "attention", "A": "attention", "-": "mlp", "G": "mlp",
@@ -631,6 +642,12 @@ class HybridModel:
         self.comm = comm or LocalComm()
         assert self.comm.tp_size == 1, "the hybrid executor is single-GPU"
         self.device = weights.final_norm.device
+        self.layer_range = range(cfg.num_hidden_layers)
+        self.I = cfg.intermediate_size
+        self.capture_layers: tuple = ()         # layer runs whose output stream a forward keeps in ``captured``
+        self.captured: list = []
+        if weights.runs is not None:
+            return self._init_stream(max_seqs, kv_bits)
         mamba_layers = [b.mamba for b in weights.blocks if b.kind in ("mamba2", "parallel")]
         mamba1_layers = [b.mamba for b in weights.blocks if b.kind == "mamba1"]
         gdn_layers = [b.mamba for b in weights.blocks if b.kind == "gdn"]
@@ -659,16 +676,75 @@ class HybridModel:
                                  comm=self.comm, kv_bits=kv_bits)
         self.Hq, self.Hkv, self.D = self.attn.Hq, self.attn.Hkv, self.attn.D
         self.num_kv_layers = len(weights.layers)
-        self.layer_range = range(cfg.num_hidden_layers)
-        self.I = cfg.intermediate_size
+
+    def _init_stream(self, max_seqs: int, kv_bits: int) -> None:
+        from .general_delta import GeneralDeltaModel
+        cfg, w = self.cfg, self.w
+        if kv_bits != 16:
+            raise ValueError("this model keeps its KV unquantized (kv_bits must be 16)")
+        self.dtype = w.embed.dtype
+        # (block, index of its KV layer or state slab, run index behind its last block or -1)
+        self.order: list = []
+        delta, n_kv, self._kv_heads = [], 0, set()
+        for r, blocks in enumerate(w.runs):
+            for blk in blocks:
+                idx = -1
+                if blk.kind == "attention_mixer":
+                    idx, n_kv = n_kv, n_kv + 1
+                    self._kv_heads.add(blk.attn.kv_heads)
+                elif blk.kind == "general_delta":
+                    idx = len(delta)
+                    delta.append(blk.mamba)
+                self.order.append((blk, idx, r if blk is blocks[-1] else -1))
+        self.num_kv_layers = n_kv
+        self.Hq, self.Hkv, self.D = cfg.num_attention_heads, cfg.num_key_value_heads, cfg.head_dim
+        # only the delta mixers carry state: a stack without them is served like any attention model
+        self.ssm = GeneralDeltaModel(delta, cfg.rms_norm_eps, self.device, max_seqs, self.comm) if delta else None
+        self.recurrent = self.ssm is not None
+        self.state_slots_on_device = self.recurrent
+
+    def decode_split_key(self, rows: int, max_len: int) -> tuple:
+        """What a captured decode graph depends on besides its rows: the KV splits of every geometry."""
+        heads = self._kv_heads if self.w.runs is not None else {self.Hkv}
+        return tuple(ops.decode_splits(rows, h, max_len) for h in sorted(heads))
+
+    def state_slot(self, seq_id: int) -> int:
+        return self.ssm.slot(seq_id)
 
     def release_seq(self, seq_id: int) -> None:
-        self.ssm.release_seq(seq_id)
+        if self.ssm is not None:
+            self.ssm.release_seq(seq_id)
+
+    def _forward_stream(self, b: StepBatch, kv_layers) -> torch.Tensor:
+        """Layer runs of the stream layout. Returns the fp32 residual stream [T, H] (before the final norm)."""
+        from ..ops import stream
+        from .attention_mixer import attention_mixer
+        cfg, eps, wb = self.cfg, self.cfg.rms_norm_eps, self.cfg.norm_weight_bias
+        if b.embeds is not None:
+            raise NotImplementedError("media embeddings with an fp32 residual stream")
+        pieces = self.ssm.pieces(b) if self.ssm is not None else None
+        self.captured = []
+        h, x = stream.embed_stream(b.token_ids, self.w.embed, cfg.embed_scale,
+                                   self.order[0][0].norm if self.order else self.w.final_norm, eps, wb)
+        for n, (blk, idx, run) in enumerate(self.order):
+            if blk.kind == "attention_mixer":
+                y = ops.linear(attention_mixer(blk.attn, x, b, kv_layers[idx], eps), blk.attn.out_proj)
+            elif blk.kind == "general_delta":
+                y = ops.linear(self.ssm.mixer(idx, blk.mamba, x, pieces), blk.mamba.out_proj)
+            else:
+                y = ops.linear(stream.polynorm(ops.linear(x, blk.up), blk.act_coef, eps), blk.down)
+            nxt = self.order[n + 1][0].norm if n + 1 < len(self.order) else None
+            x = stream.stream_norm(h, y, blk.post_norm, blk.layer_scale, nxt, eps, wb)
+            if run in self.capture_layers:
+                self.captured.append(h.clone())
+        return h
 
     @torch.inference_mode()
     def forward_hidden(self, b: StepBatch, kv_layers=None, hidden_in: torch.Tensor | None = None) -> torch.Tensor:
         cfg = self.cfg
         eps = cfg.rms_norm_eps
+        if self.w.runs is not None:
+            return self._forward_stream(b, kv_layers)
         pieces = self.ssm.pieces(b)
         h = hidden_in if hidden_in is not None else ops.embedding(b.token_ids, self.w.embed, cfg.embed_scale)
         mi = ai = 0
@@ -724,6 +800,11 @@ class HybridModel:
         return h
 
     def logits(self, h: torch.Tensor, rows: torch.Tensor | None) -> torch.Tensor:
+        if self.w.runs is not None:
+            from ..ops import stream
+            x = stream.stream_norm(h, None, None, None, self.w.final_norm, self.cfg.rms_norm_eps, self.cfg.norm_weight_bias,
+                                   dtype=self.dtype, rows=None if rows is None else rows.to(torch.int32))
+            return ops.linear(x, self.w.lm_head, out_fp32=True)
         lg = self.ssm.logits(h, rows)
         ls = self.cfg.extra.get("logits_scaling", 1.0)
         lg = lg if ls == 1.0 else (lg.float() / ls).to(lg.dtype)

@@ -80,10 +80,13 @@ def linear(x: torch.Tensor, w: torch.Tensor, bias: torch.Tensor | None = None,
     if not x.is_cuda:
         assert row_norm is None and ssq_out is None, "deferred RMSNorm is a CUDA-only path"
         return ref.linear(x, w, bias, residual, torch.float32 if out_fp32 else None)
-    assert x.dtype == torch.bfloat16 and w.dtype == torch.bfloat16
     M, K = x.shape
     N = w.shape[0]
     assert x.stride(1) == 1 and w.stride(1) == 1 and w.shape[1] == K
+    if x.dtype == torch.float32 or K % 8 or x.stride(0) % 8 or w.stride(0) % 8 or (x.data_ptr() | w.data_ptr()) % 16:
+        assert row_norm is None and ssq_out is None, "deferred RMSNorm needs the tensor-core GEMM"
+        return _linear_any(x, w, bias, residual, out, out_fp32)
+    assert x.dtype == torch.bfloat16 and w.dtype == torch.bfloat16
     if out is None:
         out = torch.empty(M, N, dtype=torch.float32 if out_fp32 else torch.bfloat16, device=x.device)
     if M == 0:
@@ -96,6 +99,21 @@ def linear(x: torch.Tensor, w: torch.Tensor, bias: torch.Tensor | None = None,
               residual.stride(0) if residual is not None else 0, epi, 1 if out_fp32 else 0, 0,
               0.0, 0.0, ws.data_ptr(), ws.numel(), force_mode, force_splits, _lib.stream(),
               _lib.ref_or_null(ex))
+    return out
+
+
+def _linear_any(x, w, bias, residual, out, out_fp32: bool) -> torch.Tensor:
+    """:func:`linear` on the SIMT kernel: fp32 operands, or bf16 rows TMA cannot address (K or a row stride that
+    is not a multiple of 8)."""
+    M, K = x.shape
+    N = w.shape[0]
+    assert w.dtype == x.dtype and x.dtype in (torch.float32, torch.bfloat16)
+    if out is None:
+        out = torch.empty(M, N, dtype=torch.float32 if out_fp32 else x.dtype, device=x.device)
+    if M:
+        _lib_call("mx_gemm_any", x.data_ptr(), w.data_ptr(), out.data_ptr(), _lib.ptr(bias), _lib.ptr(residual), M, N, K,
+                  x.stride(0), w.stride(0), out.stride(0), residual.stride(0) if residual is not None else 0,
+                  1 if x.dtype == torch.float32 else 0, 1 if out.dtype == torch.float32 else 0, _lib.stream())
     return out
 
 

@@ -21,6 +21,15 @@ def lib_path() -> Path:
     return _PKG / "lib" / "libmlxcel_b200.so"
 
 
+_UNITS: tuple | None = None
+
+
+def prefer_units(units) -> None:
+    """Restricts a build that :func:`load` has to do (no built library in the tree) to these sources."""
+    global _UNITS
+    _UNITS = tuple(units) if units else None
+
+
 def load(required: bool = True):
     """Return the loaded kernel library (building it when sources are newer and nvcc exists)."""
     global _LIB, _LIB_ERR
@@ -31,7 +40,7 @@ def load(required: bool = True):
         try:
             from .. import _build
 
-            _build.build_cuda()
+            path = _build.build_cuda(units=_UNITS)
         except Exception as e:  # pragma: no cover - build environment specific
             _LIB_ERR = f"build failed: {e}"
     if path.exists():
@@ -66,6 +75,7 @@ def _declare(lib) -> None:
     sig = {
         "mx_gemm_bf16": [_vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _i, _i, _i, _f, _f,
                          _vp, _ll, _i, _i, _vp, _vp],
+        "mx_gemm_any": [_vp, _vp, _vp, _vp, _vp, _i, _i, _i, _ll, _ll, _ll, _ll, _i, _i, _vp],
         "mx_gemm_comm": [_vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _i, _i, _i, _vp, _vp,
                          _vp, _vp, _vp, _ll, _ll, _vp, _ll, _vp, _vp],
         "mx_allreduce_comm": [_vp, _vp, _vp, _ll, _i, _i, _i, _vp, _vp, _vp, _vp, _vp, _ll, _ll, _vp, _vp,

@@ -1,0 +1,261 @@
+"""Operators of layers with an fp32 residual stream and of attention heads without rotation: sub-layer
+norms on both sides, polynomial-norm activation, q/k norm + KV append, paged attention with a logarithmic
+distance bias / sink / output gate and separate key and value widths, the generalized delta rule.
+
+Every operator exists for bf16 and fp32 activations on CUDA (``csrc/stream_norm.cu``, ``csrc/simt.cu``,
+``csrc/attention*.cu``, ``csrc/delta_rule.cu``); CPU tensors take the PyTorch statements below. Norm weights,
+layer scales and per-head constants are fp32 vectors."""
+from __future__ import annotations
+
+import ctypes
+import math
+
+import torch
+
+from . import _lib
+from .reference import _gather_kv
+
+_vp, _i, _f, _ll = ctypes.c_void_p, ctypes.c_int, ctypes.c_float, ctypes.c_longlong
+_SIG = {
+    "mx_stream_norm": [_vp] * 7 + [_i, _i, _f, _f, _i, _vp],
+    "mx_embed_stream": [_vp] * 5 + [_i, _i, _i, _f, _f, _f, _i, _vp],
+    "mx_polynorm": [_vp, _vp, _vp, _i, _i, _f, _i, _vp],
+    "mx_qk_norm_append": [_vp, _ll, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _f, _i, _vp],
+    "mx_paged_attention_any": [_vp, _ll] + [_vp] * 9 + [_ll, _vp] + [_i] * 9 + [_f, _i, _vp],
+    "mx_paged_decode_ext": [_vp, _ll] + [_vp] * 8 + [_ll, _vp, _vp] + [_i] * 8 + [_f, _i, _vp],
+    "mx_paged_prefill_ext": [_vp, _ll, _vp, _vp, _ll] + [_vp] * 7 + [_ll, _vp] + [_i] * 10 + [_f, _vp, _vp],
+    "mx_delta_rule": [_vp, _ll] + [_vp] * 11 + [_i] * 6 + [_f, _f, _f, _i, _i, _vp],
+}
+NOT_COVERED = -10        # a tensor-core kernel refuses the geometry: the shape-agnostic one takes it
+
+
+def _fn(name):
+    fn = getattr(_lib.load(), name)
+    if not fn.argtypes:
+        fn.argtypes, fn.restype = _SIG[name], _i
+    return fn
+
+
+def _call(name, *args) -> None:
+    rc = _fn(name)(*args)
+    _lib.count_launch()
+    _lib.check(rc, name)
+
+
+def _fp32(t: torch.Tensor) -> int:
+    if t.dtype not in (torch.float32, torch.bfloat16):
+        raise TypeError(f"activations must be fp32 or bf16, not {t.dtype}")
+    return 1 if t.dtype == torch.float32 else 0
+
+
+def _rms(x: torch.Tensor, eps: float) -> torch.Tensor:
+    return x * torch.rsqrt(x.pow(2).mean(-1, keepdim=True) + eps)
+
+
+# ----------------------------------------------------------------------------- residual stream
+def embed_stream(ids, table, scale: float, pre_w, eps: float, w_bias: float):
+    """``h = scale * table[ids]`` (fp32 stream) and ``x = rmsnorm(h) * (w_bias + pre_w)`` in the table's type."""
+    n, dim = ids.shape[0], table.shape[1]
+    if not table.is_cuda:
+        ok = (ids >= 0) & (ids < table.shape[0])
+        h = table[ids.clamp(0, table.shape[0] - 1).long()].float() * scale * ok[:, None]
+        return h, (_rms(h, eps) * (w_bias + pre_w)).to(table.dtype)
+    h = torch.empty(n, dim, dtype=torch.float32, device=table.device)
+    x = torch.empty(n, dim, dtype=table.dtype, device=table.device)
+    if n:
+        _call("mx_embed_stream", ids.data_ptr(), table.data_ptr(), h.data_ptr(), pre_w.data_ptr(), x.data_ptr(), n, dim,
+              table.shape[0], float(scale), float(eps), float(w_bias), _fp32(table), _lib.stream())
+    return h, x
+
+
+def stream_norm(h, y, post_w, layer_scale, pre_w, eps: float, w_bias: float, dtype=None, rows=None):
+    """One step of the stream between two sub-layers, in place on ``h`` (fp32): with a branch ``y``,
+    ``h += rmsnorm(y) * (w_bias + post_w) * layer_scale`` (layer_scale optional); with ``pre_w``, returns
+    ``rmsnorm(h) * (w_bias + pre_w)`` as ``dtype`` (default: y's type). ``rows`` (int32, no branch) selects
+    the rows of h to normalise."""
+    dtype = dtype or y.dtype
+    if not h.is_cuda:
+        if y is not None:
+            b = _rms(y.float(), eps) * (w_bias + post_w)
+            h += b if layer_scale is None else b * layer_scale
+        if pre_w is None:
+            return None
+        return (_rms(h if rows is None else h[rows.long()], eps) * (w_bias + pre_w)).to(dtype)
+    dim = h.shape[1]
+    n = h.shape[0] if rows is None else rows.shape[0]
+    x = torch.empty(n, dim, dtype=dtype, device=h.device) if pre_w is not None else None
+    assert h.is_contiguous() and (y is None or (y.is_contiguous() and y.dtype == dtype))
+    assert rows is None or rows.dtype == torch.int32
+    if n:
+        fp32 = 1 if dtype == torch.float32 else 0
+        _call("mx_stream_norm", _lib.ptr(y), h.data_ptr(), _lib.ptr(rows), _lib.ptr(post_w), _lib.ptr(layer_scale),
+              _lib.ptr(pre_w), _lib.ptr(x), n, dim, float(eps), float(w_bias), fp32, _lib.stream())
+    return x
+
+
+def polynorm(z, coef, eps: float):
+    """``a N(z) + b N(z^2) + c N(z^3) + e`` over the last dimension, N(x) = x / rms(x); coef = (a, b, c, e) fp32."""
+    if not z.is_cuda:
+        f = z.float()
+        return (coef[0] * _rms(f, eps) + coef[1] * _rms(f ** 2, eps) + coef[2] * _rms(f ** 3, eps) + coef[3]).to(z.dtype)
+    assert z.is_contiguous()
+    out = torch.empty_like(z)
+    if z.shape[0]:
+        _call("mx_polynorm", z.data_ptr(), coef.data_ptr(), out.data_ptr(), z.shape[0], z.shape[1], float(eps), _fp32(z),
+              _lib.stream())
+    return out
+
+
+# ----------------------------------------------------------------------------- attention
+def qk_norm_append(qkv, slots, kv, *, Hq: int, Hkv: int, Dk: int, Dv: int, q_norm, k_norm, eps: float) -> None:
+    """Rows ``q | k | v | ...``: per-head RMS norm of q (in place) and k, then k and v into the paged pool
+    (negative slots append nothing). No positional encoding."""
+    if not qkv.is_cuda:
+        T, nq, nk = qkv.shape[0], Hq * Dk, Hkv * Dk
+        q, k, v = qkv[:, :nq].float().view(T, Hq, Dk), qkv[:, nq:nq + nk].float().view(T, Hkv, Dk), \
+            qkv[:, nq + nk:nq + nk + Hkv * Dv].view(T, Hkv, Dv)
+        if q_norm is not None:
+            qkv[:, :nq] = (_rms(q, eps) * q_norm).reshape(T, nq).to(qkv.dtype)
+        k = _rms(k, eps) * k_norm if k_norm is not None else k
+        ok = slots >= 0
+        s = slots[ok].long()
+        blk, off = s // kv.block_size, s % kv.block_size
+        kv.k[blk, :, off] = k[ok].to(kv.k.dtype)
+        kv.v[blk, :, off] = v[ok].to(kv.v.dtype)
+        return
+    assert kv.k.dtype == qkv.dtype and qkv.stride(1) == 1 and slots.dtype == torch.int32
+    if qkv.shape[0]:
+        _call("mx_qk_norm_append", qkv.data_ptr(), qkv.stride(0), slots.data_ptr(), kv.k.data_ptr(), kv.v.data_ptr(),
+              _lib.ptr(q_norm), _lib.ptr(k_norm), qkv.shape[0], Hq, Hkv, Dk, Dv, kv.block_size, float(eps), _fp32(qkv),
+              _lib.stream())
+
+
+def paged_attention_ref(q, kv, tables, lens, cu, *, Hq, Hkv, Dk, Dv, scale, window=0, sinks=None, dist_bias=None, gate=None):
+    T, G = q.shape[0], Hq // Hkv
+    out = torch.zeros(T, Hq * Dv, dtype=q.dtype, device=q.device)
+    cu_l, lens_l = cu.tolist(), lens.tolist()
+    for s in range(len(lens_l)):
+        q0, q1, n = cu_l[s], cu_l[s + 1], lens_l[s]
+        ql = q1 - q0
+        if ql == 0 or n == 0:
+            continue
+        k, v = _gather_kv(kv, tables[s], n)
+        qs = q[q0:q1].float().reshape(ql, Hkv, G, Dk).permute(1, 2, 0, 3)
+        sc = torch.einsum("hgqd,hkd->hgqk", qs, k) * scale
+        d = torch.arange(n - ql, n, device=q.device)[:, None] - torch.arange(n, device=q.device)[None, :]
+        if dist_bias is not None:
+            r1, r2 = (t.float().reshape(Hkv, G, 1, 1) for t in dist_bias)
+            sc = sc - r1 * torch.log1p(r2 * d.clamp(min=0).float())
+        vis = (d >= 0) & (d < window) if window > 0 else d >= 0
+        sc = sc.masked_fill(~vis, float("-inf"))
+        if sinks is not None:
+            sc = torch.cat([sc, sinks.float().reshape(Hkv, G, 1, 1).expand(Hkv, G, ql, 1)], -1)
+        p = torch.softmax(sc, -1)[..., :n]
+        o = torch.einsum("hgqk,hkd->hgqd", p, v).permute(2, 0, 1, 3).reshape(ql, Hq * Dv)
+        if gate is not None:
+            o = o * torch.sigmoid(gate[q0:q1].float())
+        out[q0:q1] = o.to(q.dtype)
+    return out
+
+
+def paged_attention(q, kv, tables, lens, cu, out, *, Hq: int, Hkv: int, Dk: int, Dv: int, scale: float, max_q_len: int,
+                    max_len: int = 0, window: int = 0, sinks=None, dist_bias=None, gate=None, force_any: bool = False) -> None:
+    """Causal paged attention of the query rows of every sequence (the last ``cu[s+1] - cu[s]`` of its ``lens[s]``
+    tokens) into ``out`` [rows, Hq * Dv]. ``cu=None`` says one row per sequence (decode).
+
+    scores: ``q.k * scale - r1 ln(1 + r2 distance)`` with ``dist_bias = (r1, r2)`` per query head; ``sinks`` adds
+    ``exp(sink)`` to the denominator; ``gate`` ([rows, Hq * Dv], may be a column slice) multiplies the result by
+    its sigmoid. bf16 pools with row widths that are multiples of 8 up to 128 take the tensor-core kernels
+    (flash decoding with split KV; tcgen05 prefill); the rest the SIMT one."""
+    rows = q.shape[0]
+    if rows == 0:
+        return
+    if not q.is_cuda:
+        c = torch.arange(rows + 1) if cu is None else cu
+        out.copy_(paged_attention_ref(q, kv, tables, lens, c, Hq=Hq, Hkv=Hkv, Dk=Dk, Dv=Dv, scale=scale, window=window,
+                                      sinks=sinks, dist_bias=dist_bias, gate=gate))
+        return
+    r1, r2 = dist_bias if dist_bias is not None else (None, None)
+    assert kv.k.dtype == q.dtype and q.stride(1) == 1 and out.is_contiguous() and out.dtype == q.dtype
+    assert gate is None or (gate.stride(1) == 1 and gate.dtype == q.dtype)
+    gs = gate.stride(0) if gate is not None else 0
+    head = (q.data_ptr(), q.stride(0), kv.k.data_ptr(), kv.v.data_ptr())
+    tail = (_lib.ptr(sinks), _lib.ptr(r1), _lib.ptr(r2), _lib.ptr(gate), gs, out.data_ptr())
+    if q.dtype == torch.bfloat16 and not force_any:
+        from . import _decode_scratch, decode_splits
+        if cu is None:
+            splits = decode_splits(rows, Hkv, max_len or tables.shape[1] * kv.block_size)
+            scratch = _decode_scratch(q.device, int(_lib.load().mx_paged_decode_scratch_floats(rows, Hq, Dv, splits)))
+            rc = _fn("mx_paged_decode_ext")(*head, tables.data_ptr(), lens.data_ptr(), *tail, scratch.data_ptr(), rows, Hq,
+                                            Hkv, Dk, Dv, kv.block_size, tables.shape[1], window, float(scale), splits,
+                                            _lib.stream())
+        else:
+            rc = _fn("mx_paged_prefill_ext")(*head, kv.k.shape[0], tables.data_ptr(), cu.data_ptr(), lens.data_ptr(), *tail,
+                                             lens.shape[0], rows, max_q_len, Hq, Hkv, Dk, Dv, kv.block_size, tables.shape[1],
+                                             window, float(scale), _lib.workspace(q.device).data_ptr(), _lib.stream())
+        if rc != NOT_COVERED:
+            _lib.count_launch()
+            _lib.check(rc, "paged attention")
+            return
+    if cu is None:
+        cu = torch.arange(rows + 1, dtype=torch.int32, device=q.device)
+    _call("mx_paged_attention_any", *head, tables.data_ptr(), cu.data_ptr(), lens.data_ptr(), *tail, lens.shape[0], rows, Hq,
+          Hkv, Dk, Dv, kv.block_size, tables.shape[1], window, float(scale), _fp32(q), _lib.stream())
+
+
+# ----------------------------------------------------------------------------- generalized delta rule
+DELTA_DECAY_SCALE = math.exp(-0.5)       # largest decay exponent: w = exp(-exp(-1/2) sigmoid(.))
+DELTA_UNIT_EPS = 1e-6                    # inside the root of the unit key
+
+
+def delta_rule_ref(proj, offs, w2, w0, a_bias, norm_w, state, slots, cu, reset, D: int, norm_eps: float,
+                   decay_scale: float = DELTA_DECAY_SCALE, unit_eps: float = DELTA_UNIT_EPS):
+    H = state.shape[1]
+    HD, R = H * D, w2.shape[1]
+    f = proj.float()
+    r, k, v, g, a = (f[:, o:o + HD].reshape(-1, H, D) for o in offs[:5])
+    z = torch.tanh(f[:, offs[5]:offs[5] + R]) @ w2.float().t() + w0
+    w = torch.exp(-decay_scale * torch.sigmoid(z)).reshape(-1, H, D)
+    a = torch.sigmoid(a + a_bias.reshape(H, D))
+    u = k / torch.sqrt(k.pow(2).sum(-1, keepdim=True) + unit_eps)
+    o = torch.zeros(f.shape[0], H, D, device=proj.device)
+    sl, rs, c = slots.tolist(), reset.tolist(), cu.tolist()
+    for j in range(len(sl)):
+        if sl[j] < 0 or c[j + 1] <= c[j]:
+            continue
+        S = torch.zeros_like(state[0]) if rs[j] else state[sl[j]].clone()
+        for t in range(c[j], c[j + 1]):
+            read = (u[t][:, :, None] * S).sum(1)
+            S = w[t][:, :, None] * S - (a[t] * u[t])[:, :, None] * read[:, None, :] + k[t][:, :, None] * v[t][:, None, :]
+            o[t] = (S * r[t][:, :, None]).sum(1)
+        state[sl[j]] = S
+    y = _rms(o, norm_eps).reshape(-1, HD) * norm_w * torch.sigmoid(g.reshape(-1, HD))
+    return y.to(proj.dtype)
+
+
+def delta_rule(proj, offs, w2, w0, a_bias, norm_w, state, slots, cu, reset, *, D: int, norm_eps: float, n_short: int = 0,
+               decay_scale: float = DELTA_DECAY_SCALE, unit_eps: float = DELTA_UNIT_EPS, force_any: bool = False):
+    """Generalized delta rule over a ragged batch with its preparation, per-head output norm and gate.
+
+    ``proj`` rows hold r, k, v, gate, removal-rate and low-rank decay pre-activations at the element offsets
+    ``offs = (r, k, v, g, a, l)``; ``w2`` [H*D, R] lifts ``tanh(l)``; ``w0``, ``a_bias``, ``norm_w`` [H*D] fp32;
+    ``state`` [slots, H, D, D] fp32 is advanced in place; ``slots`` / ``reset`` [pieces], ``cu`` [pieces + 1] int32
+    (the first ``n_short`` pieces are decode rows of one token; a negative slot marks a padding row).
+    Returns [rows, H * D] in proj's type, ready for the output projection."""
+    if not proj.is_cuda:
+        return delta_rule_ref(proj, offs, w2, w0, a_bias, norm_w, state, slots, cu, reset, D, norm_eps, decay_scale, unit_eps)
+    H, rows = state.shape[1], proj.shape[0]
+    assert proj.stride(1) == 1 and w2.is_contiguous() and w2.dtype == proj.dtype and state.is_contiguous()
+    out = torch.empty(rows, H * D, dtype=proj.dtype, device=proj.device)
+    pieces = slots.shape[0]
+    scratch = None
+    if pieces > n_short and not force_any:
+        scratch = torch.empty((rows - n_short) * H * (6 * D + 2), dtype=torch.float32, device=proj.device)
+    arr = (ctypes.c_int * 6)(*[int(o) for o in offs])
+    _call("mx_delta_rule", proj.data_ptr(), proj.stride(0), ctypes.cast(arr, ctypes.c_void_p), w2.data_ptr(), w0.data_ptr(),
+          a_bias.data_ptr(), norm_w.data_ptr(), state.data_ptr(), slots.data_ptr(), cu.data_ptr(), reset.data_ptr(),
+          out.data_ptr(), _lib.ptr(scratch), pieces, n_short, rows, H, D, w2.shape[1], float(decay_scale), float(unit_eps),
+          float(norm_eps), _fp32(proj), 1 if force_any else 0, _lib.stream())
+    if not force_any:
+        _lib.count_launch((1 if n_short and pieces > n_short else 0) + (2 if pieces > n_short else 0))
+    return out

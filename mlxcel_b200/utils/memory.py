@@ -11,6 +11,8 @@ def _block_kinds(cfg: ModelConfig) -> list[str] | None:
         return ["M"] * cfg.num_hidden_layers
     if cfg.model_type == "mamba":
         return ["m"] * cfg.num_hidden_layers
+    if cfg.extra.get("layer_specs"):
+        return cfg.extra["layer_runs"]              # one entry per run: an index into the layer list
     pat = cfg.extra.get("hybrid_pattern")
     return list(pat) if pat else None
 
@@ -18,6 +20,17 @@ def _block_kinds(cfg: ModelConfig) -> list[str] | None:
 def _recurrent_block(cfg: ModelConfig, kind: str) -> tuple[int, int]:
     """(parameters, fp32 state bytes per sequence) of one block of a state-space / hybrid model."""
     h, x = cfg.hidden_size, cfg.extra
+    if x.get("layer_specs"):
+        # (a repeated layer's weights count once, its state for every run)
+        spec = x["layer_specs"][kind]
+        m, ff = spec["mixer"], (spec["mlp"] or {}).get("ff", 0)
+        if spec["type"] == "attention":
+            par = h * (m["heads"] * (m["dim"] + 2 * m["vdim"]) + m["kv_heads"] * (m["dim"] + m["vdim"]))
+            st = 0
+        else:
+            hd = m["heads"] * m["dim"]
+            par, st = 6 * h * hd + 4 * hd, 4 * hd * m["dim"]
+        return (par + 2 * h * ff + 6 * h) // x["layer_runs"].count(kind), st
     attn = h * (cfg.q_size + 2 * cfg.kv_size) + cfg.q_size * h
     if kind in ("M", "P"):
         m = x["mamba"]
@@ -70,7 +83,9 @@ def estimate_memory(cfg: ModelConfig, ctx: int = 8192, parallel: int = 4, kv_bit
         params = sum(p for p, _ in per) + emb + cfg.hidden_size
         state_seq = sum(s for _, s in per)
         n_attn = sum(k in ("*", "A", "P") for k in kinds)
-        kv_tok = cfg.kv_bytes_per_token(kv_bits) / max(cfg.num_hidden_layers, 1) * n_attn
+        kv_tok = cfg.kv_bytes_per_token(kv_bits)
+        if cfg.kv_geometry() is None:
+            kv_tok = kv_tok / max(cfg.num_hidden_layers, 1) * n_attn
     weights = (params - emb) * bpp / tp + emb * 2 / (1 if tp == 1 else 1)  # embedding replicated, head sharded
     blocks = (ctx + block_size - 1) // block_size * parallel
     kv = blocks * block_size * kv_tok
