@@ -946,6 +946,13 @@ paged_decode_mma_kernel(const DecodeParams p, const int G) {
     a[1] = pack_bf16(sacc[0][2], sacc[0][3]);
     a[2] = pack_bf16(sacc[1][0], sacc[1][1]);
     a[3] = pack_bf16(sacc[1][2], sacc[1][3]);
+    // extended form: the weights enter the second product as two bf16 terms (rounded weight + remainder)
+    uint32_t rest[4] = {0, 0, 0, 0};
+    if constexpr (EXT) {
+#pragma unroll
+      for (int i = 0; i < 4; ++i)
+        rest[i] = pack_bf16(sacc[i >> 1][(i & 1) * 2] - bf16_lo(a[i]), sacc[i >> 1][(i & 1) * 2 + 1] - bf16_hi(a[i]));
+    }
 #pragma unroll
     for (int nt = 0; nt < DV / 16; ++nt) {
       uint32_t bfr[4];
@@ -954,6 +961,10 @@ paged_decode_mma_kernel(const DecodeParams p, const int G) {
       ldmatrix_x4_trans(bfr, vs + swz<DV>(row, chunk));
       mma_bf16_16816(o_acc[nt * 2], a, bfr[0], bfr[1]);
       mma_bf16_16816(o_acc[nt * 2 + 1], a, bfr[2], bfr[3]);
+      if constexpr (EXT) {
+        mma_bf16_16816(o_acc[nt * 2], rest, bfr[0], bfr[1]);
+        mma_bf16_16816(o_acc[nt * 2 + 1], rest, bfr[2], bfr[3]);
+      }
     }
     if (++stage == kDmStages) stage = 0;
   }

@@ -60,6 +60,10 @@ struct TcPrefillParams {
 // them, so it tabulates its biases once per tile instead of taking a logarithm per score.
 constexpr int kBiasTab = 160;
 
+// The second weight term takes the room of one V stage where both heads are 128 wide: a V tile is only
+// needed once its softmax is through, so its load still has most of a tile's time.
+__host__ __device__ constexpr int tc_v_stages(int dk, int dv, bool ext) { return (ext && dk == 128 && dv == 128) ? 1 : kTcStages; }
+
 template <int DK, int DV, bool EXT>
 __global__ void __launch_bounds__(kTcThreads, 1)
 paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
@@ -69,7 +73,12 @@ paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
   constexpr int Q_BYTES = DC * SUB_BYTES;
   constexpr int K_BYTES = DC * SUB_BYTES;             // [128 keys][DK]
   constexpr int V_BYTES = DCV * SUB_BYTES;
-  constexpr int P_BYTES = 2 * SUB_BYTES;              // [128 rows][128 keys]
+  constexpr int PHALF_BYTES = 2 * SUB_BYTES;          // [128 rows][128 keys]
+  // The extended form feeds the weights to the second product as a sum of two bf16 terms (the rounded
+  // weight and what the rounding left), which keeps 16 bits of each: two MMAs per step instead of one.
+  constexpr int PTERMS = EXT ? 2 : 1;
+  constexpr int P_BYTES = PTERMS * PHALF_BYTES;
+  constexpr int VST = tc_v_stages(DK, DV, EXT);       // V ring depth
   constexpr int S_COLS = kTcKeys;                     // fp32 columns of one score buffer
   constexpr int O_COL = 2 * S_COLS;                   // first TMEM column of O
   constexpr uint32_t TMEM_COLS = 512;
@@ -82,8 +91,8 @@ paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
                                              ~static_cast<uintptr_t>(1023));
   uint8_t* q_sm = smem;
   uint8_t* k_sm = q_sm + Q_BYTES;                     // kTcStages x K_BYTES
-  uint8_t* v_sm = k_sm + kTcStages * K_BYTES;         // kTcStages x V_BYTES
-  uint8_t* p_sm = v_sm + kTcStages * V_BYTES;
+  uint8_t* v_sm = k_sm + kTcStages * K_BYTES;         // VST x V_BYTES
+  uint8_t* p_sm = v_sm + VST * V_BYTES;
   uint64_t* bars = reinterpret_cast<uint64_t*>(p_sm + P_BYTES);
   uint64_t* q_full = bars;                // 1
   uint64_t* k_full = bars + 1;            // [stages]
@@ -161,6 +170,8 @@ paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
     uint32_t phase = 0;
     bool ok = true;
     for (int j = 0; j < n_tiles && ok; ++j) {
+      const int vstage = j % VST;
+      const uint32_t vphase = static_cast<uint32_t>(j / VST) & 1u;
       // The K tile of a stage is free as soon as its score MMA has run, the V tile only after the
       // P V MMA of the same key tile: K of tile j + stages is requested a whole softmax earlier.
       // one pool block per lane; blocks past the sequence's last one repeat it (masked keys, but
@@ -181,14 +192,14 @@ paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
         for (int c = 0; c < DC; ++c) tma_load_2d(kd + c * SUB_BYTES, &map_k, &k_full[stage], c * 64, row0, pol_kv);
       }
       if (lane == 0) {
-        ok = mbar_wait(&kv_empty[stage], phase ^ 1u, p.status, kErrAttnProducer);
-        if (ok) mbar_expect_tx(&v_full[stage], V_BYTES);
+        ok = mbar_wait(&kv_empty[vstage], vphase ^ 1u, p.status, kErrAttnProducer);
+        if (ok) mbar_expect_tx(&v_full[vstage], V_BYTES);
       }
       ok = __shfl_sync(0xffffffffu, ok ? 1 : 0, 0) != 0;
       if (!ok) break;
       if (lane < kTcKeys / kTcBlock) {
-        uint8_t* vd = v_sm + stage * V_BYTES + lane * (kTcBlock * 128);
-        for (int c = 0; c < DCV; ++c) tma_load_2d(vd + c * SUB_BYTES, &map_v, &v_full[stage], c * 64, row0, pol_kv);
+        uint8_t* vd = v_sm + vstage * V_BYTES + lane * (kTcBlock * 128);
+        for (int c = 0; c < DCV; ++c) tma_load_2d(vd + c * SUB_BYTES, &map_v, &v_full[vstage], c * 64, row0, pol_kv);
       }
       __syncwarp();
       if (++stage == kTcStages) {
@@ -225,17 +236,20 @@ paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
       for (int j = 0; j < n_tiles && ok; ++j) {
         if (j + 1 < n_tiles) ok = issue_qk(j + 1);   // scores of the next tile under this softmax
         if (!ok) break;
-        const int stage = j % kTcStages;
-        const uint32_t kv_phase = static_cast<uint32_t>(j / kTcStages) & 1u;
-        if (!mbar_wait(&v_full[stage], kv_phase, p.status, kErrAttnMma)) break;
+        const int stage = j % VST;
+        const uint32_t v_phase = static_cast<uint32_t>(j / VST) & 1u;
+        if (!mbar_wait(&v_full[stage], v_phase, p.status, kErrAttnMma)) break;
         if (!mbar_wait(p_full, static_cast<uint32_t>(j) & 1u, p.status, kErrAttnMma)) break;
         tc_fence_after_sync();
         const uint32_t pa = smem_u32(p_sm), vb = smem_u32(v_sm + stage * V_BYTES);
 #pragma unroll
         for (int kk = 0; kk < kTcKeys / 16; ++kk) {
-          const uint64_t da = umma_desc_k_sw128(pa + (kk >> 2) * SUB_BYTES + (kk & 3) * 32);
           const uint64_t db = umma_desc_mn_sw128(vb + kk * (16 * 128), SUB_BYTES, 1024);
-          umma_bf16(tmem_base + O_COL, da, db, idesc_pv, (j > 0 || kk > 0) ? 1u : 0u);
+#pragma unroll
+          for (int term = 0; term < PTERMS; ++term) {
+            const uint64_t da = umma_desc_k_sw128(pa + term * PHALF_BYTES + (kk >> 2) * SUB_BYTES + (kk & 3) * 32);
+            umma_bf16(tmem_base + O_COL, da, db, idesc_pv, (j > 0 || kk > 0 || term > 0) ? 1u : 0u);
+          }
         }
         umma_commit(&kv_empty[stage]);   // the V tile of this stage is consumed
         umma_commit(pv_done);
@@ -356,7 +370,16 @@ paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
         pk.z = pack_bf16(e[4], e[5]);
         pk.w = pack_bf16(e[6], e[7]);
         const int sub = c8 >> 3, ch = c8 & 7;
-        *reinterpret_cast<uint4*>(p_sm + sub * SUB_BYTES + row * 128 + ((ch ^ (row & 7)) << 4)) = pk;
+        uint8_t* pd = p_sm + sub * SUB_BYTES + row * 128 + ((ch ^ (row & 7)) << 4);
+        *reinterpret_cast<uint4*>(pd) = pk;
+        if constexpr (EXT) {
+          uint4 rk;
+          rk.x = pack_bf16(e[0] - bf16_lo(pk.x), e[1] - bf16_hi(pk.x));
+          rk.y = pack_bf16(e[2] - bf16_lo(pk.y), e[3] - bf16_hi(pk.y));
+          rk.z = pack_bf16(e[4] - bf16_lo(pk.z), e[5] - bf16_hi(pk.z));
+          rk.w = pack_bf16(e[6] - bf16_lo(pk.w), e[7] - bf16_hi(pk.w));
+          *reinterpret_cast<uint4*>(pd + PHALF_BYTES) = rk;
+        }
       }
       l += sum;
       fence_proxy_async_smem();   // generic-proxy writes of P -> visible to the MMA's async proxy
@@ -428,8 +451,9 @@ template <int DK, int DV, bool EXT>
 static int launch_prefill_tc(const CUtensorMap& mq, const CUtensorMap& mk, const CUtensorMap& mv,
                              const TcPrefillParams& p, int grid, cudaStream_t stream) {
   constexpr int SUB = 128 * 128;
-  const int smem = (DK / 64) * SUB * (1 + kTcStages) + (DV / 64) * SUB * kTcStages + 2 * SUB + 1024 + 256 +
-                   (EXT ? 4 * kBiasTab * 4 : 0);
+  constexpr int smem = (DK / 64) * SUB * (1 + kTcStages) + (DV / 64) * SUB * tc_v_stages(DK, DV, EXT) +
+                       (EXT ? 4 : 2) * SUB + 1024 + 256 + (EXT ? 4 * kBiasTab * 4 : 0);
+  static_assert(smem <= 227 * 1024, "shared memory");
   auto kern = paged_prefill_tc_kernel<DK, DV, EXT>;
   static bool configured = false;
   if (!configured) {
