@@ -139,7 +139,13 @@ def main() -> None:
     ap.add_argument("--watchdog", type=int, default=1500,
                     help="seconds without finishing a round before every thread's stack is dumped and the "
                          "process exits (a stuck multi-rank run then ends by itself)")
+    ap.add_argument("--design", default=None, choices=["pamasun"],
+                    help="instead of the serving benchmark: prefill / decode throughput and kernel times of this design "
+                         "beside the closest existing model at equal size (one GPU, random weights)")
     args = ap.parse_args()
+    if args.design is not None:
+        import importlib
+        return importlib.import_module(f"benchmarks.{args.design}").run()
     if args.impl == "reference":
         return reference_arm(args)
     if args.warmup < 3:

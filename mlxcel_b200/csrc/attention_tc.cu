@@ -9,7 +9,7 @@
 //   warp 1     MMA issuer: S = Q K^T (M=128, N=128, K=D) into one of two TMEM score buffers, then
 //              O += P V (M=128, N=D, K=128 keys) with P read from shared memory and V consumed
 //              MN-major, exactly as it sits in the pool
-//   warps 2-5  softmax, one thread per query row: tcgen05.ld the scores, mask, running max with
+//   warps 2-5  (2-9 in the extended form) softmax, one (two) threads per query row: tcgen05.ld the scores, mask, running max with
 //              lazy rescaling (O in TMEM is rescaled only when a row maximum grows by more than
 //              2^8, the final normalisation uses the same stale maximum, so the result is exact),
 //              P = exp2(...) written as the bf16 A operand of the next MMA, and the epilogue
@@ -29,7 +29,6 @@ bool make_tensor_map_bf16(CUtensorMap* out, const void* ptr, uint64_t rows, uint
 
 constexpr int kTcRows = 128;      // query rows per CTA (UMMA M)
 constexpr int kTcKeys = 128;      // keys per tile
-constexpr int kTcThreads = 192;
 constexpr int kTcStages = 2;
 constexpr int kTcBlock = 16;      // pool block size this kernel is written for
 constexpr float kRescaleThreshold = 8.0f;   // log2 units
@@ -56,16 +55,23 @@ struct TcPrefillParams {
   long long gate_stride;
 };
 
-// Distances inside a (query tile, key tile) pair span 255 values; a softmax warp (32 rows) meets 159 of
-// them, so it tabulates its biases once per tile instead of taking a logarithm per score.
-constexpr int kBiasTab = 160;
+// The extended form runs eight softmax warps instead of four, two per 32 query rows: each takes one half of
+// a tile's keys (and of the output columns), the two exchange their row maxima once per tile and their sums
+// at the end through shared memory, under an mbarrier with the usual bounded wait.
+__host__ __device__ constexpr int tc_softmax_warps(bool ext) { return ext ? 8 : 4; }
+__host__ __device__ constexpr int tc_threads(bool ext) { return 64 + 32 * tc_softmax_warps(ext); }
+
+// Distances between a warp's 32 query rows and its 64 keys of a tile take 95 values: it tabulates their biases
+// once per tile instead of taking a logarithm per score.
+constexpr int kBiasTab = 96;
+constexpr int kExtSmem = 8 * kBiasTab * 4 + 2 * 2 * kTcRows * 4 + 2 * kTcRows * 4;   // tables, maxima (2 buffers), sums
 
 // The second weight term takes the room of one V stage where both heads are 128 wide: a V tile is only
 // needed once its softmax is through, so its load still has most of a tile's time.
 __host__ __device__ constexpr int tc_v_stages(int dk, int dv, bool ext) { return (ext && dk == 128 && dv == 128) ? 1 : kTcStages; }
 
 template <int DK, int DV, bool EXT>
-__global__ void __launch_bounds__(kTcThreads, 1)
+__global__ void __launch_bounds__(tc_threads(EXT), 1)
 paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
                         const __grid_constant__ CUtensorMap map_v, const TcPrefillParams p) {
   constexpr int DC = DK / 64, DCV = DV / 64;          // 64-column (128-byte) sub-tiles per row
@@ -103,8 +109,13 @@ paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
   uint64_t* p_full = s_empty + 2;            // 1
   uint64_t* pv_done = p_full + 1;            // 1
   uint64_t* k_empty = pv_done + 1;           // [stages] K tile consumed (after the score MMA)
-  uint32_t* tmem_ptr = reinterpret_cast<uint32_t*>(k_empty + kTcStages);
-  float* bias_tab = reinterpret_cast<float*>(p_sm + P_BYTES + 256);   // EXT: 4 warps x kBiasTab
+  uint64_t* pair_bar = k_empty + kTcStages;  // [4] EXT: the two warps of 32 rows exchange
+  uint32_t* tmem_ptr = reinterpret_cast<uint32_t*>(pair_bar + 4);
+  float* bias_tab = reinterpret_cast<float*>(p_sm + P_BYTES + 256);   // EXT: 8 warps x kBiasTab
+  float* pair_max = bias_tab + 8 * kBiasTab;                          // EXT: [2 buffers][2 halves][128 rows]
+  float* pair_sum = pair_max + 4 * kTcRows;                           // EXT: [2 halves][128 rows]
+  constexpr int SWARPS = tc_softmax_warps(EXT), HALVES = SWARPS / 4;
+  constexpr int HC = kTcKeys / HALVES;                                // key columns per softmax thread
 
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
 
@@ -139,9 +150,10 @@ paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
     }
     for (int i = 0; i < 2; ++i) {
       mbar_init(&s_full[i], 1);
-      mbar_init(&s_empty[i], 4);
+      mbar_init(&s_empty[i], SWARPS);
     }
-    mbar_init(p_full, 4);
+    mbar_init(p_full, SWARPS);
+    for (int i = 0; i < 4; ++i) mbar_init(&pair_bar[i], 2);
     mbar_init(pv_done, 1);
     fence_mbar_init();
   }
@@ -258,16 +270,22 @@ paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
     __syncwarp();
   } else {
     // ------------------------------------------------------------------ softmax + epilogue
-    const int q4 = warp & 3;
+    const int q4 = warp & 3;                        // TMEM lanes a warp may touch: 32 (warp mod 4) ..
+    const int half = HALVES == 2 ? (warp - 2) >> 2 : 0;   // EXT: keys half * 64 .. + 63 of every tile
     const int row = q4 * 32 + lane;                 // query row == TMEM lane
     const uint32_t lane_addr = tmem_base + (static_cast<uint32_t>(q4 * 32) << 16);
     const int qpos = pos_base + tok0 + row;         // absolute position of this row's token
     float m_used = -INFINITY;   // the maximum the stored exponentials refer to (scaled, log2 units)
     float l = 0.f;
-    float* tab = bias_tab + q4 * kBiasTab;
+    float* tab = bias_tab + (warp - 2) * kBiasTab;
     float r1 = 0.f, r2 = 0.f;
+    const __nv_bfloat16* gate = nullptr;            // this row's gate values, needed in the epilogue
     if constexpr (EXT) {
       if (p.bias_r1 != nullptr) r1 = p.bias_r1[hq], r2 = p.bias_r2[hq];
+      if (p.gate != nullptr && row < rows_valid) {
+        gate = p.gate + static_cast<size_t>(q0 + tok0 + row) * p.gate_stride + hq * dv;
+        for (int i = 0; i < dv; i += 64) asm volatile("prefetch.global.L2 [%0];" ::"l"(gate + i));
+      }
     }
     bool ok = true;
     for (int j = 0; j < n_tiles && ok; ++j) {
@@ -280,15 +298,16 @@ paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
       // Only tiles that cross the diagonal, the window edge or the end need the mask.
       const bool need_mask = (key0 + kTcKeys - 1 > pos_base + tok0) ||
                              (p.window > 0 && key0 < pos_base + tok0 + kTcRows - p.window);
-      int lo = 0, hi = kTcKeys;   // valid key columns of this row: [lo, hi)
+      const int hkey0 = key0 + half * HC;   // first key of this thread's columns
+      int lo = 0, hi = HC;   // valid key columns of this row: [lo, hi)
       if (need_mask) {
-        hi = min(kTcKeys, qpos - key0 + 1);
-        if (p.window > 0) lo = max(0, qpos - p.window + 1 - key0);
+        hi = min(HC, qpos - hkey0 + 1);
+        if (p.window > 0) lo = max(0, qpos - p.window + 1 - hkey0);
       }
       if constexpr (EXT) {
         // tab[i] = bias of distance base + i, where row r of this warp and key column c are at
-        // i = r - c + 127 (log2 domain: the natural logarithm's factor cancels against log2 e)
-        const int base = pos_base + tok0 + q4 * 32 - key0 - (kTcKeys - 1);
+        // i = r - c + 63 (log2 domain: the natural logarithm's factor cancels against log2 e)
+        const int base = pos_base + tok0 + q4 * 32 - hkey0 - (HC - 1);
         __syncwarp();
 #pragma unroll
         for (int i = 0; i < kBiasTab / 32; ++i) {
@@ -297,16 +316,16 @@ paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
         }
         __syncwarp();
       }
-      float sv[kTcKeys];
+      float sv[HC];
 #pragma unroll
-      for (int c = 0; c < kTcKeys / 32; ++c) {
+      for (int c = 0; c < HC / 32; ++c) {
         uint32_t r[32];
-        tmem_ld_32x32(lane_addr + sb * S_COLS + c * 32, r);
+        tmem_ld_32x32(lane_addr + sb * S_COLS + half * HC + c * 32, r);
         tmem_ld_wait();
 #pragma unroll
         for (int i = 0; i < 32; ++i) {
           sv[c * 32 + i] = __uint_as_float(r[i]) * p.scale_log2;
-          if constexpr (EXT) sv[c * 32 + i] -= tab[lane + (kTcKeys - 1) - (c * 32 + i)];
+          if constexpr (EXT) sv[c * 32 + i] -= tab[lane + (HC - 1) - (c * 32 + i)];
         }
       }
       tc_fence_before_sync();
@@ -315,13 +334,23 @@ paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
       float mx = -INFINITY;
       if (need_mask) {
 #pragma unroll
-        for (int i = 0; i < kTcKeys; ++i) {
+        for (int i = 0; i < HC; ++i) {
           if (i < lo || i >= hi) sv[i] = -INFINITY;
           mx = fmaxf(mx, sv[i]);
         }
       } else {
 #pragma unroll
-        for (int i = 0; i < kTcKeys; ++i) mx = fmaxf(mx, sv[i]);
+        for (int i = 0; i < HC; ++i) mx = fmaxf(mx, sv[i]);
+      }
+      if constexpr (HALVES == 2) {
+        // the row's maximum over both halves (two buffers: a warp is at most one exchange ahead)
+        float* xm = pair_max + (j & 1) * 2 * kTcRows;
+        xm[half * kTcRows + row] = mx;
+        __syncwarp();
+        if (lane == 0) mbar_arrive(&pair_bar[q4]);
+        ok = mbar_wait(&pair_bar[q4], static_cast<uint32_t>(j) & 1u, p.status, kErrAttnSoftmax);
+        if (!ok) break;
+        mx = fmaxf(mx, xm[(half ^ 1) * kTcRows + row]);
       }
       // lazy rescaling: keep the old reference maximum unless the row grew past it by 2^8
       float alpha = 1.0f;
@@ -341,7 +370,8 @@ paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
       }
       if (__any_sync(0xffffffffu, rescale)) {
 #pragma unroll
-        for (int c = 0; c < DV / 32; ++c) {
+        for (int cc = 0; cc < DV / 32 / HALVES; ++cc) {
+          const int c = half * (DV / 32 / HALVES) + cc;
           uint32_t r[32];
           tmem_ld_32x32(lane_addr + O_COL + c * 32, r);
           tmem_ld_wait();
@@ -357,7 +387,7 @@ paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
       float sum = 0.f;
       const float mref = (m_used == -INFINITY) ? 0.f : m_used;
 #pragma unroll
-      for (int c8 = 0; c8 < kTcKeys / 8; ++c8) {
+      for (int c8 = 0; c8 < HC / 8; ++c8) {
         float e[8];
 #pragma unroll
         for (int i = 0; i < 8; ++i) {
@@ -369,7 +399,7 @@ paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
         pk.y = pack_bf16(e[2], e[3]);
         pk.z = pack_bf16(e[4], e[5]);
         pk.w = pack_bf16(e[6], e[7]);
-        const int sub = c8 >> 3, ch = c8 & 7;
+        const int sub = half + (c8 >> 3), ch = c8 & 7;
         uint8_t* pd = p_sm + sub * SUB_BYTES + row * 128 + ((ch ^ (row & 7)) << 4);
         *reinterpret_cast<uint4*>(pd) = pk;
         if constexpr (EXT) {
@@ -387,7 +417,16 @@ paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
       __syncwarp();
       if (lane == 0) mbar_arrive(p_full);
     }
-    // ---- epilogue: O / l -> out (one row of D bf16 per thread)
+    // ---- epilogue: O / l -> out (one row of D bf16 per thread; EXT: half a row)
+    if constexpr (HALVES == 2) {
+      if (ok && n_tiles > 0) {
+        pair_sum[half * kTcRows + row] = l;
+        __syncwarp();
+        if (lane == 0) mbar_arrive(&pair_bar[q4]);
+        ok = mbar_wait(&pair_bar[q4], static_cast<uint32_t>(n_tiles) & 1u, p.status, kErrAttnSoftmax);
+        l = pair_sum[row] + pair_sum[kTcRows + row];       // (the same order in both warps)
+      }
+    }
     if (ok && n_tiles > 0) {
       ok = mbar_wait(pv_done, static_cast<uint32_t>(n_tiles - 1) & 1u, p.status, kErrAttnSoftmax);
     }
@@ -402,14 +441,19 @@ paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
       }
       const float inv = l > 0.f ? osc / l : 0.f;
       __nv_bfloat16* dst = p.out + static_cast<size_t>(q0 + tok0 + row) * p.Hq * dv + hq * dv;
-      const __nv_bfloat16* gate = nullptr;
-      if constexpr (EXT) {
-        if (p.gate != nullptr) gate = p.gate + static_cast<size_t>(q0 + tok0 + row) * p.gate_stride + hq * dv;
-      }
 #pragma unroll
-      for (int c = 0; c < DV / 32; ++c) {
+      for (int cc = 0; cc < DV / 32 / HALVES; ++cc) {
+        const int c = half * (DV / 32 / HALVES) + cc;
         uint32_t r[32];
         tmem_ld_32x32(lane_addr + O_COL + c * 32, r);
+        uint4 gv[4] = {};
+        if constexpr (EXT) {
+          if (gate != nullptr) {
+#pragma unroll
+            for (int i = 0; i < 4; ++i)
+              if (c * 32 + i * 8 < dv) gv[i] = *reinterpret_cast<const uint4*>(gate + c * 32 + i * 8);
+          }
+        }
         tmem_ld_wait();
         if (row < rows_valid) {
 #pragma unroll
@@ -417,12 +461,11 @@ paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
             if constexpr (EXT) {
               if (c * 32 + i >= dv) break;
               if (gate != nullptr) {
-                const uint4 gv = *reinterpret_cast<const uint4*>(gate + c * 32 + i);
-                const uint32_t gw[4] = {gv.x, gv.y, gv.z, gv.w};
+                const uint32_t gw[4] = {gv[i / 8].x, gv[i / 8].y, gv[i / 8].z, gv[i / 8].w};
 #pragma unroll
                 for (int e = 0; e < 4; ++e) {
-                  r[i + 2 * e] = __float_as_uint(__uint_as_float(r[i + 2 * e]) / (1.f + __expf(-bf16_lo(gw[e]))));
-                  r[i + 2 * e + 1] = __float_as_uint(__uint_as_float(r[i + 2 * e + 1]) / (1.f + __expf(-bf16_hi(gw[e]))));
+                  r[i + 2 * e] = __float_as_uint(__fdividef(__uint_as_float(r[i + 2 * e]), 1.f + __expf(-bf16_lo(gw[e]))));
+                  r[i + 2 * e + 1] = __float_as_uint(__fdividef(__uint_as_float(r[i + 2 * e + 1]), 1.f + __expf(-bf16_hi(gw[e]))));
                 }
               }
             }
@@ -452,7 +495,7 @@ static int launch_prefill_tc(const CUtensorMap& mq, const CUtensorMap& mk, const
                              const TcPrefillParams& p, int grid, cudaStream_t stream) {
   constexpr int SUB = 128 * 128;
   constexpr int smem = (DK / 64) * SUB * (1 + kTcStages) + (DV / 64) * SUB * tc_v_stages(DK, DV, EXT) +
-                       (EXT ? 4 : 2) * SUB + 1024 + 256 + (EXT ? 4 * kBiasTab * 4 : 0);
+                       (EXT ? 4 : 2) * SUB + 1024 + 256 + (EXT ? kExtSmem : 0);
   static_assert(smem <= 227 * 1024, "shared memory");
   auto kern = paged_prefill_tc_kernel<DK, DV, EXT>;
   static bool configured = false;
@@ -462,7 +505,7 @@ static int launch_prefill_tc(const CUtensorMap& mq, const CUtensorMap& mk, const
     prefer_max_shared(kern);
     configured = true;
   }
-  return static_cast<int>(launch_kernel(kern, dim3(grid), dim3(kTcThreads), smem, stream, mq, mk, mv, p));
+  return static_cast<int>(launch_kernel(kern, dim3(grid), dim3(tc_threads(EXT)), smem, stream, mq, mk, mv, p));
 }
 
 }  // namespace mx

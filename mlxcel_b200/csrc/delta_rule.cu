@@ -326,16 +326,18 @@ __device__ __forceinline__ void cp_async4_g(float* smem, const float* g) {
 }
 
 // Half a warp (16 lanes) shares kScanCols neighbouring columns of one head's state; a lane keeps RPT
-// key channels of each (channel groups of 4: 4 l .. 4 l + 3, then 64 further on; RPT = 2: 2 l, 2 l + 1).
-// A CTA of 4 warps covers kScanCta columns; the vectors of kScanChunk tokens are double-buffered in
-// shared memory. Per token: two partial dots per column, one halving exchange over the 16 lanes
-// (lanes 0-3 / 4-7 end with p of the two columns, 8-11 / 12-15 with the state part of o), the update.
-constexpr int kScanCols = 2;
-constexpr int kScanCta = 8 * kScanCols;
-constexpr int kScanTok = 16;
+// key channels of each (channel groups of 4: 4 l .. 4 l + 3, then 64 further on; RPT = 2: 2 l, 2 l + 1), so
+// that every vector element read from shared memory feeds kScanCols columns (the kernel is bound by those
+// reads and by instruction issue). A CTA of 4 warps covers kScanCta columns; the vectors of kScanTok tokens
+// are double-buffered. Per token: two partial dots per column, one halving exchange over the 16 lanes (lane
+// bit 3 ends with p or with the state part of o, bits 2 and 1 with the column), the update.
+constexpr int kScanCols = 4;
+constexpr int kScanCtaThreads = 128;
+constexpr int kScanCta = kScanCtaThreads / 16 * kScanCols;
+constexpr int kScanTok = 8;
 
 template <int RPT>
-__global__ void __launch_bounds__(128)
+__global__ void __launch_bounds__(kScanCtaThreads)
 delta_scan_kernel(const DeltaParams p, float* __restrict__ scratch, const int* __restrict__ slots,
                   const int* __restrict__ cu, const int* __restrict__ reset, int row0, int N) {
   constexpr int DP = 16 * RPT;
@@ -350,6 +352,7 @@ delta_scan_kernel(const DeltaParams p, float* __restrict__ scratch, const int* _
   const size_t HD = static_cast<size_t>(p.H) * D, arr = static_cast<size_t>(N) * HD;
   const int lane = threadIdx.x & 31, l16 = lane & 15, grp = threadIdx.x >> 4;
   const int c_in = grp * kScanCols, col0 = cb * kScanCta + c_in;
+  const int o_col = col0 + ((l16 & 4) >> 1) + ((l16 & 2) >> 1);      // output column of this lane
   // channel of this lane's row q
   const auto chan = [&](int q) { return RPT == 2 ? 2 * l16 + q : (q >> 2) * 64 + 4 * l16 + (q & 3); };
   float* S = p.state + (static_cast<size_t>(slot) * p.H + h) * D * D;
@@ -361,7 +364,7 @@ delta_scan_kernel(const DeltaParams p, float* __restrict__ scratch, const int* _
     for (int c = 0; c < kScanCols; ++c)
       s[q][c] = (chan(q) < D && col0 + c < D && !fresh) ? S[static_cast<size_t>(chan(q)) * D + col0 + c] : 0.f;
   // channels beyond D stay zero in both stages
-  for (int i = threadIdx.x; i < 2 * STAGE; i += 128) sc_smem[i] = 0.f;
+  for (int i = threadIdx.x; i < 2 * STAGE; i += kScanCtaThreads) sc_smem[i] = 0.f;
   __syncthreads();
   const float* sums = scratch + 5 * arr;
   float* o_out = scratch + 5 * arr + 2 * static_cast<size_t>(N) * p.H;
@@ -370,25 +373,27 @@ delta_scan_kernel(const DeltaParams p, float* __restrict__ scratch, const int* _
     const int nt = min(kScanTok, t1 - c0);
     if (nt > 0) {
       const size_t g0 = static_cast<size_t>(c0) * HD + static_cast<size_t>(h) * D;
+      // one warp per array: a lane copies its four channels of every token
+      const int a = threadIdx.x >> 5;
+      const float* src = scratch + a * arr + g0;
+      float* dst = st + a * DP;
       if (D % 4 == 0) {
-        const int per = D / 4;
-        for (int i = threadIdx.x; i < nt * 4 * per; i += 128) {
-          const int t = i / (4 * per), rem = i - t * 4 * per, a = rem / per, c = (rem - a * per) * 4;
-          cp_async16_g(st + (t * 4 + a) * DP + c, scratch + a * arr + g0 + t * HD + c);
-        }
+        const int c = lane * 4;
+        if (c < D)
+          for (int t = 0; t < nt; ++t) cp_async16_g(dst + t * 4 * DP + c, src + t * HD + c);
       } else {
-        for (int i = threadIdx.x; i < nt * 4 * D; i += 128) {
-          const int t = i / (4 * D), rem = i - t * 4 * D, a = rem / D, c = rem - a * D;
-          cp_async4_g(st + (t * 4 + a) * DP + c, scratch + a * arr + g0 + t * HD + c);
-        }
+        for (int t = 0; t < nt; ++t)
+          for (int c = lane; c < D; c += 32) cp_async4_g(dst + t * 4 * DP + c, src + t * HD + c);
       }
       float* vs = st + kScanTok * 4 * DP;
-      for (int i = threadIdx.x; i < nt * kScanCta; i += 128) {
-        const int t = i / kScanCta, c = i - t * kScanCta;
-        if (cb * kScanCta + c < D) cp_async4_g(vs + i, scratch + 4 * arr + g0 + t * HD + cb * kScanCta + c);
+      {
+        const int c = threadIdx.x % kScanCta, col = cb * kScanCta + c;
+        if (col < D)
+          for (int t = threadIdx.x / kScanCta; t < nt; t += kScanCtaThreads / kScanCta)
+            cp_async4_g(vs + t * kScanCta + c, scratch + 4 * arr + g0 + t * HD + col);
       }
       float* ss = vs + kScanTok * kScanCta;
-      for (int i = threadIdx.x; i < nt * 2; i += 128)
+      for (int i = threadIdx.x; i < nt * 2; i += kScanCtaThreads)
         cp_async4_g(ss + i, sums + static_cast<size_t>(i & 1) * N * p.H + static_cast<size_t>(c0 + (i >> 1)) * p.H + h);
     }
     asm volatile("cp.async.commit_group;" ::: "memory");
@@ -420,33 +425,40 @@ delta_scan_kernel(const DeltaParams p, float* __restrict__ scratch, const int* _
       };
       fetch(v4 + 2 * DP, u);
       fetch(v4 + 3 * DP, rw);
-      float p0 = 0.f, p1 = 0.f, o0 = 0.f, o1 = 0.f;
+      float pd[kScanCols], od[kScanCols];
 #pragma unroll
-      for (int q = 0; q < RPT; ++q) {
-        p0 = fmaf(u[q], s[q][0], p0);
-        p1 = fmaf(u[q], s[q][1], p1);
-        o0 = fmaf(rw[q], s[q][0], o0);
-        o1 = fmaf(rw[q], s[q][1], o1);
-      }
+      for (int c = 0; c < kScanCols; ++c) pd[c] = od[c] = 0.f;
+#pragma unroll
+      for (int q = 0; q < RPT; ++q)
+#pragma unroll
+        for (int c = 0; c < kScanCols; ++c) {
+          pd[c] = fmaf(u[q], s[q][c], pd[c]);
+          od[c] = fmaf(rw[q], s[q][c], od[c]);
+        }
       fetch(v4, w);
       fetch(v4 + DP, a);
-      const bool up8 = (l16 & 8) != 0, up4 = (l16 & 4) != 0;
-      const float x0 = (up8 ? o0 : p0) + __shfl_xor_sync(0xffffffffu, up8 ? p0 : o0, 8);
-      const float x1 = (up8 ? o1 : p1) + __shfl_xor_sync(0xffffffffu, up8 ? p1 : o1, 8);
-      float y = (up4 ? x1 : x0) + __shfl_xor_sync(0xffffffffu, up4 ? x0 : x1, 4);
-      y += __shfl_xor_sync(0xffffffffu, y, 2);
-      y += __shfl_xor_sync(0xffffffffu, y, 1);
-      const float q0 = __shfl_sync(0xffffffffu, y, lane & 16), q1 = __shfl_sync(0xffffffffu, y, (lane & 16) + 4);
-      const float2 nv = *reinterpret_cast<const float2*>(vs + t * kScanCta + c_in);
-      if (l16 == 8 && col0 < D)
-        o_out[static_cast<size_t>(c0 + t) * HD + h * D + col0] = y - ss[2 * t] * q0 + ss[2 * t + 1] * nv.x;
-      if (l16 == 12 && col0 + 1 < D)
-        o_out[static_cast<size_t>(c0 + t) * HD + h * D + col0 + 1] = y - ss[2 * t] * q1 + ss[2 * t + 1] * nv.y;
+      const bool up8 = (l16 & 8) != 0, up4 = (l16 & 4) != 0, up2 = (l16 & 2) != 0;
+      float x[4];
 #pragma unroll
-      for (int q = 0; q < RPT; ++q) {
-        s[q][0] = fmaf(w[q], s[q][0], u[q] * fmaf(-a[q], q0, nv.x));
-        s[q][1] = fmaf(w[q], s[q][1], u[q] * fmaf(-a[q], q1, nv.y));
+      for (int c = 0; c < 4; ++c) x[c] = (up8 ? od[c] : pd[c]) + __shfl_xor_sync(0xffffffffu, up8 ? pd[c] : od[c], 8);
+      const float y0 = (up4 ? x[2] : x[0]) + __shfl_xor_sync(0xffffffffu, up4 ? x[0] : x[2], 4);
+      const float y1 = (up4 ? x[3] : x[1]) + __shfl_xor_sync(0xffffffffu, up4 ? x[1] : x[3], 4);
+      float y = (up2 ? y1 : y0) + __shfl_xor_sync(0xffffffffu, up2 ? y0 : y1, 2);
+      y += __shfl_xor_sync(0xffffffffu, y, 1);
+      float pc[kScanCols];
+#pragma unroll
+      for (int c = 0; c < kScanCols; ++c) pc[c] = __shfl_sync(0xffffffffu, y, (lane & 16) + 2 * c);
+      const float4 nv4 = *reinterpret_cast<const float4*>(vs + t * kScanCta + c_in);
+      const float nv[kScanCols] = {nv4.x, nv4.y, nv4.z, nv4.w};
+      if (up8 && (l16 & 1) == 0 && o_col < D) {
+        const float pp = up4 ? (up2 ? pc[3] : pc[2]) : (up2 ? pc[1] : pc[0]);
+        const float vv = up4 ? (up2 ? nv[3] : nv[2]) : (up2 ? nv[1] : nv[0]);
+        o_out[static_cast<size_t>(c0 + t) * HD + h * D + o_col] = y - ss[2 * t] * pp + ss[2 * t + 1] * vv;
       }
+#pragma unroll
+      for (int q = 0; q < RPT; ++q)
+#pragma unroll
+        for (int c = 0; c < kScanCols; ++c) s[q][c] = fmaf(w[q], s[q][c], u[q] * fmaf(-a[q], pc[c], nv[c]));
     }
     __syncthreads();
   }
@@ -510,7 +522,7 @@ static int launch_delta_scan(const DeltaParams& p, float* scratch, const int* sl
     configured[dev] = true;
   }
   const int cbs = (p.D + kScanCta - 1) / kScanCta;
-  return static_cast<int>(launch_kernel(kern, dim3(p.H * cbs, pieces), dim3(128), smem, st, p, scratch, slots, cu, reset, row0, N));
+  return static_cast<int>(launch_kernel(kern, dim3(p.H * cbs, pieces), dim3(kScanCtaThreads), smem, st, p, scratch, slots, cu, reset, row0, N));
 }
 
 template <typename T>

@@ -165,76 +165,89 @@ polynorm_kernel(const T* __restrict__ z, const float* __restrict__ coef, T* __re
   }
 }
 
-// Rows of q | k | v (| more), `ld` elements apart. A warp handles one (token, head) of the Hq query,
-// Hkv key and Hkv value heads: queries are normalised in place, keys normalised into the pool
-// [blocks, Hkv, block_size, Dk], values copied into [blocks, Hkv, block_size, Dv]. Tokens with a
-// negative slot append nothing. A lane keeps up to 4 groups of V elements (Dk <= 128 V) in registers;
-// wider heads are read twice.
-template <typename T, int V>
+// Rows of q | k | v (| more), `ld` elements apart. One CTA per token; a warp takes every eighth of the Hq
+// query, Hkv key and Hkv value heads, kQkUnroll of them at a time so that their loads overlap: queries are
+// normalised in place, keys normalised into the pool [blocks, Hkv, block_size, Dk], values copied into
+// [blocks, Hkv, block_size, Dv]. Tokens with a negative slot append nothing. A lane keeps R groups of V
+// elements in registers; wider heads read the rest twice.
+constexpr int kQkUnroll = 3;
+
+template <typename T, int V, int R>
 __global__ void __launch_bounds__(256)
 qk_norm_append_kernel(T* __restrict__ qkv, long long ld, const int* __restrict__ slots, T* __restrict__ k_pool,
-                      T* __restrict__ v_pool, const float* __restrict__ qw, const float* __restrict__ kw, int T_,
-                      int Hq, int Hkv, int Dk, int Dv, int block_size, float eps) {
+                      T* __restrict__ v_pool, const float* __restrict__ qw, const float* __restrict__ kw, int Hq, int Hkv,
+                      int Dk, int Dv, int block_size, float eps) {
   pdl_trigger();
   pdl_wait();
-  const int lane = threadIdx.x & 31, per = Hq + 2 * Hkv;
-  const long long gw = (static_cast<long long>(blockIdx.x) * blockDim.x + threadIdx.x) >> 5;
-  if (gw >= static_cast<long long>(T_) * per) return;
-  const int t = static_cast<int>(gw / per), hd = static_cast<int>(gw - static_cast<long long>(t) * per);
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, per = Hq + 2 * Hkv, t = blockIdx.x;
   T* row = qkv + static_cast<size_t>(t) * ld;
   const int slot = slots[t];
-  T *src, *dst;
-  const float* w;
-  int D;
-  if (hd < Hq) {
-    src = dst = row + static_cast<size_t>(hd) * Dk, w = qw, D = Dk;
-    if (w == nullptr) return;
-  } else {
-    if (slot < 0) return;
-    const int blk = slot / block_size, off = slot - blk * block_size;
-    const bool key = hd < Hq + Hkv;
-    const int g = key ? hd - Hq : hd - Hq - Hkv;
-    D = key ? Dk : Dv;
-    src = row + static_cast<size_t>(Hq) * Dk + (key ? static_cast<size_t>(g) * Dk : static_cast<size_t>(Hkv) * Dk + static_cast<size_t>(g) * Dv);
-    dst = (key ? k_pool : v_pool) + ((static_cast<size_t>(blk) * Hkv + g) * block_size + off) * D;
-    w = key ? kw : nullptr;
-  }
-  constexpr int R = 4;
-  float f[R][V];
-  float s = 0.f;
+  const int blk = slot >= 0 ? slot / block_size : 0, off = slot >= 0 ? slot - blk * block_size : 0;
+  for (int h0 = warp; h0 < per; h0 += 8 * kQkUnroll) {
+    T *src[kQkUnroll], *dst[kQkUnroll];
+    const float* w[kQkUnroll];
+    int D[kQkUnroll];                       // 0: nothing to do
+    float f[kQkUnroll][R][V], s[kQkUnroll];
 #pragma unroll
-  for (int i = 0; i < R; ++i) {
-    const int c = (lane + 32 * i) * V;
-    if (c < D) {
-      load_v<V>(src + c, f[i]);
+    for (int n = 0; n < kQkUnroll; ++n) {
+      const int hd = h0 + 8 * n;
+      src[n] = dst[n] = row, w[n] = nullptr, D[n] = 0, s[n] = 0.f;
+      if (hd < Hq) {
+        src[n] = dst[n] = row + static_cast<size_t>(hd) * Dk, w[n] = qw;
+        D[n] = qw != nullptr ? Dk : 0;
+      } else if (hd < per && slot >= 0) {
+        const bool key = hd < Hq + Hkv;
+        const int g = key ? hd - Hq : hd - Hq - Hkv;
+        D[n] = key ? Dk : Dv;
+        src[n] = row + static_cast<size_t>(Hq) * Dk + (key ? static_cast<size_t>(g) * Dk : static_cast<size_t>(Hkv) * Dk + static_cast<size_t>(g) * Dv);
+        dst[n] = (key ? k_pool : v_pool) + ((static_cast<size_t>(blk) * Hkv + g) * block_size + off) * D[n];
+        w[n] = key ? kw : nullptr;
+      }
 #pragma unroll
-      for (int e = 0; e < V; ++e) s += f[i][e] * f[i][e];
+      for (int i = 0; i < R; ++i) {
+        const int c = (lane + 32 * i) * V;
+        if (c < D[n]) load_v<V>(src[n] + c, f[n][i]);
+      }
     }
-  }
-  for (int c = (lane + 32 * R) * V; c < D; c += 32 * V) {
-    float g[V];
-    load_v<V>(src + c, g);
 #pragma unroll
-    for (int e = 0; e < V; ++e) s += g[e] * g[e];
-  }
-  float r = 1.f;
-  if (w != nullptr) r = 1.f / sqrtf(warp_sum(s) / D + eps);
-  const auto emit = [&](int c, const float(&g)[V]) {
-    float o[V], wv[V];
-    if (w != nullptr) load_v<V>(w + c, wv);
+    for (int n = 0; n < kQkUnroll; ++n) {
+      if (D[n] == 0) continue;              // (the same for the whole warp)
+      float r = 1.f;
+      if (w[n] != nullptr) {
 #pragma unroll
-    for (int e = 0; e < V; ++e) o[e] = w != nullptr ? g[e] * r * wv[e] : g[e];
-    store_v<V>(dst + c, o);
-  };
+        for (int i = 0; i < R; ++i) {
+          const int c = (lane + 32 * i) * V;
+          if (c < D[n]) {
 #pragma unroll
-  for (int i = 0; i < R; ++i) {
-    const int c = (lane + 32 * i) * V;
-    if (c < D) emit(c, f[i]);
-  }
-  for (int c = (lane + 32 * R) * V; c < D; c += 32 * V) {
-    float g[V];
-    load_v<V>(src + c, g);
-    emit(c, g);
+            for (int e = 0; e < V; ++e) s[n] += f[n][i][e] * f[n][i][e];
+          }
+        }
+        for (int c = (lane + 32 * R) * V; c < D[n]; c += 32 * V) {
+          float g[V];
+          load_v<V>(src[n] + c, g);
+#pragma unroll
+          for (int e = 0; e < V; ++e) s[n] += g[e] * g[e];
+        }
+        r = 1.f / sqrtf(warp_sum(s[n]) / D[n] + eps);
+      }
+      const auto emit = [&](int c, const float(&g)[V]) {
+        float o[V], wv[V];
+        if (w[n] != nullptr) load_v<V>(w[n] + c, wv);
+#pragma unroll
+        for (int e = 0; e < V; ++e) o[e] = w[n] != nullptr ? g[e] * r * wv[e] : g[e];
+        store_v<V>(dst[n] + c, o);
+      };
+#pragma unroll
+      for (int i = 0; i < R; ++i) {
+        const int c = (lane + 32 * i) * V;
+        if (c < D[n]) emit(c, f[n][i]);
+      }
+      for (int c = (lane + 32 * R) * V; c < D[n]; c += 32 * V) {
+        float g[V];
+        load_v<V>(src[n] + c, g);
+        emit(c, g);
+      }
+    }
   }
 }
 
@@ -300,13 +313,10 @@ template <typename T>
 static int qk_norm_append_typed(void* qkv, long long ld, const int* slots, void* k_pool, void* v_pool, const float* qw,
                                 const float* kw, int n, int Hq, int Hkv, int Dk, int Dv, int bs, float eps, bool vec,
                                 cudaStream_t st) {
-  const long long warps = static_cast<long long>(n) * (Hq + 2 * Hkv);
-  const long long blocks = (warps + 7) / 8;
-  if (blocks > 0x7fffffffLL) return -1;
-  const dim3 grid(static_cast<unsigned>(blocks)), block(256);
+  const dim3 grid(n), block(256);
   T *qp = static_cast<T*>(qkv), *kp = static_cast<T*>(k_pool), *vp = static_cast<T*>(v_pool);
-  if (vec) return static_cast<int>(launch_kernel(qk_norm_append_kernel<T, 4>, grid, block, 0, st, qp, ld, slots, kp, vp, qw, kw, n, Hq, Hkv, Dk, Dv, bs, eps));
-  return static_cast<int>(launch_kernel(qk_norm_append_kernel<T, 1>, grid, block, 0, st, qp, ld, slots, kp, vp, qw, kw, n, Hq, Hkv, Dk, Dv, bs, eps));
+  auto kern = !vec ? qk_norm_append_kernel<T, 1, 4> : (Dk <= 128 && Dv <= 128) ? qk_norm_append_kernel<T, 4, 1> : qk_norm_append_kernel<T, 4, 2>;
+  return static_cast<int>(launch_kernel(kern, grid, block, 0, st, qp, ld, slots, kp, vp, qw, kw, Hq, Hkv, Dk, Dv, bs, eps));
 }
 
 }  // namespace mx
