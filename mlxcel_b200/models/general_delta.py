@@ -5,7 +5,7 @@ unit key u: ``S <- diag(w) S - (a u)(u^T S) + k v^T``, both terms from the old s
 by its root mean square per head, weighted and gated. The decay comes from a low-rank projection,
 ``w = exp(-exp(-1/2) sigmoid(w0 + W2 tanh(W1 h)))``. Kernels: ``csrc/delta_rule.cu``.
 
-State slots and the engine contract are those of :class:`Mamba2Model`; there is no convolution. Every run
+State slots and the interface to the engine are those of :class:`Mamba2Model`; there is no convolution. Every run
 of a layer that is executed several times owns a slab of its own, and layers may differ in heads and
 width, so the slabs are a list. Decode steps read the slots from a fixed device buffer when the engine
 provides one (``StepBatch.state_slots``), which makes them replayable from a CUDA graph.
