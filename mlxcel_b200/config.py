@@ -1338,6 +1338,62 @@ def _pamasun(c: ModelConfig, raw: dict) -> None:
     c.intermediate_size = max([s["mlp"]["ff"] for s in specs if s["mlp"]] or [1])
 
 
+def _rotation(rot: dict, what: str) -> dict:
+    """``rot`` record of a mixer: rotated dimensions, base, optional YaRN scaling (factor, original, fast, slow)."""
+    out = dict(dims=int(rot["dims"]), base=float(rot["base"]))
+    if out["dims"] % 2:
+        raise ValueError(f"{what}: rot.dims must be even")
+    sc = rot.get("scaling")
+    if sc:
+        out["scaling"] = {k: float(sc[k]) for k in ("factor", "original", "fast", "slow")}
+    return out
+
+
+def _govopel(c: ModelConfig, raw: dict) -> None:
+    """Govopel: an explicit layer list (grouped-query attention over chunks with values = keys, or latent attention; dense
+    clipped-GLU MLP or none), every sub-layer normalised behind it only, a normalised embedding tied to the soft-capped
+    head. Each layer owns a KV-pool layer: per-head keys and values, or one latent row per token."""
+    c.vocab_size, c.hidden_size = int(raw["vocab"]), int(raw["width"])
+    c.rms_norm_eps = float(raw["norm"]["eps"])
+    c.tie_word_embeddings = True
+    c.final_logit_softcap = float(raw.get("logit_softcap") or 0.0)
+    specs, geo = [], []
+    for i, spec in enumerate(raw["layers"]):
+        kind, m, mlp, what = spec["type"], spec["mixer"], spec.get("mlp"), f"layer {i}"
+        if kind == "attention":
+            mask = m.get("mask")
+            m = dict(heads=int(m["heads"]), kv_heads=int(m["kv_heads"]), dim=int(m["dim"]), vdim=int(m["vdim"]), scale=float(m["scale"]),
+                     softcap=float(m.get("softcap") or 0.0), rot=_rotation(m["rot"], what),
+                     mask=dict(size=int(mask["size"])) if mask else None)
+            if m["heads"] % m["kv_heads"]:
+                raise ValueError(f"{what}: heads must be a multiple of kv_heads")
+            if m["dim"] != m["vdim"]:
+                raise ValueError(f"{what}: values are the keys, so vdim must equal dim")
+            if m["rot"]["dims"] > m["dim"] or (m["mask"] and m["mask"]["size"] < 1):
+                raise ValueError(f"{what}: rot.dims above dim, or an empty chunk")
+            geo.append((m["kv_heads"], m["dim"], m["vdim"]))
+        elif kind == "latent_attention":
+            m = dict(heads=int(m["heads"]), dim=int(m["dim"]), rot_dim=int(m["rot_dim"]), vdim=int(m["vdim"]), q_rank=int(m["q_rank"]),
+                     kv_rank=int(m["kv_rank"]), scale=float(m["scale"]), rot=_rotation(m["rot"], what))
+            if m["rot"]["dims"] != m["rot_dim"]:
+                raise ValueError(f"{what}: rot.dims must equal rot_dim")
+            geo.append((1, m["kv_rank"] + m["rot_dim"], 0))
+        else:
+            raise ValueError(f"{what}: unknown mixer type {kind!r}")
+        if mlp is not None:
+            if mlp.get("kind", "dense") != "dense":
+                raise ValueError(f"{what}: unknown feed-forward kind {mlp.get('kind')!r}")
+            mlp = dict(kind="dense", ff=int(mlp["ff"]), limit=float(mlp["limit"]))
+        specs.append(dict(type=kind, mixer=m, mlp=mlp))
+    c.extra["layer_specs"], c.extra["layer_runs"], c.extra["kv_geometry"] = specs, list(range(len(specs))), geo
+    c.num_hidden_layers = len(specs)
+    # (uniform fields other parts read: the first layer's)
+    h, k, d = (specs[0]["mixer"]["heads"], *geo[0][:2]) if specs else (1, 1, 16)
+    c.num_attention_heads, c.num_key_value_heads, c.head_dim = h, k, d
+    c.partial_rotary_factor = 0.0
+    c.intermediate_size = max([s["mlp"]["ff"] for s in specs if s["mlp"]] or [1])
+
+
 def _baichuan(c: ModelConfig, raw: dict) -> None:
     """Baichuan (7B layout): Llama block with q, k, v fused in ``W_pack`` (reference src/models/baichuan.rs).
     The 13B models replace RoPE by ALiBi, which no attention kernel here implements."""
@@ -1361,7 +1417,7 @@ FAMILIES = {
     "gpt_neox": _gpt_neox, "gpt2": _gpt2, "gpt_bigcode": _gpt2, "phi": _phi, "olmo": _olmo1, "granitemoe": _granitemoe, "granitemoehybrid": _granitemoehybrid, "jamba": _jamba, "bitnet": _bitnet, "lfm2_moe": _lfm2, "exaone": _exaone, "telechat3": _telechat3, "deepseek": _deepseek_v1, "recurrent_gemma": _recurrent_gemma, "glm_moe_dsa": _glm_moe_dsa, "deepseek_v32": _glm_moe_dsa, "mistral4": _mistral4, "afmoe": _afmoe, "dbrx": _dbrx, "llama4": _llama4, "llama4_text": _llama4, "qwen3_next": _qwen3_next, "qwen3_5": _qwen3_next, "qwen3_5_text": _qwen3_next, "qwen3_5_moe": _qwen3_next, "qwen3_5_moe_text": _qwen3_next, "falcon_h1": _falcon_h1, "cohere2": _cohere2, "arcee": _arcee, "glm": _glm, "glm4": _glm4, "glm4v": _glm4v, "glm4v_text": _glm4v, "glm4v_moe": _glm4v_moe, "glm4v_moe_text": _glm4v_moe, "cohere2_vision": _cohere2, "paddleocr_vl": _paddleocr_vl, "glm_ocr": _glm_ocr, "glm_ocr_text": _glm_ocr, "paddleocr_vl_text": _paddleocr_vl, "nemotron": _nemotron,
     "ministral3": _ministral3, "granitemoeshared": _granitemoeshared, "nanochat": _nanochat, "code_llama": _plain, "cwm": _plain, "glm4_moe_lite": _deepseek_v3,
     "vaultgemma": _vaultgemma, "solar_open": _solar_open, "minimax_m2": _minimax_m2, "exaone_moe": _exaone_moe, "lfm2": _lfm2, "internlm2": _plain, "baichuan": _baichuan,
-    "pamasun": _pamasun,
+    "pamasun": _pamasun, "govopel": _govopel,
 }
 
 
@@ -1429,6 +1485,13 @@ def preset(name: str) -> ModelConfig:
         return ModelConfig.from_dict(dict(
             architecture="Pamasun", vocab=512, width=144, layers=[delta, attn, dict(delta, mlp=None), attn],
             loop=dict(start=1, stop=3, times=2), embedding=dict(scale=12.0), norm=dict(eps=1e-5)))
+    if name == "tiny-govopel":
+        lat = dict(type="latent_attention", mixer=dict(heads=4, dim=24, rot_dim=16, vdim=32, q_rank=48, kv_rank=56, scale=0.18,
+                                                       rot=dict(dims=16, base=50000.0)), mlp=dict(kind="dense", ff=160, limit=2.0))
+        att = dict(type="attention", mixer=dict(heads=6, kv_heads=2, dim=40, vdim=40, scale=0.2, softcap=12.0, mask=dict(size=48), rot=dict(
+            dims=24, base=8000.0, scaling=dict(factor=4.0, original=512, fast=16.0, slow=1.0))), mlp=dict(kind="dense", ff=144, limit=1.5))
+        return ModelConfig.from_dict(dict(architecture="Govopel", vocab=512, width=144, layers=[lat, att, dict(att, mlp=None), lat],
+                                          norm=dict(eps=1e-5), logit_softcap=20.0))
     if name == "mamba2-2.7b":
         return ModelConfig.from_dict(dict(
             model_type="mamba2", num_hidden_layers=64, hidden_size=2560, num_heads=80, head_dim=64,

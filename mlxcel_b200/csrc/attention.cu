@@ -19,6 +19,7 @@
 // chunked causal attention (src/lib/mlxcel-core/src/layers.rs:5798).
 #include "api.h"
 #include "common.cuh"
+#include "mma_sync.cuh"
 
 namespace mx {
 
@@ -48,7 +49,8 @@ struct DecodeParams {
   // elements (multiples of 8 up to the padded tile widths), a logarithmic distance bias per query head
   // (r1[h] ln(1 + r2[h] d) is taken off the score of a key d tokens back) and an output gate
   // (result *= sigmoid(gate)). bias and gate may be NULL.
-  int dk, dv;
+  // chunk > 0: a token sees only keys of its own run of `chunk` positions, counted from the sequence's start.
+  int dk, dv, chunk;
   const float* bias_r1;
   const float* bias_r2;
   const __nv_bfloat16* gate;
@@ -353,43 +355,6 @@ struct PrefillParams {
   float scale_log2, softcap;
 };
 
-__device__ __forceinline__ void ldmatrix_x4(uint32_t (&r)[4], uint32_t addr) {
-  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0, %1, %2, %3}, [%4];"
-               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3])
-               : "r"(addr));
-}
-__device__ __forceinline__ void ldmatrix_x4_trans(uint32_t (&r)[4], uint32_t addr) {
-  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0, %1, %2, %3}, [%4];"
-               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3])
-               : "r"(addr));
-}
-__device__ __forceinline__ void mma_bf16_16816(float (&c)[4], const uint32_t (&a)[4], uint32_t b0,
-                                               uint32_t b1) {
-  asm volatile(
-      "mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, "
-      "{%8, %9}, {%0, %1, %2, %3};"
-      : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
-      : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
-}
-__device__ __forceinline__ void cp_async16(uint32_t smem_addr, const void* gptr, bool pred) {
-  const int sz = pred ? 16 : 0;
-  asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(smem_addr), "l"(gptr), "r"(sz)
-               : "memory");
-}
-// 4-, 8- or 16-byte asynchronous copy (cache-all variant: the only one that takes sizes below 16);
-// a false predicate zero-fills the destination.
-template <int BYTES>
-__device__ __forceinline__ void cp_async_small(uint32_t smem_addr, const void* gptr, bool pred) {
-  const int sz = pred ? BYTES : 0;
-  asm volatile("cp.async.ca.shared.global [%0], [%1], %2, %3;" ::"r"(smem_addr), "l"(gptr), "n"(BYTES), "r"(sz)
-               : "memory");
-}
-__device__ __forceinline__ void cp_async_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
-template <int N>
-__device__ __forceinline__ void cp_async_wait() {
-  asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory");
-}
-
 // Shared tiles are [rows][D] bf16 with the 16-byte chunk index XOR-swizzled by (row & 7).
 template <int D>
 __device__ __forceinline__ uint32_t swz(int row, int chunk) {
@@ -678,6 +643,9 @@ paged_decode_mma_kernel(const DecodeParams p, const int G) {
   const int len = p.context_lens[b];
   int begin = 0;
   if (p.window > 0 && len > p.window) begin = len - p.window;
+  if constexpr (EXT) {
+    if (p.chunk > 0 && len > 0) begin = max(begin, (len - 1) / p.chunk * p.chunk);
+  }
   const int g_begin = begin / kDmKeys;                          // first key group
   const int g_end = (len + kDmKeys - 1) / kDmKeys;              // one past the last key group
   const int n_groups = max(0, g_end - g_begin);
@@ -895,8 +863,8 @@ paged_decode_mma_kernel(const DecodeParams p, const int G) {
       for (int e = 0; e < 4; ++e) {
         const int key = key0 + nt * 8 + (lane & 3) * 2 + (e & 1);
         float v = sacc[nt][e] * p.scale_log2;
-        if (p.softcap > 0.f) v = p.softcap * tanhf(v / (kLog2e * p.softcap)) * kLog2e;
-        if constexpr (EXT) {
+        if (p.softcap > 0.f) v = soft_cap_log2(v, p.softcap);
+        if (EXT && p.bias_r1 != nullptr) {
           // in the log2 domain the bias is r1 log2(1 + r2 d): the natural logarithm's factor cancels
           const float dist = static_cast<float>(max(len - 1 - key, 0));
           v -= (e < 2 ? b1_lo : b1_hi) * log2f(fmaf(e < 2 ? b2_lo : b2_hi, dist, 1.f));
@@ -1213,12 +1181,13 @@ extern "C" int mx_paged_decode(const void* q, long long q_stride, const void* k_
 }
 
 // Extended decode form over bf16 pools: key / value rows of Dk / Dv elements (multiples of 8, at most
-// 128), distance bias and output gate optional. -10 = not covered (use mx_paged_attention_any).
+// 128), soft cap, chunked visibility, distance bias and output gate optional (0 / NULL). -10 = not covered (use mx_paged_attention_any).
 extern "C" int mx_paged_decode_ext(const void* q, long long q_stride, const void* k_pool, const void* v_pool,
                                    const int* block_tables, const int* context_lens, const float* sinks,
                                    const float* bias_r1, const float* bias_r2, const void* gate, long long gate_stride,
                                    void* out, float* scratch, int B, int Hq, int Hkv, int Dk, int Dv, int block_size,
-                                   int max_blocks, int window, float scale, int num_splits, void* stream_) {
+                                   int max_blocks, int window, int chunk, float scale, float softcap, int num_splits,
+                                   void* stream_) {
   if (B <= 0) return 0;
   if (Hkv <= 0 || Hq % Hkv || (bias_r1 == nullptr) != (bias_r2 == nullptr)) return -1;
   const int G = Hq / Hkv;
@@ -1250,6 +1219,8 @@ extern "C" int mx_paged_decode_ext(const void* q, long long q_stride, const void
   p.scale_log2 = scale * kLog2e;
   p.dk = Dk;
   p.dv = Dv;
+  p.chunk = chunk;
+  p.softcap = softcap;
   p.bias_r1 = bias_r1;
   p.bias_r2 = bias_r2;
   p.gate = static_cast<const __nv_bfloat16*>(gate);

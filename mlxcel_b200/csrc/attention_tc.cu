@@ -26,6 +26,8 @@ namespace mx {
 
 bool make_tensor_map_bf16(CUtensorMap* out, const void* ptr, uint64_t rows, uint64_t cols,
                           uint64_t ld, uint32_t box_rows, uint32_t box_cols);
+bool make_tensor_map_bf16_3d(CUtensorMap* out, const void* ptr, uint64_t rows, uint64_t groups, uint64_t cols, uint64_t ld,
+                             uint64_t group_ld, uint32_t box_rows, uint32_t box_cols);
 
 constexpr int kTcRows = 128;      // query rows per CTA (UMMA M)
 constexpr int kTcKeys = 128;      // keys per tile
@@ -47,12 +49,20 @@ struct TcPrefillParams {
   // Extended form (EXT): rows of dk / dv elements inside tiles of DK / DV columns (the tensor maps end at
   // the row's width, so the missing columns arrive as zeros), a logarithmic distance bias
   // r1[h] ln(1 + r2[h] d) taken off the scores, an output gate (result *= sigmoid(gate)); bias and gate
-  // may be NULL.
-  int dk, dv;
+  // may be NULL. chunk > 0: keys of the query's own run of `chunk` positions only; softcap > 0: scores s become
+  // softcap tanh(s / softcap).
+  int dk, dv, chunk;
+  float softcap;
   const float* bias_r1;
   const float* bias_r2;
   const __nv_bfloat16* gate;
   long long gate_stride;
+  // Dense keys and values (kv_starts != NULL, no pool): the context of sequence s lies in rows kv_starts[s] .. of
+  // per-head key and value matrices, and the key's last columns (from kv_split on, one 64-column tile) come from
+  // a matrix all heads share.
+  const int* kv_starts;
+  int kv_split;
+  long long out_stride;      // elements between output rows
 };
 
 // The extended form runs eight softmax warps instead of four, two per 32 query rows: each takes one half of
@@ -68,12 +78,15 @@ constexpr int kExtSmem = 8 * kBiasTab * 4 + 2 * 2 * kTcRows * 4 + 2 * kTcRows * 
 
 // The second weight term takes the room of one V stage where both heads are 128 wide: a V tile is only
 // needed once its softmax is through, so its load still has most of a tile's time.
-__host__ __device__ constexpr int tc_v_stages(int dk, int dv, bool ext) { return (ext && dk == 128 && dv == 128) ? 1 : kTcStages; }
+__host__ __device__ constexpr int tc_v_stages(int dk, int dv, bool ext) { return (ext && dk >= 128 && dv == 128) ? 1 : kTcStages; }
+// Keys of 192 columns leave room for one K stage (free again as soon as its score MMA has run).
+__host__ __device__ constexpr int tc_k_stages(int dk) { return dk > 128 ? 1 : kTcStages; }
 
 template <int DK, int DV, bool EXT>
 __global__ void __launch_bounds__(tc_threads(EXT), 1)
 paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
-                        const __grid_constant__ CUtensorMap map_v, const TcPrefillParams p) {
+                        const __grid_constant__ CUtensorMap map_v, const __grid_constant__ CUtensorMap map_kr,
+                        const TcPrefillParams p) {
   constexpr int DC = DK / 64, DCV = DV / 64;          // 64-column (128-byte) sub-tiles per row
   constexpr int SUB_BYTES = 128 * 128;                // one [128 rows][64 cols] sub-tile
   constexpr int Q_BYTES = DC * SUB_BYTES;
@@ -85,10 +98,11 @@ paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
   constexpr int PTERMS = EXT ? 2 : 1;
   constexpr int P_BYTES = PTERMS * PHALF_BYTES;
   constexpr int VST = tc_v_stages(DK, DV, EXT);       // V ring depth
+  constexpr int KST = tc_k_stages(DK);                // K ring depth
   constexpr int S_COLS = kTcKeys;                     // fp32 columns of one score buffer
   constexpr int O_COL = 2 * S_COLS;                   // first TMEM column of O
   constexpr uint32_t TMEM_COLS = 512;
-  static_assert((DK == 64 || DK == 128) && (DV == 64 || DV == 128), "head dims");
+  static_assert((DK == 64 || DK == 128 || (EXT && DK == 192)) && (DV == 64 || DV == 128), "head dims");
   static_assert(EXT || DK == DV, "plain form: one head width");
   const int dk = EXT ? p.dk : DK, dv = EXT ? p.dv : DV;
 
@@ -96,8 +110,8 @@ paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) &
                                              ~static_cast<uintptr_t>(1023));
   uint8_t* q_sm = smem;
-  uint8_t* k_sm = q_sm + Q_BYTES;                     // kTcStages x K_BYTES
-  uint8_t* v_sm = k_sm + kTcStages * K_BYTES;         // VST x V_BYTES
+  uint8_t* k_sm = q_sm + Q_BYTES;                     // KST x K_BYTES
+  uint8_t* v_sm = k_sm + KST * K_BYTES;               // VST x V_BYTES
   uint8_t* p_sm = v_sm + VST * V_BYTES;
   uint64_t* bars = reinterpret_cast<uint64_t*>(p_sm + P_BYTES);
   uint64_t* q_full = bars;                // 1
@@ -133,6 +147,9 @@ paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
   const int kv_end = pos_base + tok0 + rows_valid;   // one past the last visible key
   int kv_begin = 0;
   if (p.window > 0) kv_begin = max(0, pos_base + tok0 - p.window + 1);
+  if constexpr (EXT) {
+    if (p.chunk > 0) kv_begin = max(kv_begin, (pos_base + tok0) / p.chunk * p.chunk);
+  }
   kv_begin = (kv_begin / kTcKeys) * kTcKeys;
   const int n_tiles = (kv_end - kv_begin + kTcKeys - 1) / kTcKeys;
   const int last_block = (ctx - 1) / kTcBlock;   // last pool block the sequence owns
@@ -176,11 +193,33 @@ paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
     if (lane == 0) {
       mbar_expect_tx(q_full, Q_BYTES);
       for (int c = 0; c < DC; ++c)
-        tma_load_2d(q_sm + c * SUB_BYTES, &map_q, q_full, hq * dk + c * 64, q0 + tok0, pol_q);
+        if (EXT && p.kv_starts != nullptr)
+          tma_load_3d(q_sm + c * SUB_BYTES, &map_q, q_full, c * 64 < p.kv_split ? c * 64 : p.kv_split, hq, q0 + tok0, pol_q);
+        else
+          tma_load_2d(q_sm + c * SUB_BYTES, &map_q, q_full, hq * dk + c * 64, q0 + tok0, pol_q);
     }
     int stage = 0;
     uint32_t phase = 0;
     bool ok = true;
+    if (EXT && p.kv_starts != nullptr) {
+      // dense rows: one box per 64-column tile (rows past the sequence belong to the next one or are filled with
+      // zeros; the mask drops them)
+      const int base = p.kv_starts[s];
+      for (int j = 0; lane == 0 && j < n_tiles; ++j) {
+        const int row0 = base + kv_begin + j * kTcKeys, ks = j % KST, vs = j % VST;
+        if (!mbar_wait(&k_empty[ks], (static_cast<uint32_t>(j / KST) & 1u) ^ 1u, p.status, kErrAttnProducer)) break;
+        mbar_expect_tx(&k_full[ks], K_BYTES);
+        for (int c = 0; c < DC; ++c) {
+          uint8_t* kd = k_sm + ks * K_BYTES + c * SUB_BYTES;
+          if (c * 64 < p.kv_split) tma_load_3d(kd, &map_k, &k_full[ks], c * 64, hkv, row0, pol_kv);
+          else tma_load_2d(kd, &map_kr, &k_full[ks], 0, row0, pol_kv);
+        }
+        if (!mbar_wait(&kv_empty[vs], (static_cast<uint32_t>(j / VST) & 1u) ^ 1u, p.status, kErrAttnProducer)) break;
+        mbar_expect_tx(&v_full[vs], V_BYTES);
+        for (int c = 0; c < DCV; ++c) tma_load_3d(v_sm + vs * V_BYTES + c * SUB_BYTES, &map_v, &v_full[vs], c * 64, hkv, row0, pol_kv);
+      }
+      ok = false;
+    }
     for (int j = 0; j < n_tiles && ok; ++j) {
       const int vstage = j % VST;
       const uint32_t vphase = static_cast<uint32_t>(j / VST) & 1u;
@@ -214,7 +253,7 @@ paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
         for (int c = 0; c < DCV; ++c) tma_load_2d(vd + c * SUB_BYTES, &map_v, &v_full[vstage], c * 64, row0, pol_kv);
       }
       __syncwarp();
-      if (++stage == kTcStages) {
+      if (++stage == KST) {
         stage = 0;
         phase ^= 1u;
       }
@@ -226,8 +265,8 @@ paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
       constexpr uint32_t idesc_pv = umma_idesc_bf16(DV, false, true);         // N = DV, V is MN-major
       bool ok = mbar_wait(q_full, 0, p.status, kErrAttnMma);
       auto issue_qk = [&](int j) -> bool {
-        const int stage = j % kTcStages;
-        const uint32_t kv_phase = static_cast<uint32_t>(j / kTcStages) & 1u;
+        const int stage = j % KST;
+        const uint32_t kv_phase = static_cast<uint32_t>(j / KST) & 1u;
         const int sb = j & 1;
         const uint32_t s_phase = static_cast<uint32_t>(j >> 1) & 1u;
         if (!mbar_wait(&k_full[stage], kv_phase, p.status, kErrAttnMma)) return false;
@@ -297,14 +336,16 @@ paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
       const int key0 = kv_begin + j * kTcKeys;
       // Only tiles that cross the diagonal, the window edge or the end need the mask.
       const bool need_mask = (key0 + kTcKeys - 1 > pos_base + tok0) ||
-                             (p.window > 0 && key0 < pos_base + tok0 + kTcRows - p.window);
+                             (p.window > 0 && key0 < pos_base + tok0 + kTcRows - p.window) ||
+                             (EXT && p.chunk > 0 && key0 < (pos_base + tok0 + rows_valid - 1) / p.chunk * p.chunk);
       const int hkey0 = key0 + half * HC;   // first key of this thread's columns
       int lo = 0, hi = HC;   // valid key columns of this row: [lo, hi)
       if (need_mask) {
         hi = min(HC, qpos - hkey0 + 1);
         if (p.window > 0) lo = max(0, qpos - p.window + 1 - hkey0);
+        if (EXT && p.chunk > 0) lo = max(lo, qpos / p.chunk * p.chunk - hkey0);
       }
-      if constexpr (EXT) {
+      if (EXT && p.bias_r1 != nullptr) {
         // tab[i] = bias of distance base + i, where row r of this warp and key column c are at
         // i = r - c + 63 (log2 domain: the natural logarithm's factor cancels against log2 e)
         const int base = pos_base + tok0 + q4 * 32 - hkey0 - (HC - 1);
@@ -325,7 +366,16 @@ paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
 #pragma unroll
         for (int i = 0; i < 32; ++i) {
           sv[c * 32 + i] = __uint_as_float(r[i]) * p.scale_log2;
-          if constexpr (EXT) sv[c * 32 + i] -= tab[lane + (HC - 1) - (c * 32 + i)];
+        }
+        if constexpr (EXT) {
+          if (p.softcap > 0.f) {
+#pragma unroll
+            for (int i = 0; i < 32; ++i) sv[c * 32 + i] = soft_cap_log2(sv[c * 32 + i], p.softcap);
+          }
+          if (p.bias_r1 != nullptr) {
+#pragma unroll
+            for (int i = 0; i < 32; ++i) sv[c * 32 + i] -= tab[lane + (HC - 1) - (c * 32 + i)];
+          }
         }
       }
       tc_fence_before_sync();
@@ -440,7 +490,7 @@ paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
         l = l * osc + exp2f(sk - m2);
       }
       const float inv = l > 0.f ? osc / l : 0.f;
-      __nv_bfloat16* dst = p.out + static_cast<size_t>(q0 + tok0 + row) * p.Hq * dv + hq * dv;
+      __nv_bfloat16* dst = p.out + static_cast<size_t>(q0 + tok0 + row) * p.out_stride + hq * dv;
 #pragma unroll
       for (int cc = 0; cc < DV / 32 / HALVES; ++cc) {
         const int c = half * (DV / 32 / HALVES) + cc;
@@ -491,10 +541,10 @@ paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
 }
 
 template <int DK, int DV, bool EXT>
-static int launch_prefill_tc(const CUtensorMap& mq, const CUtensorMap& mk, const CUtensorMap& mv,
+static int launch_prefill_tc(const CUtensorMap& mq, const CUtensorMap& mk, const CUtensorMap& mv, const CUtensorMap& mkr,
                              const TcPrefillParams& p, int grid, cudaStream_t stream) {
   constexpr int SUB = 128 * 128;
-  constexpr int smem = (DK / 64) * SUB * (1 + kTcStages) + (DV / 64) * SUB * tc_v_stages(DK, DV, EXT) +
+  constexpr int smem = (DK / 64) * SUB * (1 + tc_k_stages(DK)) + (DV / 64) * SUB * tc_v_stages(DK, DV, EXT) +
                        (EXT ? 4 : 2) * SUB + 1024 + 256 + (EXT ? kExtSmem : 0);
   static_assert(smem <= 227 * 1024, "shared memory");
   auto kern = paged_prefill_tc_kernel<DK, DV, EXT>;
@@ -505,7 +555,7 @@ static int launch_prefill_tc(const CUtensorMap& mq, const CUtensorMap& mk, const
     prefer_max_shared(kern);
     configured = true;
   }
-  return static_cast<int>(launch_kernel(kern, dim3(grid), dim3(tc_threads(EXT)), smem, stream, mq, mk, mv, p));
+  return static_cast<int>(launch_kernel(kern, dim3(grid), dim3(tc_threads(EXT)), smem, stream, mq, mk, mv, mkr, p));
 }
 
 }  // namespace mx
@@ -538,6 +588,7 @@ extern "C" int mx_paged_prefill_tc(const void* q, long long q_stride, const void
   p.Hkv = Hkv;
   p.max_blocks = max_blocks;
   p.window = window;
+  p.out_stride = static_cast<long long>(Hq) * D;
   p.tiles_per_seq = (max_q_len + kTcRows - 1) / kTcRows;
   p.scale_log2 = scale * 1.4426950408889634f;
   const long long grid = static_cast<long long>(num_seqs) * Hq * p.tiles_per_seq;
@@ -551,19 +602,19 @@ extern "C" int mx_paged_prefill_tc(const void* q, long long q_stride, const void
   const uint64_t pool_rows = static_cast<uint64_t>(pool_blocks) * Hkv * kTcBlock;
   if (!make_tensor_map_bf16(&mk, k_pool, pool_rows, D, D, kTcBlock, 64)) return -4;
   if (!make_tensor_map_bf16(&mv, v_pool, pool_rows, D, D, kTcBlock, 64)) return -4;
-  if (D == 64) return launch_prefill_tc<64, 64, false>(mq, mk, mv, p, static_cast<int>(grid), stream);
-  return launch_prefill_tc<128, 128, false>(mq, mk, mv, p, static_cast<int>(grid), stream);
+  if (D == 64) return launch_prefill_tc<64, 64, false>(mq, mk, mv, mv, p, static_cast<int>(grid), stream);
+  return launch_prefill_tc<128, 128, false>(mq, mk, mv, mv, p, static_cast<int>(grid), stream);
 }
 
-// Extended form: key / value rows of Dk / Dv elements (multiples of 8, at most 128), distance bias and
-// output gate optional. Returns -10 when not covered (use mx_paged_attention_any).
+// Extended form: key / value rows of Dk / Dv elements (multiples of 8, at most 128); distance bias, output gate,
+// chunked visibility and soft cap optional (NULL / 0). Returns -10 when not covered (use mx_paged_attention_any).
 extern "C" int mx_paged_prefill_ext(const void* q, long long q_stride, const void* k_pool, const void* v_pool,
                                     long long pool_blocks, const int* block_tables, const int* cu_q,
                                     const int* context_lens, const float* sinks, const float* bias_r1,
                                     const float* bias_r2, const void* gate, long long gate_stride, void* out,
                                     int num_seqs, int total_q, int max_q_len, int Hq, int Hkv, int Dk, int Dv,
-                                    int block_size, int max_blocks, int window, float scale, void* status,
-                                    void* stream_) {
+                                    int block_size, int max_blocks, int window, int chunk, float scale, float softcap,
+                                    void* status, void* stream_) {
   cudaStream_t stream = static_cast<cudaStream_t>(stream_);
   if (num_seqs <= 0 || total_q <= 0) return 0;
   if (Hkv <= 0 || Hq % Hkv || (bias_r1 == nullptr) != (bias_r2 == nullptr)) return -1;
@@ -583,10 +634,13 @@ extern "C" int mx_paged_prefill_ext(const void* q, long long q_stride, const voi
   p.Hkv = Hkv;
   p.max_blocks = max_blocks;
   p.window = window;
+  p.out_stride = static_cast<long long>(Hq) * Dv;
   p.tiles_per_seq = (max_q_len + kTcRows - 1) / kTcRows;
   p.scale_log2 = scale * 1.4426950408889634f;
   p.dk = Dk;
   p.dv = Dv;
+  p.chunk = chunk;
+  p.softcap = softcap;
   p.bias_r1 = bias_r1;
   p.bias_r2 = bias_r2;
   p.gate = static_cast<const __nv_bfloat16*>(gate);
@@ -603,8 +657,54 @@ extern "C" int mx_paged_prefill_ext(const void* q, long long q_stride, const voi
   if (!make_tensor_map_bf16(&mv, v_pool, pool_rows, Dv, Dv, kTcBlock, 64)) return -4;
   const int g = static_cast<int>(grid);
   if (Dk <= 64)
-    return Dv <= 64 ? launch_prefill_tc<64, 64, true>(mq, mk, mv, p, g, stream)
-                    : launch_prefill_tc<64, 128, true>(mq, mk, mv, p, g, stream);
-  return Dv <= 64 ? launch_prefill_tc<128, 64, true>(mq, mk, mv, p, g, stream)
-                  : launch_prefill_tc<128, 128, true>(mq, mk, mv, p, g, stream);
+    return Dv <= 64 ? launch_prefill_tc<64, 64, true>(mq, mk, mv, mv, p, g, stream)
+                    : launch_prefill_tc<64, 128, true>(mq, mk, mv, mv, p, g, stream);
+  return Dv <= 64 ? launch_prefill_tc<128, 64, true>(mq, mk, mv, mv, p, g, stream)
+                  : launch_prefill_tc<128, 128, true>(mq, mk, mv, mv, p, g, stream);
+}
+
+// Latent attention over expanded rows: keys [k_nope (Dn) | shared rotated part (R)], values Dv wide. Sequence s owns query
+// rows [cu_q[s], cu_q[s + 1]) of q (rows of heads of Dn + R elements), the last of its context_lens[s] tokens; its
+// context lies in rows kv_starts[s] .. of kn [kv_rows, H * Dn], kr (rows kr_stride apart, R used) and v [kv_rows, H * Dv].
+// Output rows are out_stride elements apart. -10 = not covered.
+extern "C" int mx_latent_prefill(const void* q, long long q_stride, const void* kn, const void* kr, long long kr_stride,
+                                 const void* v, long long kv_rows, const int* cu_q, const int* context_lens,
+                                 const int* kv_starts, void* out, long long out_stride, int num_seqs, int total_q,
+                                 int max_q_len, int H, int Dn, int R, int Dv, float scale, void* status, void* stream_) {
+  cudaStream_t stream = static_cast<cudaStream_t>(stream_);
+  if (num_seqs <= 0 || total_q <= 0) return 0;
+  if (H <= 0 || kv_rows <= 0) return -1;
+  const auto al16 = [](const void* a) { return (reinterpret_cast<uintptr_t>(a) & 15) == 0; };
+  if (Dn % 8 || R % 8 || Dv % 8 || Dn <= 0 || Dn > 128 || R <= 0 || R > 64 || Dv <= 0 || Dv > 128 || q_stride % 8 || kr_stride % 8 ||
+      out_stride % 8 || !al16(q) || !al16(kn) || !al16(kr) || !al16(v) || !al16(out))
+    return -10;
+  TcPrefillParams p{};
+  p.cu_q = cu_q;
+  p.context_lens = context_lens;
+  p.out = static_cast<__nv_bfloat16*>(out);
+  p.status = static_cast<int*>(status);
+  p.num_seqs = num_seqs;
+  p.Hq = p.Hkv = H;
+  p.tiles_per_seq = (max_q_len + kTcRows - 1) / kTcRows;
+  p.scale_log2 = scale * 1.4426950408889634f;
+  p.dk = Dn + R;
+  p.dv = Dv;
+  p.kv_starts = kv_starts;
+  p.kv_split = Dn;
+  p.out_stride = out_stride;
+  const long long grid = static_cast<long long>(num_seqs) * H * p.tiles_per_seq;
+  if (grid > 0x7fffffffll) return -1;
+  // a query box of the unrotated part may run into the rotated columns: the keys' columns there are zero
+  CUtensorMap mq, mk, mv, mkr;
+  if (!make_tensor_map_bf16_3d(&mq, q, total_q, H, Dn + R, q_stride, Dn + R, kTcRows, 64) ||
+      !make_tensor_map_bf16_3d(&mk, kn, kv_rows, H, Dn, static_cast<uint64_t>(H) * Dn, Dn, kTcKeys, 64) ||
+      !make_tensor_map_bf16_3d(&mv, v, kv_rows, H, Dv, static_cast<uint64_t>(H) * Dv, Dv, kTcKeys, 64) ||
+      !make_tensor_map_bf16(&mkr, kr, kv_rows, R, kr_stride, kTcKeys, 64))
+    return -4;
+  const int g = static_cast<int>(grid);
+  if (Dn <= 64)
+    return Dv <= 64 ? launch_prefill_tc<128, 64, true>(mq, mk, mv, mkr, p, g, stream)
+                    : launch_prefill_tc<128, 128, true>(mq, mk, mv, mkr, p, g, stream);
+  return Dv <= 64 ? launch_prefill_tc<192, 64, true>(mq, mk, mv, mkr, p, g, stream)
+                  : launch_prefill_tc<192, 128, true>(mq, mk, mv, mkr, p, g, stream);
 }

@@ -277,6 +277,12 @@ __device__ __forceinline__ float warp_max(float v) {
   for (int o = 16; o > 0; o >>= 1) v = fmaxf(v, __shfl_xor_sync(0xffffffffu, v, o));
   return v;
 }
+// Soft-capped score in log2 units: v = s log2(e) -> cap tanh(s / cap) log2(e), through tanh(z) = 1 - 2 / (1 + e^2z)
+// (absolute error near 1e-7 cap, which is what a softmax argument needs).
+__device__ __forceinline__ float soft_cap_log2(float v, float cap) {
+  const float t = exp2f(v * (2.0f / cap));
+  return cap * 1.4426950408889634f * (1.0f - __fdividef(2.0f, 1.0f + t));
+}
 __device__ __forceinline__ void named_bar_sync(int id, int nthreads) {
   asm volatile("bar.sync %0, %1;" ::"r"(id), "r"(nthreads) : "memory");
 }

@@ -144,6 +144,9 @@ struct GemmParams {
   int num_groups;
   int w_group_rows;
   int bias_group_stride;
+  // batched mode (group_offsets == NULL): every group multiplies all M rows, group g the columns
+  // [g * x_group_cols, + K) of x into the output columns [g * out_group_cols, + N)
+  int x_group_cols, out_group_cols;
 };
 
 // One unit of work of the persistent tile loop, in tensor-map coordinates and output indices.
@@ -154,6 +157,7 @@ struct WorkItem {
   int feat0, feat_valid;     // first output feature of the tile and how many are real
   int bias_off;
   int q_tile;                // quantized weights: index of the lane tile in the re-tiled blocks
+  int x_col0, out_col0;      // batched: first column of the group in x and in the output
 };
 struct GroupCursor {
   int e = 0, base = 0;
@@ -203,8 +207,9 @@ __device__ __forceinline__ bool decode_work(const GemmParams& p, int w, GroupCur
     constexpr int FEAT_TILE = SWAP ? kLaneRows : BN;
     const int F = (p.N + FEAT_TILE - 1) / FEAT_TILE;
     const int f = w % F, g = w / F;
+    const bool batched = p.group_offsets == nullptr;
     while (cur.e < p.num_groups) {
-      const int rows = p.group_offsets[cur.e + 1] - p.group_offsets[cur.e];
+      const int rows = batched ? p.M : p.group_offsets[cur.e + 1] - p.group_offsets[cur.e];
       const int cnt = (rows + TOK_TILE - 1) / TOK_TILE;
       if (g < cur.base + cnt) break;
       cur.base += cnt;
@@ -214,8 +219,10 @@ __device__ __forceinline__ bool decode_work(const GemmParams& p, int w, GroupCur
     const int e = cur.e;
     it.tile = w;
     it.split = 0;
-    it.out_tok0 = p.group_offsets[e] + (g - cur.base) * TOK_TILE;
-    it.tok_valid = p.group_offsets[e + 1] - it.out_tok0;
+    it.out_tok0 = (batched ? 0 : p.group_offsets[e]) + (g - cur.base) * TOK_TILE;
+    it.tok_valid = (batched ? p.M : p.group_offsets[e + 1]) - it.out_tok0;
+    it.x_col0 = e * p.x_group_cols;       // (both strides are 0 outside the batched mode)
+    it.out_col0 = e * p.out_group_cols;
     it.feat0 = f * FEAT_TILE;
     it.feat_valid = p.N - it.feat0;
     it.bias_off = e * p.bias_group_stride;
@@ -472,7 +479,7 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap map_lane,
   // producer state set up by thread 0 before the CTA-wide sync (it is also the producer thread)
   [[maybe_unused]] uint64_t pol_lane = 0, pol_col = 0;
   [[maybe_unused]] int pre = 0;   // ring stages whose weight tiles are already in flight
-  auto load_lane = [&](uint8_t* s, uint64_t* bar, int kb, int row0, [[maybe_unused]] int qtile) {
+  auto load_lane = [&](uint8_t* s, uint64_t* bar, int kb, int row0, [[maybe_unused]] int qtile, int col0) {
     if constexpr (WQ != 0) {
       // packed bytes of 128 weight rows for this k-block (byte-typed tensor map, no swizzle)
       // The packed weights were re-tiled at load time: (128-row tile, k-block) -> one contiguous
@@ -485,18 +492,18 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap map_lane,
       if (LANE_TILES == 2)
         tma_load_2d(pk + PK_BYTES, &map_lane, bar, 0, ((qtile + p.q_glu_tiles) * p.num_kb + kb) * BOX_ROWS, pol_lane);
     } else {
-      tma_load_2d(s, &map_lane, bar, kb * kBK, row0, pol_lane);
-      if (LANE_TILES == 2) tma_load_2d(s + LANE_BYTES, &map_lane, bar, kb * kBK, row0 + p.glu_offset, pol_lane);
+      tma_load_2d(s, &map_lane, bar, col0 + kb * kBK, row0, pol_lane);
+      if (LANE_TILES == 2) tma_load_2d(s + LANE_BYTES, &map_lane, bar, col0 + kb * kBK, row0 + p.glu_offset, pol_lane);
     }
   };
   // barrier the TMA loads of a stage complete on: the MMA's when the tile is ready as loaded,
   // the transform warps' when the weights still have to be dequantised
   auto load_bar = [&](int stage) -> uint64_t* { return WQ != 0 ? &raw_full[stage] : &full_bar[stage]; };
   constexpr int TX_BYTES = WQ != 0 ? RAW_BYTES : LANE_TILES * LANE_BYTES + COL_TILES * COL_BYTES;
-  auto load_col = [&](uint8_t* s, uint64_t* bar, int kb, int row0) {
+  auto load_col = [&](uint8_t* s, uint64_t* bar, int kb, int row0, int col0) {
     uint8_t* sc = s + LANE_TILES * LANE_BYTES;
-    tma_load_2d(sc, &map_col, bar, kb * kBK, row0, pol_col);
-    if (COL_TILES == 2) tma_load_2d(sc + COL_BYTES, &map_col, bar, kb * kBK, row0 + p.glu_offset, pol_col);
+    tma_load_2d(sc, &map_col, bar, col0 + kb * kBK, row0, pol_col);
+    if (COL_TILES == 2) tma_load_2d(sc + COL_BYTES, &map_col, bar, col0 + kb * kBK, row0 + p.glu_offset, pol_col);
   };
   if (threadIdx.x == 0) {
     stamp(0);
@@ -530,8 +537,8 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap map_lane,
         for (int i = 0; i < pre; ++i) {
           mbar_expect_tx(load_bar(i), TX_BYTES);
           uint8_t* s = smem + i * STAGE_BYTES;
-          if (SWAP) load_lane(s, load_bar(i), kb0 + i, it0.lane_row0, it0.q_tile);
-          else load_col(s, load_bar(i), kb0 + i, it0.col_row0);
+          if (SWAP) load_lane(s, load_bar(i), kb0 + i, it0.lane_row0, it0.q_tile, 0);
+          else load_col(s, load_bar(i), kb0 + i, it0.col_row0, 0);
         }
         // The rest of this CTA's weight slice (up to a budget) goes to L2: HBM keeps streaming
         // through the previous kernels' epilogues and the small kernels in between, and the
@@ -612,20 +619,22 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap map_lane,
         const int kb0 = it.split * p.kb_per_split;
         const int kb1 = min(p.num_kb, kb0 + p.kb_per_split);
         const int lane_row0 = it.lane_row0, col_row0 = it.col_row0;
+        const int x_col0 = GROUPED ? it.x_col0 : 0;
+        const int lane_c0 = SWAP ? 0 : x_col0, col_c0 = SWAP ? x_col0 : 0;
         for (int kb = kb0; kb < kb1; ++kb, ++seq) {
           uint8_t* s = smem + stage * STAGE_BYTES;
           if (seq < pre) {
             // weight tile already in flight: only the activation tile is missing
-            if (SWAP) load_col(s, load_bar(stage), kb, col_row0);
-            else load_lane(s, load_bar(stage), kb, lane_row0, it.q_tile);
+            if (SWAP) load_col(s, load_bar(stage), kb, col_row0, col_c0);
+            else load_lane(s, load_bar(stage), kb, lane_row0, it.q_tile, lane_c0);
           } else {
             if (!mbar_wait(&empty_bar[stage], phase ^ 1u, p.status, kErrProducerWait)) {
               ok = false;
               break;
             }
             mbar_expect_tx(load_bar(stage), TX_BYTES);
-            load_lane(s, load_bar(stage), kb, lane_row0, it.q_tile);
-            load_col(s, load_bar(stage), kb, col_row0);
+            load_lane(s, load_bar(stage), kb, lane_row0, it.q_tile, lane_c0);
+            load_col(s, load_bar(stage), kb, col_row0, col_c0);
           }
           if (seq == 0) stamp(2);
           if (++stage == p.stages) {
@@ -980,6 +989,7 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap map_lane,
           }
         };
         auto store_out = [&](size_t off, const float(&o)[8]) {
+          if constexpr (GROUPED) off += it.out_col0;
           if (p.out_fp32) {
             float* dst = reinterpret_cast<float*>(p.out) + off;
             if (vec) {
@@ -1346,7 +1356,7 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap map_lane,
                     ssq_acc += r * r;
                   }
                 }
-                const size_t off = static_cast<size_t>(m) * p.ldo + n;
+                const size_t off = static_cast<size_t>(m) * p.ldo + n + (GROUPED ? it.out_col0 : 0);
                 if (p.out_fp32) {
                   float* dst = reinterpret_cast<float*>(p.out) + off;
                   if (full8 && ((off & 3) == 0)) {
@@ -1587,6 +1597,21 @@ bool make_tensor_map_bf16(CUtensorMap* out, const void* ptr, uint64_t rows, uint
   if (cache.size() > 65536) cache.clear();
   cache.emplace(key, *out);
   return true;
+}
+
+// 3-D view [rows][groups][cols] of bf16 (row stride ld, group stride group_ld elements); box {box_cols, 1, box_rows}.
+// Columns past `cols` of a group arrive as zeros, not as the next group's.
+bool make_tensor_map_bf16_3d(CUtensorMap* out, const void* ptr, uint64_t rows, uint64_t groups, uint64_t cols, uint64_t ld,
+                             uint64_t group_ld, uint32_t box_rows, uint32_t box_cols) {
+  EncodeTiledFn enc = get_encode_fn();
+  if (enc == nullptr) return false;
+  cuuint64_t gdim[3] = {cols, groups, rows};
+  cuuint64_t gstride[2] = {group_ld * 2, ld * 2};
+  cuuint32_t box[3] = {box_cols, 1, box_rows};
+  cuuint32_t estr[3] = {1, 1, 1};
+  return enc(out, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 3, const_cast<void*>(ptr), gdim, gstride, box, estr,
+             CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B,
+             CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) == CUDA_SUCCESS;
 }
 
 // 2-D byte tensor [rows, row_bytes] with row stride ld_bytes; box {box_bytes (inner, multiple of
@@ -2086,6 +2111,54 @@ extern "C" int mx_gemm_comm(const void* x, const void* w, void* out, const void*
   return launch_gemm<128, false, false, 2>(ml, mc, p, grid, stream);
 }
 
+
+// Batched GEMM with block-diagonal weights (one matrix per head): for every group g < G
+//   out[m, g * out_group_cols + n] = sum_k x[m, g * x_group_cols + k] w[g, n, k]      ([G, N, K] contiguous)
+// on the grouped kernel: all groups have the same M rows, the tile schedule needs nothing from the device. K, N and all
+// strides multiples of 8 (-10 otherwise: use mx_batched_gemm_any).
+extern "C" int mx_batched_gemm_bf16(const void* x, const void* w, void* out, int G, int M, int N, int K, int ldx,
+                                    int x_group_cols, int ldo, int out_group_cols, void* workspace, long long ws_bytes,
+                                    void* stream_) {
+  cudaStream_t stream = static_cast<cudaStream_t>(stream_);
+  if (G <= 0 || M <= 0 || N <= 0) return 0;
+  if (K <= 0) return -1;
+  if (K % 8 || N % 8 || ldx % 8 || x_group_cols % 8 || ldo % 8 || out_group_cols % 8 || (reinterpret_cast<uintptr_t>(x) & 15) ||
+      (reinterpret_cast<uintptr_t>(w) & 15) || (reinterpret_cast<uintptr_t>(out) & 15))
+    return -10;
+  if (workspace == nullptr || ws_bytes < MX_WS_PARTIAL_OFFSET) return -2;
+  GemmParams p{};
+  p.out = out;
+  p.status = reinterpret_cast<int*>(static_cast<uint8_t*>(workspace) + MX_WS_STATUS_OFFSET);
+  p.counters = reinterpret_cast<int*>(static_cast<uint8_t*>(workspace) + MX_WS_COUNTER_OFFSET);
+  p.partials = reinterpret_cast<float*>(static_cast<uint8_t*>(workspace) + MX_WS_PARTIAL_OFFSET);
+  p.M = M;
+  p.N = N;
+  p.K = K;
+  p.ldo = ldo;
+  p.epilogue = MX_EPI_NONE;
+  p.num_kb = (K + kBK - 1) / kBK;
+  p.splits = 1;
+  p.kb_per_split = p.num_kb;
+  p.num_groups = G;
+  p.w_group_rows = N;
+  p.x_group_cols = x_group_cols;
+  p.out_group_cols = out_group_cols;
+  const bool swap = M <= 96;
+  const int bn = swap ? (M <= 16 ? 16 : M <= 32 ? 32 : 64) : (N > 128 ? 256 : 128);
+  CUtensorMap map_x, map_w;
+  if (!make_tensor_map_bf16(&map_x, x, M, static_cast<uint64_t>(G - 1) * x_group_cols + K, ldx, swap ? bn : kLaneRows, kBK)) return -4;
+  if (!make_tensor_map_bf16(&map_w, w, static_cast<uint64_t>(G) * N, K, K, swap ? kLaneRows : bn, kBK)) return -4;
+  const CUtensorMap& ml = swap ? map_w : map_x;
+  const CUtensorMap& mc = swap ? map_x : map_w;
+  const int grid = device_sm_count();
+  if (swap) {
+    if (bn == 16) return launch_gemm<16, true, false, 0, true>(ml, mc, p, grid, stream);
+    if (bn == 32) return launch_gemm<32, true, false, 0, true>(ml, mc, p, grid, stream);
+    return launch_gemm<64, true, false, 0, true>(ml, mc, p, grid, stream);
+  }
+  if (bn == 256) return launch_gemm<256, false, false, 0, true>(ml, mc, p, grid, stream);
+  return launch_gemm<128, false, false, 0, true>(ml, mc, p, grid, stream);
+}
 
 // Grouped (per-expert) GEMM: rows [off[e], off[e+1]) of x are multiplied by expert e's weight
 // matrix w[e] ([E, N or 2N, K] contiguous) with the same tcgen05 kernel; the tile schedule is

@@ -1,10 +1,11 @@
 // Shape-agnostic SIMT kernels with fp32 arithmetic, for fp32 models and for sizes the tensor-core
 // kernels do not cover (row strides that are not a multiple of 16 bytes, head widths other than
 // multiples of 8 up to 128):
-//   gemm_any       out[M, N] = x[M, K] w[N, K]^T (+ bias) (+ residual), operands bf16 or fp32
+//   gemm_any       out[M, N] = x[M, K] w[N, K]^T (+ bias) (+ residual), operands bf16 or fp32; optionally a batch of such
+//                  products at constant strides (block-diagonal weights)
 //   attention_any  causal paged attention of any query rows (decode rows are pieces of one token):
-//                  sliding window, sinks, logarithmic distance bias, output gate, key and value heads of
-//                  different width
+//                  sliding window, chunks, soft cap, sinks, logarithmic distance bias, output gate, key and value heads
+//                  of different width (which may lie in rows wider than they are)
 #include "api.h"
 #include "typed.cuh"
 
@@ -17,11 +18,12 @@ template <typename T, typename TO>
 __global__ void __launch_bounds__(kGaThreads)
 gemm_any_kernel(const T* __restrict__ x, const T* __restrict__ w, TO* __restrict__ out, const T* __restrict__ bias,
                 const T* __restrict__ residual, int M, int N, int K, long long ldx, long long ldw, long long ldo,
-                long long ldr) {
+                long long ldr, long long bx, long long bw, long long bo) {
   __shared__ __align__(16) float xs[kGaK][kGaTile + 4];
   __shared__ __align__(16) float ws[kGaK][kGaTile + 4];
   pdl_trigger();
   pdl_wait();
+  x += blockIdx.z * bx, w += blockIdx.z * bw, out += blockIdx.z * bo;
   const int m0 = blockIdx.y * kGaTile, n0 = blockIdx.x * kGaTile;
   const int tm = (threadIdx.x / 16) * 4, tn = (threadIdx.x % 16) * 4;
   float acc[4][4];
@@ -92,8 +94,8 @@ struct AnyAttnParams {
   const void* gate;        // the output is multiplied by sigmoid(gate)
   long long gate_stride;
   void* out;
-  int num_seqs, Hq, Hkv, Dk, Dv, block_size, max_blocks, window;
-  float scale;
+  int num_seqs, Hq, Hkv, Dk, Dv, ldk, ldv, block_size, max_blocks, window, chunk;   // ldk / ldv: elements of a pool row
+  float scale, softcap;
 };
 
 // One CTA per (query row, query head). The warps take the 32-key chunks in turn: scores with one key
@@ -123,11 +125,12 @@ attention_any_kernel(const AnyAttnParams p) {
   const T* q = static_cast<const T*>(p.q) + static_cast<size_t>(row) * p.q_stride + static_cast<size_t>(h) * p.Dk;
   for (int i = threadIdx.x; i < p.Dk; i += blockDim.x) q_s[i] = to_f(q[i]);
   __syncthreads();
-  const int first = (p.window > 0 && pos + 1 > p.window) ? pos + 1 - p.window : 0;
+  int first = (p.window > 0 && pos + 1 > p.window) ? pos + 1 - p.window : 0;
+  if (p.chunk > 0) first = max(first, pos / p.chunk * p.chunk);
   const float r1 = p.r1 != nullptr ? p.r1[h] : 0.f, r2 = p.r1 != nullptr ? p.r2[h] : 0.f;
   const T* kp = static_cast<const T*>(p.k_pool);
   const T* vp = static_cast<const T*>(p.v_pool);
-  const bool vec = p.Dk % 4 == 0;
+  const bool vec = p.Dk % 4 == 0 && p.ldk % 4 == 0;
   float m = -INFINITY, l = 0.f, acc[NV];
 #pragma unroll
   for (int i = 0; i < NV; ++i) acc[i] = 0.f;
@@ -139,7 +142,7 @@ attention_any_kernel(const AnyAttnParams p) {
     if (ok) {
       const int blk = table[key / p.block_size];
       prow = (static_cast<long long>(blk) * p.Hkv + hk) * p.block_size + key % p.block_size;
-      const T* kr = kp + prow * p.Dk;
+      const T* kr = kp + prow * p.ldk;
       float d = 0.f;
       if (vec) {
         float e[4] = {0.f, 0.f, 0.f, 0.f};
@@ -154,6 +157,7 @@ attention_any_kernel(const AnyAttnParams p) {
         for (int i = 0; i < p.Dk; ++i) d = fmaf(to_f(kr[i]), q_s[i], d);
       }
       sc = d * p.scale;
+      if (p.softcap > 0.f) sc = p.softcap * tanhf(sc / p.softcap);
       if (p.r1 != nullptr) sc -= r1 * log1pf(r2 * static_cast<float>(pos - key));
     }
     const float mn = fmaxf(m, warp_max(sc));
@@ -166,7 +170,7 @@ attention_any_kernel(const AnyAttnParams p) {
     const int nk = min(32, pos + 1 - c0);
     for (int t = 0; t < nk; ++t) {
       const float pt = __shfl_sync(0xffffffffu, pr, t);
-      const T* vr = vp + __shfl_sync(0xffffffffu, prow, t) * p.Dv;
+      const T* vr = vp + __shfl_sync(0xffffffffu, prow, t) * p.ldv;
 #pragma unroll
       for (int i = 0; i < NV; ++i) {
         const int d = lane + 32 * i;
@@ -219,23 +223,36 @@ static int launch_attention_any(const AnyAttnParams& p, int rows, cudaStream_t s
 
 using namespace mx;
 
-// fp32: operands fp32 (else bf16); out_fp32: result fp32 (implied by fp32 operands).
-extern "C" int mx_gemm_any(const void* x, const void* w, void* out, const void* bias, const void* residual, int M, int N,
-                           int K, long long ldx, long long ldw, long long ldo, long long ldr, int fp32, int out_fp32,
-                           void* stream) {
-  if (M <= 0 || N <= 0) return 0;
+static int gemm_any(const void* x, const void* w, void* out, const void* bias, const void* residual, int M, int N, int K,
+                    long long ldx, long long ldw, long long ldo, long long ldr, int batch, long long bx, long long bw, long long bo,
+                    int fp32, int out_fp32, void* stream) {
+  if (M <= 0 || N <= 0 || batch <= 0) return 0;
   const int gy = (M + kGaTile - 1) / kGaTile;
-  if (K <= 0 || gy > 65535) return -1;
-  const dim3 grid((N + kGaTile - 1) / kGaTile, gy), block(kGaThreads);
+  if (K <= 0 || gy > 65535 || batch > 65535) return -1;
+  const dim3 grid((N + kGaTile - 1) / kGaTile, gy, batch), block(kGaThreads);
   auto st = static_cast<cudaStream_t>(stream);
 #define MX_GA(T, TO)                                                                                                   \
   return static_cast<int>(launch_kernel(gemm_any_kernel<T, TO>, grid, block, 0, st, static_cast<const T*>(x),         \
                                         static_cast<const T*>(w), static_cast<TO*>(out), static_cast<const T*>(bias), \
-                                        static_cast<const T*>(residual), M, N, K, ldx, ldw, ldo, ldr))
+                                        static_cast<const T*>(residual), M, N, K, ldx, ldw, ldo, ldr, bx, bw, bo))
   if (fp32) MX_GA(float, float);
   if (out_fp32) MX_GA(__nv_bfloat16, float);
   MX_GA(__nv_bfloat16, __nv_bfloat16);
 #undef MX_GA
+}
+
+// fp32: operands fp32 (else bf16); out_fp32: result fp32 (implied by fp32 operands).
+extern "C" int mx_gemm_any(const void* x, const void* w, void* out, const void* bias, const void* residual, int M, int N,
+                           int K, long long ldx, long long ldw, long long ldo, long long ldr, int fp32, int out_fp32,
+                           void* stream) {
+  return gemm_any(x, w, out, bias, residual, M, N, K, ldx, ldw, ldo, ldr, 1, 0, 0, 0, fp32, out_fp32, stream);
+}
+
+// `batch` products whose operands and results lie bx / bw / bo elements apart.
+extern "C" int mx_batched_gemm_any(const void* x, const void* w, void* out, int batch, int M, int N, int K, long long ldx,
+                                   long long ldw, long long ldo, long long bx, long long bw, long long bo, int fp32,
+                                   void* stream) {
+  return gemm_any(x, w, out, nullptr, nullptr, M, N, K, ldx, ldw, ldo, 0, batch, bx, bw, bo, fp32, 0, stream);
 }
 
 // Query row r of sequence s (cu_q[s] <= r < cu_q[s + 1]) is token context_lens[s] - (cu_q[s + 1] - r) of
@@ -244,14 +261,16 @@ extern "C" int mx_paged_attention_any(const void* q, long long q_stride, const v
                                       const void* block_tables, const void* cu_q, const void* context_lens,
                                       const void* sinks, const void* r1, const void* r2, const void* gate,
                                       long long gate_stride, void* out, int num_seqs, int rows, int Hq, int Hkv, int Dk,
-                                      int Dv, int block_size, int max_blocks, int window, float scale, int fp32,
-                                      void* stream) {
+                                      int Dv, int ldk, int ldv, int block_size, int max_blocks, int window, int chunk,
+                                      float scale, float softcap, int fp32, void* stream) {
   if (num_seqs <= 0 || rows <= 0) return 0;
-  if (Hkv <= 0 || Hq % Hkv || Hq > 65535 || Dk <= 0 || Dv <= 0 || (r1 == nullptr) != (r2 == nullptr)) return -1;
+  if (Hkv <= 0 || Hq % Hkv || Hq > 65535 || Dk <= 0 || Dv <= 0 || ldk < Dk || ldv < Dv ||
+      (r1 == nullptr) != (r2 == nullptr))
+    return -1;
   AnyAttnParams p{q, q_stride, k_pool, v_pool, static_cast<const int*>(block_tables), static_cast<const int*>(cu_q),
                   static_cast<const int*>(context_lens), static_cast<const float*>(sinks), static_cast<const float*>(r1),
-                  static_cast<const float*>(r2), gate, gate_stride, out, num_seqs, Hq, Hkv, Dk, Dv, block_size,
-                  max_blocks, window, scale};
+                  static_cast<const float*>(r2), gate, gate_stride, out, num_seqs, Hq, Hkv, Dk, Dv, ldk, ldv,
+                  block_size, max_blocks, window, chunk, scale, softcap};
   auto st = static_cast<cudaStream_t>(stream);
   return fp32 ? launch_attention_any<float>(p, rows, st) : launch_attention_any<__nv_bfloat16>(p, rows, st);
 }

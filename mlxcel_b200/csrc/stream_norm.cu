@@ -1,8 +1,10 @@
 // Row kernels of layers that keep the residual stream in fp32 and normalise on both sides of a
 // sub-layer, each for bf16 and fp32 activations:
-//   embed_stream   h = scale * table[id];  x = norm(h)
-//   stream_norm    h += norm(y) * layer scale;  x = norm(h)     (either half optional)
+//   embed_stream   h = scale * table[id], optionally normalised itself;  x = norm(h) or h as it is
+//   stream_norm    h += norm(y) * layer scale;  x = norm(h) or h as it is     (either half optional)
 //   polynorm       a N(z) + b N(z^2) + c N(z^3) + e, N = division by the row's root mean square
+//   glu_rows       gated activation of rows gate | up (SwiGLU, tanh-GeGLU, clipped SwiGLU)
+//   softcap_rows   x <- cap tanh(x / cap) in fp32, in place
 //   qk_norm_append per-head RMS norm of q and k, k and v rows into the paged pool (key and value heads
 //                  may differ in width; no rotation)
 // A norm weight w acts as (w_bias + w); all norm weights and layer scales are fp32 vectors, all
@@ -62,6 +64,14 @@ stream_norm_kernel(const T* __restrict__ y, float* __restrict__ h, const int* __
     }
   }
   if (x == nullptr) return;
+  if (pre_w == nullptr) {                  // the sub-layer reads the stream itself
+#pragma unroll
+    for (int i = 0; i < VPT; ++i) {
+      const int c = (threadIdx.x + i * blockDim.x) * V;
+      if (c < dim) store_v<V>(x + row * dim + c, hv[i]);
+    }
+    return;
+  }
 #pragma unroll
   for (int i = 0; i < VPT; ++i) {
     const int c = (threadIdx.x + i * blockDim.x) * V;
@@ -88,8 +98,8 @@ stream_norm_kernel(const T* __restrict__ y, float* __restrict__ h, const int* __
 template <typename T, int V, int VPT>
 __global__ void __launch_bounds__(1024)
 embed_stream_kernel(const int* __restrict__ ids, const T* __restrict__ table, float* __restrict__ h,
-                    const float* __restrict__ pre_w, T* __restrict__ x, int dim, int vocab, float scale, float eps,
-                    float w_bias) {
+                    const float* __restrict__ own_w, const float* __restrict__ pre_w, T* __restrict__ x, int dim, int vocab,
+                    float scale, float eps, float w_bias) {
   __shared__ float red[33];
   pdl_trigger();
   pdl_wait();
@@ -109,8 +119,36 @@ embed_stream_kernel(const int* __restrict__ ids, const T* __restrict__ table, fl
         hv[i][e] = ok ? hv[i][e] * scale : 0.f;
         s[0] += hv[i][e] * hv[i][e];
       }
-      store_v<V>(h + row * dim + c, hv[i]);
+      if (own_w == nullptr) store_v<V>(h + row * dim + c, hv[i]);
     }
+  }
+  if (own_w != nullptr) {                  // the stream starts from the normalised embedding
+    block_sums<1>(s, red);
+    const float r = 1.f / sqrtf(s[0] / dim + eps);
+    s[0] = 0.f;
+#pragma unroll
+    for (int i = 0; i < VPT; ++i) {
+      const int c = (threadIdx.x + i * blockDim.x) * V;
+      if (c < dim) {
+        float w[V];
+        load_v<V>(own_w + c, w);
+#pragma unroll
+        for (int e = 0; e < V; ++e) {
+          hv[i][e] = hv[i][e] * r * (w_bias + w[e]);
+          s[0] += hv[i][e] * hv[i][e];
+        }
+        store_v<V>(h + row * dim + c, hv[i]);
+      }
+    }
+  }
+  if (x == nullptr) return;
+  if (pre_w == nullptr) {
+#pragma unroll
+    for (int i = 0; i < VPT; ++i) {
+      const int c = (threadIdx.x + i * blockDim.x) * V;
+      if (c < dim) store_v<V>(x + row * dim + c, hv[i]);
+    }
+    return;
   }
   block_sums<1>(s, red);
   const float r = 1.f / sqrtf(s[0] / dim + eps);
@@ -163,6 +201,44 @@ polynorm_kernel(const T* __restrict__ z, const float* __restrict__ coef, T* __re
       store_v<V>(out + row * dim + c, o);
     }
   }
+}
+
+// Gated activation of rows gate [dim] | up [dim], `ld` elements apart; mode as MX_EPI_SWIGLU / GEGLU / CLIPPED_SWIGLU.
+template <typename T, int V>
+__global__ void __launch_bounds__(256)
+glu_rows_kernel(const T* __restrict__ z, long long ld, T* __restrict__ out, int dim, int mode, float alpha, float limit) {
+  pdl_trigger();
+  pdl_wait();
+  const size_t row = blockIdx.x;
+  const int c = (blockIdx.y * blockDim.x + threadIdx.x) * V;
+  if (c >= dim) return;
+  float g[V], u[V];
+  load_v<V>(z + row * ld + c, g);
+  load_v<V>(z + row * ld + dim + c, u);
+#pragma unroll
+  for (int e = 0; e < V; ++e) {
+    float a = g[e], b = u[e];
+    if (mode == MX_EPI_GEGLU) {
+      g[e] = 0.5f * a * (1.f + tanhf(0.7978845608028654f * (a + 0.044715f * a * a * a))) * b;
+    } else {
+      float k = 1.f;
+      if (mode == MX_EPI_CLIPPED_SWIGLU) {
+        a = fminf(a, limit);
+        b = fminf(fmaxf(b, -limit), limit) + 1.f;
+        k = alpha;
+      }
+      g[e] = a * sigmoid_f(k * a) * b;
+    }
+  }
+  store_v<V>(out + row * dim + c, g);
+}
+
+__global__ void __launch_bounds__(256) softcap_rows_kernel(float* __restrict__ x, long long n, float cap) {
+  pdl_trigger();
+  pdl_wait();
+  const float inv = 1.f / cap;
+  for (long long i = static_cast<long long>(blockIdx.x) * blockDim.x + threadIdx.x; i < n; i += static_cast<long long>(gridDim.x) * blockDim.x)
+    x[i] = cap * tanhf(x[i] * inv);
 }
 
 // Rows of q | k | v (| more), `ld` elements apart. One CTA per token; a warp takes every eighth of the Hq
@@ -287,15 +363,15 @@ static int stream_norm_typed(const void* y, void* h, const void* rows, const flo
 }
 
 template <typename T>
-static int embed_stream_typed(const int* ids, const void* table, void* h, const float* pre_w, void* x, int n, int dim, int vocab,
+static int embed_stream_typed(const int* ids, const void* table, void* h, const float* own_w, const float* pre_w, void* x, int n, int dim, int vocab,
                               float scale, float eps, float w_bias, bool vec, cudaStream_t st) {
   const T* tp = static_cast<const T*>(table);
   if (vec) {
     const RowShape sh = row_shape(dim, 4);
-    MX_ROW_DISPATCH(embed_stream_kernel, T, 4, sh, n, st, ids, tp, static_cast<float*>(h), pre_w, static_cast<T*>(x), dim, vocab, scale, eps, w_bias)
+    MX_ROW_DISPATCH(embed_stream_kernel, T, 4, sh, n, st, ids, tp, static_cast<float*>(h), own_w, pre_w, static_cast<T*>(x), dim, vocab, scale, eps, w_bias)
   }
   const RowShape sh = row_shape(dim, 1);
-  MX_ROW_DISPATCH(embed_stream_kernel, T, 1, sh, n, st, ids, tp, static_cast<float*>(h), pre_w, static_cast<T*>(x), dim, vocab, scale, eps, w_bias)
+  MX_ROW_DISPATCH(embed_stream_kernel, T, 1, sh, n, st, ids, tp, static_cast<float*>(h), own_w, pre_w, static_cast<T*>(x), dim, vocab, scale, eps, w_bias)
 }
 
 template <typename T>
@@ -324,12 +400,12 @@ static int qk_norm_append_typed(void* qkv, long long ld, const int* slots, void*
 using namespace mx;
 
 // fp32: 1 = fp32 activations, 0 = bf16. y / rows / ls / x may be NULL (no branch to add, identity
-// row map, no layer scale, no output norm).
+// row map, no layer scale, no output); x with pre_w == NULL receives the stream itself.
 extern "C" int mx_stream_norm(const void* y, void* h, const void* rows, const void* post_w, const void* ls,
                               const void* pre_w, void* x, int n, int dim, float eps, float w_bias, int fp32,
                               void* stream) {
   if (n <= 0 || dim <= 0) return 0;
-  if (h == nullptr || (y != nullptr && (post_w == nullptr || rows != nullptr)) || (x != nullptr && pre_w == nullptr)) return -1;
+  if (h == nullptr || (y != nullptr && (post_w == nullptr || rows != nullptr))) return -1;
   const size_t ab = fp32 ? 16 : 8;
   const bool vec = dim % 4 == 0 && aligned_to(y, ab) && aligned_to(x, ab) && aligned_to(h, 16) && aligned_to(post_w, 16) &&
                    aligned_to(ls, 16) && aligned_to(pre_w, 16);
@@ -339,16 +415,17 @@ extern "C" int mx_stream_norm(const void* y, void* h, const void* rows, const vo
               : stream_norm_typed<__nv_bfloat16>(y, h, rows, pw, lp, nw, x, n, dim, eps, w_bias, vec, st);
 }
 
-extern "C" int mx_embed_stream(const void* ids, const void* table, void* h, const void* pre_w, void* x, int n, int dim,
-                               int vocab, float scale, float eps, float w_bias, int fp32, void* stream) {
+extern "C" int mx_embed_stream(const void* ids, const void* table, void* h, const void* own_w, const void* pre_w, void* x,
+                               int n, int dim, int vocab, float scale, float eps, float w_bias, int fp32, void* stream) {
   if (n <= 0 || dim <= 0) return 0;
   const size_t ab = fp32 ? 16 : 8;
-  const bool vec = dim % 4 == 0 && aligned_to(table, ab) && aligned_to(x, ab) && aligned_to(h, 16) && aligned_to(pre_w, 16);
+  const bool vec = dim % 4 == 0 && aligned_to(table, ab) && aligned_to(x, ab) && aligned_to(h, 16) && aligned_to(own_w, 16) &&
+                   aligned_to(pre_w, 16);
   auto st = static_cast<cudaStream_t>(stream);
-  const float* nw = static_cast<const float*>(pre_w);
+  const float *ow = static_cast<const float*>(own_w), *nw = static_cast<const float*>(pre_w);
   const int* ip = static_cast<const int*>(ids);
-  return fp32 ? embed_stream_typed<float>(ip, table, h, nw, x, n, dim, vocab, scale, eps, w_bias, vec, st)
-              : embed_stream_typed<__nv_bfloat16>(ip, table, h, nw, x, n, dim, vocab, scale, eps, w_bias, vec, st);
+  return fp32 ? embed_stream_typed<float>(ip, table, h, ow, nw, x, n, dim, vocab, scale, eps, w_bias, vec, st)
+              : embed_stream_typed<__nv_bfloat16>(ip, table, h, ow, nw, x, n, dim, vocab, scale, eps, w_bias, vec, st);
 }
 
 extern "C" int mx_polynorm(const void* z, const void* coef, void* out, int n, int dim, float eps, int fp32, void* stream) {
@@ -374,4 +451,34 @@ extern "C" int mx_qk_norm_append(void* qkv, long long ld, const void* slots, voi
   const float *q = static_cast<const float*>(qw), *k = static_cast<const float*>(kw);
   return fp32 ? qk_norm_append_typed<float>(qkv, ld, sp, k_pool, v_pool, q, k, n, Hq, Hkv, Dk, Dv, block_size, eps, vec, st)
               : qk_norm_append_typed<__nv_bfloat16>(qkv, ld, sp, k_pool, v_pool, q, k, n, Hq, Hkv, Dk, Dv, block_size, eps, vec, st);
+}
+
+// z rows gate | up (2 dim elements, ld apart) -> out rows of dim.
+extern "C" int mx_glu_rows(const void* z, long long ld, void* out, int n, int dim, int mode, float alpha, float limit, int fp32,
+                           void* stream) {
+  if (n <= 0 || dim <= 0) return 0;
+  if (mode < MX_EPI_SWIGLU || mode > MX_EPI_CLIPPED_SWIGLU || dim > 65535 * 256) return -1;
+  const size_t ab = fp32 ? 16 : 8;
+  const bool vec = dim % 4 == 0 && ld % 4 == 0 && aligned_to(z, ab) && aligned_to(out, ab);
+  auto st = static_cast<cudaStream_t>(stream);
+  const dim3 grid(n, (dim + (vec ? 1023 : 255)) / (vec ? 1024 : 256)), block(256);
+#define MX_GLU(T, V)                                                                                                    \
+  return static_cast<int>(launch_kernel(glu_rows_kernel<T, V>, grid, block, 0, st, static_cast<const T*>(z), ld,        \
+                                        static_cast<T*>(out), dim, mode, alpha, limit))
+  if (fp32) {
+    if (vec) MX_GLU(float, 4);
+    MX_GLU(float, 1);
+  }
+  if (vec) MX_GLU(__nv_bfloat16, 4);
+  MX_GLU(__nv_bfloat16, 1);
+#undef MX_GLU
+}
+
+// x (fp32, n contiguous values) <- cap tanh(x / cap).
+extern "C" int mx_softcap_rows(void* x, long long n, float cap, void* stream) {
+  if (n <= 0) return 0;
+  if (!(cap > 0.f)) return -1;
+  const long long blocks = (n + 255) / 256;
+  return static_cast<int>(launch_kernel(softcap_rows_kernel, dim3(static_cast<unsigned>(blocks < 4096 ? blocks : 4096)), dim3(256), 0,
+                                        static_cast<cudaStream_t>(stream), static_cast<float*>(x), n, cap));
 }

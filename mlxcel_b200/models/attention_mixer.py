@@ -1,13 +1,18 @@
-"""Attention mixer without rotation: positions enter through a logarithmic distance bias.
+"""Attention mixer with optional parts, each a field of its layer's record, so models may mix layers of different shapes:
 
-Per query head h with its key head: ``score = q.k * scale - r1_h ln(1 + r2_h (i - j))`` over all earlier
-tokens (or a window of them), softmax with ``exp(sink_h)`` in the denominator, q and k RMS-normalised per
-head, key and value heads of different widths, and a sigmoid gate computed from the mixer's input on the
-concatenated heads. Every one of bias, sink, q/k norm and gate is optional, and the geometry belongs to
-the layer, so models may mix layers of different shapes.
+* positions: a rotation of the first dimensions of q and k (``inv_freq``, ``mscale``), a logarithmic distance bias
+  (``- r1_h ln(1 + r2_h (i - j))``), or none;
+* q/k norm per head: with weights and without a rotation, or behind the rotation (``unit``: division by the root mean
+  square, weights optional);
+* visibility: all earlier tokens, a window of them, or the earlier tokens of the query's own chunk (runs of ``chunk``
+  positions counted from the sequence's start);
+* scores: ``q.k * scale``, soft-capped (``softcap tanh(s / softcap)``) where a cap is given; ``exp(sink_h)`` in the
+  denominator;
+* values: heads of their own width, or the keys as projected (``values_are_keys``: no value projection);
+* a sigmoid gate computed from the mixer's input on the concatenated heads.
 
-One GEMM produces q | k | v | gate; one kernel normalises q and k and appends k, v to the paged pool; the
-attention kernels apply the gate on the way out. Scores, bias, softmax and accumulation are fp32.
+One GEMM produces q | k | v | gate; one kernel rotates and normalises q and k and appends k, v to the paged pool; the
+attention kernels cap, mask and gate. Scores, bias, softmax and accumulation are fp32.
 """
 from __future__ import annotations
 
@@ -21,7 +26,7 @@ from ..ops import stream
 
 @dataclass
 class AttentionMixerWeights:
-    w_in: torch.Tensor                    # rows q | k | v (| gate), zero rows up to a multiple of 8
+    w_in: torch.Tensor                    # rows q | k (| v) (| gate), zero rows up to a multiple of 8
     out_proj: torch.Tensor                # [H, heads * vdim]
     heads: int
     kv_heads: int
@@ -35,6 +40,12 @@ class AttentionMixerWeights:
     r2: torch.Tensor | None = None
     sinks: torch.Tensor | None = None     # fp32 [heads]
     window: int = 0
+    chunk: int = 0
+    softcap: float = 0.0
+    inv_freq: torch.Tensor | None = None  # fp32 [rotated dimensions / 2]
+    mscale: float = 1.0
+    unit: bool = False                    # with a rotation: q and k divided by their root mean square behind it
+    values_are_keys: bool = False
 
 
 def stack_rows(parts: list[torch.Tensor]) -> torch.Tensor:
@@ -51,12 +62,17 @@ def attention_mixer(w: AttentionMixerWeights, x: torch.Tensor, b, kv, eps: float
     T, nd = x.shape[0], b.num_decode
     row = ops.linear(x, w.w_in)
     geo = dict(Hq=w.heads, Hkv=w.kv_heads, Dk=w.dim, Dv=w.vdim)
-    stream.qk_norm_append(row, b.slot_mapping, kv, q_norm=w.q_norm, k_norm=w.k_norm, eps=eps, **geo)
+    if w.inv_freq is not None:
+        stream.rope_norm_append(row, b.positions, b.slot_mapping, kv, inv_freq=w.inv_freq, mscale=w.mscale, unit=w.unit,
+                                values_are_keys=w.values_are_keys, q_norm=w.q_norm, k_norm=w.k_norm, eps=eps, **geo)
+    else:
+        stream.qk_norm_append(row, b.slot_mapping, kv, q_norm=w.q_norm, k_norm=w.k_norm, eps=eps, **geo)
     q = row[:, : w.heads * w.dim]
-    g0 = w.heads * w.dim + w.kv_heads * (w.dim + w.vdim)
+    g0 = w.heads * w.dim + w.kv_heads * (w.dim + (0 if w.values_are_keys else w.vdim))
     gate = row[:, g0:g0 + w.heads * w.vdim] if w.gated else None
     out = torch.empty(T, w.heads * w.vdim, dtype=row.dtype, device=row.device)
-    common = dict(scale=w.scale, window=w.window, sinks=w.sinks, dist_bias=None if w.r1 is None else (w.r1, w.r2), **geo)
+    common = dict(scale=w.scale, window=w.window, chunk=w.chunk, softcap=w.softcap, sinks=w.sinks,
+                  dist_bias=None if w.r1 is None else (w.r1, w.r2), **geo)
     if nd > 0:
         stream.paged_attention(q[:nd], kv, b.dec_block_tables, b.dec_context_lens, None, out[:nd], max_q_len=1,
                                max_len=b.dec_max_len, gate=None if gate is None else gate[:nd], **common)

@@ -15,10 +15,11 @@ A model is a flat list of pre-norm residual blocks; the family decides the list 
 =====  ===============================================================================================
 
 A second layout ("stream") serves designs that keep the residual in fp32 and normalise every sub-layer on
-both sides: ``h <- h + layer_scale * norm(branch(norm(h)))``. Its blocks carry ``post_norm`` / ``layer_scale``, its
-mixers are ``attention_mixer`` (``models/attention_mixer.py``) and ``general_delta`` (``models/general_delta.py``),
-and ``HybridWeights.runs`` lists the layers in execution order: a layer may run several times with the same
-weights, each run with a KV-pool layer or state slab of its own (Pamasun).
+both sides or behind it only: ``h <- h + layer_scale * norm(branch(norm(h)))``, the inner norm left out where a block's
+``norm`` is None. Its blocks carry ``post_norm`` / ``layer_scale``, its mixers are ``attention_mixer``
+(``models/attention_mixer.py``), ``latent_mixer`` (``models/latent_mixer.py``) and ``general_delta``
+(``models/general_delta.py``), and ``HybridWeights.runs`` lists the layers in execution order: a layer may run several times
+with the same weights, each run with a KV-pool layer or state slab of its own (Pamasun, Govopel).
 
 Nemotron-H gives one block per layer through ``hybrid_override_pattern`` (``"M-M-M*-..."``); the other
 families have a mixer block and an MLP / MoE block per layer. Reference: src/models/nemotron_h.rs,
@@ -45,7 +46,7 @@ from .weights import LayerWeights, ModelWeights
 @dataclass
 class HybridBlock:
     kind: str                                   # "mamba2" | "mamba1" | "attention" | "mlp" | "moe"
-    norm: torch.Tensor
+    norm: torch.Tensor | None                   # None (stream layout): the branch reads the residual stream itself
     mamba: object | None = None                 # Mamba2LayerWeights or Mamba1LayerWeights
     moe: LayerWeights | None = None             # router + stacked experts (block kind "moe")
     attn: LayerWeights | None = None            # wqkv / wo (+ biases)
@@ -62,6 +63,8 @@ class HybridBlock:
     post_norm: torch.Tensor | None = None       # norm of the branch's result
     layer_scale: torch.Tensor | None = None     # element-wise factor behind it
     act_coef: torch.Tensor | None = None        # polynomial-norm activation (a, b, c, e)
+    act_alpha: float = 1.702                    # clipped gated activation: slope of the gate's sigmoid, clip
+    act_limit: float = 7.0
 
 
 @dataclass
@@ -72,6 +75,7 @@ class HybridWeights:
     lm_head: torch.Tensor
     layers: list = field(default_factory=list)  # the attention blocks' LayerWeights (= KV-pool layers)
     runs: list | None = None                    # stream layout: the layers (lists of blocks) in execution order
+    embed_norm: torch.Tensor | None = None      # stream layout: norm of the embedding itself
 
 
 _KINDS = {"M": "mamba2", "m": "mamba1", "L": "gdn", "C": "shortconv", "R": "rglru", "P": "parallel", "*": "attention", "A": "attention", "-": "mlp", "G": "mlp",
@@ -685,13 +689,16 @@ class HybridModel:
         self.dtype = w.embed.dtype
         # (block, index of its KV layer or state slab, run index behind its last block or -1)
         self.order: list = []
-        delta, n_kv, self._kv_heads = [], 0, set()
+        delta, n_kv, self._kv_heads, self._latent_heads = [], 0, set(), set()
         for r, blocks in enumerate(w.runs):
             for blk in blocks:
                 idx = -1
                 if blk.kind == "attention_mixer":
                     idx, n_kv = n_kv, n_kv + 1
                     self._kv_heads.add(blk.attn.kv_heads)
+                elif blk.kind == "latent_mixer":
+                    idx, n_kv = n_kv, n_kv + 1
+                    self._latent_heads.add(blk.attn.heads)
                 elif blk.kind == "general_delta":
                     idx = len(delta)
                     delta.append(blk.mamba)
@@ -705,8 +712,11 @@ class HybridModel:
 
     def decode_split_key(self, rows: int, max_len: int) -> tuple:
         """What a captured decode graph depends on besides its rows: the KV splits of every geometry."""
-        heads = self._kv_heads if self.w.runs is not None else {self.Hkv}
-        return tuple(ops.decode_splits(rows, h, max_len) for h in sorted(heads))
+        if self.w.runs is None:
+            return (ops.decode_splits(rows, self.Hkv, max_len),)
+        from ..ops.latent import latent_splits
+        return tuple(ops.decode_splits(rows, h, max_len) for h in sorted(self._kv_heads)) + \
+            tuple(latent_splits(rows, h, max_len) for h in sorted(self._latent_heads))
 
     def state_slot(self, seq_id: int) -> int:
         return self.ssm.slot(seq_id)
@@ -719,22 +729,28 @@ class HybridModel:
         """Layer runs of the stream layout. Returns the fp32 residual stream [T, H] (before the final norm)."""
         from ..ops import stream
         from .attention_mixer import attention_mixer
+        from .latent_mixer import latent_mixer
         cfg, eps, wb = self.cfg, self.cfg.rms_norm_eps, self.cfg.norm_weight_bias
         if b.embeds is not None:
             raise NotImplementedError("media embeddings with an fp32 residual stream")
         pieces = self.ssm.pieces(b) if self.ssm is not None else None
         self.captured = []
         h, x = stream.embed_stream(b.token_ids, self.w.embed, cfg.embed_scale,
-                                   self.order[0][0].norm if self.order else self.w.final_norm, eps, wb)
+                                   self.order[0][0].norm if self.order else self.w.final_norm, eps, wb, self.w.embed_norm)
         for n, (blk, idx, run) in enumerate(self.order):
             if blk.kind == "attention_mixer":
                 y = ops.linear(attention_mixer(blk.attn, x, b, kv_layers[idx], eps), blk.attn.out_proj)
+            elif blk.kind == "latent_mixer":
+                y = ops.linear(latent_mixer(blk.attn, x, b, kv_layers[idx], eps), blk.attn.out_proj)
             elif blk.kind == "general_delta":
                 y = ops.linear(self.ssm.mixer(idx, blk.mamba, x, pieces), blk.mamba.out_proj)
-            else:
+            elif blk.act == "polynorm":
                 y = ops.linear(stream.polynorm(ops.linear(x, blk.up), blk.act_coef, eps), blk.down)
-            nxt = self.order[n + 1][0].norm if n + 1 < len(self.order) else None
-            x = stream.stream_norm(h, y, blk.post_norm, blk.layer_scale, nxt, eps, wb)
+            else:
+                y = ops.linear(ops.glu_linear(x, blk.up, blk.up.shape[0] // 2, blk.act, alpha=blk.act_alpha, limit=blk.act_limit), blk.down)
+            last = n + 1 == len(self.order)
+            nxt = None if last else self.order[n + 1][0].norm
+            x = stream.stream_norm(h, y, blk.post_norm, blk.layer_scale, nxt, eps, wb, plain=not last)
             if run in self.capture_layers:
                 self.captured.append(h.clone())
         return h
@@ -804,7 +820,9 @@ class HybridModel:
             from ..ops import stream
             x = stream.stream_norm(h, None, None, None, self.w.final_norm, self.cfg.rms_norm_eps, self.cfg.norm_weight_bias,
                                    dtype=self.dtype, rows=None if rows is None else rows.to(torch.int32))
-            return ops.linear(x, self.w.lm_head, out_fp32=True)
+            lg = ops.linear(x, self.w.lm_head, out_fp32=True)
+            cap = self.cfg.final_logit_softcap
+            return lg if cap <= 0 else stream.softcap_(lg, cap)
         lg = self.ssm.logits(h, rows)
         ls = self.cfg.extra.get("logits_scaling", 1.0)
         lg = lg if ls == 1.0 else (lg.float() / ls).to(lg.dtype)

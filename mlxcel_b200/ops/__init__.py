@@ -128,6 +128,9 @@ def glu_linear(x: torch.Tensor, w: torch.Tensor, inter: int, act: str = "silu",
         return ref.glu_linear(x, w, inter, epi, bias, alpha, limit)
     M, K = x.shape
     assert w.shape[0] == 2 * inter and x.stride(1) == 1 and w.stride(1) == 1
+    if x.dtype == torch.float32 or inter % 8 or K % 8 or x.stride(0) % 8 or w.stride(0) % 8 or (x.data_ptr() | w.data_ptr()) % 16:
+        assert row_norm is None and bias is None, "this form has no bias and no deferred RMSNorm"
+        return _glu_any(x, w, inter, epi, alpha, limit, out)
     if out is None:
         out = torch.empty(M, inter, dtype=torch.bfloat16, device=x.device)
     if M == 0:
@@ -138,6 +141,42 @@ def glu_linear(x: torch.Tensor, w: torch.Tensor, inter: int, act: str = "silu",
               inter, K, x.stride(0), w.stride(0), out.stride(0), 0, epi, 0, inter, float(alpha),
               float(limit), ws.data_ptr(), ws.numel(), force_mode, force_splits, _lib.stream(),
               _lib.ref_or_null(ex))
+    return out
+
+
+def _glu_any(x, w, inter: int, epi: int, alpha: float, limit: float, out) -> torch.Tensor:
+    """:func:`glu_linear` as projection and activation kernel, for fp32 operands and sizes the fused form does not take."""
+    z = linear(x, w)
+    out = torch.empty(x.shape[0], inter, dtype=x.dtype, device=x.device) if out is None else out
+    if x.shape[0]:
+        _lib_call("mx_glu_rows", z.data_ptr(), z.stride(0), out.data_ptr(), x.shape[0], inter, epi, float(alpha), float(limit),
+                  1 if x.dtype == torch.float32 else 0, _lib.stream())
+    return out
+
+
+def batched_linear(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, x_cols: int, out_cols: int) -> torch.Tensor:
+    """Block-diagonal projection: group g of ``w`` [G, N, K] takes the columns ``[g * x_cols, + K)`` of x and writes the
+    columns ``[g * out_cols, + N)`` of ``out`` (both may be wider than what is used; other columns keep their values)."""
+    G, N, K = w.shape
+    M = x.shape[0]
+    assert x.shape[1] >= (G - 1) * x_cols + K and out.shape[1] >= (G - 1) * out_cols + N and out.shape[0] == M and w.is_contiguous()
+    if not x.is_cuda:
+        for g in range(G):
+            out[:, g * out_cols:g * out_cols + N] = ref.linear(x[:, g * x_cols:g * x_cols + K], w[g])
+        return out
+    assert x.stride(1) == 1 and out.stride(1) == 1 and x.dtype == w.dtype == out.dtype
+    if M == 0:
+        return out
+    if x.dtype == torch.bfloat16:
+        ws = _lib.workspace(x.device)
+        rc = _lib.load().mx_batched_gemm_bf16(x.data_ptr(), w.data_ptr(), out.data_ptr(), G, M, N, K, x.stride(0), x_cols,
+                                              out.stride(0), out_cols, ws.data_ptr(), ws.numel(), _lib.stream())
+        if rc != -10:
+            _lib.count_launch()
+            _lib.check(rc, "mx_batched_gemm_bf16")
+            return out
+    _lib_call("mx_batched_gemm_any", x.data_ptr(), w.data_ptr(), out.data_ptr(), G, M, N, K, x.stride(0), K, out.stride(0),
+              x_cols, N * K, out_cols, 1 if x.dtype == torch.float32 else 0, _lib.stream())
     return out
 
 

@@ -76,6 +76,9 @@ def _declare(lib) -> None:
         "mx_gemm_bf16": [_vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _i, _i, _i, _f, _f,
                          _vp, _ll, _i, _i, _vp, _vp],
         "mx_gemm_any": [_vp, _vp, _vp, _vp, _vp, _i, _i, _i, _ll, _ll, _ll, _ll, _i, _i, _vp],
+        "mx_batched_gemm_bf16": [_vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _i, _vp, _ll, _vp],
+        "mx_batched_gemm_any": [_vp, _vp, _vp, _i, _i, _i, _i, _ll, _ll, _ll, _ll, _ll, _ll, _i, _vp],
+        "mx_glu_rows": [_vp, _ll, _vp, _i, _i, _i, _f, _f, _i, _vp],
         "mx_gemm_comm": [_vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _i, _i, _i, _vp, _vp,
                          _vp, _vp, _vp, _ll, _ll, _vp, _ll, _vp, _vp],
         "mx_allreduce_comm": [_vp, _vp, _vp, _ll, _i, _i, _i, _vp, _vp, _vp, _vp, _vp, _ll, _ll, _vp, _vp,

@@ -93,7 +93,7 @@ def rope_inv_freq(head_dim_rot: int, theta: float, scaling: dict | None,
             if truncate:
                 lo, hi = math.floor(lo), math.ceil(hi)
             lo, hi = max(lo, 0), min(hi, head_dim_rot - 1)
-            if hi == lo:
+            if hi <= lo:
                 hi = lo + 0.001
             ramp = ((torch.arange(half, dtype=torch.float64) - lo) / (hi - lo)).clamp(0, 1)
             extrap_w = 1.0 - ramp

@@ -1,9 +1,10 @@
-"""Operators of layers with an fp32 residual stream and of attention heads without rotation: sub-layer
-norms on both sides, polynomial-norm activation, q/k norm + KV append, paged attention with a logarithmic
-distance bias / sink / output gate and separate key and value widths, the generalized delta rule.
+"""Operators of layers with an fp32 residual stream: sub-layer norms before and / or behind a branch,
+polynomial-norm activation, soft cap, q/k norm (before or behind a rotation) + KV append, paged attention with
+chunks, soft cap, a logarithmic distance bias, sink, output gate and separate key and value widths, the
+generalized delta rule.
 
-Every operator exists for bf16 and fp32 activations on CUDA (``csrc/stream_norm.cu``, ``csrc/simt.cu``,
-``csrc/attention*.cu``, ``csrc/delta_rule.cu``); CPU tensors take the PyTorch statements below. Norm weights,
+Every operator exists for bf16 and fp32 activations on CUDA (``csrc/stream_norm.cu``, ``csrc/rope_norm.cu``,
+``csrc/simt.cu``, ``csrc/attention*.cu``, ``csrc/delta_rule.cu``); CPU tensors take the PyTorch statements below. Norm weights,
 layer scales and per-head constants are fp32 vectors."""
 from __future__ import annotations
 
@@ -18,12 +19,14 @@ from .reference import _gather_kv
 _vp, _i, _f, _ll = ctypes.c_void_p, ctypes.c_int, ctypes.c_float, ctypes.c_longlong
 _SIG = {
     "mx_stream_norm": [_vp] * 7 + [_i, _i, _f, _f, _i, _vp],
-    "mx_embed_stream": [_vp] * 5 + [_i, _i, _i, _f, _f, _f, _i, _vp],
+    "mx_embed_stream": [_vp] * 6 + [_i, _i, _i, _f, _f, _f, _i, _vp],
     "mx_polynorm": [_vp, _vp, _vp, _i, _i, _f, _i, _vp],
+    "mx_softcap_rows": [_vp, _ll, _f, _vp],
+    "mx_rope_norm_append": [_vp, _ll, _vp, _vp, _vp, _f] + [_vp] * 4 + [_i] * 9 + [_f, _i, _vp],
     "mx_qk_norm_append": [_vp, _ll, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _f, _i, _vp],
-    "mx_paged_attention_any": [_vp, _ll] + [_vp] * 9 + [_ll, _vp] + [_i] * 9 + [_f, _i, _vp],
-    "mx_paged_decode_ext": [_vp, _ll] + [_vp] * 8 + [_ll, _vp, _vp] + [_i] * 8 + [_f, _i, _vp],
-    "mx_paged_prefill_ext": [_vp, _ll, _vp, _vp, _ll] + [_vp] * 7 + [_ll, _vp] + [_i] * 10 + [_f, _vp, _vp],
+    "mx_paged_attention_any": [_vp, _ll] + [_vp] * 9 + [_ll, _vp] + [_i] * 12 + [_f, _f, _i, _vp],
+    "mx_paged_decode_ext": [_vp, _ll] + [_vp] * 8 + [_ll, _vp, _vp] + [_i] * 9 + [_f, _f, _i, _vp],
+    "mx_paged_prefill_ext": [_vp, _ll, _vp, _vp, _ll] + [_vp] * 7 + [_ll, _vp] + [_i] * 11 + [_f, _f, _vp, _vp],
     "mx_delta_rule": [_vp, _ll] + [_vp] * 11 + [_i] * 6 + [_f, _f, _f, _i, _i, _vp],
 }
 NOT_COVERED = -10        # a tensor-core kernel refuses the geometry: the shape-agnostic one takes it
@@ -53,44 +56,52 @@ def _rms(x: torch.Tensor, eps: float) -> torch.Tensor:
 
 
 # ----------------------------------------------------------------------------- residual stream
-def embed_stream(ids, table, scale: float, pre_w, eps: float, w_bias: float):
-    """``h = scale * table[ids]`` (fp32 stream) and ``x = rmsnorm(h) * (w_bias + pre_w)`` in the table's type."""
+def embed_stream(ids, table, scale: float, pre_w, eps: float, w_bias: float, own_w=None):
+    """``h = scale * table[ids]`` (fp32 stream; with ``own_w`` the embedding's own norm: ``rmsnorm(.) * (w_bias + own_w)``)
+    and ``x = rmsnorm(h) * (w_bias + pre_w)`` in the table's type; without ``pre_w``, x is h itself."""
     n, dim = ids.shape[0], table.shape[1]
     if not table.is_cuda:
         ok = (ids >= 0) & (ids < table.shape[0])
         h = table[ids.clamp(0, table.shape[0] - 1).long()].float() * scale * ok[:, None]
-        return h, (_rms(h, eps) * (w_bias + pre_w)).to(table.dtype)
+        h = h if own_w is None else _rms(h, eps) * (w_bias + own_w)
+        return h, _stream_as(h, table.dtype) if pre_w is None else (_rms(h, eps) * (w_bias + pre_w)).to(table.dtype)
     h = torch.empty(n, dim, dtype=torch.float32, device=table.device)
-    x = torch.empty(n, dim, dtype=table.dtype, device=table.device)
+    alias = pre_w is None and table.dtype == torch.float32       # (the branch has read the stream before it is added to it)
+    x = None if alias else torch.empty(n, dim, dtype=table.dtype, device=table.device)
     if n:
-        _call("mx_embed_stream", ids.data_ptr(), table.data_ptr(), h.data_ptr(), pre_w.data_ptr(), x.data_ptr(), n, dim,
-              table.shape[0], float(scale), float(eps), float(w_bias), _fp32(table), _lib.stream())
-    return h, x
+        _call("mx_embed_stream", ids.data_ptr(), table.data_ptr(), h.data_ptr(), _lib.ptr(own_w), _lib.ptr(pre_w), _lib.ptr(x),
+              n, dim, table.shape[0], float(scale), float(eps), float(w_bias), _fp32(table), _lib.stream())
+    return h, h if alias else x
 
 
-def stream_norm(h, y, post_w, layer_scale, pre_w, eps: float, w_bias: float, dtype=None, rows=None):
+def _stream_as(h, dtype):
+    return h if h.dtype == dtype else h.to(dtype)
+
+
+def stream_norm(h, y, post_w, layer_scale, pre_w, eps: float, w_bias: float, dtype=None, rows=None, plain: bool = False):
     """One step of the stream between two sub-layers, in place on ``h`` (fp32): with a branch ``y``,
     ``h += rmsnorm(y) * (w_bias + post_w) * layer_scale`` (layer_scale optional); with ``pre_w``, returns
-    ``rmsnorm(h) * (w_bias + pre_w)`` as ``dtype`` (default: y's type). ``rows`` (int32, no branch) selects
-    the rows of h to normalise."""
+    ``rmsnorm(h) * (w_bias + pre_w)`` as ``dtype`` (default: y's type); with ``plain`` (and no ``pre_w``) the
+    stream itself as ``dtype``. ``rows`` (int32, no branch) selects the rows of h to normalise."""
     dtype = dtype or y.dtype
     if not h.is_cuda:
         if y is not None:
             b = _rms(y.float(), eps) * (w_bias + post_w)
             h += b if layer_scale is None else b * layer_scale
         if pre_w is None:
-            return None
+            return _stream_as(h, dtype) if plain else None
         return (_rms(h if rows is None else h[rows.long()], eps) * (w_bias + pre_w)).to(dtype)
     dim = h.shape[1]
     n = h.shape[0] if rows is None else rows.shape[0]
-    x = torch.empty(n, dim, dtype=dtype, device=h.device) if pre_w is not None else None
+    alias = plain and pre_w is None and dtype == torch.float32
+    x = torch.empty(n, dim, dtype=dtype, device=h.device) if pre_w is not None or (plain and not alias) else None
     assert h.is_contiguous() and (y is None or (y.is_contiguous() and y.dtype == dtype))
     assert rows is None or rows.dtype == torch.int32
     if n:
         fp32 = 1 if dtype == torch.float32 else 0
         _call("mx_stream_norm", _lib.ptr(y), h.data_ptr(), _lib.ptr(rows), _lib.ptr(post_w), _lib.ptr(layer_scale),
               _lib.ptr(pre_w), _lib.ptr(x), n, dim, float(eps), float(w_bias), fp32, _lib.stream())
-    return x
+    return h if alias else x
 
 
 def polynorm(z, coef, eps: float):
@@ -106,7 +117,57 @@ def polynorm(z, coef, eps: float):
     return out
 
 
+def softcap_(x, cap: float):
+    """``cap tanh(x / cap)`` on fp32 values, in place."""
+    if not x.is_cuda:
+        return x.copy_(cap * torch.tanh(x / cap))
+    assert x.dtype == torch.float32 and x.is_contiguous()
+    if x.numel():
+        _call("mx_softcap_rows", x.data_ptr(), x.numel(), float(cap), _lib.stream())
+    return x
+
+
 # ----------------------------------------------------------------------------- attention
+def rotate_half(x, positions, inv_freq, mscale: float):
+    """x [T, H, D] fp32: dimension i turned with i + R / 2 by ``positions * inv_freq[i]`` (R = 2 len(inv_freq)), both
+    times ``mscale``; dimensions from R on pass."""
+    half = inv_freq.shape[0]
+    a = (positions.float()[:, None] * inv_freq)[:, None]
+    c, s = a.cos() * mscale, a.sin() * mscale
+    u, v = x[..., :half], x[..., half:2 * half]
+    return torch.cat([u * c - v * s, v * c + u * s, x[..., 2 * half:]], -1)
+
+
+def rope_norm_append(row, positions, slots, kv, *, Hq: int, Hkv: int, Dk: int, Dv: int, inv_freq, mscale: float = 1.0,
+                     unit: bool = True, values_are_keys: bool = False, q_norm=None, k_norm=None, eps: float = 1e-6) -> None:
+    """Rows ``q | k (| v)``: q (in place) and k are rotated by their positions, then divided per head by their root
+    mean square (``unit``) and multiplied by an optional weight; k and v go into the paged pool (negative slots append
+    nothing). ``values_are_keys``: no v columns, the values are the keys as projected."""
+    if not row.is_cuda:
+        T, nq, nk = row.shape[0], Hq * Dk, Hkv * Dk
+        q, k = row[:, :nq].float().view(T, Hq, Dk), row[:, nq:nq + nk].float().view(T, Hkv, Dk)
+        v = row[:, nq:nq + nk] if values_are_keys else row[:, nq + nk:nq + nk + Hkv * Dv]
+        v = v.reshape(T, Hkv, Dv).clone()
+
+        def turned(x, w):
+            x = rotate_half(x, positions, inv_freq, mscale)
+            x = _rms(x, eps) if unit else x
+            return x if w is None else x * w
+        row[:, :nq] = turned(q, q_norm).reshape(T, nq).to(row.dtype)
+        ok = slots >= 0
+        s = slots[ok].long()
+        blk, off = s // kv.block_size, s % kv.block_size
+        kv.k[blk, :, off] = turned(k, k_norm)[ok].to(kv.k.dtype)
+        kv.v[blk, :, off] = v[ok].to(kv.v.dtype)
+        return
+    assert kv.k.dtype == row.dtype and row.stride(1) == 1 and slots.dtype == torch.int32 and positions.dtype == torch.int32
+    if row.shape[0]:
+        _call("mx_rope_norm_append", row.data_ptr(), row.stride(0), positions.data_ptr(), slots.data_ptr(), inv_freq.data_ptr(),
+              float(mscale), kv.k.data_ptr(), kv.v.data_ptr(), _lib.ptr(q_norm), _lib.ptr(k_norm), row.shape[0], Hq, Hkv, Dk, Dv,
+              2 * inv_freq.shape[0], 1 if values_are_keys else 0, 1 if unit else 0, kv.block_size, float(eps), _fp32(row),
+              _lib.stream())
+
+
 def qk_norm_append(qkv, slots, kv, *, Hq: int, Hkv: int, Dk: int, Dv: int, q_norm, k_norm, eps: float) -> None:
     """Rows ``q | k | v | ...``: per-head RMS norm of q (in place) and k, then k and v into the paged pool
     (negative slots append nothing). No positional encoding."""
@@ -130,7 +191,8 @@ def qk_norm_append(qkv, slots, kv, *, Hq: int, Hkv: int, Dk: int, Dv: int, q_nor
               _lib.stream())
 
 
-def paged_attention_ref(q, kv, tables, lens, cu, *, Hq, Hkv, Dk, Dv, scale, window=0, sinks=None, dist_bias=None, gate=None):
+def paged_attention_ref(q, kv, tables, lens, cu, *, Hq, Hkv, Dk, Dv, scale, window=0, sinks=None, dist_bias=None, gate=None,
+                        softcap=0.0, chunk=0):
     T, G = q.shape[0], Hq // Hkv
     out = torch.zeros(T, Hq * Dv, dtype=q.dtype, device=q.device)
     cu_l, lens_l = cu.tolist(), lens.tolist()
@@ -142,11 +204,14 @@ def paged_attention_ref(q, kv, tables, lens, cu, *, Hq, Hkv, Dk, Dv, scale, wind
         k, v = _gather_kv(kv, tables[s], n)
         qs = q[q0:q1].float().reshape(ql, Hkv, G, Dk).permute(1, 2, 0, 3)
         sc = torch.einsum("hgqd,hkd->hgqk", qs, k) * scale
-        d = torch.arange(n - ql, n, device=q.device)[:, None] - torch.arange(n, device=q.device)[None, :]
+        sc = softcap * torch.tanh(sc / softcap) if softcap > 0 else sc
+        qp, kp = torch.arange(n - ql, n, device=q.device)[:, None], torch.arange(n, device=q.device)[None, :]
+        d = qp - kp
         if dist_bias is not None:
             r1, r2 = (t.float().reshape(Hkv, G, 1, 1) for t in dist_bias)
             sc = sc - r1 * torch.log1p(r2 * d.clamp(min=0).float())
         vis = (d >= 0) & (d < window) if window > 0 else d >= 0
+        vis = vis & (kp // chunk == qp // chunk) if chunk > 0 else vis
         sc = sc.masked_fill(~vis, float("-inf"))
         if sinks is not None:
             sc = torch.cat([sc, sinks.float().reshape(Hkv, G, 1, 1).expand(Hkv, G, ql, 1)], -1)
@@ -159,12 +224,14 @@ def paged_attention_ref(q, kv, tables, lens, cu, *, Hq, Hkv, Dk, Dv, scale, wind
 
 
 def paged_attention(q, kv, tables, lens, cu, out, *, Hq: int, Hkv: int, Dk: int, Dv: int, scale: float, max_q_len: int,
-                    max_len: int = 0, window: int = 0, sinks=None, dist_bias=None, gate=None, force_any: bool = False) -> None:
+                    max_len: int = 0, window: int = 0, sinks=None, dist_bias=None, gate=None, softcap: float = 0.0, chunk: int = 0,
+                    force_any: bool = False) -> None:
     """Causal paged attention of the query rows of every sequence (the last ``cu[s+1] - cu[s]`` of its ``lens[s]``
     tokens) into ``out`` [rows, Hq * Dv]. ``cu=None`` says one row per sequence (decode).
 
-    scores: ``q.k * scale - r1 ln(1 + r2 distance)`` with ``dist_bias = (r1, r2)`` per query head; ``sinks`` adds
-    ``exp(sink)`` to the denominator; ``gate`` ([rows, Hq * Dv], may be a column slice) multiplies the result by
+    scores: ``q.k * scale``, with ``softcap`` > 0 ``softcap tanh(. / softcap)``, then ``- r1 ln(1 + r2 distance)`` with
+    ``dist_bias = (r1, r2)`` per query head; ``chunk`` > 0: a token sees only keys of its own run of ``chunk`` positions
+    (counted from the sequence's start); ``sinks`` adds ``exp(sink)`` to the denominator; ``gate`` ([rows, Hq * Dv], may be a column slice) multiplies the result by
     its sigmoid. bf16 pools with row widths that are multiples of 8 up to 128 take the tensor-core kernels
     (flash decoding with split KV; tcgen05 prefill); the rest the SIMT one."""
     rows = q.shape[0]
@@ -173,7 +240,7 @@ def paged_attention(q, kv, tables, lens, cu, out, *, Hq: int, Hkv: int, Dk: int,
     if not q.is_cuda:
         c = torch.arange(rows + 1) if cu is None else cu
         out.copy_(paged_attention_ref(q, kv, tables, lens, c, Hq=Hq, Hkv=Hkv, Dk=Dk, Dv=Dv, scale=scale, window=window,
-                                      sinks=sinks, dist_bias=dist_bias, gate=gate))
+                                      sinks=sinks, dist_bias=dist_bias, gate=gate, softcap=softcap, chunk=chunk))
         return
     r1, r2 = dist_bias if dist_bias is not None else (None, None)
     assert kv.k.dtype == q.dtype and q.stride(1) == 1 and out.is_contiguous() and out.dtype == q.dtype
@@ -187,12 +254,13 @@ def paged_attention(q, kv, tables, lens, cu, out, *, Hq: int, Hkv: int, Dk: int,
             splits = decode_splits(rows, Hkv, max_len or tables.shape[1] * kv.block_size)
             scratch = _decode_scratch(q.device, int(_lib.load().mx_paged_decode_scratch_floats(rows, Hq, Dv, splits)))
             rc = _fn("mx_paged_decode_ext")(*head, tables.data_ptr(), lens.data_ptr(), *tail, scratch.data_ptr(), rows, Hq,
-                                            Hkv, Dk, Dv, kv.block_size, tables.shape[1], window, float(scale), splits,
-                                            _lib.stream())
+                                            Hkv, Dk, Dv, kv.block_size, tables.shape[1], window, chunk, float(scale),
+                                            float(softcap), splits, _lib.stream())
         else:
             rc = _fn("mx_paged_prefill_ext")(*head, kv.k.shape[0], tables.data_ptr(), cu.data_ptr(), lens.data_ptr(), *tail,
                                              lens.shape[0], rows, max_q_len, Hq, Hkv, Dk, Dv, kv.block_size, tables.shape[1],
-                                             window, float(scale), _lib.workspace(q.device).data_ptr(), _lib.stream())
+                                             window, chunk, float(scale), float(softcap), _lib.workspace(q.device).data_ptr(),
+                                             _lib.stream())
         if rc != NOT_COVERED:
             _lib.count_launch()
             _lib.check(rc, "paged attention")
@@ -200,7 +268,7 @@ def paged_attention(q, kv, tables, lens, cu, out, *, Hq: int, Hkv: int, Dk: int,
     if cu is None:
         cu = torch.arange(rows + 1, dtype=torch.int32, device=q.device)
     _call("mx_paged_attention_any", *head, tables.data_ptr(), cu.data_ptr(), lens.data_ptr(), *tail, lens.shape[0], rows, Hq,
-          Hkv, Dk, Dv, kv.block_size, tables.shape[1], window, float(scale), _fp32(q), _lib.stream())
+          Hkv, Dk, Dv, Dk, Dv, kv.block_size, tables.shape[1], window, chunk, float(scale), float(softcap), _fp32(q), _lib.stream())
 
 
 # ----------------------------------------------------------------------------- generalized delta rule

@@ -24,6 +24,13 @@ def _recurrent_block(cfg: ModelConfig, kind: str) -> tuple[int, int]:
         # (a repeated layer's weights count once, its state for every run)
         spec = x["layer_specs"][kind]
         m, ff = spec["mixer"], (spec["mlp"] or {}).get("ff", 0)
+        if cfg.model_type == "govopel":
+            if spec["type"] == "attention":                       # values are the keys
+                par = h * m["dim"] * (2 * m["heads"] + m["kv_heads"])
+            else:
+                par = h * (m["q_rank"] + m["kv_rank"] + m["rot_dim"] + m["heads"] * m["vdim"]) + m["q_rank"] + m["kv_rank"] + m["heads"] * (
+                    m["q_rank"] * (m["dim"] + m["rot_dim"]) + m["kv_rank"] * (m["dim"] + m["vdim"]))
+            return par + 3 * h * ff + (2 if ff else 1) * h, 0
         if spec["type"] == "attention":
             par = h * (m["heads"] * (m["dim"] + 2 * m["vdim"]) + m["kv_heads"] * (m["dim"] + m["vdim"]))
             st = 0
