@@ -1,12 +1,14 @@
-"""Shared driver of the Pamasun tests: an engine over random weights, fed token by token or in portions, with
-small pools so that pages and state slots come round again."""
+"""Shared driver of the tests of designs without a library implementation: an engine over random weights, fed token by
+token or in portions, with small pools so that pages and state slots come round again. ``O`` is the design's plain model."""
 import torch
 
-import oracle_pamasun as O
 from mlxcel_b200.config import ModelConfig
 from mlxcel_b200.engine import EngineConfig
 from mlxcel_b200.llm import LLM
+from mlxcel_b200.models.govopel import build_govopel_weights
 from mlxcel_b200.models.pamasun import build_pamasun_weights
+
+BUILDERS = {"pamasun": build_pamasun_weights, "govopel": build_govopel_weights}
 
 
 def llm_for(raw, tensors, device, dtype, **ecfg):
@@ -14,7 +16,7 @@ def llm_for(raw, tensors, device, dtype, **ecfg):
     kw = dict(max_batch=4, max_prefill_seqs=4, state_slots=4, block_size=16, num_blocks=48, max_num_batched_tokens=768,
               max_model_len=768, prefix_cache=False, watermark=0.0)
     kw.update(ecfg)
-    return LLM(cfg, build_pamasun_weights(tensors.__getitem__, cfg, dtype, device), EngineConfig(**kw))
+    return LLM(cfg, BUILDERS[cfg.model_type](tensors.__getitem__, cfg, dtype, device), EngineConfig(**kw))
 
 
 def tokens_for(raw, n, seed):
@@ -98,7 +100,7 @@ def _errors(got, want):
     return d.pow(2).mean(-1).sqrt() / (want - want.mean(-1, keepdim=True)).pow(2).mean().sqrt()
 
 
-def bf16_ok(raw, tensors, toks, got, want):
+def bf16_ok(O, raw, tensors, toks, got, want):
     """A bf16 run against what rounding the activations alone causes: the mean error stays near that of
     rounding, and all but a few positions (ill-conditioned ones, where rounding decides a sign) stay within
     three times its largest error."""
@@ -108,7 +110,7 @@ def bf16_ok(raw, tensors, toks, got, want):
     return float(e.median()) < 1.3 * float(r.median()) + 1e-3 and int((e > 3 * r.max()).sum()) <= max(1, len(toks) // 50)
 
 
-def oracle_greedy(raw, tensors, prompt, n):
+def oracle_greedy(O, raw, tensors, prompt, n):
     toks = list(prompt)
     for _ in range(n):
         toks.append(int(O.forward(raw, tensors, toks)[-1].argmax()))

@@ -136,3 +136,63 @@ def forward(cfg, tensors, tokens, dtype=torch.float64, want_layers=False):
         stream.append(x)
     logits = soft_cap(act(norm(x, t["final.norm"], eps)) @ t["embed"].T, cfg["logit_softcap"])
     return (logits, torch.stack(stream)) if want_layers else logits
+
+
+def random_tensors(cfg, seed, dtype=torch.float32):
+    """Checkpoint of a configuration with random values: sharp query latents and projections of unit gain."""
+    g = torch.Generator().manual_seed(seed)
+    n = lambda *s: torch.randn(*s, generator=g)          # noqa: E731
+    lin = lambda o, i: n(o, i) * i ** -0.5               # noqa: E731
+    H, V = cfg["width"], cfg["vocab"]
+    t = {"embed": lin(V, H) * 2, "embed.norm": 1 + 0.3 * n(H), "final.norm": 1 + 0.3 * n(H)}
+    for i, spec in enumerate(cfg["layers"]):
+        p, m = f"l{i}.", spec["mixer"]
+        x, h, d = p + "mix.", m["heads"], m["dim"]
+        t[p + "norm1"] = 1 + 0.3 * n(H)
+        if spec["type"] == "attention":
+            t.update({x + "q": lin(h * d, H), x + "k": lin(m["kv_heads"] * d, H), x + "o": lin(H, h * m["vdim"])})
+        else:
+            q, c, r, v = m["q_rank"], m["kv_rank"], m["rot_dim"], m["vdim"]
+            t.update({x + "dq": lin(q, H), x + "dq.norm": 1.5 + 0.3 * n(q), x + "uq": lin(h * (d + r), q), x + "dkv": lin(c + r, H),
+                      x + "dkv.norm": 1 + 0.3 * n(c), x + "uk": lin(h * d, c), x + "uv": lin(h * v, c), x + "o": lin(H, h * v)})
+        if spec.get("mlp"):
+            ff = spec["mlp"]["ff"]
+            t.update({p + "norm2": 1 + 0.3 * n(H), p + "mlp.gate": lin(ff, H), p + "mlp.up": lin(ff, H), p + "mlp.down": lin(H, ff)})
+    return {k: v.to(torch.bfloat16).to(dtype) for k, v in t.items()}
+
+
+def _mlp(ff, limit):
+    return None if ff is None else dict(kind="dense", ff=ff, limit=limit)
+
+
+def attn_spec(heads, kv_heads, dim, rot, chunk, scale, softcap, ff, limit=1.5, base=3000.0, scaling=(2.5, 300, 20.0, 1.5)):
+    r = dict(dims=rot, base=base)
+    if scaling:
+        r["scaling"] = dict(zip(("factor", "original", "fast", "slow"), scaling))
+    return dict(type="attention", mixer=dict(heads=heads, kv_heads=kv_heads, dim=dim, vdim=dim, scale=scale, softcap=softcap, rot=r,
+                                             mask=dict(size=chunk)), mlp=_mlp(ff, limit))
+
+
+def latent_spec(heads, dim, rot, vdim, q_rank, kv_rank, scale, ff, limit=1.5, base=20000.0):
+    return dict(type="latent_attention", mixer=dict(heads=heads, dim=dim, rot_dim=rot, vdim=vdim, q_rank=q_rank, kv_rank=kv_rank,
+                                                    scale=scale, rot=dict(dims=rot, base=base)), mlp=_mlp(ff, limit))
+
+
+def model_config(vocab, width, layers, eps=1e-5, logit_softcap=9.0):
+    return dict(architecture="Govopel", vocab=vocab, width=width, layers=layers, norm=dict(eps=eps), logit_softcap=logit_softcap)
+
+
+# Configurations of the tests: mixed orders, unequal layers, layers without feed-forward, chunks that do and do not fall on
+# page borders, sizes no tensor-core tile or vector access divides, and values that happen to be equal or one.
+CONFIGS = {
+    "mixed": model_config(160, 96, [latent_spec(3, 32, 16, 24, 40, 56, 0.3, 112), attn_spec(6, 2, 48, 24, 20, 0.15, 6.0, 72),
+                                    latent_spec(5, 24, 24, 40, 24, 32, 0.25, None), attn_spec(4, 1, 32, 32, 16, 0.2, 15.0, 80, 0.7)]),
+    "odd": model_config(101, 75, [attn_spec(3, 3, 20, 10, 13, 0.3, 4.0, 50), latent_spec(3, 9, 6, 11, 17, 13, 0.5, 33, 3.0),
+                                  attn_spec(5, 1, 33, 22, 1, 0.1, 2.0, None, scaling=None)], eps=1e-3, logit_softcap=25.0),
+    "attention_only": model_config(128, 64, [attn_spec(2, 2, 64, 64, 64, 0.125, 10.0, 64, scaling=(1.0, 64, 1.0, 1.0)),
+                                             attn_spec(8, 1, 16, 2, 129, 0.6, 30.0, 96, base=10.0, scaling=(40.0, 50, 32.0, 1.0))]),
+    "latent_only": model_config(96, 64, [latent_spec(1, 8, 8, 8, 8, 8, 0.9, 64), latent_spec(8, 64, 64, 64, 64, 64, 0.12, 64, 1.0),
+                                         latent_spec(2, 16, 2, 72, 120, 104, 0.4, None)]),
+    "wide": model_config(264, 256, [latent_spec(20, 128, 64, 128, 96, 512, 0.1, 320), attn_spec(10, 2, 128, 64, 200, 0.1, 20.0, 256),
+                                    latent_spec(4, 96, 40, 80, 160, 200, 0.12, 192)]),
+}

@@ -7,7 +7,7 @@ import oracle_pamasun as O
 from mlxcel_b200 import ops
 from mlxcel_b200.engine import SamplingParams
 from mlxcel_b200.ops import KVLayer, stream
-from pamasun_runs import bf16_ok, interleave, llm_for, oracle_greedy, run_alone, run_mixed, tokens_for, worst
+from design_runs import bf16_ok, interleave, llm_for, oracle_greedy, run_alone, run_mixed, tokens_for, worst
 
 pytestmark = pytest.mark.gpu
 DEV = "cuda"
@@ -248,7 +248,7 @@ def test_prompts_portions_and_decoding(name, dtype):
     want, layers = O.forward(raw, t, toks, want_layers=True)
     llm = llm_for(raw, t, DEV, dtype)
     whole = run_alone(llm.engine, toks, [150])
-    ok = (lambda got: worst(got, want) < 1e-4) if dtype == F32 else (lambda got: bf16_ok(raw, t, toks, got, want))   # noqa: E731
+    ok = (lambda got: worst(got, want) < 1e-4) if dtype == F32 else (lambda got: bf16_ok(O, raw, t, toks, got, want))   # noqa: E731
     assert ok(whole)
     for sizes in ([1], [130, 1], [2], [17, 3, 1, 64, 16]):
         assert ok(run_alone(llm.engine, toks, sizes)), sizes
@@ -271,7 +271,7 @@ def test_mixed_batches_on_reused_pages_and_slots(name):
     for dtype in (F32, BF16):
         llm = llm_for(raw, t, DEV, dtype, num_blocks=34, max_model_len=544)
         for s, got, want in zip(seqs, run_mixed(llm.engine, seqs, sched), wants):
-            assert worst(got, want) < 1e-4 if dtype == F32 else bf16_ok(raw, t, s, got, want)
+            assert worst(got, want) < 1e-4 if dtype == F32 else bf16_ok(O, raw, t, s, got, want)
         assert llm.engine.bm.num_free == 34 and len(llm.model.ssm.free) == 4
 
 
@@ -282,14 +282,14 @@ def test_long_decoding_keeps_state_and_cache():
     want = O.forward(raw, t, toks)
     for dtype in (F32, BF16):
         got = run_alone(llm_for(raw, t, DEV, dtype).engine, toks, [40] + [1] * 660)
-        assert worst(got, want) < 1e-4 if dtype == F32 else bf16_ok(raw, t, toks, got, want)
+        assert worst(got, want) < 1e-4 if dtype == F32 else bf16_ok(O, raw, t, toks, got, want)
 
 
 def test_greedy_generation_through_the_scheduler():
     raw = O.CONFIGS["mixed"]
     t = O.random_tensors(raw, seed=9)
     prompts = [tokens_for(raw, n, 40 + n) for n in (23, 1, 9, 30, 4)]
-    want = [oracle_greedy(raw, t, p, 12) for p in prompts]
+    want = [oracle_greedy(O, raw, t, p, 12) for p in prompts]
     sp = SamplingParams(max_tokens=12, temperature=0.0, ignore_eos=True)
     # decode graphs with the lookahead pipeline; without graphs; queueing, prompt portions and preemption
     for kw in (dict(max_batch=8, state_slots=8), dict(cuda_graphs=False), dict(max_batch=2, max_num_batched_tokens=8, num_blocks=6)):

@@ -12,7 +12,7 @@ import oracle_pamasun as O
 from mlxcel_b200.config import ModelConfig, preset
 from mlxcel_b200.engine import SamplingParams
 from mlxcel_b200.ops import stream
-from pamasun_runs import cut, interleave, llm_for, oracle_greedy, run_alone, run_mixed, tokens_for, worst
+from design_runs import cut, interleave, llm_for, oracle_greedy, run_alone, run_mixed, tokens_for, worst
 
 TOL = 2e-5
 ROOT = Path(__file__).resolve().parent.parent
@@ -157,7 +157,7 @@ def test_greedy_generation_through_the_scheduler():
     raw = O.CONFIGS["mixed"]
     t = O.random_tensors(raw, seed=9)
     prompts = [tokens_for(raw, n, 40 + n) for n in (23, 1, 9, 30, 4)]
-    want = [oracle_greedy(raw, t, p, 6) for p in prompts]
+    want = [oracle_greedy(O, raw, t, p, 6) for p in prompts]
     sp = SamplingParams(max_tokens=6, temperature=0.0, ignore_eos=True)
     for kw in (dict(), dict(max_batch=2, max_num_batched_tokens=8, num_blocks=6)):       # roomy; queueing, portions, preemption
         llm = llm_for(raw, t, "cpu", torch.float32, **kw)
@@ -174,7 +174,7 @@ def test_prefix_cache_serves_stacks_without_state():
     sp = SamplingParams(max_tokens=4, temperature=0.0, ignore_eos=True)
     first = llm.generate(prompt_token_ids=[p], sampling_params=sp)[0].output
     again = llm.generate(prompt_token_ids=[p], sampling_params=sp)[0].output
-    assert first == again == oracle_greedy(raw, t, p, 4) and llm.engine.stats["prefix_hit_tokens"] == 32
+    assert first == again == oracle_greedy(O, raw, t, p, 4) and llm.engine.stats["prefix_hit_tokens"] == 32
 
 
 def test_loglikelihoods_and_checkpoint_round_trip(tmp_path):
