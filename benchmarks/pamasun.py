@@ -10,26 +10,17 @@ bandwidth or tensor-core peak (``MEASURED_PEAKS.json``)."""
 from __future__ import annotations
 
 import json
-import time
-from pathlib import Path
 
 import torch
 
-DEV = "cuda"
+from .design_common import DEV, VOCAB, Table, engine_rates, peaks
+
 SIZES = {
     # width, ff, layers of [delta x3, attention] groups, query / kv heads x 128, delta heads x 128
     "w2048": dict(width=2048, ff=8192, groups=4, heads=16, kv=4, delta=16),
     "w4096": dict(width=4096, ff=16384, groups=2, heads=32, kv=8, delta=32),
 }
-VOCAB, DIM = 32768, 128
-
-
-def _peaks():
-    p = Path(__file__).resolve().parent.parent / "MEASURED_PEAKS.json"
-    if p.exists():
-        d = json.loads(p.read_text())
-        return float(d["hbm_gbs"]), float(d["bf16_tflops"]), "measured"
-    return 6650.0, 1590.0, "fallback"
+DIM = 128
 
 
 def pamasun_llm(s, ecfg):
@@ -80,78 +71,16 @@ def closest_llm(s, ecfg):
     return LLM(cfg, w, ecfg)
 
 
-def engine_rates(make, s, decode_rows=64, decode_new=128, prompt=1024, prompts=8):
-    """Output tok/s of a decoding batch and prompt tok/s of a prefill, through the engine."""
-    from mlxcel_b200.engine import EngineConfig, SamplingParams
-    ml = prompt + decode_new + 64
-    ecfg = EngineConfig(max_batch=decode_rows, max_num_batched_tokens=8192, prefill_chunk_alone=prompt, prefill_chunk_contended=prompt,
-                        max_prefill_seqs=8, block_size=16, num_blocks=(ml // 16 + 2) * decode_rows, max_model_len=ml, prefix_cache=False)
-    llm = make(s, ecfg)
-    g = torch.Generator().manual_seed(0)
-    draw = lambda n, ln: torch.randint(0, VOCAB, (n, ln), generator=g).tolist()            # noqa: E731
-    sp = lambda n: SamplingParams(max_tokens=n, temperature=0.0, ignore_eos=True)          # noqa: E731
-
-    def timed(n, ln, new):
-        p = draw(n, ln)
-        torch.cuda.synchronize()
-        e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
-        t0 = time.perf_counter()
-        e0.record()
-        outs = llm.generate(prompt_token_ids=p, sampling_params=sp(new))
-        e1.record()
-        torch.cuda.synchronize()
-        return e0.elapsed_time(e1) / 1e3, time.perf_counter() - t0, outs
-    for _ in range(2):                                     # kernels' first launches, decode graphs
-        timed(prompts, 64, 1), timed(decode_rows, 8, 8)
-    pre = min(timed(prompts, prompt, 1)[0] for _ in range(2))
-    # decode: the difference between two generation lengths from the same short prompts
-    short, long = min(timed(decode_rows, 8, 8)[0] for _ in range(2)), min(timed(decode_rows, 8, 8 + decode_new)[0] for _ in range(2))
-    st = llm.engine.stats
-    out = dict(prefill_tok_s=round(prompts * prompt / pre), decode_tok_s=round(decode_rows * decode_new / (long - short)),
-               decode_step_us=round((long - short) / decode_new * 1e6, 1), graph_replays=st["graph_replays"])
-    del llm
-    torch.cuda.empty_cache()
-    return out
-
-
-class Timer:
-    def __init__(self):
-        self.flush = torch.empty(256 << 20, dtype=torch.uint8, device=DEV)
-
-    def __call__(self, fn, iters=9, warm=3):
-        for _ in range(warm):
-            fn()
-        ts = []
-        for _ in range(iters):
-            self.flush.zero_()
-            e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
-            e0.record()
-            fn()
-            e1.record()
-            torch.cuda.synchronize()
-            ts.append(e0.elapsed_time(e1))
-        return sorted(ts)[len(ts) // 2] * 1e3              # us
-
-
 def kernel_rows(s, rows=64, ctx=1024, pieces=8, piece=1024):
     """(name, new kernel us, share of roofline, its counterpart, us, share) per role."""
     from mlxcel_b200 import ops
     from mlxcel_b200.ops import KVLayer, recurrent as R, stream
-    hbm, tf, _ = _peaks()
-    t = Timer()
     W, ff, Hq, Hkv, H = s["width"], s["ff"], s["heads"], s["kv"], s["delta"]
     bf = lambda *sh: torch.randn(*sh, device=DEV).to(torch.bfloat16)                       # noqa: E731
     i32 = lambda x: torch.tensor(x, dtype=torch.int32, device=DEV)                         # noqa: E731
     f32 = lambda *sh: torch.randn(*sh, device=DEV)                                         # noqa: E731
-    mem = lambda nbytes, us: round(nbytes / us / 1e3 / hbm, 3)                             # noqa: E731
-    out = []
-
-    def add(role, bound, new, new_work, old, old_work):
-        share = (lambda w, us: mem(w, us)) if bound == "hbm" else (lambda w, us: round(w / us / 1e6 / tf, 3))
-        a, b = t(new[1]), t(old[1]) if old else None
-        out.append(dict(role=role, bound=bound, kernel=new[0], us=round(a, 1), frac=share(new_work, a),
-                        counterpart=old[0] if old else None, counterpart_us=round(b, 1) if old else None,
-                        counterpart_frac=share(old_work, b) if old else None))
+    table = Table()
+    add = table.add
     # ---- row kernels (prefill and decode rows)
     for n in (rows, pieces * piece):
         h, y, w, x = f32(n, W), bf(n, W), f32(W), bf(n, W)
@@ -224,11 +153,11 @@ def kernel_rows(s, rows=64, ctx=1024, pieces=8, piece=1024):
                                                                             D=D, norm_eps=1e-6)), flops,
         ("ssm_scan (Mamba2, same state; the delta rule of the closest model runs token by token)",
          lambda: R.ssm_scan_varlen(mst, sl[:pieces], cu, z0[:pieces], mx, mdt, A, mB[:, :N], mB[:, N:])), T * H * D * N * 5)
-    return out
+    return table.rows
 
 
 def run() -> None:
-    hbm, tf, how = _peaks()
+    how = peaks()[2]
     for name, s in SIZES.items():
         for k in kernel_rows(s):
             print(json.dumps(dict(design="pamasun", size=name, peaks=how, **k)), flush=True)

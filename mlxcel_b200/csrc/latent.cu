@@ -14,9 +14,10 @@
 namespace mx {
 
 // ----------------------------------------------------------------------------- append
-constexpr int kLaThreads = 128;
+constexpr int kLaThreads = 256;
 
-template <typename T>
+// One CTA per token, V elements per access.
+template <typename T, int V>
 __global__ void __launch_bounds__(kLaThreads)
 latent_append_kernel(T* __restrict__ a, long long ld, const int* __restrict__ positions, const int* __restrict__ slots,
                      const float* __restrict__ inv_freq, float mscale, const float* __restrict__ qw,
@@ -26,24 +27,33 @@ latent_append_kernel(T* __restrict__ a, long long ld, const int* __restrict__ po
   pdl_wait();
   const int t = blockIdx.x;
   T* row = a + static_cast<size_t>(t) * ld;
+  const int slot = slots[t];
+  const float pos = static_cast<float>(positions[t]);
   float s[2] = {0.f, 0.f};
-  for (int i = threadIdx.x; i < Q + C; i += kLaThreads) {
-    const float f = to_f(row[i]);
-    s[i < Q ? 0 : 1] += f * f;
+#pragma unroll 4
+  for (int i = threadIdx.x * V; i < Q + C; i += kLaThreads * V) {
+    float f[V];
+    load_v<V>(row + i, f);
+#pragma unroll
+    for (int e = 0; e < V; ++e) s[i < Q ? 0 : 1] += f[e] * f[e];
   }
   block_sums<2>(s, red);
-  if (Q > 0) {
-    const float r = 1.f / sqrtf(s[0] / Q + eps);
-    for (int i = threadIdx.x; i < Q; i += kLaThreads) row[i] = from_f<T>(to_f(row[i]) * r * qw[i]);
+  const float rq = 1.f / sqrtf(s[0] / max(Q, 1) + eps), rc = 1.f / sqrtf(s[1] / C + eps);
+  T* dst = pool + static_cast<size_t>(max(slot, 0)) * (C + R);
+#pragma unroll 4
+  for (int i = threadIdx.x * V; i < Q + C; i += kLaThreads * V) {
+    const bool query = i < Q;
+    if (!query && slot < 0) break;
+    float f[V], w[V];
+    load_v<V>(row + i, f);
+    load_v<V>(query ? qw + i : cw + (i - Q), w);
+#pragma unroll
+    for (int e = 0; e < V; ++e) f[e] *= (query ? rq : rc) * w[e];
+    store_v<V>(query ? row + i : dst + (i - Q), f);
   }
-  const int slot = slots[t];
   if (slot < 0) return;
-  const float r = 1.f / sqrtf(s[1] / C + eps);
-  T* dst = pool + static_cast<size_t>(slot) * (C + R);
-  for (int i = threadIdx.x; i < C; i += kLaThreads) dst[i] = from_f<T>(to_f(row[Q + i]) * r * cw[i]);
-  const float pos = static_cast<float>(positions[t]);
   const int half = R / 2;
-  for (int i = threadIdx.x; i < half; i += kLaThreads) {
+  for (int i = kLaThreads - 1 - threadIdx.x; i < half; i += kLaThreads) {      // (the last threads: they have the fewest columns)
     float sn, cs;
     sincosf(pos * inv_freq[i], &sn, &cs);
     cs *= mscale, sn *= mscale;
@@ -112,7 +122,7 @@ latent_gather_kernel(const uint8_t* __restrict__ pool, const int* __restrict__ t
 // cp.async. Per tile: the eight warps take 16 tokens x half of the row's columns each for the scores (the halves are
 // added in shared memory), the softmax runs over 16 threads per head, and for the values each warp owns an eighth of the
 // latent columns of the SAME shared tile. Weights enter the value product as two bf16 terms (rounded weight and
-// remainder). The last split to arrive merges.
+// remainder). Splits leave fp32 partial results for a merge kernel (one CTA per head row).
 constexpr float kLdLog2e = 1.4426950408889634f;
 constexpr int kLdThreads = 256, kLdKeys = 64, kLdMaxRow = 576, kLdMaxLatent = 512;
 constexpr int kLdSRow = kLdKeys + 4;      // floats per score row
@@ -127,7 +137,6 @@ struct LatentDecodeParams {
   __nv_bfloat16* out;                     // [B, H, C]
   float* scratch_o;                       // [B, head tiles, splits, 16 MT, C]
   float* scratch_ml;                      // [B, head tiles, splits, 16 MT, 2]
-  int* counters;                          // [B * head tiles]
   int H, W, C, block_size, max_blocks, num_splits, head_tiles;
   float scale_log2;
 };
@@ -147,7 +156,6 @@ __global__ void __launch_bounds__(kLdThreads, 1) latent_decode_kernel(const Late
   float* s_s = reinterpret_cast<float*>(k_s + 2 * kLdKeys * RS);                       // [2 halves][HR][kLdSRow]
   __nv_bfloat16* p_s = reinterpret_cast<__nv_bfloat16*>(s_s + 2 * HR * kLdSRow);       // [2 terms][HR][kLdPRow]
   __shared__ float alpha_s[HR], m_s[HR], l_s[HR];
-  __shared__ int last_s;
   pdl_trigger();
 
   const int split = blockIdx.x % p.num_splits, bt = blockIdx.x / p.num_splits;
@@ -207,24 +215,35 @@ __global__ void __launch_bounds__(kLdThreads, 1) latent_decode_kernel(const Late
       // ---- scores: tokens kg .. + 15, columns of half kh
       const int kg = (warp & 3) * 16, kh = warp >> 2;
       const int k0 = kh == 0 ? 0 : KS / 2, k1 = kh == 0 ? KS / 2 : KS;
-      float sc[MT][2][4];
+      float sc[MT][2][4], sd[MT][2][4];   // even and odd steps: independent accumulation chains
 #pragma unroll
       for (int m = 0; m < MT; ++m)
 #pragma unroll
-        for (int e = 0; e < 8; ++e) sc[m][e >> 2][e & 3] = 0.f;
+        for (int e = 0; e < 8; ++e) sc[m][e >> 2][e & 3] = sd[m][e >> 2][e & 3] = 0.f;
       const uint32_t ka = kb + (kg + (lane & 7) + (lane >> 4) * 8) * RS + ((lane >> 3) & 1) * 16;
       const uint32_t qa = smem_u32(q_s) + ((lane & 7) + ((lane >> 3) & 1) * 8) * RS + (lane >> 4) * 16;
-      for (int kk = k0; kk < k1; ++kk) {
+      const auto step = [&](int kk, float(&acc)[MT][2][4]) {
         uint32_t kf[4];
         ldmatrix_x4(kf, ka + kk * 32);
 #pragma unroll
         for (int m = 0; m < MT; ++m) {
           uint32_t qf[4];
           ldmatrix_x4(qf, qa + m * 16 * RS + kk * 32);
-          mma_bf16_16816(sc[m][0], qf, kf[0], kf[1]);
-          mma_bf16_16816(sc[m][1], qf, kf[2], kf[3]);
+          mma_bf16_16816(acc[m][0], qf, kf[0], kf[1]);
+          mma_bf16_16816(acc[m][1], qf, kf[2], kf[3]);
         }
+      };
+      int kk = k0;
+#pragma unroll 3
+      for (; kk + 1 < k1; kk += 2) {
+        step(kk, sc);
+        step(kk + 1, sd);
       }
+      if (kk < k1) step(kk, sc);
+#pragma unroll
+      for (int m = 0; m < MT; ++m)
+#pragma unroll
+        for (int e = 0; e < 8; ++e) sc[m][e >> 2][e & 3] += sd[m][e >> 2][e & 3];
 #pragma unroll
       for (int m = 0; m < MT; ++m)
 #pragma unroll
@@ -295,7 +314,7 @@ __global__ void __launch_bounds__(kLdThreads, 1) latent_decode_kernel(const Late
 #pragma unroll
       for (int n = 0; n < 4; ++n) {
         const int nt = warp + n * 8;
-        if (nt >= NT) break;
+        if (nt >= NT) continue;           // (the same for the whole warp)
         uint32_t vf[4];
         ldmatrix_x4_trans(vf, va + kk * 16 * RS + nt * 32);
 #pragma unroll
@@ -333,38 +352,46 @@ __global__ void __launch_bounds__(kLdThreads, 1) latent_decode_kernel(const Late
     p.scratch_ml[(part * HR + threadIdx.x) * 2] = m_s[threadIdx.x];
     p.scratch_ml[(part * HR + threadIdx.x) * 2 + 1] = l_s[threadIdx.x];
   }
-  __threadfence();
-  __syncthreads();
-  if (threadIdx.x == 0) {
-    const int last = atomicAdd(&p.counters[bt], 1) == p.num_splits - 1;
-    if (last) atomicExch(&p.counters[bt], 0);
-    last_s = last;
+}
+
+// out[b, h, :] from the partial results of its splits; one CTA per (sequence, head), two columns per thread.
+__global__ void __launch_bounds__(256) latent_merge_kernel(const LatentDecodeParams p, int HR) {
+  __shared__ float f_s[64];
+  __shared__ float inv_s;
+  pdl_trigger();
+  pdl_wait();
+  const int b = blockIdx.x / p.H, h = blockIdx.x - b * p.H, ht = h / HR, r = h - ht * HR;
+  const size_t base = (static_cast<size_t>(b) * p.head_tiles + ht) * p.num_splits;
+  if (threadIdx.x < 32) {
+    float m[2], l[2], mx = -INFINITY;
+#pragma unroll
+    for (int i = 0; i < 2; ++i) {
+      const int s = threadIdx.x + i * 32;
+      m[i] = s < p.num_splits ? p.scratch_ml[((base + s) * HR + r) * 2] : -INFINITY;
+      l[i] = s < p.num_splits ? p.scratch_ml[((base + s) * HR + r) * 2 + 1] : 0.f;
+      mx = fmaxf(mx, m[i]);
+    }
+    mx = warp_max(mx);
+    float sum = 0.f;
+#pragma unroll
+    for (int i = 0; i < 2; ++i) {
+      const float f = m[i] > -INFINITY ? exp2f(m[i] - mx) : 0.f;
+      f_s[threadIdx.x + i * 32] = f;
+      sum += f * l[i];
+    }
+    sum = warp_sum(sum);
+    if (threadIdx.x == 0) inv_s = sum > 0.f ? 1.f / sum : 0.f;
   }
   __syncthreads();
-  if (!last_s) return;
-  __threadfence();
-  const size_t base = static_cast<size_t>(bt) * p.num_splits;
-  float* f_s = s_s;                       // [splits][HR]: factor of every split's partial result (splits <= 64)
-  for (int r = threadIdx.x; r < heads; r += kLdThreads) {
-    float m = -INFINITY, l = 0.f;
-    for (int s = 0; s < p.num_splits; ++s) m = fmaxf(m, __ldcg(&p.scratch_ml[((base + s) * HR + r) * 2]));
+  for (int c = threadIdx.x * 2; c < p.C; c += 512) {
+    const float* o = p.scratch_o + (base * HR + r) * static_cast<size_t>(p.C) + c;
+    float x = 0.f, y = 0.f;
+#pragma unroll 8
     for (int s = 0; s < p.num_splits; ++s) {
-      const float ms = __ldcg(&p.scratch_ml[((base + s) * HR + r) * 2]);
-      const float f = ms > -INFINITY ? exp2f(ms - m) : 0.f;
-      f_s[s * HR + r] = f;
-      l += f * __ldcg(&p.scratch_ml[((base + s) * HR + r) * 2 + 1]);
+      const float2 v = *reinterpret_cast<const float2*>(o + static_cast<size_t>(s) * HR * p.C);
+      x += f_s[s] * v.x, y += f_s[s] * v.y;
     }
-    l_s[r] = l > 0.f ? 1.f / l : 0.f;
-  }
-  __syncthreads();
-  for (int i = threadIdx.x; i < heads * p.C; i += kLdThreads) {
-    const int r = i / p.C, c = i - r * p.C;
-    float v = 0.f;
-    for (int s = 0; s < p.num_splits; ++s) {
-      const float f = f_s[s * HR + r];
-      if (f > 0.f) v += f * __ldcg(&p.scratch_o[((base + s) * HR + r) * static_cast<size_t>(p.C) + c]);
-    }
-    p.out[(static_cast<size_t>(b) * p.H + h0 + r) * p.C + c] = __float2bfloat16(v * l_s[r]);
+    *reinterpret_cast<uint32_t*>(p.out + (static_cast<size_t>(b) * p.H + h) * p.C + c) = pack_bf16(x * inv_s, y * inv_s);
   }
 }
 
@@ -378,14 +405,16 @@ static int launch_latent_decode(const LatentDecodeParams& p, int grid, cudaStrea
     prefer_max_shared(kern);
     configured = true;
   }
-  return static_cast<int>(launch_kernel(kern, dim3(grid), dim3(kLdThreads), ld_smem(p.W, MT), st, p));
+  cudaError_t e = launch_kernel(kern, dim3(grid), dim3(kLdThreads), ld_smem(p.W, MT), st, p);
+  if (e != cudaSuccess || p.num_splits == 1) return static_cast<int>(e);
+  return static_cast<int>(launch_kernel(latent_merge_kernel, dim3(grid / p.num_splits / p.head_tiles * p.H), dim3(256), 0, st, p, 16 * MT));
 }
 
 }  // namespace mx
 
 using namespace mx;
 
-constexpr int kLatentCounters = 65536;    // the region the paged decode kernels share (see mx_paged_decode_scratch_floats)
+constexpr int kLatentScratch0 = 65536;    // the scratch buffer starts with the counters of the paged decode kernels
 
 // a: rows q_latent [Q] | latent [C] | key part [R], ld elements apart. Q may be 0.
 extern "C" int mx_latent_append(void* a, long long ld, const void* positions, const void* slots, const void* inv_freq, float mscale,
@@ -394,13 +423,20 @@ extern "C" int mx_latent_append(void* a, long long ld, const void* positions, co
   if (n <= 0) return 0;
   if (Q < 0 || C <= 0 || R < 0 || R % 2 || (Q > 0 && qw == nullptr)) return -1;
   auto st = static_cast<cudaStream_t>(stream);
-#define MX_LA(T)                                                                                                              \
-  return static_cast<int>(launch_kernel(latent_append_kernel<T>, dim3(n), dim3(kLaThreads), 0, st, static_cast<T*>(a), ld,    \
+  const size_t ab = fp32 ? 16 : 8;
+  const bool vec = Q % 4 == 0 && C % 4 == 0 && R % 4 == 0 && ld % 4 == 0 && aligned_to(a, ab) && aligned_to(pool, ab) && aligned_to(qw, 16) &&
+                   aligned_to(cw, 16);
+#define MX_LA(T, V)                                                                                                           \
+  return static_cast<int>(launch_kernel(latent_append_kernel<T, V>, dim3(n), dim3(kLaThreads), 0, st, static_cast<T*>(a), ld,    \
                                         static_cast<const int*>(positions), static_cast<const int*>(slots),                   \
                                         static_cast<const float*>(inv_freq), mscale, static_cast<const float*>(qw),           \
                                         static_cast<const float*>(cw), static_cast<T*>(pool), Q, C, R, eps))
-  if (fp32) MX_LA(float);
-  MX_LA(__nv_bfloat16);
+  if (fp32) {
+    if (vec) MX_LA(float, 4);
+    MX_LA(float, 1);
+  }
+  if (vec) MX_LA(__nv_bfloat16, 4);
+  MX_LA(__nv_bfloat16, 1);
 #undef MX_LA
 }
 
@@ -430,11 +466,11 @@ extern "C" int mx_latent_gather(const void* pool, const void* tables, const void
                                         unit, block_size, max_blocks));
 }
 
-// Heads per CTA tile and the scratch floats of a call (counters included).
+// Heads per CTA tile and the scratch floats of a call.
 extern "C" int mx_latent_head_tile(int H) { return H > 16 ? 32 : 16; }
 extern "C" long long mx_latent_decode_scratch_floats(int B, int H, int C, int num_splits) {
   const int hr = mx_latent_head_tile(H);
-  return kLatentCounters + static_cast<long long>(B) * ((H + hr - 1) / hr) * hr * num_splits * (C + 2);
+  return kLatentScratch0 + static_cast<long long>(B) * ((H + hr - 1) / hr) * hr * num_splits * (C + 2);
 }
 
 // Absorbed queries [B, H, W] (token stride q_stride) over the latent pool -> out [B, H, C]. bf16; W at most 576, C at most
@@ -459,9 +495,8 @@ extern "C" int mx_latent_decode(const void* q, long long q_stride, const void* p
   p.head_tiles = (H + hr - 1) / hr;
   p.scale_log2 = scale * kLdLog2e;
   const long long pairs = static_cast<long long>(B) * p.head_tiles;
-  if (pairs > kLatentCounters || pairs * num_splits > 0x7fffffffll) return -1;
-  p.counters = reinterpret_cast<int*>(scratch);
-  p.scratch_ml = scratch + kLatentCounters;
+  if (pairs * num_splits > 0x7fffffffll || static_cast<long long>(B) * H > 0x7fffffffll) return -1;
+  p.scratch_ml = scratch + kLatentScratch0;
   p.scratch_o = p.scratch_ml + pairs * num_splits * hr * 2;
   const int grid = static_cast<int>(pairs * num_splits);
   auto st = static_cast<cudaStream_t>(stream);

@@ -12,7 +12,7 @@ namespace mx {
 
 constexpr int kRnWarps = 8;
 
-// One CTA per token; the token's cosines and sines are computed once into shared memory, then a warp takes every
+// One CTA per token (several, over the heads, when there are few tokens); the token's cosines and sines are computed once into shared memory, then a warp takes every
 // eighth head: it stages the head in shared memory (the partner of a dimension sits in another lane), rotates,
 // sums squares and writes. `unit`: divide by the root mean square (mean over D, eps inside the root).
 template <typename T, int V>
@@ -41,7 +41,7 @@ rope_norm_append_kernel(T* __restrict__ qkv, long long ld, const int* __restrict
   const int slot = slots[t];
   const int blk = slot >= 0 ? slot / block_size : 0, off = slot >= 0 ? slot - blk * block_size : 0;
   const int nv = values_are_keys ? 0 : Hkv;
-  for (int hd = warp; hd < Hq + Hkv + nv; hd += kRnWarps) {
+  for (int hd = blockIdx.y * kRnWarps + warp; hd < Hq + Hkv + nv; hd += kRnWarps * gridDim.y) {
     if (hd >= Hq && slot < 0) break;
     if (hd >= Hq + Hkv) {                  // plain value head
       const int g = hd - Hq - Hkv;
@@ -109,7 +109,8 @@ extern "C" int mx_rope_norm_append(void* qkv, long long ld, const void* position
   const size_t ab = fp32 ? 16 : 8;
   const bool vec = Dk % 4 == 0 && Dv % 4 == 0 && ld % 4 == 0 && aligned_to(qkv, ab) && aligned_to(k_pool, ab) && aligned_to(v_pool, ab);
   auto st = static_cast<cudaStream_t>(stream);
-  const dim3 grid(n), block(kRnWarps * 32);
+  const int groups = (Hq + (values_are_keys ? 1 : 2) * Hkv + kRnWarps - 1) / kRnWarps;
+  const dim3 grid(n, n >= 512 ? 1 : groups), block(kRnWarps * 32);
 #define MX_RN(T, V)                                                                                                         \
   return static_cast<int>(launch_kernel(rope_norm_append_kernel<T, V>, grid, block, smem, st, static_cast<T*>(qkv), ld,     \
                                         static_cast<const int*>(positions), static_cast<const int*>(slots),                 \

@@ -233,12 +233,18 @@ glu_rows_kernel(const T* __restrict__ z, long long ld, T* __restrict__ out, int 
   store_v<V>(out + row * dim + c, g);
 }
 
+template <int V>
 __global__ void __launch_bounds__(256) softcap_rows_kernel(float* __restrict__ x, long long n, float cap) {
   pdl_trigger();
   pdl_wait();
   const float inv = 1.f / cap;
-  for (long long i = static_cast<long long>(blockIdx.x) * blockDim.x + threadIdx.x; i < n; i += static_cast<long long>(gridDim.x) * blockDim.x)
-    x[i] = cap * tanhf(x[i] * inv);
+  for (long long i = (static_cast<long long>(blockIdx.x) * blockDim.x + threadIdx.x) * V; i < n; i += static_cast<long long>(gridDim.x) * blockDim.x * V) {
+    float f[V];
+    load_v<V>(x + i, f);
+#pragma unroll
+    for (int e = 0; e < V; ++e) f[e] = cap * tanhf(f[e] * inv);
+    store_v<V>(x + i, f);
+  }
 }
 
 // Rows of q | k | v (| more), `ld` elements apart. One CTA per token; a warp takes every eighth of the Hq
@@ -478,7 +484,8 @@ extern "C" int mx_glu_rows(const void* z, long long ld, void* out, int n, int di
 extern "C" int mx_softcap_rows(void* x, long long n, float cap, void* stream) {
   if (n <= 0) return 0;
   if (!(cap > 0.f)) return -1;
-  const long long blocks = (n + 255) / 256;
-  return static_cast<int>(launch_kernel(softcap_rows_kernel, dim3(static_cast<unsigned>(blocks < 4096 ? blocks : 4096)), dim3(256), 0,
+  const bool vec = n % 4 == 0 && aligned_to(x, 16);
+  const long long blocks = (n + (vec ? 1023 : 255)) / (vec ? 1024 : 256);
+  return static_cast<int>(launch_kernel(vec ? softcap_rows_kernel<4> : softcap_rows_kernel<1>, dim3(static_cast<unsigned>(blocks < 4096 ? blocks : 4096)), dim3(256), 0,
                                         static_cast<cudaStream_t>(stream), static_cast<float*>(x), n, cap));
 }

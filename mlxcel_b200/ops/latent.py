@@ -102,7 +102,7 @@ def latent_attention(q, kv, tables, lens, cu, out, *, H: int, C: int, scale: flo
                                      scratch.data_ptr(), rows, H, W, C, kv.block_size, tables.shape[1], float(scale), splits,
                                      _lib.stream())
         if rc != NOT_COVERED:
-            _lib.count_launch()
+            _lib.count_launch(2 if splits > 1 else 1)
             _lib.check(rc, "mx_latent_decode")
             return
     if cu is None:
