@@ -8,6 +8,7 @@
 //                   columns of the same rows as values; every row is read once for all heads
 // Norms, angles, scores, softmax and accumulation are fp32.
 #include "api.h"
+#include "latent.cuh"
 #include "mma_sync.cuh"
 #include "typed.cuh"
 
@@ -127,19 +128,6 @@ constexpr float kLdLog2e = 1.4426950408889634f;
 constexpr int kLdThreads = 256, kLdKeys = 64, kLdMaxRow = 576, kLdMaxLatent = 512;
 constexpr int kLdSRow = kLdKeys + 4;      // floats per score row
 constexpr int kLdPRow = kLdKeys + 8;      // bf16 per weight row (an odd number of 16-byte chunks)
-
-struct LatentDecodeParams {
-  const __nv_bfloat16* q;
-  long long q_stride;                     // between tokens; heads are W apart
-  const __nv_bfloat16* pool;
-  const int* block_tables;
-  const int* context_lens;
-  __nv_bfloat16* out;                     // [B, H, C]
-  float* scratch_o;                       // [B, head tiles, splits, 16 MT, C]
-  float* scratch_ml;                      // [B, head tiles, splits, 16 MT, 2]
-  int H, W, C, block_size, max_blocks, num_splits, head_tiles;
-  float scale_log2;
-};
 
 __host__ __device__ inline int ld_row_bytes(int W) { return (W + 15) / 16 * 32 + 16; }   // an odd number of 16-byte chunks
 __host__ inline int ld_smem(int W, int mt) {
@@ -355,12 +343,12 @@ __global__ void __launch_bounds__(kLdThreads, 1) latent_decode_kernel(const Late
 }
 
 // out[b, h, :] from the partial results of its splits; one CTA per (sequence, head), two columns per thread.
-__global__ void __launch_bounds__(256) latent_merge_kernel(const LatentDecodeParams p, int HR) {
+__global__ void __launch_bounds__(256) latent_merge_kernel(const LatentDecodeParams p) {
   __shared__ float f_s[64];
   __shared__ float inv_s;
   pdl_trigger();
   pdl_wait();
-  const int b = blockIdx.x / p.H, h = blockIdx.x - b * p.H, ht = h / HR, r = h - ht * HR;
+  const int HR = p.head_tile, b = blockIdx.x / p.H, h = blockIdx.x - b * p.H, ht = h / HR, r = h - ht * HR;
   const size_t base = (static_cast<size_t>(b) * p.head_tiles + ht) * p.num_splits;
   if (threadIdx.x < 32) {
     float m[2], l[2], mx = -INFINITY;
@@ -389,7 +377,7 @@ __global__ void __launch_bounds__(256) latent_merge_kernel(const LatentDecodePar
 #pragma unroll 8
     for (int s = 0; s < p.num_splits; ++s) {
       const float2 v = *reinterpret_cast<const float2*>(o + static_cast<size_t>(s) * HR * p.C);
-      x += f_s[s] * v.x, y += f_s[s] * v.y;
+      x += f_s[s] > 0.f ? f_s[s] * v.x : 0.f, y += f_s[s] > 0.f ? f_s[s] * v.y : 0.f;   // (a split without tokens wrote nothing)
     }
     *reinterpret_cast<uint32_t*>(p.out + (static_cast<size_t>(b) * p.H + h) * p.C + c) = pack_bf16(x * inv_s, y * inv_s);
   }
@@ -405,9 +393,7 @@ static int launch_latent_decode(const LatentDecodeParams& p, int grid, cudaStrea
     prefer_max_shared(kern);
     configured = true;
   }
-  cudaError_t e = launch_kernel(kern, dim3(grid), dim3(kLdThreads), ld_smem(p.W, MT), st, p);
-  if (e != cudaSuccess || p.num_splits == 1) return static_cast<int>(e);
-  return static_cast<int>(launch_kernel(latent_merge_kernel, dim3(grid / p.num_splits / p.head_tiles * p.H), dim3(256), 0, st, p, 16 * MT));
+  return static_cast<int>(launch_kernel(kern, dim3(grid), dim3(kLdThreads), ld_smem(p.W, MT), st, p));
 }
 
 }  // namespace mx
@@ -473,11 +459,12 @@ extern "C" long long mx_latent_decode_scratch_floats(int B, int H, int C, int nu
   return kLatentScratch0 + static_cast<long long>(B) * ((H + hr - 1) / hr) * hr * num_splits * (C + 2);
 }
 
-// Absorbed queries [B, H, W] (token stride q_stride) over the latent pool -> out [B, H, C]. bf16; W at most 576, C at most
+// Absorbed queries [B, H, W] (token stride q_stride) over the latent pool (pool_rows rows) -> out [B, H, C]. form 0: the
+// tcgen05 kernel where it applies (16-token blocks), else the mma.sync one; 1: the mma.sync one. bf16; W at most 576, C at most
 // 512, multiples of 8. -10 = not covered (use mx_paged_attention_any).
-extern "C" int mx_latent_decode(const void* q, long long q_stride, const void* pool, const void* block_tables,
+extern "C" int mx_latent_decode(const void* q, long long q_stride, const void* pool, long long pool_rows, const void* block_tables,
                                 const void* context_lens, void* out, float* scratch, int B, int H, int W, int C, int block_size,
-                                int max_blocks, float scale, int num_splits, void* stream) {
+                                int max_blocks, float scale, int num_splits, int form, void* status, void* stream) {
   if (B <= 0) return 0;
   if (H <= 0 || C <= 0 || C > W || block_size <= 0) return -1;
   if (W % 8 || C % 8 || W > kLdMaxRow || C > kLdMaxLatent || q_stride % 8 || !aligned_to(q, 16) || !aligned_to(pool, 16)) return -10;
@@ -492,7 +479,7 @@ extern "C" int mx_latent_decode(const void* q, long long q_stride, const void* p
   p.context_lens = static_cast<const int*>(context_lens);
   p.out = static_cast<__nv_bfloat16*>(out);
   p.H = H, p.W = W, p.C = C, p.block_size = block_size, p.max_blocks = max_blocks, p.num_splits = num_splits;
-  p.head_tiles = (H + hr - 1) / hr;
+  p.head_tile = hr, p.head_tiles = (H + hr - 1) / hr;
   p.scale_log2 = scale * kLdLog2e;
   const long long pairs = static_cast<long long>(B) * p.head_tiles;
   if (pairs * num_splits > 0x7fffffffll || static_cast<long long>(B) * H > 0x7fffffffll) return -1;
@@ -500,5 +487,8 @@ extern "C" int mx_latent_decode(const void* q, long long q_stride, const void* p
   p.scratch_o = p.scratch_ml + pairs * num_splits * hr * 2;
   const int grid = static_cast<int>(pairs * num_splits);
   auto st = static_cast<cudaStream_t>(stream);
-  return hr == 32 ? launch_latent_decode<2>(p, grid, st) : launch_latent_decode<1>(p, grid, st);
+  int rc = form == 1 ? -10 : latent_decode_tc(p, B, pool_rows, static_cast<int*>(status), st);
+  if (rc == -10) rc = hr == 32 ? launch_latent_decode<2>(p, grid, st) : launch_latent_decode<1>(p, grid, st);
+  if (rc != 0 || num_splits == 1) return rc;
+  return static_cast<int>(launch_kernel(latent_merge_kernel, dim3(static_cast<unsigned>(B) * H), dim3(256), 0, st, p));
 }

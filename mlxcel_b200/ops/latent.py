@@ -17,7 +17,7 @@ _SIG.update({
     "mx_latent_q_rope": [_vp, _ll, _i, _vp, _ll, _i, _vp, _vp, _f, _i, _i, _i, _i, _vp],
     "mx_latent_gather": [_vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _vp],
     "mx_latent_head_tile": [_i],
-    "mx_latent_decode": [_vp, _ll, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _f, _i, _vp],
+    "mx_latent_decode": [_vp, _ll, _vp, _ll, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _f, _i, _i, _vp, _vp],
     "mx_latent_prefill": [_vp, _ll, _vp, _vp, _ll, _vp, _ll, _vp, _vp, _vp, _vp, _ll] + [_i] * 7 + [_f, _vp, _vp],
 })
 
@@ -80,10 +80,12 @@ def latent_attention_ref(q, kv, tables, lens, cu, *, H: int, C: int, scale: floa
     return out
 
 
-def latent_attention(q, kv, tables, lens, cu, out, *, H: int, C: int, scale: float, max_len: int = 0, force_any: bool = False) -> None:
+def latent_attention(q, kv, tables, lens, cu, out, *, H: int, C: int, scale: float, max_len: int = 0, force_any: bool = False,
+                     form: int = 0) -> None:
     """Causal attention of absorbed query rows [rows, H * (C + R)] over the latent pool into ``out`` [rows, H * C].
-    ``cu=None`` says one row per sequence (decode): bf16 rows of at most 576 (latent 512) take the tensor-core kernel, which
-    reads every pool row once for up to 32 heads; the rest the SIMT one."""
+    ``cu=None`` says one row per sequence (decode): bf16 rows of at most 576 (latent 512) take the tensor-core kernels, which
+    read every pool row once for up to 32 heads (tcgen05 for pages of 16 tokens; ``form`` 1: the mma.sync one everywhere); the
+    rest the SIMT one."""
     rows, W = q.shape[0], kv.k.shape[-1]
     if rows == 0:
         return
@@ -98,9 +100,9 @@ def latent_attention(q, kv, tables, lens, cu, out, *, H: int, C: int, scale: flo
         if not floats.argtypes:
             floats.argtypes, floats.restype = [_i] * 4, _ll
         scratch = _decode_scratch(q.device, int(floats(rows, H, C, splits)) if splits > 1 else 0)
-        rc = _fn("mx_latent_decode")(q.data_ptr(), q.stride(0), kv.k.data_ptr(), tables.data_ptr(), lens.data_ptr(), out.data_ptr(),
-                                     scratch.data_ptr(), rows, H, W, C, kv.block_size, tables.shape[1], float(scale), splits,
-                                     _lib.stream())
+        rc = _fn("mx_latent_decode")(q.data_ptr(), q.stride(0), kv.k.data_ptr(), kv.k.shape[0] * kv.block_size, tables.data_ptr(),
+                                     lens.data_ptr(), out.data_ptr(), scratch.data_ptr(), rows, H, W, C, kv.block_size, tables.shape[1],
+                                     float(scale), splits, form, _lib.workspace(q.device).data_ptr(), _lib.stream())
         if rc != NOT_COVERED:
             _lib.count_launch(2 if splits > 1 else 1)
             _lib.check(rc, "mx_latent_decode")

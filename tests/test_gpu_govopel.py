@@ -238,14 +238,37 @@ def test_absorbed_latent_attention(H, D, R, V, C, bs, dtype):
         if n:
             want[s] = torch.softmax(q[s].double() @ rows[s].double().T * scale, -1) @ rows[s][:, :C].double()
     kv = KVLayer(pool.to(DEV), pool[..., :0].to(DEV), None, None, bs)
-    for max_len in (100, 5000):
-        out = torch.full((len(lens), H * C), 9.0, dtype=dtype, device=DEV)
-        latent.latent_attention(q.reshape(-1, H * W).to(DEV), kv, tab.to(DEV), _i32(lens), None, out, H=H, C=C, scale=scale, max_len=max_len)
-        _close(out.view(-1, H, C), want, dtype, f32=5e-5)
     big = torch.cat([q] * 30).reshape(-1, H * W).to(DEV)                   # more rows than SMs: no split
-    out = torch.empty(big.shape[0], H * C, dtype=dtype, device=DEV)
-    latent.latent_attention(big, kv, tab.repeat(30, 1).to(DEV), _i32(lens * 30), None, out, H=H, C=C, scale=scale, max_len=700)
-    _close(out.view(30, -1, H, C), want.expand(30, -1, -1, -1), dtype, f32=5e-5)
+    for form in (0, 1):                                                    # tcgen05 where it applies; mma.sync
+        for max_len in (100, 400, 5000):
+            out = torch.full((len(lens), H * C), 9.0, dtype=dtype, device=DEV)
+            latent.latent_attention(q.reshape(-1, H * W).to(DEV), kv, tab.to(DEV), _i32(lens), None, out, H=H, C=C, scale=scale,
+                                    max_len=max_len, form=form)
+            _close(out.view(-1, H, C), want, dtype, f32=5e-5)
+        out = torch.empty(big.shape[0], H * C, dtype=dtype, device=DEV)
+        latent.latent_attention(big, kv, tab.repeat(30, 1).to(DEV), _i32(lens * 30), None, out, H=H, C=C, scale=scale, max_len=700, form=form)
+        _close(out.view(30, -1, H, C), want.expand(30, -1, -1, -1), dtype, f32=5e-5)
+    assert _lib.read_status(torch.device(DEV, 0)) == 0
+
+
+def test_latent_decode_follows_growing_scores():
+    """Scores that grow along the context by far more than the lazy rescaling's threshold, and fall again."""
+    H, C, R, n = 16, 128, 64, 1000
+    W, g = C + R, _gen(1)
+    tab, blocks = _paged([n], 16)
+    rows, q = torch.randn(n, W, generator=g), torch.zeros(1, H, W)
+    rows[:, 0] = 40 * torch.sin(torch.arange(n) / 150.0) + torch.arange(n) / 50.0
+    q[:, :, 0] = torch.linspace(-1, 1, H)
+    rows, q = rows.to(BF16), q.to(BF16)
+    pool = torch.zeros(blocks, 1, 16, W, dtype=BF16)
+    _fill(pool, tab, 0, rows[:, None])
+    want = torch.softmax(q[0].double() @ rows.double().T, -1) @ rows[:, :C].double()
+    kv = KVLayer(pool.to(DEV), pool[..., :0].to(DEV), None, None, 16)
+    for form in (0, 1):
+        for max_len in (128, 1000):
+            out = torch.empty(1, H * C, dtype=BF16, device=DEV)
+            latent.latent_attention(q.view(1, -1).to(DEV), kv, tab.to(DEV), _i32([n]), None, out, H=H, C=C, scale=1.0, max_len=max_len, form=form)
+            _close(out.view(H, C), want, BF16)
 
 
 @pytest.mark.parametrize("H,D,R,V,C,bs", [x for x in LAT if x[4] % 8 == 0])
