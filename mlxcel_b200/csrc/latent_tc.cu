@@ -6,7 +6,7 @@
 //   values  O^T [128 columns, N] += rows [64 tokens, 128 columns]^T x weights [N, 64 tokens]^T, per 128 latent columns
 //                                   (the SAME shared tile, read MN-major)
 //
-//   warp 0     TMA producer: the queries once; per tile ceil(W / 128) slots of [64 tokens][128 columns] (two 64-column
+//   warp 0 and the last two: TMA producers, taking slots in turn: the queries once; per tile ceil(W / 128) slots of [64 tokens][128 columns] (two 64-column
 //              128-byte-swizzled sub-tiles, four pool blocks each) through a ring that holds at least two tiles where it
 //              can; a slot of latent columns is free again when its value MMA has run, one of the rotated part already
 //              after the scores
@@ -30,7 +30,8 @@ bool make_tensor_map_bf16_3d(CUtensorMap* out, const void* ptr, uint64_t rows, u
 
 constexpr int kLtKeys = 64, kLtBlock = 16;
 constexpr int kLtHeads = 16;                         // heads per softmax thread
-__host__ __device__ constexpr int lt_threads(int N) { return 64 + 128 * (N / kLtHeads); }
+constexpr int kLtProducers = 3;                      // one warp's issue rate does not keep up with boxes of one pool block
+__host__ __device__ constexpr int lt_threads(int N) { return 32 * (1 + kLtProducers) + 128 * (N / kLtHeads); }
 constexpr int kLtSub = kLtKeys * 128;                // one [64 tokens][64 columns] sub-tile
 constexpr int kLtSlot = 2 * kLtSub;
 constexpr int kLtMaxSlots = 20;
@@ -103,36 +104,39 @@ latent_decode_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
   pdl_trigger();
   pdl_wait();                                        // the queries and the newest rows come from the previous kernels
 
-  if (warp == 0) {
-    // ------------------------------------------------------------------ TMA producer
+  // warps: producer, MMA issuer, softmax groups, the other producers
+  const int producer = warp == 0 ? 0 : warp - (2 + 4 * GROUPS) + 1;
+  if (warp == 0 || warp >= 2 + 4 * GROUPS) {
+    // ------------------------------------------------------------------ TMA producers
     const int* table = p.block_tables + static_cast<size_t>(b) * p.max_blocks;
     const uint64_t pol_q = l2_policy_evict_first(), pol_k = p.head_tiles > 1 ? l2_policy_evict_last() : l2_policy_evict_first();
-    if (lane == 0 && n_tiles > 0) {
+    if (warp == 0 && lane == 0 && n_tiles > 0) {
       mbar_expect_tx(q_full, subs * Q_SUB);
       for (int c = 0; c < subs; ++c) tma_load_3d(q_sm + c * Q_SUB, &map_q, q_full, c * 64, b, h0, pol_q);
     }
-    int slot = 0;
-    uint32_t phase = 0;
-    bool ok = true;
-    const int last = (len - 1) / kLtBlock;
-    for (int j = 0; j < n_tiles && ok; ++j) {
-      constexpr int BL = kLtKeys / kLtBlock;         // lanes 0-7: sub-tile lane / 4, pool block lane % 4 (past the end: the last
-      int row0 = 0;                                  // one, masked)
-      if (lane < 2 * BL) row0 = table[min((t0 + j) * BL + lane % BL, last)] * kLtBlock;
-      for (int i = 0; i < np; ++i) {
-        const int ns = min(2, subs - 2 * i);
-        if (lane == 0) {
-          ok = mbar_wait(&empty[slot], phase ^ 1u, t.status, kErrLatentProducer);
-          if (ok) mbar_expect_tx(&full[slot], ns * kLtSub);
-        }
-        ok = __shfl_sync(0xffffffffu, ok ? 1 : 0, 0) != 0;
-        if (!ok) break;
-        if (lane < BL * ns)
-          tma_load_2d(k_sm + slot * kLtSlot + (lane / BL) * kLtSub + (lane % BL) * (kLtBlock * 128), &map_pool, &full[slot],
-                      (2 * i + lane / BL) * 64, row0, pol_k);
-        __syncwarp();
-        if (++slot == t.slots) slot = 0, phase ^= 1u;
+    constexpr int BL = kLtKeys / kLtBlock;           // lanes 0-7: sub-tile lane / 4, pool block lane % 4
+    const int last = (len - 1) / kLtBlock, total = n_tiles * np;
+    const auto row_of = [&](int j) {                 // blocks past the sequence's end: the last one (masked)
+      return lane < 2 * BL && j < n_tiles ? table[min((t0 + j) * BL + lane % BL, last)] * kLtBlock : 0;
+    };
+    int cur = producer / np, row = row_of(cur), next = row_of(cur + 1);
+    for (int g = producer; g < total; g += kLtProducers) {   // this warp's slots
+      const int j = g / np, i = g - j * np, slot = g % t.slots, ns = min(2, subs - 2 * i);
+      while (cur < j) {                              // (the next tile's rows were asked for a tile ahead)
+        row = next;
+        next = row_of(++cur + 1);
       }
+      bool ok = true;
+      if (lane == 0) {
+        ok = mbar_wait(&empty[slot], (static_cast<uint32_t>(g / t.slots) & 1u) ^ 1u, t.status, kErrLatentProducer);
+        if (ok) mbar_expect_tx(&full[slot], ns * kLtSub);
+      }
+      ok = __shfl_sync(0xffffffffu, ok ? 1 : 0, 0) != 0;
+      if (!ok) break;
+      if (lane < BL * ns)
+        tma_load_2d(k_sm + slot * kLtSlot + (lane / BL) * kLtSub + (lane % BL) * (kLtBlock * 128), &map_pool, &full[slot],
+                    (2 * i + lane / BL) * 64, row, pol_k);
+      __syncwarp();
     }
   } else if (warp == 1) {
     // ------------------------------------------------------------------ MMA issuer
