@@ -186,13 +186,13 @@ def model_config(vocab, width, layers, eps=1e-5, logit_softcap=9.0):
 # page borders, sizes no tensor-core tile or vector access divides, and values that happen to be equal or one.
 CONFIGS = {
     "mixed": model_config(160, 96, [latent_spec(3, 32, 16, 24, 40, 56, 0.3, 112), attn_spec(6, 2, 48, 24, 20, 0.15, 6.0, 72),
-                                    latent_spec(5, 24, 24, 40, 24, 32, 0.25, None), attn_spec(4, 1, 32, 32, 16, 0.2, 15.0, 80, 0.7)]),
+                                    latent_spec(5, 24, 24, 40, 24, 32, 0.25, None), attn_spec(4, 1, 32, 32, 16, 0.2, 14.0, 80, 0.7)]),
     "odd": model_config(101, 75, [attn_spec(3, 3, 20, 10, 13, 0.3, 4.0, 50), latent_spec(3, 9, 6, 11, 17, 13, 0.5, 33, 3.0),
                                   attn_spec(5, 1, 33, 22, 1, 0.1, 2.0, None, scaling=None)], eps=1e-3, logit_softcap=25.0),
     "attention_only": model_config(128, 64, [attn_spec(2, 2, 64, 64, 64, 0.125, 10.0, 64, scaling=(1.0, 64, 1.0, 1.0)),
                                              attn_spec(8, 1, 16, 2, 129, 0.6, 30.0, 96, base=10.0, scaling=(40.0, 50, 32.0, 1.0))]),
     "latent_only": model_config(96, 64, [latent_spec(1, 8, 8, 8, 8, 8, 0.9, 64), latent_spec(8, 64, 64, 64, 64, 64, 0.12, 64, 1.0),
                                          latent_spec(2, 16, 2, 72, 120, 104, 0.4, None)]),
-    "wide": model_config(264, 256, [latent_spec(20, 128, 64, 128, 96, 512, 0.1, 320), attn_spec(10, 2, 128, 64, 200, 0.1, 20.0, 256),
+    "wide": model_config(264, 256, [latent_spec(20, 128, 64, 128, 96, 512, 0.1, 320), attn_spec(10, 2, 128, 64, 184, 0.1, 18.0, 256),
                                     latent_spec(4, 96, 40, 80, 160, 200, 0.12, 192)]),
 }
