@@ -38,6 +38,7 @@ NVCC_FLAGS = [
 MODEL_UNITS = {
     "govopel": ("attention", "attention_tc", "gemm", "latent", "latent_tc", "misc", "rope_norm", "sampling", "simt", "stream_norm"),
     "pamasun": ("attention", "attention_tc", "delta_rule", "gemm", "misc", "sampling", "simt", "stream_norm"),
+    "vavadra": ("attention", "attention_tc", "gated_delta", "gemm", "latent", "latent_tc", "misc", "moe", "sampling", "simt", "stream_norm"),
 }
 
 

@@ -1094,7 +1094,7 @@ def cmd_inspect(a):
 
 
 _HYBRID = {"nemotron_h", "granitemoehybrid", "jamba", "qwen3_next", "qwen3_5", "qwen3_5_text", "qwen3_5_moe",
-           "qwen3_5_moe_text", "falcon_h1", "lfm2", "lfm2_moe", "recurrent_gemma", "pamasun", "govopel"}
+           "qwen3_5_moe_text", "falcon_h1", "lfm2", "lfm2_moe", "recurrent_gemma", "pamasun", "govopel", "vavadra"}
 _STATE_SPACE = {"mamba", "mamba2"}
 _CHECKED_BY_READING = {"internlm3", "minicpm", "mimo", "yi", "kimi_k2", "deepseek"}       # no independent implementation at hand
 _CHECKED_BY_LAYOUT = {"internlm2", "baichuan", "exaone", "telechat3"}                                 # round trip against the Llama form
@@ -1116,7 +1116,7 @@ def arch_catalog() -> dict:
             how = f"transformers logits (as {name}_text)"
         if name == "deepseek_v32":
             how = "transformers logits (as glm_moe_dsa)"
-        if name in ("pamasun", "govopel"):
+        if name in ("pamasun", "govopel", "vavadra"):
             how = "a plain PyTorch statement of the model (no library has it)"
         if name == "dbrx":
             how = "a plain PyTorch statement of the model (the transformers implementation is not usable)"
@@ -1174,6 +1174,11 @@ def cmd_random_init(a):
     if cfg.model_type == "govopel":
         from .models.govopel import random_govopel_tensors, save_govopel_checkpoint
         save_govopel_checkpoint(a.out, cfg, random_govopel_tensors(cfg, seed=a.seed))
+        print("wrote", a.out)
+        return
+    if cfg.model_type == "vavadra":
+        from .models.vavadra import random_vavadra_tensors, save_vavadra_checkpoint
+        save_vavadra_checkpoint(a.out, cfg, random_vavadra_tensors(cfg, seed=a.seed))
         print("wrote", a.out)
         return
     w = random_weights(cfg, seed=a.seed, dtype=torch.bfloat16)

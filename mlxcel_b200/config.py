@@ -1292,6 +1292,18 @@ def _lfm2(c: ModelConfig, raw: dict) -> None:
     c.layer_types = None
 
 
+def _looped_runs(c: ModelConfig, loop: dict | None, n: int) -> list[int]:
+    """Layer index of every run in order; layers ``start .. stop - 1`` run ``times`` times in a row."""
+    runs = list(range(n))
+    if not loop:
+        return runs
+    a, b, times = int(loop["start"]), int(loop["stop"]), int(loop["times"])
+    if not (0 <= a <= b <= n) or times < 0:
+        raise ValueError(f"loop {loop} does not fit {n} layers")
+    c.extra["loop"] = dict(start=a, stop=b, times=times)
+    return runs[:a] + runs[a:b] * times + runs[b:]
+
+
 def _pamasun(c: ModelConfig, raw: dict) -> None:
     """Pamasun: an explicit layer list (attention or generalized-delta mixer, dense MLP or none), every
     sub-layer normalised on both sides with a layer scale, and optionally a run of layers repeated with
@@ -1319,15 +1331,8 @@ def _pamasun(c: ModelConfig, raw: dict) -> None:
             mlp = dict(kind="dense", ff=int(mlp["ff"]))
         specs.append(dict(type=kind, mixer=m, mlp=mlp))
     n = len(specs)
-    runs = list(range(n))
-    loop = raw.get("loop")
-    if loop:
-        a, b, times = int(loop["start"]), int(loop["stop"]), int(loop["times"])
-        if not (0 <= a <= b <= n) or times < 0:
-            raise ValueError(f"loop {loop} does not fit {n} layers")
-        runs = runs[:a] + runs[a:b] * times + runs[b:]
-        c.extra["loop"] = dict(start=a, stop=b, times=times)
-    c.extra["layer_specs"], c.extra["layer_runs"] = specs, runs
+    c.extra["layer_specs"], c.extra["layer_runs"] = specs, _looped_runs(c, raw.get("loop"), n)
+    runs = c.extra["layer_runs"]
     c.num_hidden_layers = n
     att = [specs[i]["mixer"] for i in runs if specs[i]["type"] == "attention"]
     c.extra["kv_geometry"] = [(m["kv_heads"], m["dim"], m["vdim"]) for m in att]
@@ -1394,6 +1399,70 @@ def _govopel(c: ModelConfig, raw: dict) -> None:
     c.intermediate_size = max([s["mlp"]["ff"] for s in specs if s["mlp"]] or [1])
 
 
+def _moe_feed_forward(mlp: dict, what: str) -> dict:
+    """``mlp`` record of a mixture of clipped-GLU experts: routed experts, identity experts behind them (their output is
+    the input), a shared expert or none."""
+    if mlp.get("kind", "moe") != "moe":
+        raise ValueError(f"{what}: unknown feed-forward kind {mlp.get('kind')!r}")
+    r, e, sh = mlp["router"], mlp["expert"], mlp.get("shared")
+    out = dict(kind="moe", expert=dict(ff=int(e["ff"]), limit=float(e["limit"])),
+               router=dict(experts=int(r["experts"]), identity=int(r.get("identity") or 0), top=int(r["top"]), scale=float(r["scale"])),
+               shared=dict(ff=int(sh["ff"]), limit=float(sh["limit"])) if sh else None)
+    n = out["router"]
+    if n["experts"] < 1 or n["identity"] < 0 or not 1 <= n["top"] <= n["experts"] + n["identity"]:
+        raise ValueError(f"{what}: the router chooses {n['top']} of {n['experts']} + {n['identity']} experts")
+    return out
+
+
+def _vavadra(c: ModelConfig, raw: dict) -> None:
+    """Vavadra: an explicit layer list (differential attention over chunks, latent attention with a window and a sink, or
+    the gated delta rule; mixture of experts or none), pre-norm, an optional run of layers repeated with the same weights
+    (``loop``) into which every pass adds a step vector and, from the second on, the embedding. Attention runs own a
+    KV-pool layer (per-head keys and values, or one latent row per token), delta runs a state slab."""
+    c.vocab_size, c.hidden_size = int(raw["vocab"]), int(raw["width"])
+    c.embed_scale = float((raw.get("embedding") or {}).get("scale", 1.0))
+    c.rms_norm_eps = float(raw["norm"]["eps"])
+    c.tie_word_embeddings = True
+    c.extra["logit_scale"] = float(raw.get("logit_scale", 1.0))
+    specs = []
+    for i, spec in enumerate(raw["layers"]):
+        kind, m, mlp, what = spec["type"], spec["mixer"], spec.get("mlp"), f"layer {i}"
+        if kind == "attention":
+            m = dict(heads=int(m["heads"]), kv_heads=int(m["kv_heads"]), dim=int(m["dim"]), vdim=int(m["vdim"]), scale=float(m["scale"]),
+                     diff=float(m["diff"]), mask=dict(size=int(m["mask"]["size"])))
+        elif kind == "latent_attention":
+            m = dict(heads=int(m["heads"]), dim=int(m["dim"]), rot_dim=int(m["rot_dim"]), vdim=int(m["vdim"]), kv_rank=int(m["kv_rank"]),
+                     scale=float(m["scale"]), mask=dict(size=int(m["mask"]["size"])), rot=_rotation(m["rot"], what))
+            if m["rot"]["dims"] != m["rot_dim"]:
+                raise ValueError(f"{what}: rot.dims must equal rot_dim")
+        elif kind == "delta":
+            m = dict(heads=int(m["heads"]), kv_heads=int(m["kv_heads"]), dim=int(m["dim"]), vdim=int(m["vdim"]), conv=int(m["conv"]))
+            if m["conv"] < 1:
+                raise ValueError(f"{what}: the convolution needs a tap")
+        else:
+            raise ValueError(f"{what}: unknown mixer type {kind!r}")
+        if m["heads"] % m.get("kv_heads", 1):
+            raise ValueError(f"{what}: heads must be a multiple of kv_heads")
+        if "mask" in m and m["mask"]["size"] < 1:
+            raise ValueError(f"{what}: an empty chunk or window")
+        specs.append(dict(type=kind, mixer=m, mlp=None if mlp is None else _moe_feed_forward(mlp, what)))
+    c.extra["layer_specs"], c.extra["layer_runs"] = specs, _looped_runs(c, raw.get("loop"), len(specs))
+    c.num_hidden_layers = len(specs)
+    geo = []
+    for i in c.extra["layer_runs"]:
+        m, kind = specs[i]["mixer"], specs[i]["type"]
+        if kind == "attention":                           # a key row holds both maps
+            geo.append((m["kv_heads"], 2 * m["dim"], m["vdim"]))
+        elif kind == "latent_attention":
+            geo.append((1, m["kv_rank"] + m["rot_dim"], 0))
+    c.extra["kv_geometry"] = geo
+    # (uniform fields other parts read: the first layer's, or the minimum a pool accepts)
+    c.num_attention_heads = next((s["mixer"]["heads"] for s in specs if s["type"] != "delta"), 1)
+    c.num_key_value_heads, c.head_dim = geo[0][:2] if geo else (1, 16)
+    c.partial_rotary_factor = 0.0
+    c.intermediate_size = max([s["mlp"]["expert"]["ff"] for s in specs if s["mlp"]] or [1])
+
+
 def _baichuan(c: ModelConfig, raw: dict) -> None:
     """Baichuan (7B layout): Llama block with q, k, v fused in ``W_pack`` (reference src/models/baichuan.rs).
     The 13B models replace RoPE by ALiBi, which no attention kernel here implements."""
@@ -1417,7 +1486,7 @@ FAMILIES = {
     "gpt_neox": _gpt_neox, "gpt2": _gpt2, "gpt_bigcode": _gpt2, "phi": _phi, "olmo": _olmo1, "granitemoe": _granitemoe, "granitemoehybrid": _granitemoehybrid, "jamba": _jamba, "bitnet": _bitnet, "lfm2_moe": _lfm2, "exaone": _exaone, "telechat3": _telechat3, "deepseek": _deepseek_v1, "recurrent_gemma": _recurrent_gemma, "glm_moe_dsa": _glm_moe_dsa, "deepseek_v32": _glm_moe_dsa, "mistral4": _mistral4, "afmoe": _afmoe, "dbrx": _dbrx, "llama4": _llama4, "llama4_text": _llama4, "qwen3_next": _qwen3_next, "qwen3_5": _qwen3_next, "qwen3_5_text": _qwen3_next, "qwen3_5_moe": _qwen3_next, "qwen3_5_moe_text": _qwen3_next, "falcon_h1": _falcon_h1, "cohere2": _cohere2, "arcee": _arcee, "glm": _glm, "glm4": _glm4, "glm4v": _glm4v, "glm4v_text": _glm4v, "glm4v_moe": _glm4v_moe, "glm4v_moe_text": _glm4v_moe, "cohere2_vision": _cohere2, "paddleocr_vl": _paddleocr_vl, "glm_ocr": _glm_ocr, "glm_ocr_text": _glm_ocr, "paddleocr_vl_text": _paddleocr_vl, "nemotron": _nemotron,
     "ministral3": _ministral3, "granitemoeshared": _granitemoeshared, "nanochat": _nanochat, "code_llama": _plain, "cwm": _plain, "glm4_moe_lite": _deepseek_v3,
     "vaultgemma": _vaultgemma, "solar_open": _solar_open, "minimax_m2": _minimax_m2, "exaone_moe": _exaone_moe, "lfm2": _lfm2, "internlm2": _plain, "baichuan": _baichuan,
-    "pamasun": _pamasun, "govopel": _govopel,
+    "pamasun": _pamasun, "govopel": _govopel, "vavadra": _vavadra,
 }
 
 
@@ -1492,6 +1561,14 @@ def preset(name: str) -> ModelConfig:
             dims=24, base=8000.0, scaling=dict(factor=4.0, original=512, fast=16.0, slow=1.0))), mlp=dict(kind="dense", ff=144, limit=1.5))
         return ModelConfig.from_dict(dict(architecture="Govopel", vocab=512, width=144, layers=[lat, att, dict(att, mlp=None), lat],
                                           norm=dict(eps=1e-5), logit_softcap=20.0))
+    if name == "tiny-vavadra":
+        mlp = dict(kind="moe", expert=dict(ff=48, limit=1.5), router=dict(experts=6, identity=2, top=3, scale=1.5), shared=dict(ff=80, limit=2.0))
+        lat = dict(type="latent_attention", mlp=mlp, mixer=dict(heads=4, dim=24, rot_dim=16, vdim=32, kv_rank=56, scale=0.18, mask=dict(size=40),
+                                                                rot=dict(dims=16, base=50000.0)))
+        att = dict(type="attention", mlp=None, mixer=dict(heads=6, kv_heads=2, dim=16, vdim=40, scale=0.25, diff=0.4, mask=dict(size=48)))
+        delta = dict(type="delta", mlp=mlp, mixer=dict(heads=4, kv_heads=2, dim=32, vdim=24, conv=3))
+        return ModelConfig.from_dict(dict(architecture="Vavadra", vocab=512, width=144, layers=[delta, lat, att, delta], norm=dict(eps=1e-5),
+                                          embedding=dict(scale=4.0), logit_scale=1.5, loop=dict(start=1, stop=3, times=2)))
     if name == "mamba2-2.7b":
         return ModelConfig.from_dict(dict(
             model_type="mamba2", num_hidden_layers=64, hidden_size=2560, num_heads=80, head_dim=64,

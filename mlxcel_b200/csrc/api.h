@@ -58,6 +58,26 @@ typedef struct MxGemmExtras {
   void* out_mc;
 } MxGemmExtras;
 
+// What a step of the fp32 residual stream adds besides a branch (NULL fields: nothing). In this order: the weighted sum of
+// a token's chosen experts (pair t * moe_k + s went to expert moe_ids[.] with weight moe_w[.]; its result is row moe_inv[.] of
+// moe_y, or the row t of moe_x itself for ids from moe_experts on) and the shared expert's row; the embedding
+// emb_scale * table[ids[t]]; an fp32 vector.
+typedef struct MxStreamExtras {
+  const void* moe_y;
+  const void* moe_shared;
+  const void* moe_x;
+  const int* moe_ids;
+  const int* moe_inv;
+  const float* moe_w;
+  int moe_k;
+  int moe_experts;
+  const float* vec;
+  const int* ids;
+  const void* table;
+  int vocab;
+  float emb_scale;
+} MxStreamExtras;
+
 // out[M, N] = epilogue(x[M, K] @ w[N(+N), K]^T). bf16 operands, fp32 accumulation on the
 // 5th-generation tensor cores (tcgen05.mma, accumulators in TMEM, operand tiles brought by TMA).
 // For the gated epilogues `w` holds gate rows at [0, N) and up rows at [glu_offset, glu_offset + N).

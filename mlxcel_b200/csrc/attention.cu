@@ -55,6 +55,11 @@ struct DecodeParams {
   const float* bias_r2;
   const __nv_bfloat16* gate;
   long long gate_stride;
+  // maps == 2: differential heads. A query and key head of dk elements holds two maps of dk / 2, attentions of their own
+  // over the same values; the result is (a1 - lambda a2) / rms(.) * gain. The maps are rows of the same tile (row 2 g +
+  // map of head g, zero in the other map's columns), so keys and values are still read once per key head. Hq counts heads.
+  int maps;
+  float lambda, gain, eps;
 };
 
 // Loads 8 consecutive elements of a K/V row as floats.
@@ -607,7 +612,7 @@ constexpr int kDmKeys = 16;  // keys per group (one MMA k-step of P V)
 
 template <int DK, int DV, int KV_BITS, bool BS16, bool EXT>
 __global__ void __launch_bounds__(kDmThreads)
-paged_decode_mma_kernel(const DecodeParams p, const int G) {
+paged_decode_mma_kernel(const DecodeParams p, const int heads_per_key) {
   // DK / DV: tile widths of keys and values; the plain form has rows of exactly D = DK = DV elements,
   // the extended one rows of p.dk / p.dv whose missing columns are zero-filled on load.
   constexpr int D = DK;
@@ -618,6 +623,8 @@ paged_decode_mma_kernel(const DecodeParams p, const int G) {
   constexpr int VTILE_BYTES = kDmKeys * DV * 2;          // one V group
   constexpr int STAGE_BYTES = TILE_BYTES + VTILE_BYTES;
   const int dk = EXT ? p.dk : DK, dv = EXT ? p.dv : DV;
+  const bool two_maps = EXT && p.maps == 2;
+  const int G = two_maps ? 2 * heads_per_key : heads_per_key;   // query rows of the tile
   constexpr int WARP_BYTES = kDmStages * STAGE_BYTES;
   // Quantized pools: a ring stage holds the RAW group (K codes, V codes, K and V scale/offset
   // pairs), fetched with cp.async like the bf16 tiles so that the ring keeps several groups in
@@ -675,9 +682,14 @@ paged_decode_mma_kernel(const DecodeParams p, const int G) {
   for (int i = threadIdx.x; i < 16 * CH; i += kDmThreads) {
     const int r = i / CH, c = i - r * CH;
     uint4 v = make_uint4(0, 0, 0, 0);
-    if (r < G && (!EXT || c * 8 < dk))
+    if (EXT && two_maps) {
+      if (r < G && c * 8 < dk && (c * 16 >= dk) == (r & 1))    // (dk / 2 is a multiple of 8)
+        v = *reinterpret_cast<const uint4*>(p.q + static_cast<size_t>(b) * p.q_stride +
+                                            static_cast<size_t>(h * heads_per_key + (r >> 1)) * dk + c * 8);
+    } else if (r < G && (!EXT || c * 8 < dk)) {
       v = *reinterpret_cast<const uint4*>(p.q + static_cast<size_t>(b) * p.q_stride +
                                           static_cast<size_t>(h * G + r) * dk + c * 8);
+    }
     *reinterpret_cast<uint4*>(q_sm + swz<D>(r, c)) = v;
   }
   __syncthreads();
@@ -976,6 +988,42 @@ paged_decode_mma_kernel(const DecodeParams p, const int G) {
     p.out[static_cast<size_t>(b) * p.Hq * dv + col] = __float2bfloat16(r);
   };
   float* part_ml = p.scratch_ml + part_idx * (static_cast<size_t>(G) * 2);
+  // differential heads: row 2 g of the first warp's part holds a1 - lambda a2 of head g (each column is written by the one
+  // thread that has read it); one warp per head norms it
+  const auto finish_maps = [&]() {
+    __syncthreads();
+    for (int g = warp; g < heads_per_key; g += kDmWarps) {
+      const float* o = o_s + 2 * g * DV;
+      float ss = 0.f;
+      for (int d = lane; d < dv; d += 32) ss += o[d] * o[d];
+      const float r = p.gain / sqrtf(warp_sum(ss) / dv + p.eps);
+      __nv_bfloat16* dst = p.out + static_cast<size_t>(b) * p.Hq * dv + static_cast<size_t>(h * heads_per_key + g) * dv;
+      for (int d = lane; d < dv; d += 32) dst[d] = __float2bfloat16(o[d] * r);
+    }
+  };
+  if (EXT && two_maps && p.num_splits == 1) {
+    for (int i = threadIdx.x; i < heads_per_key * dv; i += kDmThreads) {
+      const int g = i / dv, d = i - g * dv;
+      float a[2];
+#pragma unroll
+      for (int map = 0; map < 2; ++map) {
+        const int r = 2 * g + map;
+        float m = -INFINITY, l = 0.f, o = 0.f;
+#pragma unroll
+        for (int w = 0; w < kDmWarps; ++w) m = fmaxf(m, m_s[w][r]);
+#pragma unroll
+        for (int w = 0; w < kDmWarps; ++w) {
+          const float sc = (m_s[w][r] > -INFINITY) ? exp2f(m_s[w][r] - m) : 0.f;
+          l += l_s[w][r] * sc;
+          o += o_s[(w * 16 + r) * DV + d] * sc;
+        }
+        a[map] = l > 0.f ? o / l : 0.f;
+      }
+      o_s[2 * g * DV + d] = a[0] - p.lambda * a[1];
+    }
+    finish_maps();
+    return;
+  }
   for (int i = threadIdx.x; i < G * dv; i += kDmThreads) {
     const int g = i / dv, d = i - g * dv;
     float m = -INFINITY;
@@ -1018,8 +1066,7 @@ paged_decode_mma_kernel(const DecodeParams p, const int G) {
   if (!last_s) return;
   __threadfence();
   const size_t base_idx = (static_cast<size_t>(b) * p.Hkv + h) * p.num_splits;
-  for (int i = threadIdx.x; i < G * dv; i += kDmThreads) {
-    const int g = i / dv, d = i - g * dv;
+  const auto merged = [&](int g, int d) -> float {      // row g, column d over the splits
     float m = -INFINITY;
     for (int s2 = 0; s2 < p.num_splits; ++s2)
       m = fmaxf(m, __ldcg(&p.scratch_ml[(base_idx + s2) * (G * 2) + g * 2]));
@@ -1034,11 +1081,20 @@ paged_decode_mma_kernel(const DecodeParams p, const int G) {
       const float ls = __ldcg(&p.scratch_ml[(base_idx + s2) * (G * 2) + g * 2 + 1]);
       const float sc = (ms > -INFINITY) ? exp2f(ms - m) : 0.f;
       l += ls * sc;
-      o += __ldcg(&p.scratch_o[(base_idx + s2) * (static_cast<size_t>(G) * dv) + i]) * sc;
+      o += __ldcg(&p.scratch_o[(base_idx + s2) * (static_cast<size_t>(G) * dv) + g * dv + d]) * sc;
     }
     if (p.sinks != nullptr) l += exp2f(sk - m);
-    finish(g, d, l > 0.f ? o / l : 0.f);
+    return l > 0.f ? o / l : 0.f;
+  };
+  if (EXT && two_maps) {
+    for (int i = threadIdx.x; i < heads_per_key * dv; i += kDmThreads) {
+      const int g = i / dv, d = i - g * dv;
+      o_s[2 * g * DV + d] = merged(2 * g, d) - p.lambda * merged(2 * g + 1, d);
+    }
+    finish_maps();
+    return;
   }
+  for (int i = threadIdx.x; i < G * dv; i += kDmThreads) finish(i / dv, i % dv, merged(i / dv, i % dv));
 }
 
 template <int DK, int DV, int KV_BITS, bool BS16, bool EXT>
@@ -1181,16 +1237,19 @@ extern "C" int mx_paged_decode(const void* q, long long q_stride, const void* k_
 }
 
 // Extended decode form over bf16 pools: key / value rows of Dk / Dv elements (multiples of 8, at most
-// 128), soft cap, chunked visibility, distance bias and output gate optional (0 / NULL). -10 = not covered (use mx_paged_attention_any).
+// 128), soft cap, chunked visibility, distance bias and output gate optional (0 / NULL). maps == 2: differential heads (Hq
+// heads whose Dk columns are both maps; scratch for 2 Hq heads; no sinks, bias or gate). -10 = not covered (use mx_paged_attention_any).
 extern "C" int mx_paged_decode_ext(const void* q, long long q_stride, const void* k_pool, const void* v_pool,
                                    const int* block_tables, const int* context_lens, const float* sinks,
                                    const float* bias_r1, const float* bias_r2, const void* gate, long long gate_stride,
                                    void* out, float* scratch, int B, int Hq, int Hkv, int Dk, int Dv, int block_size,
-                                   int max_blocks, int window, int chunk, float scale, float softcap, int num_splits,
-                                   void* stream_) {
+                                   int max_blocks, int window, int chunk, float scale, float softcap, int maps, float lambda,
+                                   float gain, float eps, int num_splits, void* stream_) {
   if (B <= 0) return 0;
   if (Hkv <= 0 || Hq % Hkv || (bias_r1 == nullptr) != (bias_r2 == nullptr)) return -1;
+  if ((maps != 1 && maps != 2) || (maps == 2 && (sinks != nullptr || bias_r1 != nullptr || gate != nullptr))) return -1;
   const int G = Hq / Hkv;
+  if (maps == 2 && (G > 8 || Dk % 16)) return -10;
   const auto al16 = [](const void* a) { return (reinterpret_cast<uintptr_t>(a) & 15) == 0; };
   if (G > 16 || Dk % 8 || Dv % 8 || Dk > 128 || Dv > 128 || block_size % 16 || q_stride % 8 || !al16(q) || !al16(k_pool) ||
       !al16(v_pool))
@@ -1208,7 +1267,9 @@ extern "C" int mx_paged_decode_ext(const void* q, long long q_stride, const void
   p.counters = reinterpret_cast<int*>(scratch);
   if (num_splits > 1 && static_cast<long long>(B) * Hkv > kDecodeCounters) return -1;
   p.scratch_ml = scratch + kDecodeCounters;
-  p.scratch_o = p.scratch_ml + static_cast<size_t>(B) * Hkv * num_splits * G * 2;
+  p.scratch_o = p.scratch_ml + static_cast<size_t>(B) * Hkv * num_splits * maps * G * 2;
+  p.maps = maps;
+  p.lambda = lambda, p.gain = gain, p.eps = eps;
   p.B = B;
   p.Hq = Hq;
   p.Hkv = Hkv;

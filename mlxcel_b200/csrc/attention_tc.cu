@@ -63,6 +63,8 @@ struct TcPrefillParams {
   const int* kv_starts;
   int kv_split;
   long long out_stride;      // elements between output rows
+  // Differential heads (MAPS == 2): the result is (a1 - lambda a2) / rms(.) * gain.
+  float lambda, gain, eps;
 };
 
 // The extended form runs eight softmax warps instead of four, two per 32 query rows: each takes one half of
@@ -76,13 +78,18 @@ __host__ __device__ constexpr int tc_threads(bool ext) { return 64 + 32 * tc_sof
 constexpr int kBiasTab = 96;
 constexpr int kExtSmem = 8 * kBiasTab * 4 + 2 * 2 * kTcRows * 4 + 2 * kTcRows * 4;   // tables, maxima (2 buffers), sums
 
+// Differential heads (MAPS == 2, no sinks, bias or gate): query and key heads are two maps of dk columns each. The CTA walks
+// its key tiles twice, first with map 1, then with map 2 (tile j of the walk is key tile j mod n of map j / n), with running
+// maxima and sums per map and an accumulator each in TMEM; the epilogue combines the two in registers. Scores of map
+// 2's first tile run under the softmax of map 1's last one, as between any two tiles.
+//
 // The second weight term takes the room of one V stage where both heads are 128 wide: a V tile is only
 // needed once its softmax is through, so its load still has most of a tile's time.
 __host__ __device__ constexpr int tc_v_stages(int dk, int dv, bool ext) { return (ext && dk >= 128 && dv == 128) ? 1 : kTcStages; }
-// Keys of 192 columns leave room for one K stage (free again as soon as its score MMA has run).
-__host__ __device__ constexpr int tc_k_stages(int dk) { return dk > 128 ? 1 : kTcStages; }
+// Keys of 192 columns (and two maps of queries of 128) leave room for one K stage (free again as soon as its score MMA has run).
+__host__ __device__ constexpr int tc_k_stages(int dk, int maps) { return dk > 128 || (dk == 128 && maps == 2) ? 1 : kTcStages; }
 
-template <int DK, int DV, bool EXT>
+template <int DK, int DV, bool EXT, int MAPS>
 __global__ void __launch_bounds__(tc_threads(EXT), 1)
 paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
                         const __grid_constant__ CUtensorMap map_v, const __grid_constant__ CUtensorMap map_kr,
@@ -98,19 +105,20 @@ paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
   constexpr int PTERMS = EXT ? 2 : 1;
   constexpr int P_BYTES = PTERMS * PHALF_BYTES;
   constexpr int VST = tc_v_stages(DK, DV, EXT);       // V ring depth
-  constexpr int KST = tc_k_stages(DK);                // K ring depth
+  constexpr int KST = tc_k_stages(DK, MAPS);          // K ring depth
   constexpr int S_COLS = kTcKeys;                     // fp32 columns of one score buffer
-  constexpr int O_COL = 2 * S_COLS;                   // first TMEM column of O
+  constexpr int O_COL = 2 * S_COLS;                   // first TMEM column of O (DV columns per map)
   constexpr uint32_t TMEM_COLS = 512;
   static_assert((DK == 64 || DK == 128 || (EXT && DK == 192)) && (DV == 64 || DV == 128), "head dims");
   static_assert(EXT || DK == DV, "plain form: one head width");
+  static_assert(MAPS == 1 || EXT, "differential heads: extended form");
   const int dk = EXT ? p.dk : DK, dv = EXT ? p.dv : DV;
 
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) &
                                              ~static_cast<uintptr_t>(1023));
   uint8_t* q_sm = smem;
-  uint8_t* k_sm = q_sm + Q_BYTES;                     // KST x K_BYTES
+  uint8_t* k_sm = q_sm + MAPS * Q_BYTES;              // KST x K_BYTES
   uint8_t* v_sm = k_sm + KST * K_BYTES;               // VST x V_BYTES
   uint8_t* p_sm = v_sm + VST * V_BYTES;
   uint64_t* bars = reinterpret_cast<uint64_t*>(p_sm + P_BYTES);
@@ -151,7 +159,10 @@ paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
     if (p.chunk > 0) kv_begin = max(kv_begin, (pos_base + tok0) / p.chunk * p.chunk);
   }
   kv_begin = (kv_begin / kTcKeys) * kTcKeys;
-  const int n_tiles = (kv_end - kv_begin + kTcKeys - 1) / kTcKeys;
+  const int key_tiles = (kv_end - kv_begin + kTcKeys - 1) / kTcKeys;
+  const int n_tiles = MAPS * key_tiles;               // tiles of the walk
+  const auto key_tile = [&](int j) { return MAPS == 2 && j >= key_tiles ? j - key_tiles : j; };
+  const auto map_of = [&](int j) { return MAPS == 2 && j >= key_tiles ? 1 : 0; };
   const int last_block = (ctx - 1) / kTcBlock;   // last pool block the sequence owns
 
   if (threadIdx.x == 0) {
@@ -191,9 +202,11 @@ paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
     const uint64_t pol_q = l2_policy_evict_first();
     const uint64_t pol_kv = l2_policy_evict_last();   // re-read by the other heads / token tiles
     if (lane == 0) {
-      mbar_expect_tx(q_full, Q_BYTES);
-      for (int c = 0; c < DC; ++c)
-        if (EXT && p.kv_starts != nullptr)
+      mbar_expect_tx(q_full, MAPS * Q_BYTES);
+      for (int c = 0; c < MAPS * DC; ++c)
+        if (MAPS == 2)
+          tma_load_3d(q_sm + c * SUB_BYTES, &map_q, q_full, (c % DC) * 64, hq * 2 + c / DC, q0 + tok0, pol_q);
+        else if (EXT && p.kv_starts != nullptr)
           tma_load_3d(q_sm + c * SUB_BYTES, &map_q, q_full, c * 64 < p.kv_split ? c * 64 : p.kv_split, hq, q0 + tok0, pol_q);
         else
           tma_load_2d(q_sm + c * SUB_BYTES, &map_q, q_full, hq * dk + c * 64, q0 + tok0, pol_q);
@@ -201,7 +214,7 @@ paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
     int stage = 0;
     uint32_t phase = 0;
     bool ok = true;
-    if (EXT && p.kv_starts != nullptr) {
+    if (EXT && MAPS == 1 && p.kv_starts != nullptr) {
       // dense rows: one box per 64-column tile (rows past the sequence belong to the next one or are filled with
       // zeros; the mask drops them)
       const int base = p.kv_starts[s];
@@ -229,7 +242,7 @@ paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
       // the values multiplied by P = 0 must be finite)
       int row0 = 0;
       if (lane < kTcKeys / kTcBlock) {
-        const int b = min((kv_begin + j * kTcKeys) / kTcBlock + lane, last_block);
+        const int b = min((kv_begin + key_tile(j) * kTcKeys) / kTcBlock + lane, last_block);
         row0 = (table[b] * p.Hkv + hkv) * kTcBlock;
       }
       if (lane == 0) {
@@ -240,7 +253,10 @@ paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
       if (!ok) break;
       if (lane < kTcKeys / kTcBlock) {
         uint8_t* kd = k_sm + stage * K_BYTES + lane * (kTcBlock * 128);
-        for (int c = 0; c < DC; ++c) tma_load_2d(kd + c * SUB_BYTES, &map_k, &k_full[stage], c * 64, row0, pol_kv);
+        for (int c = 0; c < DC; ++c) {
+          if (MAPS == 2) tma_load_3d(kd + c * SUB_BYTES, &map_k, &k_full[stage], c * 64, map_of(j), row0, pol_kv);
+          else tma_load_2d(kd + c * SUB_BYTES, &map_k, &k_full[stage], c * 64, row0, pol_kv);
+        }
       }
       if (lane == 0) {
         ok = mbar_wait(&kv_empty[vstage], vphase ^ 1u, p.status, kErrAttnProducer);
@@ -272,7 +288,7 @@ paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
         if (!mbar_wait(&k_full[stage], kv_phase, p.status, kErrAttnMma)) return false;
         if (!mbar_wait(&s_empty[sb], s_phase ^ 1u, p.status, kErrAttnMma)) return false;
         tc_fence_after_sync();
-        const uint32_t qa = smem_u32(q_sm), kb = smem_u32(k_sm + stage * K_BYTES);
+        const uint32_t qa = smem_u32(q_sm) + map_of(j) * Q_BYTES, kb = smem_u32(k_sm + stage * K_BYTES);
 #pragma unroll
         for (int kk = 0; kk < DK / 16; ++kk) {
           const uint32_t off = (kk >> 2) * SUB_BYTES + (kk & 3) * 32;
@@ -299,7 +315,7 @@ paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
 #pragma unroll
           for (int term = 0; term < PTERMS; ++term) {
             const uint64_t da = umma_desc_k_sw128(pa + term * PHALF_BYTES + (kk >> 2) * SUB_BYTES + (kk & 3) * 32);
-            umma_bf16(tmem_base + O_COL, da, db, idesc_pv, (j > 0 || kk > 0 || term > 0) ? 1u : 0u);
+            umma_bf16(tmem_base + O_COL + map_of(j) * DV, da, db, idesc_pv, (key_tile(j) > 0 || kk > 0 || term > 0) ? 1u : 0u);
           }
         }
         umma_commit(&kv_empty[stage]);   // the V tile of this stage is consumed
@@ -315,7 +331,7 @@ paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
     const uint32_t lane_addr = tmem_base + (static_cast<uint32_t>(q4 * 32) << 16);
     const int qpos = pos_base + tok0 + row;         // absolute position of this row's token
     float m_used = -INFINITY;   // the maximum the stored exponentials refer to (scaled, log2 units)
-    float l = 0.f;
+    float l = 0.f, l_first = 0.f;                   // (MAPS == 2: the first map's sum)
     float* tab = bias_tab + (warp - 2) * kBiasTab;
     float r1 = 0.f, r2 = 0.f;
     const __nv_bfloat16* gate = nullptr;            // this row's gate values, needed in the epilogue
@@ -330,10 +346,16 @@ paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
     for (int j = 0; j < n_tiles && ok; ++j) {
       const int sb = j & 1;
       const uint32_t s_phase = static_cast<uint32_t>(j >> 1) & 1u;
+      if (MAPS == 2 && j == key_tiles) {
+        l_first = l;
+        l = 0.f;
+        m_used = -INFINITY;
+      }
       ok = mbar_wait(&s_full[sb], s_phase, p.status, kErrAttnSoftmax);
       if (!ok) break;
       tc_fence_after_sync();
-      const int key0 = kv_begin + j * kTcKeys;
+      const int o_col = O_COL + map_of(j) * DV;
+      const int key0 = kv_begin + key_tile(j) * kTcKeys;
       // Only tiles that cross the diagonal, the window edge or the end need the mask.
       const bool need_mask = (key0 + kTcKeys - 1 > pos_base + tok0) ||
                              (p.window > 0 && key0 < pos_base + tok0 + kTcRows - p.window) ||
@@ -423,11 +445,11 @@ paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
         for (int cc = 0; cc < DV / 32 / HALVES; ++cc) {
           const int c = half * (DV / 32 / HALVES) + cc;
           uint32_t r[32];
-          tmem_ld_32x32(lane_addr + O_COL + c * 32, r);
+          tmem_ld_32x32(lane_addr + o_col + c * 32, r);
           tmem_ld_wait();
 #pragma unroll
           for (int i = 0; i < 32; ++i) r[i] = __float_as_uint(__uint_as_float(r[i]) * alpha);
-          tmem_st_32x32(lane_addr + O_COL + c * 32, r);
+          tmem_st_32x32(lane_addr + o_col + c * 32, r);
         }
         tmem_st_wait();
       }
@@ -468,6 +490,54 @@ paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
       if (lane == 0) mbar_arrive(p_full);
     }
     // ---- epilogue: O / l -> out (one row of D bf16 per thread; EXT: half a row)
+    if constexpr (MAPS == 2) {
+      // sums of both maps over the two halves, then the combined row: its square sum takes one more exchange
+      constexpr int CW = DV / 2;                    // columns of a thread
+      float inv1 = 0.f, inv2 = 0.f, av[CW];
+      if (ok) {
+        pair_sum[half * kTcRows + row] = l;
+        pair_max[half * kTcRows + row] = l_first;   // (the maxima of the tiles before the last are through: see below)
+        __syncwarp();
+        if (lane == 0) mbar_arrive(&pair_bar[q4]);
+        ok = mbar_wait(&pair_bar[q4], static_cast<uint32_t>(n_tiles) & 1u, p.status, kErrAttnSoftmax);
+        const float l1 = pair_max[row] + pair_max[kTcRows + row], l2 = pair_sum[row] + pair_sum[kTcRows + row];
+        inv1 = l1 > 0.f ? 1.f / l1 : 0.f;
+        inv2 = l2 > 0.f ? p.lambda / l2 : 0.f;
+      }
+      if (ok) ok = mbar_wait(pv_done, static_cast<uint32_t>(n_tiles - 1) & 1u, p.status, kErrAttnSoftmax);
+      if (ok) {
+        tc_fence_after_sync();
+        float ss = 0.f;
+#pragma unroll
+        for (int c = 0; c < CW / 32; ++c) {
+          uint32_t r1_[32], r2_[32];
+          tmem_ld_32x32(lane_addr + O_COL + half * CW + c * 32, r1_);
+          tmem_ld_32x32(lane_addr + O_COL + DV + half * CW + c * 32, r2_);
+          tmem_ld_wait();
+#pragma unroll
+          for (int i = 0; i < 32; ++i) {            // (columns past the row's width are zero)
+            const float a = __uint_as_float(r1_[i]) * inv1 - __uint_as_float(r2_[i]) * inv2;
+            av[c * 32 + i] = a;
+            ss = fmaf(a, a, ss);
+          }
+        }
+        float* xs = pair_max + 2 * kTcRows;         // the other buffer
+        xs[half * kTcRows + row] = ss;
+        __syncwarp();
+        if (lane == 0) mbar_arrive(&pair_bar[q4]);
+        ok = mbar_wait(&pair_bar[q4], static_cast<uint32_t>(n_tiles + 1) & 1u, p.status, kErrAttnSoftmax);
+        const float rs = p.gain / sqrtf((xs[row] + xs[kTcRows + row]) / dv + p.eps);
+        if (ok && row < rows_valid) {
+          __nv_bfloat16* dst = p.out + static_cast<size_t>(q0 + tok0 + row) * p.out_stride + hq * dv + half * CW;
+#pragma unroll
+          for (int i = 0; i < CW; i += 8) {
+            if (half * CW + i < dv)
+              *reinterpret_cast<uint4*>(dst + i) = make_uint4(pack_bf16(av[i] * rs, av[i + 1] * rs), pack_bf16(av[i + 2] * rs, av[i + 3] * rs),
+                                                              pack_bf16(av[i + 4] * rs, av[i + 5] * rs), pack_bf16(av[i + 6] * rs, av[i + 7] * rs));
+          }
+        }
+      }
+    } else {
     if constexpr (HALVES == 2) {
       if (ok && n_tiles > 0) {
         pair_sum[half * kTcRows + row] = l;
@@ -529,6 +599,7 @@ paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
         }
       }
     }
+    }
   }
 
   // ------------------------------------------------------------------ teardown
@@ -540,14 +611,14 @@ paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
   }
 }
 
-template <int DK, int DV, bool EXT>
+template <int DK, int DV, bool EXT, int MAPS = 1>
 static int launch_prefill_tc(const CUtensorMap& mq, const CUtensorMap& mk, const CUtensorMap& mv, const CUtensorMap& mkr,
                              const TcPrefillParams& p, int grid, cudaStream_t stream) {
   constexpr int SUB = 128 * 128;
-  constexpr int smem = (DK / 64) * SUB * (1 + tc_k_stages(DK)) + (DV / 64) * SUB * tc_v_stages(DK, DV, EXT) +
+  constexpr int smem = (DK / 64) * SUB * (MAPS + tc_k_stages(DK, MAPS)) + (DV / 64) * SUB * tc_v_stages(DK, DV, EXT) +
                        (EXT ? 4 : 2) * SUB + 1024 + 256 + (EXT ? kExtSmem : 0);
   static_assert(smem <= 227 * 1024, "shared memory");
-  auto kern = paged_prefill_tc_kernel<DK, DV, EXT>;
+  auto kern = paged_prefill_tc_kernel<DK, DV, EXT, MAPS>;
   static bool configured = false;
   if (!configured) {
     cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
@@ -607,18 +678,21 @@ extern "C" int mx_paged_prefill_tc(const void* q, long long q_stride, const void
 }
 
 // Extended form: key / value rows of Dk / Dv elements (multiples of 8, at most 128); distance bias, output gate,
-// chunked visibility and soft cap optional (NULL / 0). Returns -10 when not covered (use mx_paged_attention_any).
+// chunked visibility and soft cap optional (NULL / 0). maps == 2: differential heads, Dk columns hold both maps. Returns -10 when not covered (use mx_paged_attention_any).
 extern "C" int mx_paged_prefill_ext(const void* q, long long q_stride, const void* k_pool, const void* v_pool,
                                     long long pool_blocks, const int* block_tables, const int* cu_q,
                                     const int* context_lens, const float* sinks, const float* bias_r1,
                                     const float* bias_r2, const void* gate, long long gate_stride, void* out,
                                     int num_seqs, int total_q, int max_q_len, int Hq, int Hkv, int Dk, int Dv,
                                     int block_size, int max_blocks, int window, int chunk, float scale, float softcap,
-                                    void* status, void* stream_) {
+                                    int maps, float lambda, float gain, float eps, void* status, void* stream_) {
   cudaStream_t stream = static_cast<cudaStream_t>(stream_);
   if (num_seqs <= 0 || total_q <= 0) return 0;
   if (Hkv <= 0 || Hq % Hkv || (bias_r1 == nullptr) != (bias_r2 == nullptr)) return -1;
+  if ((maps != 1 && maps != 2) || (maps == 2 && (sinks != nullptr || bias_r1 != nullptr || gate != nullptr))) return -1;
   const auto al16 = [](const void* a) { return (reinterpret_cast<uintptr_t>(a) & 15) == 0; };
+  if (Dk % maps) return -10;
+  Dk /= maps;                          // columns of one map
   if (block_size != kTcBlock || Dk % 8 || Dv % 8 || Dk > 128 || Dv > 128 || q_stride % 8 || gate_stride % 8 || !al16(q) ||
       !al16(out) || !al16(gate) || !al16(k_pool) || !al16(v_pool))
     return -10;
@@ -648,6 +722,21 @@ extern "C" int mx_paged_prefill_ext(const void* q, long long q_stride, const voi
   const long long grid = static_cast<long long>(num_seqs) * Hq * p.tiles_per_seq;
   if (grid > 0x7fffffffll) return -1;
   CUtensorMap mq, mk, mv;
+  if (maps == 2) {
+    // maps as groups of their own: a box that is wider than a map ends in zeros
+    p.lambda = lambda, p.gain = gain, p.eps = eps;
+    const uint64_t rows = static_cast<uint64_t>(pool_blocks) * Hkv * kTcBlock;
+    if (!make_tensor_map_bf16_3d(&mq, q, total_q, 2ull * Hq, Dk, q_stride, Dk, kTcRows, 64) ||
+        !make_tensor_map_bf16_3d(&mk, k_pool, rows, 2, Dk, 2ull * Dk, Dk, kTcBlock, 64) ||
+        !make_tensor_map_bf16(&mv, v_pool, rows, Dv, Dv, kTcBlock, 64))
+      return -4;
+    const int g2 = static_cast<int>(grid);
+    if (Dk <= 64)
+      return Dv <= 64 ? launch_prefill_tc<64, 64, true, 2>(mq, mk, mv, mv, p, g2, stream)
+                      : launch_prefill_tc<64, 128, true, 2>(mq, mk, mv, mv, p, g2, stream);
+    return Dv <= 64 ? launch_prefill_tc<128, 64, true, 2>(mq, mk, mv, mv, p, g2, stream)
+                    : launch_prefill_tc<128, 128, true, 2>(mq, mk, mv, mv, p, g2, stream);
+  }
   // a query box may run into the next head's columns: the keys' columns there are zero
   if (!make_tensor_map_bf16(&mq, q, static_cast<uint64_t>(total_q), static_cast<uint64_t>(Hq) * Dk,
                             static_cast<uint64_t>(q_stride), kTcRows, 64))
@@ -665,12 +754,13 @@ extern "C" int mx_paged_prefill_ext(const void* q, long long q_stride, const voi
 
 // Latent attention over expanded rows: keys [k_nope (Dn) | shared rotated part (R)], values Dv wide. Sequence s owns query
 // rows [cu_q[s], cu_q[s + 1]) of q (rows of heads of Dn + R elements), the last of its context_lens[s] tokens; its
-// context lies in rows kv_starts[s] .. of kn [kv_rows, H * Dn], kr (rows kr_stride apart, R used) and v [kv_rows, H * Dv].
+// context lies in rows kv_starts[s] .. (the first of them, that of token 0, may be before the matrices where the window is not) of kn [kv_rows, H * Dn], kr (rows kr_stride apart, R used) and v [kv_rows, H * Dv].
 // Output rows are out_stride elements apart. -10 = not covered.
 extern "C" int mx_latent_prefill(const void* q, long long q_stride, const void* kn, const void* kr, long long kr_stride,
                                  const void* v, long long kv_rows, const int* cu_q, const int* context_lens,
-                                 const int* kv_starts, void* out, long long out_stride, int num_seqs, int total_q,
-                                 int max_q_len, int H, int Dn, int R, int Dv, float scale, void* status, void* stream_) {
+                                 const int* kv_starts, const float* sinks, void* out, long long out_stride, int num_seqs,
+                                 int total_q, int max_q_len, int H, int Dn, int R, int Dv, int window, float scale, void* status,
+                                 void* stream_) {
   cudaStream_t stream = static_cast<cudaStream_t>(stream_);
   if (num_seqs <= 0 || total_q <= 0) return 0;
   if (H <= 0 || kv_rows <= 0) return -1;
@@ -690,6 +780,8 @@ extern "C" int mx_latent_prefill(const void* q, long long q_stride, const void* 
   p.dk = Dn + R;
   p.dv = Dv;
   p.kv_starts = kv_starts;
+  p.sinks = sinks;
+  p.window = window;
   p.kv_split = Dn;
   p.out_stride = out_stride;
   const long long grid = static_cast<long long>(num_seqs) * H * p.tiles_per_seq;

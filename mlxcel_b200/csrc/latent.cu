@@ -2,10 +2,11 @@
 // shared by all heads (pool [blocks, 1, block_size, C + R]).
 //   latent_append   projection row q_latent | latent | key part: q_latent normalised in place, the latent normalised and
 //                   the key part rotated into the pool
-//   latent_q_rope   rotates the last R dimensions of every query head (in place, or into the absorbed query row)
+//   latent_q_rope   rotates the last R dimensions of every query head (in place, or into the absorbed query row); dimensions
+//                   are paired with those half the width on, or neighbours with each other
 //   latent_gather   the pool rows of several sequences as one dense matrix (input of the key / value up-projections)
 //   latent_decode   attention in the absorbed form: queries [q W_uk | q_rot] against the pool rows, the first C
-//                   columns of the same rows as values; every row is read once for all heads
+//                   columns of the same rows as values; every row is read once for all heads; optional window and sinks
 // Norms, angles, scores, softmax and accumulation are fp32.
 #include "api.h"
 #include "latent.cuh"
@@ -22,7 +23,7 @@ template <typename T, int V>
 __global__ void __launch_bounds__(kLaThreads)
 latent_append_kernel(T* __restrict__ a, long long ld, const int* __restrict__ positions, const int* __restrict__ slots,
                      const float* __restrict__ inv_freq, float mscale, const float* __restrict__ qw,
-                     const float* __restrict__ cw, T* __restrict__ pool, int Q, int C, int R, float eps) {
+                     const float* __restrict__ cw, T* __restrict__ pool, int Q, int C, int R, float eps, int adjacent) {
   __shared__ float red[2 * 33];
   pdl_trigger();
   pdl_wait();
@@ -58,9 +59,10 @@ latent_append_kernel(T* __restrict__ a, long long ld, const int* __restrict__ po
     float sn, cs;
     sincosf(pos * inv_freq[i], &sn, &cs);
     cs *= mscale, sn *= mscale;
-    const float u = to_f(row[Q + C + i]), v = to_f(row[Q + C + half + i]);
-    dst[C + i] = from_f<T>(u * cs - v * sn);
-    dst[C + half + i] = from_f<T>(v * cs + u * sn);
+    const int iu = C + (adjacent ? 2 * i : i), iv = C + (adjacent ? 2 * i + 1 : half + i);
+    const float u = to_f(row[Q + iu]), v = to_f(row[Q + iv]);
+    dst[iu] = from_f<T>(u * cs - v * sn);
+    dst[iv] = from_f<T>(v * cs + u * sn);
   }
 }
 
@@ -68,7 +70,7 @@ latent_append_kernel(T* __restrict__ a, long long ld, const int* __restrict__ po
 template <typename T>
 __global__ void __launch_bounds__(kLaThreads)
 latent_q_rope_kernel(const T* __restrict__ q, long long ldq, int q_head, T* __restrict__ dst, long long ldd, int d_head,
-                     const int* __restrict__ positions, const float* __restrict__ inv_freq, float mscale, int H, int R) {
+                     const int* __restrict__ positions, const float* __restrict__ inv_freq, float mscale, int H, int R, int adjacent) {
   extern __shared__ float lr_smem[];
   const int half = R / 2;
   float *cs = lr_smem, *sn = lr_smem + half;
@@ -84,18 +86,19 @@ latent_q_rope_kernel(const T* __restrict__ q, long long ldq, int q_head, T* __re
   __syncthreads();
   for (int i = threadIdx.x; i < H * half; i += kLaThreads) {
     const int h = i / half, j = i - h * half;
-    const T* src = q + t * ldq + static_cast<size_t>(h) * q_head + j;
-    T* out = dst + t * ldd + static_cast<size_t>(h) * d_head + j;
-    const float u = to_f(src[0]), v = to_f(src[half]);
-    out[0] = from_f<T>(u * cs[j] - v * sn[j]);
-    out[half] = from_f<T>(v * cs[j] + u * sn[j]);
+    const int iu = adjacent ? 2 * j : j, iv = adjacent ? 2 * j + 1 : half + j;
+    const T* src = q + t * ldq + static_cast<size_t>(h) * q_head;
+    T* out = dst + t * ldd + static_cast<size_t>(h) * d_head;
+    const float u = to_f(src[iu]), v = to_f(src[iv]);
+    out[iu] = from_f<T>(u * cs[j] - v * sn[j]);
+    out[iv] = from_f<T>(v * cs[j] + u * sn[j]);
   }
 }
 
-// Row r of the dense matrix is token r - starts[s] of sequence s (starts[s] <= r < starts[s + 1]).
+// Row r of the dense matrix is token r - zero[s] of sequence s (starts[s] <= r < starts[s + 1]).
 __global__ void __launch_bounds__(256)
 latent_gather_kernel(const uint8_t* __restrict__ pool, const int* __restrict__ tables, const int* __restrict__ starts,
-                     uint8_t* __restrict__ out, int rows, int num_seqs, int row_bytes, int unit, int block_size, int max_blocks) {
+                     const int* __restrict__ zero, uint8_t* __restrict__ out, int rows, int num_seqs, int row_bytes, int unit, int block_size, int max_blocks) {
   pdl_trigger();
   pdl_wait();
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -107,7 +110,7 @@ latent_gather_kernel(const uint8_t* __restrict__ pool, const int* __restrict__ t
     if (starts[mid] <= r) lo = mid;
     else hi = mid;
   }
-  const int tok = r - starts[lo];
+  const int tok = r - zero[lo];
   const int blk = tables[static_cast<size_t>(lo) * max_blocks + tok / block_size];
   const uint8_t* src = pool + (static_cast<size_t>(blk) * block_size + tok % block_size) * row_bytes;
   uint8_t* dst = out + static_cast<size_t>(r) * row_bytes;
@@ -151,9 +154,8 @@ __global__ void __launch_bounds__(kLdThreads, 1) latent_decode_kernel(const Late
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int h0 = ht * HR, heads = min(HR, p.H - h0);
   const int len = p.context_lens[b];
-  const int tiles = (len + kLdKeys - 1) / kLdKeys;
-  const int per = (tiles + p.num_splits - 1) / p.num_splits;
-  const int t0 = split * per, t1 = min(tiles, t0 + per);
+  const LatentSpan span = latent_span(p, len, split, kLdKeys);
+  const int t0 = span.t0, t1 = span.t1;
   const int* table = p.block_tables + static_cast<size_t>(b) * p.max_blocks;
   const int chunks = p.W / 8, row_chunks = KS * 2;          // real and padded 16-byte chunks of a row
   pdl_wait();
@@ -252,7 +254,8 @@ __global__ void __launch_bounds__(kLdThreads, 1) latent_decode_kernel(const Late
       float mx = -INFINITY;
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
-        v[e] = tile * kLdKeys + c + e < len ? v[e] * p.scale_log2 : -INFINITY;
+        const int key = tile * kLdKeys + c + e;
+        v[e] = key < len && key >= span.begin ? v[e] * p.scale_log2 : -INFINITY;
         mx = fmaxf(mx, v[e]);
       }
 #pragma unroll
@@ -332,8 +335,13 @@ __global__ void __launch_bounds__(kLdThreads, 1) latent_decode_kernel(const Late
         const int c = (warp + n * 8) * 16 + (e >> 2) * 8 + (lane & 3) * 2 + (e & 1);
         if (r >= heads || c >= p.C) continue;
         const float v = o[m][n][e >> 2][e & 3];
-        if (p.num_splits > 1) po[r * p.C + c] = v;
-        else p.out[(static_cast<size_t>(b) * p.H + h0 + r) * p.C + c] = __float2bfloat16(l_s[r] > 0.f ? v / l_s[r] : 0.f);
+        if (p.num_splits > 1) {
+          po[r * p.C + c] = v;
+        } else {
+          float f;
+          const float l = latent_denominator(p, h0 + r, m_s[r], l_s[r], f);
+          p.out[(static_cast<size_t>(b) * p.H + h0 + r) * p.C + c] = __float2bfloat16(l > 0.f ? v * f / l : 0.f);
+        }
       }
   if (p.num_splits == 1) return;
   if (threadIdx.x < HR) {
@@ -368,7 +376,11 @@ __global__ void __launch_bounds__(256) latent_merge_kernel(const LatentDecodePar
       sum += f * l[i];
     }
     sum = warp_sum(sum);
-    if (threadIdx.x == 0) inv_s = sum > 0.f ? 1.f / sum : 0.f;
+    if (threadIdx.x == 0) {
+      float f;
+      const float l = latent_denominator(p, h, mx, sum, f);
+      inv_s = l > 0.f ? f / l : 0.f;
+    }
   }
   __syncthreads();
   for (int c = threadIdx.x * 2; c < p.C; c += 512) {
@@ -404,8 +416,8 @@ constexpr int kLatentScratch0 = 65536;    // the scratch buffer starts with the 
 
 // a: rows q_latent [Q] | latent [C] | key part [R], ld elements apart. Q may be 0.
 extern "C" int mx_latent_append(void* a, long long ld, const void* positions, const void* slots, const void* inv_freq, float mscale,
-                                const void* qw, const void* cw, void* pool, int n, int Q, int C, int R, float eps, int fp32,
-                                void* stream) {
+                                const void* qw, const void* cw, void* pool, int n, int Q, int C, int R, float eps, int adjacent,
+                                int fp32, void* stream) {
   if (n <= 0) return 0;
   if (Q < 0 || C <= 0 || R < 0 || R % 2 || (Q > 0 && qw == nullptr)) return -1;
   auto st = static_cast<cudaStream_t>(stream);
@@ -416,7 +428,7 @@ extern "C" int mx_latent_append(void* a, long long ld, const void* positions, co
   return static_cast<int>(launch_kernel(latent_append_kernel<T, V>, dim3(n), dim3(kLaThreads), 0, st, static_cast<T*>(a), ld,    \
                                         static_cast<const int*>(positions), static_cast<const int*>(slots),                   \
                                         static_cast<const float*>(inv_freq), mscale, static_cast<const float*>(qw),           \
-                                        static_cast<const float*>(cw), static_cast<T*>(pool), Q, C, R, eps))
+                                        static_cast<const float*>(cw), static_cast<T*>(pool), Q, C, R, eps, adjacent))
   if (fp32) {
     if (vec) MX_LA(float, 4);
     MX_LA(float, 1);
@@ -428,27 +440,27 @@ extern "C" int mx_latent_append(void* a, long long ld, const void* positions, co
 
 // q / dst point at the first rotated dimension of the first head; heads are q_head / d_head, tokens ldq / ldd elements apart.
 extern "C" int mx_latent_q_rope(const void* q, long long ldq, int q_head, void* dst, long long ldd, int d_head, const void* positions,
-                                const void* inv_freq, float mscale, int n, int H, int R, int fp32, void* stream) {
+                                const void* inv_freq, float mscale, int n, int H, int R, int adjacent, int fp32, void* stream) {
   if (n <= 0 || R == 0) return 0;
   if (H <= 0 || R < 0 || R % 2 || R > 8192) return -1;
   auto st = static_cast<cudaStream_t>(stream);
 #define MX_LQ(T)                                                                                                              \
   return static_cast<int>(launch_kernel(latent_q_rope_kernel<T>, dim3(n), dim3(kLaThreads), R * sizeof(float), st,            \
                                         static_cast<const T*>(q), ldq, q_head, static_cast<T*>(dst), ldd, d_head,             \
-                                        static_cast<const int*>(positions), static_cast<const float*>(inv_freq), mscale, H, R))
+                                        static_cast<const int*>(positions), static_cast<const float*>(inv_freq), mscale, H, R, adjacent))
   if (fp32) MX_LQ(float);
   MX_LQ(__nv_bfloat16);
 #undef MX_LQ
 }
 
-extern "C" int mx_latent_gather(const void* pool, const void* tables, const void* starts, void* out, int rows, int num_seqs,
-                                int row_bytes, int block_size, int max_blocks, void* stream) {
+extern "C" int mx_latent_gather(const void* pool, const void* tables, const void* starts, const void* zero, void* out, int rows,
+                                int num_seqs, int row_bytes, int block_size, int max_blocks, void* stream) {
   if (rows <= 0) return 0;
   if (num_seqs <= 0 || row_bytes <= 0 || row_bytes % 2 || block_size <= 0) return -1;
   const int unit = row_bytes % 16 == 0 && aligned_to(pool, 16) && aligned_to(out, 16) ? 16 : 2;
   return static_cast<int>(launch_kernel(latent_gather_kernel, dim3((rows + 7) / 8), dim3(256), 0, static_cast<cudaStream_t>(stream),
                                         static_cast<const uint8_t*>(pool), static_cast<const int*>(tables),
-                                        static_cast<const int*>(starts), static_cast<uint8_t*>(out), rows, num_seqs, row_bytes,
+                                        static_cast<const int*>(starts), static_cast<const int*>(zero), static_cast<uint8_t*>(out), rows, num_seqs, row_bytes,
                                         unit, block_size, max_blocks));
 }
 
@@ -463,8 +475,8 @@ extern "C" long long mx_latent_decode_scratch_floats(int B, int H, int C, int nu
 // tcgen05 kernel where it applies (16-token blocks), else the mma.sync one; 1: the mma.sync one. bf16; W at most 576, C at most
 // 512, multiples of 8. -10 = not covered (use mx_paged_attention_any).
 extern "C" int mx_latent_decode(const void* q, long long q_stride, const void* pool, long long pool_rows, const void* block_tables,
-                                const void* context_lens, void* out, float* scratch, int B, int H, int W, int C, int block_size,
-                                int max_blocks, float scale, int num_splits, int form, void* status, void* stream) {
+                                const void* context_lens, const void* sinks, void* out, float* scratch, int B, int H, int W, int C,
+                                int block_size, int max_blocks, int window, float scale, int num_splits, int form, void* status, void* stream) {
   if (B <= 0) return 0;
   if (H <= 0 || C <= 0 || C > W || block_size <= 0) return -1;
   if (W % 8 || C % 8 || W > kLdMaxRow || C > kLdMaxLatent || q_stride % 8 || !aligned_to(q, 16) || !aligned_to(pool, 16)) return -10;
@@ -477,6 +489,8 @@ extern "C" int mx_latent_decode(const void* q, long long q_stride, const void* p
   p.pool = static_cast<const __nv_bfloat16*>(pool);
   p.block_tables = static_cast<const int*>(block_tables);
   p.context_lens = static_cast<const int*>(context_lens);
+  p.sinks = static_cast<const float*>(sinks);
+  p.window = window;
   p.out = static_cast<__nv_bfloat16*>(out);
   p.H = H, p.W = W, p.C = C, p.block_size = block_size, p.max_blocks = max_blocks, p.num_splits = num_splits;
   p.head_tile = hr, p.head_tiles = (H + hr - 1) / hr;

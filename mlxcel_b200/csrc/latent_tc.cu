@@ -73,8 +73,8 @@ latent_decode_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
   const int split = blockIdx.x % p.num_splits, bt = blockIdx.x / p.num_splits;
   const int ht = bt % p.head_tiles, b = bt / p.head_tiles, h0 = ht * N;
   const int len = p.context_lens[b];
-  const int tiles = (len + kLtKeys - 1) / kLtKeys, per = (tiles + p.num_splits - 1) / p.num_splits;
-  const int t0 = split * per, n_tiles = max(0, min(tiles, t0 + per) - t0);
+  const LatentSpan span = latent_span(p, len, split, kLtKeys);
+  const int t0 = span.t0, n_tiles = max(0, span.t1 - t0);
 
   if (threadIdx.x == 0) {
     tma_prefetch_desc(&map_q);
@@ -220,7 +220,8 @@ latent_decode_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
 #pragma unroll
         for (int kk = 0; kk < 4; ++kk) tmem_ld_32x16(lane_addr + ((j & 1) * 4 + kk) * N, r[kk]);
         tmem_ld_wait();
-        const bool in = holds && (t0 + j) * kLtKeys + key < len;
+        const int at = (t0 + j) * kLtKeys + key;
+        const bool in = holds && at < len && at >= span.begin;
 #pragma unroll
         for (int n = 0; n < HT; ++n) {
           const float s = (__uint_as_float(r[0][n]) + __uint_as_float(r[1][n])) + (__uint_as_float(r[2][n]) + __uint_as_float(r[3][n]));
@@ -352,8 +353,9 @@ latent_decode_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
               if (p.num_splits > 1) {
                 p.scratch_o[(part * N + g0 + n) * p.C + c] = o[n];
               } else {
-                const float s = xs[n] + xs[HT + n] + xs[2 * HT + n] + xs[3 * HT + n];
-                p.out[(static_cast<size_t>(b) * p.H + h0 + g0 + n) * p.C + c] = __float2bfloat16(s > 0.f ? o[n] / s : 0.f);
+                float f;
+                const float s = latent_denominator(p, h0 + g0 + n, m_used[n], xs[n] + xs[HT + n] + xs[2 * HT + n] + xs[3 * HT + n], f);
+                p.out[(static_cast<size_t>(b) * p.H + h0 + g0 + n) * p.C + c] = __float2bfloat16(s > 0.f ? o[n] * f / s : 0.f);
               }
             }
           }

@@ -4,6 +4,7 @@
 //                       all experts, then top-k (optionally renormalised; Qwen-MoE). mode 1: top-k
 //                       on the logits, then softmax over the k selected logits (Mixtral, GPT-OSS:
 //                       src/models/gpt_oss.rs:402-446 of the reference).
+//   mx_moe_route_choice fp32 logits: chosen by softmax score + correction, weighted by the score * scale.
 //   mx_moe_align        counts the (token, slot) pairs routed to each LOCAL expert
 //                       [e_begin, e_end), builds exclusive offsets and the permutation that sorts
 //                       pairs by expert (stable in token order, so results are deterministic).
@@ -96,13 +97,67 @@ __global__ void moe_route_kernel(const __nv_bfloat16* __restrict__ logits, int* 
   }
 }
 
+// One warp per token, fp32 logits: softmax over all experts (identity experts included), the k largest score + correction
+// (ties: lowest id), weight = score * scale.
+__global__ void __launch_bounds__(128)
+moe_route_choice_kernel(const float* __restrict__ logits, long long ld, const float* __restrict__ correction, int* __restrict__ ids,
+                        float* __restrict__ wts, int T, int E, int k, float scale) {
+  pdl_trigger();
+  pdl_wait();
+  const int t = (blockIdx.x * blockDim.x + threadIdx.x) >> 5, lane = threadIdx.x & 31;
+  if (t >= T) return;
+  const float* row = logits + static_cast<size_t>(t) * ld;
+  float p[16], c[16], mx = -INFINITY, sum = 0.f;
+#pragma unroll
+  for (int i = 0; i < 16; ++i) {
+    const int e = lane + 32 * i;
+    float v = e < E ? row[e] : -INFINITY;
+    if (!(v == v)) v = -INFINITY;
+    p[i] = v;
+    mx = fmaxf(mx, v);
+  }
+  mx = warp_max(mx);
+  if (mx == -INFINITY) mx = 0.f;                             // (a row without a number: every score is zero)
+#pragma unroll
+  for (int i = 0; i < 16; ++i) p[i] = expf(p[i] - mx), sum += p[i];
+  sum = warp_sum(sum);
+  const float inv = sum > 0.f ? 1.f / sum : 0.f;
+#pragma unroll
+  for (int i = 0; i < 16; ++i) {
+    const int e = lane + 32 * i;
+    p[i] *= inv;
+    c[i] = e < E ? p[i] + (correction != nullptr ? correction[e] : 0.f) : -INFINITY;
+  }
+  for (int s = 0; s < k; ++s) {
+    float best = -INFINITY, score = 0.f;
+    int best_e = 0x7fffffff;
+#pragma unroll
+    for (int i = 0; i < 16; ++i)
+      if (c[i] > best) best = c[i], score = p[i], best_e = lane + 32 * i;
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) {
+      const float ob = __shfl_xor_sync(0xffffffffu, best, o), os = __shfl_xor_sync(0xffffffffu, score, o);
+      const int oe = __shfl_xor_sync(0xffffffffu, best_e, o);
+      if (ob > best || (ob == best && oe < best_e)) best = ob, score = os, best_e = oe;
+    }
+    if (best_e == 0x7fffffff) best_e = s, score = 0.f;       // nothing left above -inf
+#pragma unroll
+    for (int i = 0; i < 16; ++i)
+      if (lane + 32 * i == best_e) c[i] = -INFINITY;
+    if (lane == 0) {
+      ids[static_cast<size_t>(t) * k + s] = best_e;
+      wts[static_cast<size_t>(t) * k + s] = score * scale;
+    }
+  }
+}
+
 // Single CTA: histogram -> exclusive scan -> stable scatter. T * k pairs are at most a few
 // tens of thousands (8192 tokens x top-8), which one 1024-thread CTA sorts in microseconds.
 __global__ void __launch_bounds__(1024)
 moe_align_kernel(const int* __restrict__ topk_ids, int* __restrict__ expert_offsets,
                  int* __restrict__ sorted_pair, int* __restrict__ sorted_token, int pairs, int k,
                  int e_begin, int e_end, const int* __restrict__ n_pairs_dev,
-                 const int* __restrict__ token_map) {
+                 const int* __restrict__ token_map, int* __restrict__ inv) {
   extern __shared__ int sh[];
   // n_pairs_dev: the pair count lives on the device (at most ``pairs``); token_map: the row of x that
   // token i stands for (a compacted list of rows of a larger buffer)
@@ -115,6 +170,7 @@ moe_align_kernel(const int* __restrict__ topk_ids, int* __restrict__ expert_offs
   for (int i = threadIdx.x; i < pairs; i += blockDim.x) {
     const int e = topk_ids[i];
     if (e >= e_begin && e < e_end) atomicAdd(&count[e - e_begin], 1);
+    else if (inv) inv[i] = -1;
   }
   __syncthreads();
   if (threadIdx.x == 0) {
@@ -142,6 +198,7 @@ moe_align_kernel(const int* __restrict__ topk_ids, int* __restrict__ expert_offs
         const int r = pos + __popc(m & ((1u << lane) - 1u));
         sorted_pair[r] = i;
         sorted_token[r] = token_map ? token_map[i / k] : i / k;
+        if (inv) inv[i] = r;
       }
       pos += __popc(m);
     }
@@ -160,7 +217,7 @@ __global__ void __launch_bounds__(1024)
 moe_align_fast_kernel(const int* __restrict__ topk_ids, int* __restrict__ expert_offsets,
                       int* __restrict__ sorted_pair, int* __restrict__ sorted_token, int pairs, int k,
                       int e_begin, int e_end, const int* __restrict__ n_pairs_dev,
-                      const int* __restrict__ token_map) {
+                      const int* __restrict__ token_map, int* __restrict__ inv) {
   extern __shared__ int sh[];
   const int El = e_end - e_begin;
   if (n_pairs_dev) pairs = min(pairs, max(*n_pairs_dev, 0));
@@ -241,7 +298,10 @@ moe_align_fast_kernel(const int* __restrict__ topk_ids, int* __restrict__ expert
       if (hit) {
         sorted_pair[r] = i;
         sorted_token[r] = token_map ? token_map[i / k] : i / k;
+        if (inv) inv[i] = r;
         if (before == 0u) mine[key] += __popc(m);
+      } else if (inv && i < end) {
+        inv[i] = -1;
       }
       __syncwarp();
     }
@@ -363,11 +423,37 @@ extern "C" int mx_moe_align(const int* topk_ids, int* expert_offsets, int* sorte
   if (g_align_fast && El <= kAlignFastMaxExperts)
     moe_align_fast_kernel<<<1, 1024, 33 * El * sizeof(int), stream>>>(topk_ids, expert_offsets, sorted_row,
                                                                      sorted_token, T * k, k, e_begin, e_end,
-                                                                     nullptr, nullptr);
+                                                                     nullptr, nullptr, nullptr);
   else
     moe_align_kernel<<<1, 1024, 2 * El * sizeof(int), stream>>>(topk_ids, expert_offsets, sorted_row,
                                                                 sorted_token, T * k, k, e_begin, e_end,
-                                                                nullptr, nullptr);
+                                                                nullptr, nullptr, nullptr);
+  return static_cast<int>(cudaGetLastError());
+}
+
+// logits fp32 [T, E], rows ld apart; correction fp32 [E] or NULL. E at most 512, k at most 16.
+extern "C" int mx_moe_route_choice(const void* logits, long long ld, const void* correction, int* ids, float* wts, int T, int E, int k,
+                                   float scale, void* stream) {
+  if (T <= 0) return 0;
+  if (E > 512 || k > kMaxTopK || k > E || k < 1) return -1;
+  return static_cast<int>(launch_kernel(moe_route_choice_kernel, dim3((T + 3) / 4), dim3(128), 0, static_cast<cudaStream_t>(stream),
+                                        static_cast<const float*>(logits), ld, static_cast<const float*>(correction), ids, wts, T, E, k,
+                                        scale));
+}
+
+// As mx_moe_align, and the inverse: inv_row[pair] = sorted row of the pair, -1 when its expert is not local.
+extern "C" int mx_moe_align_inv(const int* topk_ids, int* expert_offsets, int* sorted_row, int* sorted_token, int* inv_row, int T, int k,
+                                int e_begin, int e_end, void* stream_) {
+  cudaStream_t stream = static_cast<cudaStream_t>(stream_);
+  const int El = e_end - e_begin;
+  if (T <= 0) return 0;
+  if (El <= 0 || El > 4096) return -1;
+  if (g_align_fast && El <= kAlignFastMaxExperts)
+    moe_align_fast_kernel<<<1, 1024, 33 * El * sizeof(int), stream>>>(topk_ids, expert_offsets, sorted_row, sorted_token, T * k, k, e_begin,
+                                                                     e_end, nullptr, nullptr, inv_row);
+  else
+    moe_align_kernel<<<1, 1024, 2 * El * sizeof(int), stream>>>(topk_ids, expert_offsets, sorted_row, sorted_token, T * k, k, e_begin, e_end,
+                                                                nullptr, nullptr, inv_row);
   return static_cast<int>(cudaGetLastError());
 }
 
@@ -382,11 +468,11 @@ extern "C" int mx_moe_align_n(const int* topk_ids, const int* n_pairs_dev, const
   if (g_align_fast && El <= kAlignFastMaxExperts)
     moe_align_fast_kernel<<<1, 1024, 33 * El * sizeof(int), stream>>>(topk_ids, expert_offsets, sorted_row,
                                                                      sorted_token, max_tokens * k, k, e_begin,
-                                                                     e_end, n_pairs_dev, token_map);
+                                                                     e_end, n_pairs_dev, token_map, nullptr);
   else
     moe_align_kernel<<<1, 1024, 2 * El * sizeof(int), stream>>>(topk_ids, expert_offsets, sorted_row,
                                                                 sorted_token, max_tokens * k, k, e_begin,
-                                                                e_end, n_pairs_dev, token_map);
+                                                                e_end, n_pairs_dev, token_map, nullptr);
   return static_cast<int>(cudaGetLastError());
 }
 

@@ -1,7 +1,8 @@
 // Row kernels of layers that keep the residual stream in fp32 and normalise on both sides of a
 // sub-layer, each for bf16 and fp32 activations:
-//   embed_stream   h = scale * table[id], optionally normalised itself;  x = norm(h) or h as it is
-//   stream_norm    h += norm(y) * layer scale;  x = norm(h) or h as it is     (either half optional)
+//   embed_stream   h = scale * table[id], optionally normalised itself, plus a vector;  x = norm(h) or h as it is
+//   stream_norm    h += norm(y) * layer scale, or y as it is;  h += a token's weighted experts, the embedding again, a
+//                  vector;  x = norm(h) or h as it is                          (every part optional)
 //   polynorm       a N(z) + b N(z^2) + c N(z^3) + e, N = division by the row's root mean square
 //   glu_rows       gated activation of rows gate | up (SwiGLU, tanh-GeGLU, clipped SwiGLU)
 //   softcap_rows   x <- cap tanh(x / cap) in fp32, in place
@@ -16,11 +17,11 @@ namespace mx {
 
 // One CTA per row, V elements per access, up to VPT accesses per thread kept in registers: every
 // input is read once and every output written once.
-template <typename T, int V, int VPT>
-__global__ void __launch_bounds__(1024)
-stream_norm_kernel(const T* __restrict__ y, float* __restrict__ h, const int* __restrict__ rows,
-                   const float* __restrict__ post_w, const float* __restrict__ ls,
-                   const float* __restrict__ pre_w, T* __restrict__ x, int dim, float eps, float w_bias) {
+template <typename T, int V, int VPT, bool EX>
+__device__ __forceinline__ void stream_step(const T* __restrict__ y, float* __restrict__ h, const int* __restrict__ rows,
+                                            const float* __restrict__ post_w, const float* __restrict__ ls,
+                                            const float* __restrict__ pre_w, T* __restrict__ x, int dim, float eps, float w_bias,
+                                            const MxStreamExtras& ex) {
   __shared__ float red[33];
   pdl_trigger();
   pdl_wait();
@@ -33,6 +34,19 @@ stream_norm_kernel(const T* __restrict__ y, float* __restrict__ h, const int* __
     const int c = (threadIdx.x + i * blockDim.x) * V;
     if (c < dim) load_v<V>(hr + c, hv[i]);
   }
+  // hv += f * src[.] over this thread's columns
+  const auto add = [&](const auto* src, float f) {
+#pragma unroll
+    for (int i = 0; i < VPT; ++i) {
+      const int c = (threadIdx.x + i * blockDim.x) * V;
+      if (c < dim) {
+        float a[V];
+        load_v<V>(src + c, a);
+#pragma unroll
+        for (int e = 0; e < V; ++e) hv[i][e] = fmaf(f, a[e], hv[i][e]);
+      }
+    }
+  };
   if (y != nullptr) {
     float yv[VPT][V];
 #pragma unroll
@@ -44,23 +58,47 @@ stream_norm_kernel(const T* __restrict__ y, float* __restrict__ h, const int* __
         for (int e = 0; e < V; ++e) s[0] += yv[i][e] * yv[i][e];
       }
     }
-    block_sums<1>(s, red);
-    const float r = 1.f / sqrtf(s[0] / dim + eps);
+    float r = 1.f;
+    if (post_w != nullptr) {
+      block_sums<1>(s, red);
+      r = 1.f / sqrtf(s[0] / dim + eps);
+    }
     s[0] = 0.f;
 #pragma unroll
     for (int i = 0; i < VPT; ++i) {
       const int c = (threadIdx.x + i * blockDim.x) * V;
       if (c < dim) {
         float w[V], l[V];
-        load_v<V>(post_w + c, w);
+        if (post_w != nullptr) load_v<V>(post_w + c, w);
         if (ls != nullptr) load_v<V>(ls + c, l);
 #pragma unroll
         for (int e = 0; e < V; ++e) {
-          const float b = yv[i][e] * r * (w_bias + w[e]);
+          const float b = post_w != nullptr ? yv[i][e] * r * (w_bias + w[e]) : yv[i][e];
           hv[i][e] += ls != nullptr ? b * l[e] : b;
         }
-        store_v<V>(hr + c, hv[i]);
       }
+    }
+  }
+  if (EX && ex.moe_ids != nullptr) {
+#pragma unroll 4
+    for (int k = 0; k < ex.moe_k; ++k) {
+      const size_t pair = row * ex.moe_k + k;
+      const T* src = ex.moe_ids[pair] >= ex.moe_experts ? static_cast<const T*>(ex.moe_x) + row * dim
+                                                        : static_cast<const T*>(ex.moe_y) + static_cast<size_t>(ex.moe_inv[pair]) * dim;
+      add(src, ex.moe_w[pair]);
+    }
+    if (ex.moe_shared != nullptr) add(static_cast<const T*>(ex.moe_shared) + row * dim, 1.f);
+  }
+  if (EX && ex.ids != nullptr) {
+    const int id = ex.ids[row];
+    if (id >= 0 && id < ex.vocab) add(static_cast<const T*>(ex.table) + static_cast<size_t>(id) * dim, ex.emb_scale);
+  }
+  if (EX && ex.vec != nullptr) add(ex.vec, 1.f);
+  if (EX || y != nullptr) {
+#pragma unroll
+    for (int i = 0; i < VPT; ++i) {
+      const int c = (threadIdx.x + i * blockDim.x) * V;
+      if (c < dim) store_v<V>(hr + c, hv[i]);
     }
   }
   if (x == nullptr) return;
@@ -97,8 +135,23 @@ stream_norm_kernel(const T* __restrict__ y, float* __restrict__ h, const int* __
 
 template <typename T, int V, int VPT>
 __global__ void __launch_bounds__(1024)
+stream_norm_kernel(const T* __restrict__ y, float* __restrict__ h, const int* __restrict__ rows, const float* __restrict__ post_w,
+                   const float* __restrict__ ls, const float* __restrict__ pre_w, T* __restrict__ x, int dim, float eps, float w_bias) {
+  stream_step<T, V, VPT, false>(y, h, rows, post_w, ls, pre_w, x, dim, eps, w_bias, MxStreamExtras{});
+}
+
+template <typename T, int V, int VPT>
+__global__ void __launch_bounds__(1024)
+stream_sum_kernel(const T* __restrict__ y, float* __restrict__ h, const float* __restrict__ post_w, const float* __restrict__ ls,
+                  const float* __restrict__ pre_w, T* __restrict__ x, int dim, float eps, float w_bias, const MxStreamExtras ex) {
+  stream_step<T, V, VPT, true>(y, h, nullptr, post_w, ls, pre_w, x, dim, eps, w_bias, ex);
+}
+
+template <typename T, int V, int VPT>
+__global__ void __launch_bounds__(1024)
 embed_stream_kernel(const int* __restrict__ ids, const T* __restrict__ table, float* __restrict__ h,
-                    const float* __restrict__ own_w, const float* __restrict__ pre_w, T* __restrict__ x, int dim, int vocab,
+                    const float* __restrict__ own_w, const float* __restrict__ vec, const float* __restrict__ pre_w, T* __restrict__ x,
+                    int dim, int vocab,
                     float scale, float eps, float w_bias) {
   __shared__ float red[33];
   pdl_trigger();
@@ -115,10 +168,15 @@ embed_stream_kernel(const int* __restrict__ ids, const T* __restrict__ table, fl
     if (c < dim) {
       load_v<V>(tr + c, hv[i]);
 #pragma unroll
-      for (int e = 0; e < V; ++e) {
-        hv[i][e] = ok ? hv[i][e] * scale : 0.f;
-        s[0] += hv[i][e] * hv[i][e];
+      for (int e = 0; e < V; ++e) hv[i][e] = ok ? hv[i][e] * scale : 0.f;
+      if (own_w == nullptr && vec != nullptr) {
+        float a[V];
+        load_v<V>(vec + c, a);
+#pragma unroll
+        for (int e = 0; e < V; ++e) hv[i][e] += a[e];
       }
+#pragma unroll
+      for (int e = 0; e < V; ++e) s[0] += hv[i][e] * hv[i][e];
       if (own_w == nullptr) store_v<V>(h + row * dim + c, hv[i]);
     }
   }
@@ -130,11 +188,12 @@ embed_stream_kernel(const int* __restrict__ ids, const T* __restrict__ table, fl
     for (int i = 0; i < VPT; ++i) {
       const int c = (threadIdx.x + i * blockDim.x) * V;
       if (c < dim) {
-        float w[V];
+        float w[V], a[V];
         load_v<V>(own_w + c, w);
+        if (vec != nullptr) load_v<V>(vec + c, a);
 #pragma unroll
         for (int e = 0; e < V; ++e) {
-          hv[i][e] = hv[i][e] * r * (w_bias + w[e]);
+          hv[i][e] = hv[i][e] * r * (w_bias + w[e]) + (vec != nullptr ? a[e] : 0.f);
           s[0] += hv[i][e] * hv[i][e];
         }
         store_v<V>(h + row * dim + c, hv[i]);
@@ -357,27 +416,30 @@ static RowShape row_shape(int dim, int v) {
 
 template <typename T>
 static int stream_norm_typed(const void* y, void* h, const void* rows, const float* post_w, const float* ls, const float* pre_w,
-                             void* x, int n, int dim, float eps, float w_bias, bool vec, cudaStream_t st) {
+                             void* x, int n, int dim, float eps, float w_bias, const MxStreamExtras* ex, bool vec, cudaStream_t st) {
   const T* yp = static_cast<const T*>(y);
   const int* rp = static_cast<const int*>(rows);
-  if (vec) {
-    const RowShape sh = row_shape(dim, 4);
-    MX_ROW_DISPATCH(stream_norm_kernel, T, 4, sh, n, st, yp, static_cast<float*>(h), rp, post_w, ls, pre_w, static_cast<T*>(x), dim, eps, w_bias)
+  const RowShape sh = row_shape(dim, vec ? 4 : 1);
+  auto *hp = static_cast<float*>(h);
+  auto *xp = static_cast<T*>(x);
+  if (ex != nullptr) {
+    if (vec) MX_ROW_DISPATCH(stream_sum_kernel, T, 4, sh, n, st, yp, hp, post_w, ls, pre_w, xp, dim, eps, w_bias, *ex)
+    MX_ROW_DISPATCH(stream_sum_kernel, T, 1, sh, n, st, yp, hp, post_w, ls, pre_w, xp, dim, eps, w_bias, *ex)
   }
-  const RowShape sh = row_shape(dim, 1);
-  MX_ROW_DISPATCH(stream_norm_kernel, T, 1, sh, n, st, yp, static_cast<float*>(h), rp, post_w, ls, pre_w, static_cast<T*>(x), dim, eps, w_bias)
+  if (vec) MX_ROW_DISPATCH(stream_norm_kernel, T, 4, sh, n, st, yp, hp, rp, post_w, ls, pre_w, xp, dim, eps, w_bias)
+  MX_ROW_DISPATCH(stream_norm_kernel, T, 1, sh, n, st, yp, hp, rp, post_w, ls, pre_w, xp, dim, eps, w_bias)
 }
 
 template <typename T>
-static int embed_stream_typed(const int* ids, const void* table, void* h, const float* own_w, const float* pre_w, void* x, int n, int dim, int vocab,
+static int embed_stream_typed(const int* ids, const void* table, void* h, const float* own_w, const float* add, const float* pre_w, void* x, int n, int dim, int vocab,
                               float scale, float eps, float w_bias, bool vec, cudaStream_t st) {
   const T* tp = static_cast<const T*>(table);
   if (vec) {
     const RowShape sh = row_shape(dim, 4);
-    MX_ROW_DISPATCH(embed_stream_kernel, T, 4, sh, n, st, ids, tp, static_cast<float*>(h), own_w, pre_w, static_cast<T*>(x), dim, vocab, scale, eps, w_bias)
+    MX_ROW_DISPATCH(embed_stream_kernel, T, 4, sh, n, st, ids, tp, static_cast<float*>(h), own_w, add, pre_w, static_cast<T*>(x), dim, vocab, scale, eps, w_bias)
   }
   const RowShape sh = row_shape(dim, 1);
-  MX_ROW_DISPATCH(embed_stream_kernel, T, 1, sh, n, st, ids, tp, static_cast<float*>(h), own_w, pre_w, static_cast<T*>(x), dim, vocab, scale, eps, w_bias)
+  MX_ROW_DISPATCH(embed_stream_kernel, T, 1, sh, n, st, ids, tp, static_cast<float*>(h), own_w, add, pre_w, static_cast<T*>(x), dim, vocab, scale, eps, w_bias)
 }
 
 template <typename T>
@@ -405,33 +467,37 @@ static int qk_norm_append_typed(void* qkv, long long ld, const int* slots, void*
 
 using namespace mx;
 
-// fp32: 1 = fp32 activations, 0 = bf16. y / rows / ls / x may be NULL (no branch to add, identity
-// row map, no layer scale, no output); x with pre_w == NULL receives the stream itself.
+// fp32: 1 = fp32 activations, 0 = bf16. y / rows / post_w / ls / extras / x may be NULL (no branch to add, identity row
+// map, the branch is not normalised, no layer scale, nothing else to add, no output); x with pre_w == NULL receives the stream itself.
 extern "C" int mx_stream_norm(const void* y, void* h, const void* rows, const void* post_w, const void* ls,
                               const void* pre_w, void* x, int n, int dim, float eps, float w_bias, int fp32,
-                              void* stream) {
+                              const MxStreamExtras* extras, void* stream) {
   if (n <= 0 || dim <= 0) return 0;
-  if (h == nullptr || (y != nullptr && (post_w == nullptr || rows != nullptr))) return -1;
+  const MxStreamExtras ex = extras != nullptr ? *extras : MxStreamExtras{};
+  if (h == nullptr || (rows != nullptr && (y != nullptr || extras != nullptr))) return -1;
+  if (ex.moe_ids != nullptr && (ex.moe_x == nullptr || ex.moe_y == nullptr || ex.moe_inv == nullptr || ex.moe_w == nullptr)) return -1;
+  if (ex.ids != nullptr && (ex.table == nullptr || ex.vec == nullptr)) return -1;
   const size_t ab = fp32 ? 16 : 8;
   const bool vec = dim % 4 == 0 && aligned_to(y, ab) && aligned_to(x, ab) && aligned_to(h, 16) && aligned_to(post_w, 16) &&
-                   aligned_to(ls, 16) && aligned_to(pre_w, 16);
+                   aligned_to(ls, 16) && aligned_to(pre_w, 16) && aligned_to(ex.moe_y, ab) && aligned_to(ex.moe_x, ab) &&
+                   aligned_to(ex.moe_shared, ab) && aligned_to(ex.table, ab) && aligned_to(ex.vec, 16);
   auto st = static_cast<cudaStream_t>(stream);
   const float *pw = static_cast<const float*>(post_w), *lp = static_cast<const float*>(ls), *nw = static_cast<const float*>(pre_w);
-  return fp32 ? stream_norm_typed<float>(y, h, rows, pw, lp, nw, x, n, dim, eps, w_bias, vec, st)
-              : stream_norm_typed<__nv_bfloat16>(y, h, rows, pw, lp, nw, x, n, dim, eps, w_bias, vec, st);
+  return fp32 ? stream_norm_typed<float>(y, h, rows, pw, lp, nw, x, n, dim, eps, w_bias, extras, vec, st)
+              : stream_norm_typed<__nv_bfloat16>(y, h, rows, pw, lp, nw, x, n, dim, eps, w_bias, extras, vec, st);
 }
 
-extern "C" int mx_embed_stream(const void* ids, const void* table, void* h, const void* own_w, const void* pre_w, void* x,
-                               int n, int dim, int vocab, float scale, float eps, float w_bias, int fp32, void* stream) {
+extern "C" int mx_embed_stream(const void* ids, const void* table, void* h, const void* own_w, const void* add, const void* pre_w,
+                               void* x, int n, int dim, int vocab, float scale, float eps, float w_bias, int fp32, void* stream) {
   if (n <= 0 || dim <= 0) return 0;
   const size_t ab = fp32 ? 16 : 8;
   const bool vec = dim % 4 == 0 && aligned_to(table, ab) && aligned_to(x, ab) && aligned_to(h, 16) && aligned_to(own_w, 16) &&
-                   aligned_to(pre_w, 16);
+                   aligned_to(pre_w, 16) && aligned_to(add, 16);
   auto st = static_cast<cudaStream_t>(stream);
-  const float *ow = static_cast<const float*>(own_w), *nw = static_cast<const float*>(pre_w);
+  const float *ow = static_cast<const float*>(own_w), *av = static_cast<const float*>(add), *nw = static_cast<const float*>(pre_w);
   const int* ip = static_cast<const int*>(ids);
-  return fp32 ? embed_stream_typed<float>(ip, table, h, ow, nw, x, n, dim, vocab, scale, eps, w_bias, vec, st)
-              : embed_stream_typed<__nv_bfloat16>(ip, table, h, ow, nw, x, n, dim, vocab, scale, eps, w_bias, vec, st);
+  return fp32 ? embed_stream_typed<float>(ip, table, h, ow, av, nw, x, n, dim, vocab, scale, eps, w_bias, vec, st)
+              : embed_stream_typed<__nv_bfloat16>(ip, table, h, ow, av, nw, x, n, dim, vocab, scale, eps, w_bias, vec, st);
 }
 
 extern "C" int mx_polynorm(const void* z, const void* coef, void* out, int n, int dim, float eps, int fp32, void* stream) {

@@ -28,13 +28,14 @@ class LLM:
         if model is not None:
             self.model = model
         elif cfg.model_type in ("mamba", "mamba2", "nemotron_h", "granitemoehybrid", "jamba", "qwen3_next", "qwen3_5", "qwen3_5_text",
-                                "qwen3_5_moe", "qwen3_5_moe_text", "falcon_h1", "lfm2", "lfm2_moe", "recurrent_gemma", "pamasun", "govopel"):
+                                "qwen3_5_moe", "qwen3_5_moe_text", "falcon_h1", "lfm2", "lfm2_moe", "recurrent_gemma", "pamasun", "govopel",
+                                "vavadra"):
             from .models.hybrid import HybridModel
             from .models.mamba1 import Mamba1Model
             from .models.mamba2 import Mamba2Model
             cls = {"mamba": Mamba1Model, "mamba2": Mamba2Model}.get(cfg.model_type, HybridModel)
             ec = engine_config or EngineConfig()
-            kw = dict(kv_bits=ec.kv_bits) if cfg.model_type in ("pamasun", "govopel") else {}
+            kw = dict(kv_bits=ec.kv_bits) if cfg.model_type in ("pamasun", "govopel", "vavadra") else {}
             self.model = cls(cfg, weights, comm=comm, max_seqs=ec.state_slots or 2 * ec.max_batch, **kw)
         else:
             self.model = DecoderModel(cfg, weights, comm=comm,
@@ -65,6 +66,9 @@ class LLM:
         if cfg.model_type == "govopel":
             from .models.govopel import random_govopel_weights
             return LLM(cfg, random_govopel_weights(cfg, seed=seed, dtype=dtype, device=device), engine_config, comm=comm)
+        if cfg.model_type == "vavadra":
+            from .models.vavadra import random_vavadra_weights
+            return LLM(cfg, random_vavadra_weights(cfg, seed=seed, dtype=dtype, device=device), engine_config, comm=comm)
         tp = comm.tp_size if comm is not None else 1
         rank = comm.tp_rank if comm is not None else 0
         hook = None
@@ -101,6 +105,10 @@ class LLM:
         if cfg.model_type == "govopel":
             from .models.govopel import load_govopel_weights
             return LLM(cfg, load_govopel_weights(path, cfg, dtype=dtype or torch.bfloat16, device=device), engine_config,
+                       comm=comm, tokenizer=load_tokenizer(path))
+        if cfg.model_type == "vavadra":
+            from .models.vavadra import load_vavadra_weights
+            return LLM(cfg, load_vavadra_weights(path, cfg, dtype=dtype or torch.bfloat16, device=device), engine_config,
                        comm=comm, tokenizer=load_tokenizer(path))
         if dtype not in (None, torch.bfloat16):
             raise ValueError(f"{cfg.model_type} models are served in bf16")

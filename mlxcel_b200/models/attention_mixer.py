@@ -9,10 +9,12 @@
 * scores: ``q.k * scale``, soft-capped (``softcap tanh(s / softcap)``) where a cap is given; ``exp(sink_h)`` in the
   denominator;
 * values: heads of their own width, or the keys as projected (``values_are_keys``: no value projection);
-* a sigmoid gate computed from the mixer's input on the concatenated heads.
+* a sigmoid gate computed from the mixer's input on the concatenated heads;
+* differential heads (``diff``): query and key rows hold two maps of ``dim / 2`` each, attentions of their own over the same
+  values; the head is ``a1 - factor * a2``, divided by its root mean square, times a gain.
 
 One GEMM produces q | k | v | gate; one kernel rotates and normalises q and k and appends k, v to the paged pool; the
-attention kernels cap, mask and gate. Scores, bias, softmax and accumulation are fp32.
+attention kernels cap, mask, gate and combine the maps. Scores, bias, softmax and accumulation are fp32.
 """
 from __future__ import annotations
 
@@ -46,6 +48,8 @@ class AttentionMixerWeights:
     mscale: float = 1.0
     unit: bool = False                    # with a rotation: q and k divided by their root mean square behind it
     values_are_keys: bool = False
+    b_in: torch.Tensor | None = None      # biases of w_in's rows
+    diff: tuple | None = None             # (factor of the second map, gain)
 
 
 def stack_rows(parts: list[torch.Tensor]) -> torch.Tensor:
@@ -60,7 +64,7 @@ def attention_mixer(w: AttentionMixerWeights, x: torch.Tensor, b, kv, eps: float
     """x [T, H] normalised input, ``b`` the step's batch, ``kv`` this run's pool layer. Returns the gated heads
     [T, heads * vdim] (the input of ``out_proj``)."""
     T, nd = x.shape[0], b.num_decode
-    row = ops.linear(x, w.w_in)
+    row = ops.linear(x, w.w_in, bias=w.b_in)
     geo = dict(Hq=w.heads, Hkv=w.kv_heads, Dk=w.dim, Dv=w.vdim)
     if w.inv_freq is not None:
         stream.rope_norm_append(row, b.positions, b.slot_mapping, kv, inv_freq=w.inv_freq, mscale=w.mscale, unit=w.unit,
@@ -72,7 +76,7 @@ def attention_mixer(w: AttentionMixerWeights, x: torch.Tensor, b, kv, eps: float
     gate = row[:, g0:g0 + w.heads * w.vdim] if w.gated else None
     out = torch.empty(T, w.heads * w.vdim, dtype=row.dtype, device=row.device)
     common = dict(scale=w.scale, window=w.window, chunk=w.chunk, softcap=w.softcap, sinks=w.sinks,
-                  dist_bias=None if w.r1 is None else (w.r1, w.r2), **geo)
+                  dist_bias=None if w.r1 is None else (w.r1, w.r2), diff=None if w.diff is None else (*w.diff, eps), **geo)
     if nd > 0:
         stream.paged_attention(q[:nd], kv, b.dec_block_tables, b.dec_context_lens, None, out[:nd], max_q_len=1,
                                max_len=b.dec_max_len, gate=None if gate is None else gate[:nd], **common)

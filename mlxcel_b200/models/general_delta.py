@@ -47,11 +47,14 @@ class GeneralDeltaModel(Mamba2Model):
         self.comm = comm or LocalComm()
         if self.comm.tp_size != 1:
             raise NotImplementedError("the delta-rule executor is single-GPU")
-        self.state = [torch.zeros(max_seqs, w.heads, w.dim, w.dim, dtype=torch.float32, device=device) for w in runs]
+        self.state = self._slabs(runs, max_seqs)
         self.slot_of: dict[int, int] = {}
         self.free = list(range(max_seqs - 1, -1, -1))
         self._iota = torch.arange(max_seqs + 1, dtype=torch.int32, device=device)
         self._no_reset = torch.zeros(max_seqs + 1, dtype=torch.int32, device=device)
+
+    def _slabs(self, runs: list, max_seqs: int) -> list:
+        return [torch.zeros(max_seqs, w.heads, w.dim, w.dim, dtype=torch.float32, device=self.device) for w in runs]
 
     def _slot(self, seq_id: int, resets: bool) -> int:
         s = self.slot_of.get(seq_id)

@@ -15,11 +15,13 @@ A model is a flat list of pre-norm residual blocks; the family decides the list 
 =====  ===============================================================================================
 
 A second layout ("stream") serves designs that keep the residual in fp32 and normalise every sub-layer on
-both sides or behind it only: ``h <- h + layer_scale * norm(branch(norm(h)))``, the inner norm left out where a block's
-``norm`` is None. Its blocks carry ``post_norm`` / ``layer_scale``, its mixers are ``attention_mixer``
-(``models/attention_mixer.py``), ``latent_mixer`` (``models/latent_mixer.py``) and ``general_delta``
-(``models/general_delta.py``), and ``HybridWeights.runs`` lists the layers in execution order: a layer may run several times
-with the same weights, each run with a KV-pool layer or state slab of its own (Pamasun, Govopel).
+both sides, behind it or in front of it only: ``h <- h + layer_scale * norm(branch(norm(h)))``, the inner norm left out
+where a block's ``norm`` is None, the outer one where its ``post_norm`` is. Its mixers are ``attention_mixer``
+(``models/attention_mixer.py``), ``latent_mixer`` (``models/latent_mixer.py``), ``general_delta``
+(``models/general_delta.py``) and ``gated_delta`` (``models/gated_delta.py``), its feed-forwards ``mlp`` and ``moe_stream``
+(``models/moe.py``), and ``HybridWeights.runs`` lists the layers in execution order: a layer may run several times
+with the same weights, each run with a KV-pool layer or state slab of its own; ``run_entries`` adds a vector, and the
+embedding once more, in front of a run (Pamasun, Govopel, Vavadra).
 
 Nemotron-H gives one block per layer through ``hybrid_override_pattern`` (``"M-M-M*-..."``); the other
 families have a mixer block and an MLP / MoE block per layer. Reference: src/models/nemotron_h.rs,
@@ -76,6 +78,7 @@ class HybridWeights:
     layers: list = field(default_factory=list)  # the attention blocks' LayerWeights (= KV-pool layers)
     runs: list | None = None                    # stream layout: the layers (lists of blocks) in execution order
     embed_norm: torch.Tensor | None = None      # stream layout: norm of the embedding itself
+    run_entries: dict = field(default_factory=dict)   # stream layout: run index -> (add the embedding, fp32 vector to add) ahead of it
 
 
 _KINDS = {"M": "mamba2", "m": "mamba1", "L": "gdn", "C": "shortconv", "R": "rglru", "P": "parallel", "*": "attention", "A": "attention", "-": "mlp", "G": "mlp",
@@ -682,6 +685,7 @@ class HybridModel:
         self.num_kv_layers = len(weights.layers)
 
     def _init_stream(self, max_seqs: int, kv_bits: int) -> None:
+        from .gated_delta import GatedDeltaModel
         from .general_delta import GeneralDeltaModel
         cfg, w = self.cfg, self.w
         if kv_bits != 16:
@@ -689,24 +693,29 @@ class HybridModel:
         self.dtype = w.embed.dtype
         # (block, index of its KV layer or state slab, run index behind its last block or -1)
         self.order: list = []
-        delta, n_kv, self._kv_heads, self._latent_heads = [], 0, set(), set()
+        # KV splits of decode depend on (key heads, tokens a query sees at most or 0)
+        delta, n_kv, self._kv_spans, self._latent_spans = [], 0, set(), set()
         for r, blocks in enumerate(w.runs):
             for blk in blocks:
                 idx = -1
                 if blk.kind == "attention_mixer":
                     idx, n_kv = n_kv, n_kv + 1
-                    self._kv_heads.add(blk.attn.kv_heads)
+                    self._kv_spans.add((blk.attn.kv_heads, blk.attn.window or blk.attn.chunk))
                 elif blk.kind == "latent_mixer":
                     idx, n_kv = n_kv, n_kv + 1
-                    self._latent_heads.add(blk.attn.heads)
-                elif blk.kind == "general_delta":
+                    self._latent_spans.add((blk.attn.heads, blk.attn.window))
+                elif blk.kind in ("general_delta", "gated_delta"):
                     idx = len(delta)
-                    delta.append(blk.mamba)
+                    delta.append(blk)
                 self.order.append((blk, idx, r if blk is blocks[-1] else -1))
+        kinds = {blk.kind for blk in delta}
+        if len(kinds) > 1:
+            raise ValueError(f"one kind of recurrent mixer per model, not {sorted(kinds)}")
         self.num_kv_layers = n_kv
         self.Hq, self.Hkv, self.D = cfg.num_attention_heads, cfg.num_key_value_heads, cfg.head_dim
         # only the delta mixers carry state: a stack without them is served like any attention model
-        self.ssm = GeneralDeltaModel(delta, cfg.rms_norm_eps, self.device, max_seqs, self.comm) if delta else None
+        cls = GatedDeltaModel if kinds == {"gated_delta"} else GeneralDeltaModel
+        self.ssm = cls([blk.mamba for blk in delta], cfg.rms_norm_eps, self.device, max_seqs, self.comm) if delta else None
         self.recurrent = self.ssm is not None
         self.state_slots_on_device = self.recurrent
 
@@ -715,8 +724,9 @@ class HybridModel:
         if self.w.runs is None:
             return (ops.decode_splits(rows, self.Hkv, max_len),)
         from ..ops.latent import latent_splits
-        return tuple(ops.decode_splits(rows, h, max_len) for h in sorted(self._kv_heads)) + \
-            tuple(latent_splits(rows, h, max_len) for h in sorted(self._latent_heads))
+        from ..ops.stream import visible
+        return tuple(ops.decode_splits(rows, h, visible(max_len, n)) for h, n in sorted(self._kv_spans)) + \
+            tuple(latent_splits(rows, h, visible(max_len, n)) for h, n in sorted(self._latent_spans))
 
     def state_slot(self, seq_id: int) -> int:
         return self.ssm.slot(seq_id)
@@ -730,29 +740,41 @@ class HybridModel:
         from ..ops import stream
         from .attention_mixer import attention_mixer
         from .latent_mixer import latent_mixer
+        from .moe import moe_stream
         cfg, eps, wb = self.cfg, self.cfg.rms_norm_eps, self.cfg.norm_weight_bias
         if b.embeds is not None:
             raise NotImplementedError("media embeddings with an fp32 residual stream")
         pieces = self.ssm.pieces(b) if self.ssm is not None else None
         self.captured = []
+        entries = {r: stream.Entry(vec, b.token_ids if again else None, self.w.embed, cfg.embed_scale)
+                   for r, (again, vec) in self.w.run_entries.items()}
+        first = entries.get(0)
         h, x = stream.embed_stream(b.token_ids, self.w.embed, cfg.embed_scale,
-                                   self.order[0][0].norm if self.order else self.w.final_norm, eps, wb, self.w.embed_norm)
+                                   self.order[0][0].norm if self.order else self.w.final_norm, eps, wb, self.w.embed_norm,
+                                   vec=None if first is None else first.vec)
         for n, (blk, idx, run) in enumerate(self.order):
+            rows = None
             if blk.kind == "attention_mixer":
                 y = ops.linear(attention_mixer(blk.attn, x, b, kv_layers[idx], eps), blk.attn.out_proj)
             elif blk.kind == "latent_mixer":
                 y = ops.linear(latent_mixer(blk.attn, x, b, kv_layers[idx], eps), blk.attn.out_proj)
-            elif blk.kind == "general_delta":
+            elif blk.kind in ("general_delta", "gated_delta"):
                 y = ops.linear(self.ssm.mixer(idx, blk.mamba, x, pieces), blk.mamba.out_proj)
+            elif blk.kind == "moe_stream":
+                y, rows = None, moe_stream(blk.moe, x)
             elif blk.act == "polynorm":
                 y = ops.linear(stream.polynorm(ops.linear(x, blk.up), blk.act_coef, eps), blk.down)
             else:
                 y = ops.linear(ops.glu_linear(x, blk.up, blk.up.shape[0] // 2, blk.act, alpha=blk.act_alpha, limit=blk.act_limit), blk.down)
             last = n + 1 == len(self.order)
             nxt = None if last else self.order[n + 1][0].norm
-            x = stream.stream_norm(h, y, blk.post_norm, blk.layer_scale, nxt, eps, wb, plain=not last)
-            if run in self.capture_layers:
+            entry = entries.get(run + 1) if run >= 0 and not last else None
+            if run in self.capture_layers:        # (what comes ahead of the next run is a step of its own then)
+                stream.stream_norm(h, y, blk.post_norm, blk.layer_scale, None, eps, wb, dtype=self.dtype, moe=rows)
                 self.captured.append(h.clone())
+                y = rows = None
+            x = stream.stream_norm(h, y, blk.post_norm, blk.layer_scale, nxt, eps, wb, dtype=self.dtype, plain=not last, moe=rows,
+                                   entry=entry)
         return h
 
     @torch.inference_mode()

@@ -9,6 +9,8 @@ Reference: MLPBlock.forward (src/models/gpt_oss.rs:402-446), SwitchGLU
 """
 from __future__ import annotations
 
+from dataclasses import dataclass
+
 import torch
 
 from .. import ops
@@ -93,3 +95,32 @@ def moe_forward(cfg, lw: LayerWeights, x: torch.Tensor, h: torch.Tensor, comm) -
     if ep > 1:
         out = comm.all_reduce(out)
     return out
+
+
+# ----------------------------------------------------------------------------- stream layout
+@dataclass
+class MoeBlockWeights:
+    """Mixture of clipped-GLU experts of the stream layout: softmax scores over all experts, chosen by score + correction,
+    weighted by score * scale. Experts from ``len(gate_up)`` on are identity experts; the shared expert is optional."""
+
+    router: torch.Tensor                      # [experts + identity experts, H]
+    correction: torch.Tensor                  # fp32, per expert
+    gate_up: torch.Tensor                     # [experts, 2 * ff, H], gate rows first
+    down: torch.Tensor                        # [experts, H, ff]
+    top: int
+    scale: float
+    limit: float
+    alpha: float
+    shared_gate_up: torch.Tensor | None = None
+    shared_down: torch.Tensor | None = None
+    shared_limit: float = 0.0
+
+
+def moe_stream(w: MoeBlockWeights, x: torch.Tensor) -> moe_ops.MoeRows:
+    """x [T, H] normalised input. Returns the chosen experts' rows for the step of the stream that sums them up."""
+    ids, wts = moe_ops.route_choice(ops.linear(x, w.router, out_fp32=True), w.correction, w.top, w.scale)
+    rows = moe_ops.expert_rows(x, ids, wts, w.gate_up, w.down, w.alpha, w.limit)
+    if w.shared_gate_up is not None:
+        a = ops.glu_linear(x, w.shared_gate_up, w.shared_gate_up.shape[0] // 2, "clipped_swiglu", alpha=w.alpha, limit=w.shared_limit)
+        rows.shared = ops.linear(a, w.shared_down)
+    return rows

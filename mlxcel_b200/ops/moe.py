@@ -8,6 +8,7 @@ src/models/gpt_oss.rs:402-446 of the reference.
 from __future__ import annotations
 
 import os
+from dataclasses import dataclass
 
 import torch
 
@@ -283,3 +284,96 @@ def moe_experts_rows(x: torch.Tensor, ids_c: torch.Tensor, row_map: torch.Tensor
     _lib.check(rc, "mx_moe_scatter_rows_n")
     _lib.count_launch(3)
     return out
+
+
+# ----------------------------------------------------------------------------- stream layout
+@dataclass
+class MoeRows:
+    """What a token's chosen experts returned, before they are summed: pair (t, s) went to expert ``ids[t, s]`` with weight
+    ``wts[t, s]``; its result is row ``inv[t * k + s]`` of ``y``, or the input row ``x[t]`` itself for an identity expert
+    (``ids >= experts``). ``shared`` rows are added as they are."""
+
+    y: torch.Tensor                       # [pairs, H]
+    x: torch.Tensor                       # [T, H]
+    ids: torch.Tensor                     # [T, k] int32
+    inv: torch.Tensor                     # [T * k] int32
+    wts: torch.Tensor                     # [T, k] fp32
+    experts: int
+    shared: torch.Tensor | None = None    # [T, H]
+
+    def summed(self) -> torch.Tensor:
+        """fp32 [T, H] (plain statement of what the stream kernel adds)."""
+        T, k = self.ids.shape
+        own = self.ids >= self.experts
+        rows = self.y[self.inv.clamp(min=0).long()].view(T, k, -1).float() if self.y.shape[0] else torch.zeros(T, k, self.x.shape[1])
+        out = (torch.where(own[..., None], self.x[:, None].float(), rows) * self.wts[..., None]).sum(1)
+        return out if self.shared is None else out + self.shared.float()
+
+
+def route_choice_ref(logits, correction, k: int, scale: float):
+    p = torch.softmax(logits.float(), -1)
+    ids = (p if correction is None else p + correction).topk(k, -1)[1]
+    return ids.to(torch.int32).contiguous(), (p.gather(1, ids) * scale).contiguous()
+
+
+def route_choice(logits: torch.Tensor, correction: torch.Tensor | None, k: int, scale: float):
+    """Router logits [T, E] fp32 -> (ids [T, k] int32, weights [T, k] fp32): the k experts with the largest softmax score plus
+    ``correction`` (fp32 [E]), weighted by the score itself times ``scale``, not renormalised."""
+    T, E = logits.shape
+    if not logits.is_cuda or E > 512 or k > 16:
+        return route_choice_ref(logits, correction, k, scale)
+    assert logits.dtype == torch.float32 and logits.stride(1) == 1
+    ids = torch.empty(T, k, dtype=torch.int32, device=logits.device)
+    wts = torch.empty(T, k, dtype=torch.float32, device=logits.device)
+    rc = _lib.load().mx_moe_route_choice(logits.data_ptr(), logits.stride(0), _lib.ptr(correction), ids.data_ptr(), wts.data_ptr(), T, E,
+                                         k, float(scale), _lib.stream())
+    _lib.count_launch()
+    _lib.check(rc, "mx_moe_route_choice")
+    return ids, wts
+
+
+def expert_rows(x: torch.Tensor, ids: torch.Tensor, wts: torch.Tensor, w_gate_up: torch.Tensor, w_down: torch.Tensor, alpha: float,
+                limit: float, force_any: bool = False) -> MoeRows:
+    """The chosen experts' clipped-GLU rows of every token, unsummed. ``w_gate_up`` [E, 2 I, H] (gate rows first), ``w_down``
+    [E, H, I]; ids from E on are identity experts and cost nothing here. bf16 rows of widths TMA can address run the
+    grouped tcgen05 GEMMs, the rest the SIMT ones."""
+    T, k = ids.shape
+    E, I, H = w_gate_up.shape[0], w_gate_up.shape[1] // 2, x.shape[1]
+    if not x.is_cuda:
+        y, inv = [], torch.full((T * k,), -1, dtype=torch.int32)
+        for e in range(E):
+            tok, slot = torch.nonzero(ids == e, as_tuple=True)
+            inv[tok * k + slot] = torch.arange(tok.numel(), dtype=torch.int32) + sum(r.shape[0] for r in y)
+            a = ref.glu_linear(x[tok], w_gate_up[e], I, ref.EPI_CLIPPED_SWIGLU, None, alpha, limit)
+            y.append(ref.linear(a, w_down[e]))
+        return MoeRows(torch.cat(y), x, ids, inv, wts, E)
+    lib, st, dev, pairs = _lib.load(), _lib.stream(), x.device, T * k
+    meta = torch.empty(E + 1 + 3 * pairs, dtype=torch.int32, device=dev)
+    offsets, pair, token, inv = meta[:E + 1], meta[E + 1:E + 1 + pairs], meta[E + 1 + pairs:E + 1 + 2 * pairs], meta[E + 1 + 2 * pairs:]
+    if T == 0:
+        return MoeRows(x.new_empty(0, H), x, ids, inv, wts, E)
+    assert x.is_contiguous() and w_gate_up.is_contiguous() and w_down.is_contiguous()
+    _lib.check(lib.mx_moe_align_inv(ids.data_ptr(), offsets.data_ptr(), pair.data_ptr(), token.data_ptr(), inv.data_ptr(), T, k, 0, E, st),
+               "mx_moe_align_inv")
+    _lib.count_launch()
+    if x.dtype == torch.bfloat16 and H % 8 == 0 and I % 8 == 0 and not force_any:
+        xs = torch.empty(pairs, H, dtype=x.dtype, device=dev)
+        _lib.check(lib.mx_moe_gather_rows_n(x.data_ptr(), token.data_ptr(), offsets[E:].data_ptr(), xs.data_ptr(), pairs, H, st),
+                   "mx_moe_gather_rows_n")
+        _lib.count_launch()
+        a = grouped_linear(xs, w_gate_up, offsets, I, None, "clipped_swiglu", alpha, limit)
+        return MoeRows(grouped_linear(a, w_down, offsets, H), x, ids, inv, wts, E)
+
+    def grouped(rows, w, row_map):
+        out = torch.empty(pairs, w.shape[1], dtype=x.dtype, device=dev)
+        _lib.check(lib.mx_grouped_gemm_any(rows.data_ptr(), w.data_ptr(), out.data_ptr(), offsets.data_ptr(), _lib.ptr(row_map), E, T,
+                                           w.shape[1], w.shape[2], rows.stride(0), 1 if x.dtype == torch.float32 else 0, st),
+                   "mx_grouped_gemm_any")
+        _lib.count_launch()
+        return out
+    z = grouped(x, w_gate_up, token)
+    a = torch.empty(pairs, I, dtype=x.dtype, device=dev)
+    _lib.check(lib.mx_glu_rows(z.data_ptr(), z.stride(0), a.data_ptr(), pairs, I, ref.EPI_CLIPPED_SWIGLU, float(alpha), float(limit),
+                               1 if x.dtype == torch.float32 else 0, st), "mx_glu_rows")
+    _lib.count_launch()
+    return MoeRows(grouped(a, w_down, None), x, ids, inv, wts, E)

@@ -10,6 +10,7 @@ from __future__ import annotations
 
 import ctypes
 import math
+from dataclasses import dataclass
 
 import torch
 
@@ -18,15 +19,15 @@ from .reference import _gather_kv
 
 _vp, _i, _f, _ll = ctypes.c_void_p, ctypes.c_int, ctypes.c_float, ctypes.c_longlong
 _SIG = {
-    "mx_stream_norm": [_vp] * 7 + [_i, _i, _f, _f, _i, _vp],
-    "mx_embed_stream": [_vp] * 6 + [_i, _i, _i, _f, _f, _f, _i, _vp],
+    "mx_stream_norm": [_vp] * 7 + [_i, _i, _f, _f, _i, _vp, _vp],
+    "mx_embed_stream": [_vp] * 7 + [_i, _i, _i, _f, _f, _f, _i, _vp],
     "mx_polynorm": [_vp, _vp, _vp, _i, _i, _f, _i, _vp],
     "mx_softcap_rows": [_vp, _ll, _f, _vp],
     "mx_rope_norm_append": [_vp, _ll, _vp, _vp, _vp, _f] + [_vp] * 4 + [_i] * 9 + [_f, _i, _vp],
     "mx_qk_norm_append": [_vp, _ll, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _f, _i, _vp],
-    "mx_paged_attention_any": [_vp, _ll] + [_vp] * 9 + [_ll, _vp] + [_i] * 12 + [_f, _f, _i, _vp],
-    "mx_paged_decode_ext": [_vp, _ll] + [_vp] * 8 + [_ll, _vp, _vp] + [_i] * 9 + [_f, _f, _i, _vp],
-    "mx_paged_prefill_ext": [_vp, _ll, _vp, _vp, _ll] + [_vp] * 7 + [_ll, _vp] + [_i] * 11 + [_f, _f, _vp, _vp],
+    "mx_paged_attention_any": [_vp, _ll] + [_vp] * 9 + [_ll, _vp] + [_i] * 12 + [_f, _f, _i, _f, _f, _f, _i, _vp],
+    "mx_paged_decode_ext": [_vp, _ll] + [_vp] * 8 + [_ll, _vp, _vp] + [_i] * 9 + [_f, _f, _i, _f, _f, _f, _i, _vp],
+    "mx_paged_prefill_ext": [_vp, _ll, _vp, _vp, _ll] + [_vp] * 7 + [_ll, _vp] + [_i] * 11 + [_f, _f, _i, _f, _f, _f, _vp, _vp],
     "mx_delta_rule": [_vp, _ll] + [_vp] * 11 + [_i] * 6 + [_f, _f, _f, _i, _i, _vp],
 }
 NOT_COVERED = -10        # a tensor-core kernel refuses the geometry: the shape-agnostic one takes it
@@ -51,26 +52,55 @@ def _fp32(t: torch.Tensor) -> int:
     return 1 if t.dtype == torch.float32 else 0
 
 
+def visible(max_len: int, span: int) -> int:
+    """Tokens a query sees at most: a window or chunk of ``span`` (0: all) of ``max_len``."""
+    return min(max_len, span) if span > 0 else max_len
+
+
 def _rms(x: torch.Tensor, eps: float) -> torch.Tensor:
     return x * torch.rsqrt(x.pow(2).mean(-1, keepdim=True) + eps)
 
 
 # ----------------------------------------------------------------------------- residual stream
-def embed_stream(ids, table, scale: float, pre_w, eps: float, w_bias: float, own_w=None):
-    """``h = scale * table[ids]`` (fp32 stream; with ``own_w`` the embedding's own norm: ``rmsnorm(.) * (w_bias + own_w)``)
-    and ``x = rmsnorm(h) * (w_bias + pre_w)`` in the table's type; without ``pre_w``, x is h itself."""
+class _StreamExtras(ctypes.Structure):
+    """Mirror of ``MxStreamExtras`` (csrc/api.h): what a step of the stream adds besides a branch."""
+
+    _fields_ = [("moe_y", _vp), ("moe_shared", _vp), ("moe_x", _vp), ("moe_ids", _vp), ("moe_inv", _vp), ("moe_w", _vp),
+                ("moe_k", _i), ("moe_experts", _i), ("vec", _vp), ("ids", _vp), ("table", _vp), ("vocab", _i), ("emb_scale", _f)]
+
+
+@dataclass
+class Entry:
+    """What is added to the stream ahead of a run of layers: a vector and, with ``ids``, the tokens' embedding again."""
+
+    vec: torch.Tensor                     # fp32 [dim]
+    ids: torch.Tensor | None = None
+    table: torch.Tensor | None = None
+    scale: float = 1.0
+
+    def add_to(self, h) -> None:
+        if self.ids is not None:
+            ok = (self.ids >= 0) & (self.ids < self.table.shape[0])
+            h += self.table[self.ids.clamp(0, self.table.shape[0] - 1).long()].float() * self.scale * ok[:, None]
+        h += self.vec
+
+
+def embed_stream(ids, table, scale: float, pre_w, eps: float, w_bias: float, own_w=None, vec=None):
+    """``h = scale * table[ids]`` (fp32 stream; with ``own_w`` the embedding's own norm: ``rmsnorm(.) * (w_bias + own_w)``;
+    plus the fp32 vector ``vec``) and ``x = rmsnorm(h) * (w_bias + pre_w)`` in the table's type; without ``pre_w``, x is h itself."""
     n, dim = ids.shape[0], table.shape[1]
     if not table.is_cuda:
         ok = (ids >= 0) & (ids < table.shape[0])
         h = table[ids.clamp(0, table.shape[0] - 1).long()].float() * scale * ok[:, None]
         h = h if own_w is None else _rms(h, eps) * (w_bias + own_w)
+        h = h if vec is None else h + vec
         return h, _stream_as(h, table.dtype) if pre_w is None else (_rms(h, eps) * (w_bias + pre_w)).to(table.dtype)
     h = torch.empty(n, dim, dtype=torch.float32, device=table.device)
     alias = pre_w is None and table.dtype == torch.float32       # (the branch has read the stream before it is added to it)
     x = None if alias else torch.empty(n, dim, dtype=table.dtype, device=table.device)
     if n:
-        _call("mx_embed_stream", ids.data_ptr(), table.data_ptr(), h.data_ptr(), _lib.ptr(own_w), _lib.ptr(pre_w), _lib.ptr(x),
-              n, dim, table.shape[0], float(scale), float(eps), float(w_bias), _fp32(table), _lib.stream())
+        _call("mx_embed_stream", ids.data_ptr(), table.data_ptr(), h.data_ptr(), _lib.ptr(own_w), _lib.ptr(vec), _lib.ptr(pre_w),
+              _lib.ptr(x), n, dim, table.shape[0], float(scale), float(eps), float(w_bias), _fp32(table), _lib.stream())
     return h, h if alias else x
 
 
@@ -78,16 +108,23 @@ def _stream_as(h, dtype):
     return h if h.dtype == dtype else h.to(dtype)
 
 
-def stream_norm(h, y, post_w, layer_scale, pre_w, eps: float, w_bias: float, dtype=None, rows=None, plain: bool = False):
+def stream_norm(h, y, post_w, layer_scale, pre_w, eps: float, w_bias: float, dtype=None, rows=None, plain: bool = False,
+                moe=None, entry: Entry | None = None):
     """One step of the stream between two sub-layers, in place on ``h`` (fp32): with a branch ``y``,
-    ``h += rmsnorm(y) * (w_bias + post_w) * layer_scale`` (layer_scale optional); with ``pre_w``, returns
-    ``rmsnorm(h) * (w_bias + pre_w)`` as ``dtype`` (default: y's type); with ``plain`` (and no ``pre_w``) the
-    stream itself as ``dtype``. ``rows`` (int32, no branch) selects the rows of h to normalise."""
+    ``h += rmsnorm(y) * (w_bias + post_w) * layer_scale`` (without ``post_w``, y as it is; layer_scale optional); with ``moe``
+    (:class:`~mlxcel_b200.ops.moe.MoeRows`) the weighted sum of a token's experts; then what ``entry`` adds. With ``pre_w``,
+    returns ``rmsnorm(h) * (w_bias + pre_w)`` as ``dtype`` (default: y's type); with ``plain`` (and no ``pre_w``) the
+    stream itself as ``dtype``. ``rows`` (int32, nothing to add) selects the rows of h to normalise."""
     dtype = dtype or y.dtype
+    assert rows is None or (y is None and moe is None and entry is None)
     if not h.is_cuda:
         if y is not None:
-            b = _rms(y.float(), eps) * (w_bias + post_w)
+            b = y.float() if post_w is None else _rms(y.float(), eps) * (w_bias + post_w)
             h += b if layer_scale is None else b * layer_scale
+        if moe is not None:
+            h += moe.summed()
+        if entry is not None:
+            entry.add_to(h)
         if pre_w is None:
             return _stream_as(h, dtype) if plain else None
         return (_rms(h if rows is None else h[rows.long()], eps) * (w_bias + pre_w)).to(dtype)
@@ -97,10 +134,22 @@ def stream_norm(h, y, post_w, layer_scale, pre_w, eps: float, w_bias: float, dty
     x = torch.empty(n, dim, dtype=dtype, device=h.device) if pre_w is not None or (plain and not alias) else None
     assert h.is_contiguous() and (y is None or (y.is_contiguous() and y.dtype == dtype))
     assert rows is None or rows.dtype == torch.int32
+    ex = None
+    if moe is not None or entry is not None:
+        ex = _StreamExtras()
+        if moe is not None:
+            assert moe.x.dtype == dtype and moe.x.is_contiguous() and moe.y.dtype == dtype and moe.x.shape == h.shape
+            ex.moe_y, ex.moe_x, ex.moe_ids, ex.moe_inv, ex.moe_w = (t.data_ptr() for t in (moe.y, moe.x, moe.ids, moe.inv, moe.wts))
+            ex.moe_shared, ex.moe_k, ex.moe_experts = _lib.ptr(moe.shared), moe.ids.shape[1], moe.experts
+        if entry is not None:
+            ex.vec = entry.vec.data_ptr()
+            if entry.ids is not None:
+                assert entry.table.dtype == dtype
+                ex.ids, ex.table, ex.vocab, ex.emb_scale = entry.ids.data_ptr(), entry.table.data_ptr(), entry.table.shape[0], entry.scale
     if n:
         fp32 = 1 if dtype == torch.float32 else 0
         _call("mx_stream_norm", _lib.ptr(y), h.data_ptr(), _lib.ptr(rows), _lib.ptr(post_w), _lib.ptr(layer_scale),
-              _lib.ptr(pre_w), _lib.ptr(x), n, dim, float(eps), float(w_bias), fp32, _lib.stream())
+              _lib.ptr(pre_w), _lib.ptr(x), n, dim, float(eps), float(w_bias), fp32, _lib.ref_or_null(ex), _lib.stream())
     return h if alias else x
 
 
@@ -128,12 +177,16 @@ def softcap_(x, cap: float):
 
 
 # ----------------------------------------------------------------------------- attention
-def rotate_half(x, positions, inv_freq, mscale: float):
+def rotate_half(x, positions, inv_freq, mscale: float, adjacent: bool = False):
     """x [T, H, D] fp32: dimension i turned with i + R / 2 by ``positions * inv_freq[i]`` (R = 2 len(inv_freq)), both
-    times ``mscale``; dimensions from R on pass."""
+    times ``mscale``; dimensions from R on pass. ``adjacent``: dimension 2 i turned with 2 i + 1 instead."""
     half = inv_freq.shape[0]
     a = (positions.float()[:, None] * inv_freq)[:, None]
     c, s = a.cos() * mscale, a.sin() * mscale
+    if adjacent:
+        u, v = x[..., 0:2 * half:2], x[..., 1:2 * half:2]
+        turned = torch.stack([u * c - v * s, v * c + u * s], -1).flatten(-2)
+        return torch.cat([turned, x[..., 2 * half:]], -1)
     u, v = x[..., :half], x[..., half:2 * half]
     return torch.cat([u * c - v * s, v * c + u * s, x[..., 2 * half:]], -1)
 
@@ -192,7 +245,16 @@ def qk_norm_append(qkv, slots, kv, *, Hq: int, Hkv: int, Dk: int, Dv: int, q_nor
 
 
 def paged_attention_ref(q, kv, tables, lens, cu, *, Hq, Hkv, Dk, Dv, scale, window=0, sinks=None, dist_bias=None, gate=None,
-                        softcap=0.0, chunk=0):
+                        softcap=0.0, chunk=0, diff=None):
+    if diff is not None:
+        # the maps as two attentions whose queries are zero in the other map's columns
+        factor, gain, eps = diff
+        q3, a, common = q.reshape(-1, Hq, 2, Dk // 2), [], dict(Hq=Hq, Hkv=Hkv, Dk=Dk, Dv=Dv, scale=scale, window=window, chunk=chunk)
+        for i in (0, 1):
+            one = torch.zeros_like(q3)
+            one[:, :, i] = q3[:, :, i]
+            a.append(paged_attention_ref(one.reshape(q.shape[0], -1).float(), kv, tables, lens, cu, **common).view(-1, Hq, Dv))
+        return (_rms(a[0] - factor * a[1], eps) * gain).reshape(-1, Hq * Dv).to(q.dtype)
     T, G = q.shape[0], Hq // Hkv
     out = torch.zeros(T, Hq * Dv, dtype=q.dtype, device=q.device)
     cu_l, lens_l = cu.tolist(), lens.tolist()
@@ -225,14 +287,16 @@ def paged_attention_ref(q, kv, tables, lens, cu, *, Hq, Hkv, Dk, Dv, scale, wind
 
 def paged_attention(q, kv, tables, lens, cu, out, *, Hq: int, Hkv: int, Dk: int, Dv: int, scale: float, max_q_len: int,
                     max_len: int = 0, window: int = 0, sinks=None, dist_bias=None, gate=None, softcap: float = 0.0, chunk: int = 0,
-                    force_any: bool = False) -> None:
+                    diff: tuple | None = None, force_any: bool = False) -> None:
     """Causal paged attention of the query rows of every sequence (the last ``cu[s+1] - cu[s]`` of its ``lens[s]``
     tokens) into ``out`` [rows, Hq * Dv]. ``cu=None`` says one row per sequence (decode).
 
     scores: ``q.k * scale``, with ``softcap`` > 0 ``softcap tanh(. / softcap)``, then ``- r1 ln(1 + r2 distance)`` with
     ``dist_bias = (r1, r2)`` per query head; ``chunk`` > 0: a token sees only keys of its own run of ``chunk`` positions
     (counted from the sequence's start); ``sinks`` adds ``exp(sink)`` to the denominator; ``gate`` ([rows, Hq * Dv], may be a column slice) multiplies the result by
-    its sigmoid. bf16 pools with row widths that are multiples of 8 up to 128 take the tensor-core kernels
+    its sigmoid; ``diff = (factor, gain, eps)``: differential heads, the Dk columns of a query and key head are two maps of
+    Dk / 2 (scores and softmax of their own, the same values) and the result is ``a1 - factor a2`` over its root mean square,
+    times ``gain``. bf16 pools with row widths that are multiples of 8 up to 128 take the tensor-core kernels
     (flash decoding with split KV; tcgen05 prefill); the rest the SIMT one."""
     rows = q.shape[0]
     if rows == 0:
@@ -240,8 +304,11 @@ def paged_attention(q, kv, tables, lens, cu, out, *, Hq: int, Hkv: int, Dk: int,
     if not q.is_cuda:
         c = torch.arange(rows + 1) if cu is None else cu
         out.copy_(paged_attention_ref(q, kv, tables, lens, c, Hq=Hq, Hkv=Hkv, Dk=Dk, Dv=Dv, scale=scale, window=window,
-                                      sinks=sinks, dist_bias=dist_bias, gate=gate, softcap=softcap, chunk=chunk))
+                                      sinks=sinks, dist_bias=dist_bias, gate=gate, softcap=softcap, chunk=chunk, diff=diff))
         return
+    assert diff is None or (Dk % 2 == 0 and sinks is None and dist_bias is None and gate is None), "differential heads: plain scores"
+    maps, (lam, gain, eps) = (1, (0.0, 1.0, 0.0)) if diff is None else (2, diff)
+    dargs = (maps, float(lam), float(gain), float(eps))
     r1, r2 = dist_bias if dist_bias is not None else (None, None)
     assert kv.k.dtype == q.dtype and q.stride(1) == 1 and out.is_contiguous() and out.dtype == q.dtype
     assert gate is None or (gate.stride(1) == 1 and gate.dtype == q.dtype)
@@ -251,15 +318,15 @@ def paged_attention(q, kv, tables, lens, cu, out, *, Hq: int, Hkv: int, Dk: int,
     if q.dtype == torch.bfloat16 and not force_any:
         from . import _decode_scratch, decode_splits
         if cu is None:
-            splits = decode_splits(rows, Hkv, max_len or tables.shape[1] * kv.block_size)
-            scratch = _decode_scratch(q.device, int(_lib.load().mx_paged_decode_scratch_floats(rows, Hq, Dv, splits)))
+            splits = decode_splits(rows, Hkv, visible(max_len or tables.shape[1] * kv.block_size, window or chunk))
+            scratch = _decode_scratch(q.device, int(_lib.load().mx_paged_decode_scratch_floats(rows, maps * Hq, Dv, splits)))
             rc = _fn("mx_paged_decode_ext")(*head, tables.data_ptr(), lens.data_ptr(), *tail, scratch.data_ptr(), rows, Hq,
                                             Hkv, Dk, Dv, kv.block_size, tables.shape[1], window, chunk, float(scale),
-                                            float(softcap), splits, _lib.stream())
+                                            float(softcap), *dargs, splits, _lib.stream())
         else:
             rc = _fn("mx_paged_prefill_ext")(*head, kv.k.shape[0], tables.data_ptr(), cu.data_ptr(), lens.data_ptr(), *tail,
                                              lens.shape[0], rows, max_q_len, Hq, Hkv, Dk, Dv, kv.block_size, tables.shape[1],
-                                             window, chunk, float(scale), float(softcap), _lib.workspace(q.device).data_ptr(),
+                                             window, chunk, float(scale), float(softcap), *dargs, _lib.workspace(q.device).data_ptr(),
                                              _lib.stream())
         if rc != NOT_COVERED:
             _lib.count_launch()
@@ -268,7 +335,7 @@ def paged_attention(q, kv, tables, lens, cu, out, *, Hq: int, Hkv: int, Dk: int,
     if cu is None:
         cu = torch.arange(rows + 1, dtype=torch.int32, device=q.device)
     _call("mx_paged_attention_any", *head, tables.data_ptr(), cu.data_ptr(), lens.data_ptr(), *tail, lens.shape[0], rows, Hq,
-          Hkv, Dk, Dv, Dk, Dv, kv.block_size, tables.shape[1], window, chunk, float(scale), float(softcap), _fp32(q), _lib.stream())
+          Hkv, Dk, Dv, Dk, Dv, kv.block_size, tables.shape[1], window, chunk, float(scale), float(softcap), *dargs, _fp32(q), _lib.stream())
 
 
 # ----------------------------------------------------------------------------- generalized delta rule

@@ -18,7 +18,7 @@ import os
 import sys
 
 LIVE_REQUESTS = 4
-FP32_MODELS = ("govopel", "pamasun")
+FP32_MODELS = ("govopel", "pamasun", "vavadra")
 
 
 def build_engine(model_dir: str, dtype: str, max_tokens: int, device: str):

@@ -24,6 +24,21 @@ def _recurrent_block(cfg: ModelConfig, kind: str) -> tuple[int, int]:
         # (a repeated layer's weights count once, its state for every run)
         spec = x["layer_specs"][kind]
         m, ff = spec["mixer"], (spec["mlp"] or {}).get("ff", 0)
+        if cfg.model_type == "vavadra":
+            st, mlp, d, v, n = 0, spec["mlp"], m["dim"], m["vdim"], m["heads"]
+            if spec["type"] == "attention":
+                par = (h + 1) * (2 * d * (n + m["kv_heads"]) + v * m["kv_heads"]) + h * n * v + 4 * d
+            elif spec["type"] == "latent_attention":
+                c, r = m["kv_rank"], m["rot_dim"]
+                par = h * (n * (d + r + v) + c + r) + c * (1 + n * (d + v)) + n
+            else:
+                conv = 2 * m["kv_heads"] * d + n * v
+                par = h * (conv + 2 * n * v + 2 * n) + conv * m["conv"] + 2 * n + v
+                st = 4 * ((m["conv"] - 1) * conv + n * d * v)
+            if mlp:
+                e = mlp["router"]["experts"] + mlp["router"]["identity"]
+                par += e * (h + 1) + 3 * h * (mlp["router"]["experts"] * mlp["expert"]["ff"] + (mlp["shared"] or {"ff": 0})["ff"]) + h
+            return (par + h) // x["layer_runs"].count(kind), st
         if cfg.model_type == "govopel":
             if spec["type"] == "attention":                       # values are the keys
                 par = h * m["dim"] * (2 * m["heads"] + m["kv_heads"])

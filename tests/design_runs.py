@@ -7,8 +7,9 @@ from mlxcel_b200.engine import EngineConfig
 from mlxcel_b200.llm import LLM
 from mlxcel_b200.models.govopel import build_govopel_weights
 from mlxcel_b200.models.pamasun import build_pamasun_weights
+from mlxcel_b200.models.vavadra import build_vavadra_weights
 
-BUILDERS = {"pamasun": build_pamasun_weights, "govopel": build_govopel_weights}
+BUILDERS = {"pamasun": build_pamasun_weights, "govopel": build_govopel_weights, "vavadra": build_vavadra_weights}
 
 
 def llm_for(raw, tensors, device, dtype, **ecfg):
