@@ -116,3 +116,37 @@ def oracle_greedy(O, raw, tensors, prompt, n):
     for _ in range(n):
         toks.append(int(O.forward(raw, tensors, toks)[-1].argmax()))
     return toks[len(prompt):]
+
+
+# ----------------------------------------------------------------------------- kernels on paged pools
+def assert_close(got, want, dtype, f32=2e-5, bf16=1.5e-2):
+    """Error of every element relative to its size plus the tensor's root mean square."""
+    tol = f32 if dtype == torch.float32 else bf16
+    got, want = got.double().cpu(), want.double()
+    err = (got - want).abs() / (want.abs() + want.pow(2).mean().sqrt())
+    assert torch.isfinite(got).all() and err.max() < tol, float(err.max())
+
+
+def paged_tables(lens, bs, seed=0):
+    """Block tables of sequences of these lengths over a shuffled pool; (tables, blocks in the pool)."""
+    need = [-(-n // bs) for n in lens]
+    perm = torch.randperm(sum(need) + 3, generator=torch.Generator().manual_seed(seed)).tolist()
+    tab, at = torch.zeros(len(lens), max(max(need), 1), dtype=torch.int32), 0
+    for s, k in enumerate(need):
+        tab[s, :k] = torch.tensor(perm[at:at + k], dtype=torch.int32)
+        at += k
+    return tab, len(perm)
+
+
+def fill_pages(pool, tab, s, rows):
+    """rows [n, heads, width] as the first n entries of sequence s."""
+    bs = pool.shape[2]
+    for i in range(rows.shape[0]):
+        pool[int(tab[s, i // bs]), :, i % bs] = rows[i].to(pool.dtype)
+
+
+def bounds(sizes):
+    out = [0]
+    for n in sizes:
+        out.append(out[-1] + n)
+    return out
