@@ -39,7 +39,8 @@ struct GatedParams {
 };
 
 __device__ __forceinline__ int gd_channels(const GatedParams& p) { return 2 * p.G * p.D + p.H * p.V; }
-__device__ __forceinline__ float silu_f(float x) { return x * sigmoid_f(x); }
+// (within two units in the last place of the exponential)
+__device__ __forceinline__ float silu_f(float x) { return __fdividef(x, 1.f + __expf(fminf(-x, 80.f))); }
 
 // Decay of a head. Slow heads sit just below one and are multiplied into the state at every token: 1 + expm1 is within half
 // a unit in the last place there.
@@ -86,7 +87,7 @@ __device__ __forceinline__ float conv_input(const GatedParams& p, int c, int t, 
 constexpr int kGsThreads = 256;
 
 template <typename T, int RPW>
-__global__ void __launch_bounds__(kGsThreads) gated_step_kernel(const GatedParams p) {
+__global__ void __launch_bounds__(kGsThreads, 2) gated_step_kernel(const GatedParams p) {
   extern __shared__ __align__(16) float gs_v[];             // [heads of the group][V]
   __shared__ float red[3 * 33];
   __shared__ float k_s[128], q_s[128];
@@ -230,6 +231,7 @@ __device__ __forceinline__ int piece_of(const GatedParams& p, int t) {   // piec
 }
 
 constexpr int kGpTok = 16;         // tokens a warp takes
+constexpr int kGpBatch = 4;        // of which it requests so many at a time
 constexpr int kGpThreads = 128;
 
 // Silu of the convolution of four neighbouring channels over a run of tokens: the taps' inputs slide through registers.
@@ -254,14 +256,13 @@ struct ConvRun {
 #pragma unroll
       for (int e = 0; e < 4; ++e) x[i][e] = conv_input<T>(p, c + e, t - TAPS + i, t0, slot, fresh);
   }
-  __device__ void next(int t, float (&y)[4]) {
+  __device__ void input(int t, float (&in)[4]) const { load_v<4>(static_cast<const T*>(p.proj) + static_cast<size_t>(t) * p.ld + c, in); }
+  __device__ void next(int t, const float (&in)[4], float (&y)[4]) {
     if (t >= t1) {
       int n = j + 1;
       while (p.cu[n + 1] <= t) ++n;
       enter(n, t);
     }
-    float in[4];
-    load_v<4>(static_cast<const T*>(p.proj) + static_cast<size_t>(t) * p.ld + c, in);
 #pragma unroll
     for (int e = 0; e < 4; ++e) {
       float s = 0.f;
@@ -301,32 +302,48 @@ gated_prep_kernel(const GatedParams p, float* __restrict__ scratch, int row0, in
     const bool in = c < D;
     ConvRun<T, TAPS> q(p, unit * D + (in ? c : 0), row0 + n0), k(p, (p.G + unit) * D + (in ? c : 0), row0 + n0);
     const float dq = rsqrtf(static_cast<float>(D));
-    for (int n = n0; n < n1; ++n) {
-      float a[4], b[4];
-      q.next(row0 + n, a);
-      k.next(row0 + n, b);
-      float aa = 0.f, bb = 0.f, ab = 0.f;
-      if (in) {
+    for (int m0 = n0; m0 < n1; m0 += kGpBatch) {
+      float qi[kGpBatch][4], ki[kGpBatch][4];
 #pragma unroll
-        for (int e = 0; e < 4; ++e) aa = fmaf(a[e], a[e], aa), bb = fmaf(b[e], b[e], bb), ab = fmaf(a[e], b[e], ab);
-      }
-      aa = warp_sum(aa), bb = warp_sum(bb), ab = warp_sum(ab);
-      const float iq = dq / sqrtf(aa + p.unit_eps), ik = 1.f / sqrtf(bb + p.unit_eps);
-      if (in) {
+      for (int i = 0; i < kGpBatch; ++i) q.input(row0 + min(m0 + i, n1 - 1), qi[i]), k.input(row0 + min(m0 + i, n1 - 1), ki[i]);
 #pragma unroll
-        for (int e = 0; e < 4; ++e) a[e] *= iq, b[e] *= ik;
-        store_v<4>(sc.q + (static_cast<size_t>(n) * p.G + unit) * D + c, a);
-        store_v<4>(sc.k + (static_cast<size_t>(n) * p.G + unit) * D + c, b);
+      for (int i = 0; i < kGpBatch; ++i) {
+        const int n = m0 + i;
+        if (n >= n1) break;
+        float a[4], b[4];
+        q.next(row0 + n, qi[i], a);
+        k.next(row0 + n, ki[i], b);
+        float aa = 0.f, bb = 0.f, ab = 0.f;
+        if (in) {
+#pragma unroll
+          for (int e = 0; e < 4; ++e) aa = fmaf(a[e], a[e], aa), bb = fmaf(b[e], b[e], bb), ab = fmaf(a[e], b[e], ab);
+        }
+        aa = warp_sum(aa), bb = warp_sum(bb), ab = warp_sum(ab);
+        const float iq = dq / sqrtf(aa + p.unit_eps), ik = 1.f / sqrtf(bb + p.unit_eps);
+        if (in) {
+#pragma unroll
+          for (int e = 0; e < 4; ++e) a[e] *= iq, b[e] *= ik;
+          store_v<4>(sc.q + (static_cast<size_t>(n) * p.G + unit) * D + c, a);
+          store_v<4>(sc.k + (static_cast<size_t>(n) * p.G + unit) * D + c, b);
+        }
+        write_rates(p, sc, row0 + n, n, unit, ab * iq * ik, lane);
       }
-      write_rates(p, sc, row0 + n, n, unit, ab * iq * ik, lane);
     }
   } else if (c < V) {
     const int h = unit - p.G;
     ConvRun<T, TAPS> v(p, 2 * p.G * D + h * V + c, row0 + n0);
-    for (int n = n0; n < n1; ++n) {
-      float a[4];
-      v.next(row0 + n, a);
-      store_v<4>(sc.v + (static_cast<size_t>(n) * p.H + h) * V + c, a);
+    for (int m0 = n0; m0 < n1; m0 += kGpBatch) {
+      float vi[kGpBatch][4];
+#pragma unroll
+      for (int i = 0; i < kGpBatch; ++i) v.input(row0 + min(m0 + i, n1 - 1), vi[i]);
+#pragma unroll
+      for (int i = 0; i < kGpBatch; ++i) {
+        const int n = m0 + i;
+        if (n >= n1) break;
+        float a[4];
+        v.next(row0 + n, vi[i], a);
+        store_v<4>(sc.v + (static_cast<size_t>(n) * p.H + h) * V + c, a);
+      }
     }
   }
 }
@@ -388,127 +405,129 @@ __device__ __forceinline__ void gd_copy16(float* smem, const float* g) {
   asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(smem_u32(smem)), "l"(g) : "memory");
 }
 
-// Half a warp (16 lanes) shares 4 neighbouring columns of one head's state; a lane keeps RPT key channels of each (groups of 4:
-// 4 l .. 4 l + 3, then 64 further on; RPT = 2: 2 l, 2 l + 1) as packed pairs of channels. A CTA of 4 warps covers 32 columns;
-// the vectors of kGcTok tokens are double-buffered. Per token: two partial dots per column, one halving exchange over the 16
-// lanes (lane bit 3 ends with k.S or q.S, bits 2 and 1 with the column), the update. D and V multiples of 4.
-constexpr int kGcCols = 4, kGcThreads = 128, kGcCta = kGcThreads / 16 * kGcCols, kGcTok = 8;
+// Eight lanes share COLS neighbouring columns of one head's state; a lane keeps RPT key channels of each (groups of 4: 4 l ..
+// 4 l + 3, then 32 further on) as packed pairs of channels. A CTA of 2 warps covers 8 COLS columns; the vectors of kGcTok
+// tokens are double-buffered. Per token: two partial dots per column, a halving exchange over the eight lanes (lane bit 2 ends
+// with k.S or q.S, the lower bits with the column), u by the lane that has k.S, its broadcast, the update. A lane numbers its
+// columns so that the ones it hands on in the exchange always have the same registers: number c stands for column c ^ (the
+// lane's column bits). Four columns a lane need the fewest instructions; with two a lone sequence's tokens follow one
+// another faster. D and V multiples of 4.
+constexpr int kGcThreads = 64, kGcTok = 8;
 
-template <typename T, int RPT>
+template <typename T, int RPT, int COLS>
 __global__ void __launch_bounds__(kGcThreads)
 gated_scan_kernel(const GatedParams p, float* __restrict__ scratch, int row0, int N) {
-  constexpr int DP = 16 * RPT, P2 = RPT / 2;
-  constexpr int STAGE = kGcTok * (2 * DP + kGcCta + 4);
+  constexpr int DP = 8 * RPT, P2 = RPT / 2, CTA = kGcThreads / 8 * COLS;
+  constexpr int STAGE = kGcTok * (2 * DP + CTA + 4);
+  static_assert(COLS == 4 || COLS == 2, "columns of a lane");
   extern __shared__ __align__(16) float gc_smem[];
   pdl_trigger();
   pdl_wait();
-  const int D = p.D, V = p.V, cbs = (V + kGcCta - 1) / kGcCta;
+  const int D = p.D, V = p.V, cbs = (V + CTA - 1) / CTA;
   const int h = blockIdx.x / cbs, cb = blockIdx.x - h * cbs, j = blockIdx.y, grp = h / (p.H / p.G);
   const int t0 = p.cu[j] - row0, t1 = p.cu[j + 1] - row0, slot = p.slots[j];
   if (t1 <= t0) return;
   const GatedScratch sc = gd_scratch(scratch, N, p.H, p.G, D, V);
-  const int lane = threadIdx.x & 31, l16 = lane & 15, c_in = (threadIdx.x >> 4) * kGcCols, col0 = cb * kGcCta + c_in;
-  const int o_col = col0 + ((l16 & 4) >> 1) + ((l16 & 2) >> 1);      // output column of this lane
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, l8 = lane & 7;
   if (slot < 0) {
-    for (int i = threadIdx.x; i < (t1 - t0) * kGcCta; i += kGcThreads) {
-      const int c = cb * kGcCta + i % kGcCta;
-      if (c < V) sc.o[(static_cast<size_t>(t0 + i / kGcCta) * p.H + h) * V + c] = 0.f;
+    for (int i = threadIdx.x; i < (t1 - t0) * CTA; i += kGcThreads) {
+      const int c = cb * CTA + i % CTA;
+      if (c < V) sc.o[(static_cast<size_t>(t0 + i / CTA) * p.H + h) * V + c] = 0.f;
     }
     return;
   }
   const bool fresh = p.reset[j] != 0;
   if (cb == 0) write_tail<T>(p, h, t0 + row0, t1 + row0, slot, fresh);
-  // channel of this lane's row r
-  const auto chan = [&](int r) { return RPT == 2 ? 2 * l16 + r : (r >> 2) * 64 + 4 * l16 + (r & 3); };
+  const int flip = COLS == 4 ? l8 & 3 : (l8 >> 1) & 1;                 // the lane's column bits
+  const int c_in = (threadIdx.x >> 3) * COLS, col0 = cb * CTA + c_in, own = col0 + flip;
+  const bool reads_q = (l8 & 4) != 0, writes = reads_q && (COLS == 4 || (l8 & 1) == 0) && own < V;
+  const auto chan = [&](int r) { return (r >> 2) * 32 + 4 * l8 + (r & 3); };
   float* S = p.memory + (static_cast<size_t>(slot) * p.H + h) * D * V;
-  f32x2 s[P2][kGcCols];
+  f32x2 s[P2][COLS];
 #pragma unroll
   for (int r = 0; r < P2; ++r)
 #pragma unroll
-    for (int c = 0; c < kGcCols; ++c) {
-      const bool ok = chan(2 * r) < D && col0 + c < V && !fresh;       // (D is even: both channels of a pair are in or out)
-      s[r][c] = ok ? pack2(S[static_cast<size_t>(chan(2 * r)) * V + col0 + c], S[static_cast<size_t>(chan(2 * r + 1)) * V + col0 + c]) : 0ull;
+    for (int c = 0; c < COLS; ++c) {
+      const int col = col0 + (c ^ flip);
+      const bool ok = chan(2 * r) < D && col < V && !fresh;            // (D is even: both channels of a pair are in or out)
+      s[r][c] = ok ? pack2(S[static_cast<size_t>(chan(2 * r)) * V + col], S[static_cast<size_t>(chan(2 * r + 1)) * V + col]) : 0ull;
     }
   for (int i = threadIdx.x; i < 2 * STAGE; i += kGcThreads) gc_smem[i] = 0.f;     // channels beyond D stay zero
   __syncthreads();
   const auto load = [&](int c0, int buf) {
     float* st = gc_smem + buf * STAGE;
-    const int nt = min(kGcTok, t1 - c0), d4 = D / 4;
-    for (int i = threadIdx.x; i < nt * d4; i += kGcThreads) {
-      const int t = i / d4, c = (i - t * d4) * 4;
-      const size_t src = (static_cast<size_t>(c0 + t) * p.G + grp) * D + c;
-      gd_copy16(st + t * 2 * DP + c, sc.k + src);
-      gd_copy16(st + t * 2 * DP + DP + c, sc.q + src);
+    const int nt = min(kGcTok, t1 - c0);
+    if (4 * lane < D) {
+      const size_t src = (static_cast<size_t>(c0) * p.G + grp) * D + 4 * lane;
+      for (int t = warp; t < nt; t += kGcThreads / 32) {
+        gd_copy16(st + t * 2 * DP + 4 * lane, sc.k + src + static_cast<size_t>(t) * p.G * D);
+        gd_copy16(st + t * 2 * DP + DP + 4 * lane, sc.q + src + static_cast<size_t>(t) * p.G * D);
+      }
     }
     float* vs = st + kGcTok * 2 * DP;
-    for (int i = threadIdx.x; i < nt * (kGcCta / 4); i += kGcThreads) {
-      const int t = i / (kGcCta / 4), c = (i - t * (kGcCta / 4)) * 4;
-      if (cb * kGcCta + c < V) gd_copy16(vs + t * kGcCta + c, sc.v + (static_cast<size_t>(c0 + t) * p.H + h) * V + cb * kGcCta + c);
+    constexpr int Q = CTA / 4;
+    for (int i = threadIdx.x; i < nt * Q; i += kGcThreads) {
+      const int t = i / Q, c = (i - t * Q) * 4;
+      if (cb * CTA + c < V) gd_copy16(vs + t * CTA + c, sc.v + (static_cast<size_t>(c0 + t) * p.H + h) * V + cb * CTA + c);
     }
-    float* rs = vs + kGcTok * kGcCta;
+    float* rs = vs + kGcTok * CTA;
     if (static_cast<int>(threadIdx.x) < nt) gd_copy16(rs + threadIdx.x * 4, sc.rates + (static_cast<size_t>(c0 + threadIdx.x) * p.H + h) * 4);
-    asm volatile("cp.async.commit_group;" ::: "memory");
   };
   load(t0, 0);
+  asm volatile("cp.async.commit_group;" ::: "memory");
   int buf = 0;
   for (int c0 = t0; c0 < t1; c0 += kGcTok, buf ^= 1) {
     if (c0 + kGcTok < t1) load(c0 + kGcTok, buf ^ 1);
-    else asm volatile("cp.async.commit_group;" ::: "memory");
+    asm volatile("cp.async.commit_group;" ::: "memory");
     asm volatile("cp.async.wait_group 1;" ::: "memory");
     __syncthreads();
-    const float* st = gc_smem + buf * STAGE;
-    const float* vs = st + kGcTok * 2 * DP;
-    const float* rs = vs + kGcTok * kGcCta;
+    const float* st = gc_smem + buf * STAGE + 4 * l8;
+    const float* vs = gc_smem + buf * STAGE + kGcTok * 2 * DP + c_in + flip;
+    const float* rs = gc_smem + buf * STAGE + kGcTok * (2 * DP + CTA);
+    float* o = sc.o + (static_cast<size_t>(c0) * p.H + h) * V + own;
     const int nt = min(kGcTok, t1 - c0);
-    for (int t = 0; t < nt; ++t) {
+    for (int t = 0; t < nt; ++t, st += 2 * DP, vs += CTA, rs += 4, o += static_cast<size_t>(p.H) * V) {
       f32x2 k[P2], q[P2];
-      const auto fetch = [&](const float* src, f32x2(&dst)[P2]) {
-        if constexpr (RPT == 2) {
-          dst[0] = *reinterpret_cast<const f32x2*>(src + 2 * l16);
-        } else {
 #pragma unroll
-          for (int r = 0; r < P2; r += 2) {
-            const ulonglong2 x = *reinterpret_cast<const ulonglong2*>(src + r * 32 + 4 * l16);
-            dst[r] = x.x, dst[r + 1] = x.y;
-          }
-        }
-      };
-      fetch(st + t * 2 * DP, k);
-      fetch(st + t * 2 * DP + DP, q);
-      f32x2 kd[kGcCols], qd[kGcCols];
+      for (int r = 0; r < P2; r += 2) {
+        const ulonglong2 a = *reinterpret_cast<const ulonglong2*>(st + r * 16), b = *reinterpret_cast<const ulonglong2*>(st + DP + r * 16);
+        k[r] = a.x, k[r + 1] = a.y, q[r] = b.x, q[r + 1] = b.y;
+      }
+      const float4 rate = *reinterpret_cast<const float4*>(rs);        // g, beta, q.k
+      const float v = *vs;
+      f32x2 kd[COLS], qd[COLS];
 #pragma unroll
-      for (int c = 0; c < kGcCols; ++c) kd[c] = qd[c] = 0ull;
+      for (int c = 0; c < COLS; ++c) kd[c] = mul2(k[0], s[0][c]), qd[c] = mul2(q[0], s[0][c]);
 #pragma unroll
-      for (int r = 0; r < P2; ++r)
+      for (int r = 1; r < P2; ++r)
 #pragma unroll
-        for (int c = 0; c < kGcCols; ++c) {
+        for (int c = 0; c < COLS; ++c) {
           kd[c] = fma2(k[r], s[r][c], kd[c]);
           qd[c] = fma2(q[r], s[r][c], qd[c]);
         }
-      const bool up8 = (l16 & 8) != 0, up4 = (l16 & 4) != 0, up2 = (l16 & 2) != 0;
-      float x[4];
+      float x[COLS];
 #pragma unroll
-      for (int c = 0; c < 4; ++c) {
+      for (int c = 0; c < COLS; ++c) {
         const float a = sum2(kd[c]), b = sum2(qd[c]);
-        x[c] = (up8 ? b : a) + __shfl_xor_sync(0xffffffffu, up8 ? a : b, 8);
+        x[c] = (reads_q ? b : a) + __shfl_xor_sync(0xffffffffu, reads_q ? a : b, 4);
       }
-      const float y0 = (up4 ? x[2] : x[0]) + __shfl_xor_sync(0xffffffffu, up4 ? x[0] : x[2], 4);
-      const float y1 = (up4 ? x[3] : x[1]) + __shfl_xor_sync(0xffffffffu, up4 ? x[1] : x[3], 4);
-      float y = (up2 ? y1 : y0) + __shfl_xor_sync(0xffffffffu, up2 ? y0 : y1, 2);
-      y += __shfl_xor_sync(0xffffffffu, y, 1);
-      const float4 rate = *reinterpret_cast<const float4*>(rs + 4 * t);           // g, beta, q.k
-      const float4 v4 = *reinterpret_cast<const float4*>(vs + t * kGcCta + c_in);
-      const float v[kGcCols] = {v4.x, v4.y, v4.z, v4.w};
-      float u[kGcCols];
+      float y;
+      if constexpr (COLS == 4) {
+        const float y0 = x[0] + __shfl_xor_sync(0xffffffffu, x[2], 2), y1 = x[1] + __shfl_xor_sync(0xffffffffu, x[3], 2);
+        y = y0 + __shfl_xor_sync(0xffffffffu, y1, 1);
+      } else {
+        y = x[0] + __shfl_xor_sync(0xffffffffu, x[1], 2);
+        y += __shfl_xor_sync(0xffffffffu, y, 1);
+      }
+      y *= rate.x;                                                     // column `own` of the decayed state with k or q
+      const float mine = rate.y * (v - y);                             // (of use where this lane has k.S)
+      float u[COLS];
 #pragma unroll
-      for (int c = 0; c < kGcCols; ++c) u[c] = rate.y * (v[c] - rate.x * __shfl_sync(0xffffffffu, y, (lane & 16) + 2 * c));
-      if (up8 && (l16 & 1) == 0 && o_col < V) {
-        const float uu = up4 ? (up2 ? u[3] : u[2]) : (up2 ? u[1] : u[0]);
-        sc.o[(static_cast<size_t>(c0 + t) * p.H + h) * V + o_col] = fmaf(rate.x, y, rate.z * uu);
-      }
+      for (int c = 0; c < COLS; ++c) u[c] = __shfl_sync(0xffffffffu, mine, (lane & 24) + (COLS == 4 ? c ^ flip : 2 * (c ^ flip)));
+      if (writes) *o = fmaf(rate.z, u[0], y);
       const f32x2 g2 = pack2(rate.x, rate.x);
 #pragma unroll
-      for (int c = 0; c < kGcCols; ++c) {
+      for (int c = 0; c < COLS; ++c) {
         const f32x2 u2 = pack2(u[c], u[c]);
 #pragma unroll
         for (int r = 0; r < P2; ++r) s[r][c] = fma2(k[r], u2, mul2(g2, s[r][c]));
@@ -520,12 +539,13 @@ gated_scan_kernel(const GatedParams p, float* __restrict__ scratch, int row0, in
 #pragma unroll
   for (int r = 0; r < P2; ++r)
 #pragma unroll
-    for (int c = 0; c < kGcCols; ++c) {
-      if (chan(2 * r) >= D || col0 + c >= V) continue;
+    for (int c = 0; c < COLS; ++c) {
+      const int col = col0 + (c ^ flip);
+      if (chan(2 * r) >= D || col >= V) continue;
       float a, b;
       asm("mov.b64 {%0, %1}, %2;" : "=f"(a), "=f"(b) : "l"(s[r][c]));
-      S[static_cast<size_t>(chan(2 * r)) * V + col0 + c] = a;
-      S[static_cast<size_t>(chan(2 * r + 1)) * V + col0 + c] = b;
+      S[static_cast<size_t>(chan(2 * r)) * V + col] = a;
+      S[static_cast<size_t>(chan(2 * r + 1)) * V + col] = b;
     }
 }
 
@@ -576,9 +596,9 @@ gated_post_kernel(const GatedParams p, float* __restrict__ scratch, int row0, in
   pdl_trigger();
   pdl_wait();
   const int lane = threadIdx.x & 31, V = p.V;
-  const long long gw = (static_cast<long long>(blockIdx.x) * blockDim.x + threadIdx.x) >> 5;
-  if (gw >= static_cast<long long>(N) * p.H) return;
-  const int n = static_cast<int>(gw / p.H), h = static_cast<int>(gw - static_cast<long long>(n) * p.H);
+  const unsigned gw = blockIdx.x * (blockDim.x / 32) + (threadIdx.x >> 5);
+  if (gw >= static_cast<unsigned>(N) * p.H) return;
+  const int n = static_cast<int>(gw / p.H), h = static_cast<int>(gw - static_cast<unsigned>(n) * p.H);
   const GatedScratch sc = gd_scratch(scratch, N, p.H, p.G, p.D, V);
   const float* o = sc.o + (static_cast<size_t>(n) * p.H + h) * V;
   const T* z = static_cast<const T*>(p.proj) + static_cast<size_t>(row0 + n) * p.ld + gd_channels(p) + h * V;
@@ -617,12 +637,19 @@ static int launch_gated_step(const GatedParams& p, int pieces, cudaStream_t st) 
   return static_cast<int>(launch_kernel(gated_step_kernel<T, 16>, grid, block, smem, st, p));
 }
 
+template <typename T, int RPT, int COLS>
+static int launch_gated_scan_cols(const GatedParams& p, float* scratch, int pieces, int row0, int N, cudaStream_t st) {
+  constexpr int CTA = kGcThreads / 8 * COLS, smem = 2 * kGcTok * (2 * 8 * RPT + CTA + 4) * 4;
+  static_assert(smem <= 48 * 1024, "fits the default limit");
+  const int cbs = (p.V + CTA - 1) / CTA;
+  return static_cast<int>(launch_kernel(gated_scan_kernel<T, RPT, COLS>, dim3(p.H * cbs, pieces), dim3(kGcThreads), smem, st, p, scratch, row0, N));
+}
+
 template <typename T, int RPT>
 static int launch_gated_scan(const GatedParams& p, float* scratch, int pieces, int row0, int N, cudaStream_t st) {
-  constexpr int smem = 2 * kGcTok * (2 * 16 * RPT + kGcCta + 4) * 4;
-  static_assert(smem <= 48 * 1024, "fits the default limit");
-  const int cbs = (p.V + kGcCta - 1) / kGcCta;
-  return static_cast<int>(launch_kernel(gated_scan_kernel<T, RPT>, dim3(p.H * cbs, pieces), dim3(kGcThreads), smem, st, p, scratch, row0, N));
+  // columns of a lane: two while that leaves every SM no more than one CTA
+  const bool few = static_cast<long long>(pieces) * p.H * ((p.V + 15) / 16) <= 148;
+  return few ? launch_gated_scan_cols<T, RPT, 2>(p, scratch, pieces, row0, N, st) : launch_gated_scan_cols<T, RPT, 4>(p, scratch, pieces, row0, N, st);
 }
 
 static bool gated_step_covered(int H, int G, int D, int V) {
@@ -653,11 +680,12 @@ static int gated_delta_typed(GatedParams p, int pieces, int n_short, int rows, f
   else rc = static_cast<int>(launch_kernel(gated_prep_any_kernel<T>, one, dim3(kGpThreads), 0, st, p, scratch, n_short, N));
   if (rc) return rc;
   if (!fast) rc = static_cast<int>(launch_kernel(gated_scan_any_kernel<T>, dim3(p.H, np), dim3(p.V <= 128 ? 128 : 256), 0, st, p, scratch, n_short, N));
-  else if (p.D <= 32) rc = launch_gated_scan<T, 2>(p, scratch, np, n_short, N, st);
-  else if (p.D <= 64) rc = launch_gated_scan<T, 4>(p, scratch, np, n_short, N, st);
-  else rc = launch_gated_scan<T, 8>(p, scratch, np, n_short, N, st);
+  else if (p.D <= 32) rc = launch_gated_scan<T, 4>(p, scratch, np, n_short, N, st);
+  else if (p.D <= 64) rc = launch_gated_scan<T, 8>(p, scratch, np, n_short, N, st);
+  else rc = launch_gated_scan<T, 16>(p, scratch, np, n_short, N, st);
   if (rc) return rc;
   const long long warps = static_cast<long long>(N) * p.H;
+  if (warps > 0x7fffffffll) return -1;
   return static_cast<int>(launch_kernel(gated_post_kernel<T>, dim3(static_cast<unsigned>((warps + 7) / 8)), dim3(256), 0, st, p, scratch, n_short, N));
 }
 

@@ -6,6 +6,7 @@
 //   polynorm       a N(z) + b N(z^2) + c N(z^3) + e, N = division by the row's root mean square
 //   glu_rows       gated activation of rows gate | up (SwiGLU, tanh-GeGLU, clipped SwiGLU)
 //   softcap_rows   x <- cap tanh(x / cap) in fp32, in place
+//   kv_append      k and v rows as projected into the paged pool
 //   qk_norm_append per-head RMS norm of q and k, k and v rows into the paged pool (key and value heads
 //                  may differ in width; no rotation)
 // A norm weight w acts as (w_bias + w); all norm weights and layer scales are fp32 vectors, all
@@ -392,6 +393,27 @@ qk_norm_append_kernel(T* __restrict__ qkv, long long ld, const int* __restrict__
   }
 }
 
+// Keys and values as projected into the paged pool (no norm): one 16-byte group per thread over tokens and heads.
+template <int BYTES>
+__global__ void __launch_bounds__(256)
+kv_append_kernel(const uint8_t* __restrict__ src, long long ld, const int* __restrict__ slots, uint8_t* __restrict__ k_pool,
+                 uint8_t* __restrict__ v_pool, int n, int Hkv, int kb, int vb, int block_size) {      // ld, kb, vb: bytes
+  pdl_trigger();
+  pdl_wait();
+  const int kg = Hkv * (kb / BYTES), per = kg + Hkv * (vb / BYTES);
+  const unsigned i = blockIdx.x * 256u + threadIdx.x, t = i / per;
+  if (t >= static_cast<unsigned>(n)) return;
+  const int g = static_cast<int>(i - t * per), slot = slots[t];
+  if (slot < 0) return;
+  const bool key = g < kg;
+  const int b = key ? kb : vb, j = key ? g : g - kg, head = j / (b / BYTES), at = (j - head * (b / BYTES)) * BYTES;
+  const int blk = slot / block_size, off = slot - blk * block_size;
+  const uint8_t* s = src + static_cast<size_t>(t) * ld + static_cast<size_t>(g) * BYTES;
+  uint8_t* d = (key ? k_pool : v_pool) + ((static_cast<size_t>(blk) * Hkv + head) * block_size + off) * b + at;
+  if constexpr (BYTES == 16) *reinterpret_cast<uint4*>(d) = *reinterpret_cast<const uint4*>(s);
+  else *reinterpret_cast<uint16_t*>(d) = *reinterpret_cast<const uint16_t*>(s);
+}
+
 // Launch shape of a row kernel: groups of V elements per row -> threads and accesses per thread.
 struct RowShape {
   int threads, vpt;
@@ -515,6 +537,16 @@ extern "C" int mx_qk_norm_append(void* qkv, long long ld, const void* slots, voi
                                  int fp32, void* stream) {
   if (n <= 0) return 0;
   if (Hq <= 0 || Hkv <= 0 || Dk <= 0 || Dv <= 0 || block_size <= 0) return -1;
+  if (qw == nullptr && kw == nullptr) {
+    const int es = fp32 ? 4 : 2, kb = Dk * es, vb = Dv * es;
+    const auto* src = static_cast<const uint8_t*>(qkv) + static_cast<size_t>(Hq) * Dk * es;
+    const bool wide = kb % 16 == 0 && vb % 16 == 0 && ld * es % 16 == 0 && aligned_to(src, 16) && aligned_to(k_pool, 16) && aligned_to(v_pool, 16);
+    const long long groups = static_cast<long long>(n) * Hkv * (kb + vb) / (wide ? 16 : 2);
+    if (groups > 0x7fffffffll) return -1;
+    return static_cast<int>(launch_kernel(wide ? kv_append_kernel<16> : kv_append_kernel<2>, dim3(static_cast<unsigned>((groups + 255) / 256)),
+                                          dim3(256), 0, static_cast<cudaStream_t>(stream), src, ld * es, static_cast<const int*>(slots),
+                                          static_cast<uint8_t*>(k_pool), static_cast<uint8_t*>(v_pool), n, Hkv, kb, vb, block_size));
+  }
   const size_t ab = fp32 ? 16 : 8;
   const bool vec = Dk % 4 == 0 && Dv % 4 == 0 && ld % 4 == 0 && aligned_to(qkv, ab) && aligned_to(k_pool, ab) &&
                    aligned_to(v_pool, ab) && aligned_to(qw, 16) && aligned_to(kw, 16);
