@@ -253,9 +253,10 @@ class ModelWorker:
         reason = seq.finish_reason.value if seq.finish_reason else "stop"
         usage = dict(prompt_tokens=n_prompt, completion_tokens=n_out, total_tokens=n_prompt + n_out,
                      prompt_tokens_details=dict(cached_tokens=seq.num_cached))
-        self._emit(req, GenEvent("done", text=tail, finish_reason=reason, usage=usage, timings=timings))
-        # token stream of the slot's last occupant (what /slots/{id}?action=save writes out)
+        # token stream of the slot's last occupant (what /slots/{id}?action=save writes out), there before the client
+        # can ask for it
         self.recent[seq.seq_id % max(1, self.engine.ecfg.max_batch)] = list(seq.prompt) + list(seq.output)
+        self._emit(req, GenEvent("done", text=tail, finish_reason=reason, usage=usage, timings=timings))
         self.engine.release(seq.seq_id)
 
     # ------------------------------------------------------------------ loop
