@@ -13,7 +13,8 @@ instead of 2 * heads * head_dim), in the K slab with a single head; the V slab i
 (the reference's MLA cache, src/lib/mlxcel-core/src/mla/cache.rs:253).
 
 Models with ``cfg.kv_geometry()`` (attention layers of different head counts, keys and values of
-different widths) get one slab pair per attention run with exactly those sizes.
+different widths) get one slab pair per attention run with exactly those sizes, and with ``cfg.kv_means()`` a second, smaller
+pair for the means of blocks of tokens.
 """
 from __future__ import annotations
 
@@ -21,6 +22,8 @@ import torch
 
 from ..config import ModelConfig
 from ..ops import KVLayer
+
+SLABS = ("k", "v", "k_meta", "v_meta", "k_mean", "v_mean")
 
 
 class KVPool:
@@ -42,10 +45,13 @@ class KVPool:
             if tp_size != 1:
                 raise ValueError("per-layer attention geometry is not sharded across tensor-parallel ranks")
             self.latent = False
-            for h, dk, dv in geo:
-                k = torch.zeros((num_blocks, h, block_size, dk), dtype=dtype, device=device)
-                v = torch.zeros((num_blocks, h, block_size, dv), dtype=dtype, device=device)
-                self.layers.append(KVLayer(k, v, None, None, block_size, kv_bits))
+            for (h, dk, dv), m in zip(geo, cfg.kv_means() or [0] * len(geo)):
+                slab = lambda rows, width: torch.zeros((num_blocks, h, rows, width), dtype=dtype, device=device)    # noqa: E731,B023
+                layer = KVLayer(slab(block_size, dk), slab(block_size, dv), None, None, block_size, kv_bits)
+                if m:
+                    rows = -(-block_size // m)
+                    layer.k_mean, layer.v_mean, layer.mean_of = slab(rows, dk), slab(rows, dv), m
+                self.layers.append(layer)
             return
         self.latent = bool(cfg.extra.get("mla_latent"))
         if self.latent:
@@ -82,8 +88,10 @@ class KVPool:
                         num_layers: int | None = None) -> int:
         Hkv = max(1, cfg.num_key_value_heads // tp_size)
         L = cfg.num_hidden_layers if num_layers is None else num_layers
-        if cfg.kv_geometry() is not None:
-            return cfg.kv_bytes_per_token(kv_bits) * block_size
+        geo = cfg.kv_geometry()
+        if geo is not None:
+            rows = [block_size + (-(-block_size // m) if m else 0) for m in cfg.kv_means() or [0] * len(geo)]
+            return sum(h * (dk + dv) * n for (h, dk, dv), n in zip(geo, rows)) * kv_bits // 8
         if cfg.extra.get("mla_latent"):
             return KVPool.latent_width(cfg) * 2 * block_size * L
         per_tok = Hkv * cfg.head_dim * kv_bits // 8
@@ -98,7 +106,8 @@ class KVPool:
         src = torch.tensor([p[0] for p in pairs], device=self.layers[0].k.device)
         dst = torch.tensor([p[1] for p in pairs], device=self.layers[0].k.device)
         for l in self.layers:
-            for t in (l.k, l.v, l.k_meta, l.v_meta):
+            for n in SLABS:
+                t = getattr(l, n)
                 if t is not None:
                     t[dst] = t[src]
 
@@ -107,8 +116,7 @@ class KVPool:
         idx = torch.tensor(block_ids, device=self.layers[0].k.device)
         out = []
         for l in self.layers:
-            out.append({n: getattr(l, n)[idx].cpu() for n in ("k", "v", "k_meta", "v_meta")
-                        if getattr(l, n) is not None})
+            out.append({n: getattr(l, n)[idx].cpu() for n in SLABS if getattr(l, n) is not None})
         return out
 
     def restore_blocks(self, block_ids: list[int], data: list[dict]) -> None:

@@ -15,6 +15,8 @@ import os
 import sys
 import time
 
+from .models.designs import DESIGNS, design_fn
+
 
 def _add_model_args(p):
     p.add_argument("-m", "--model", required=True, help="checkpoint directory or preset:<name>")
@@ -1094,7 +1096,7 @@ def cmd_inspect(a):
 
 
 _HYBRID = {"nemotron_h", "granitemoehybrid", "jamba", "qwen3_next", "qwen3_5", "qwen3_5_text", "qwen3_5_moe",
-           "qwen3_5_moe_text", "falcon_h1", "lfm2", "lfm2_moe", "recurrent_gemma", "pamasun", "govopel", "vavadra"}
+           "qwen3_5_moe_text", "falcon_h1", "lfm2", "lfm2_moe", "recurrent_gemma", *DESIGNS}
 _STATE_SPACE = {"mamba", "mamba2"}
 _CHECKED_BY_READING = {"internlm3", "minicpm", "mimo", "yi", "kimi_k2", "deepseek"}       # no independent implementation at hand
 _CHECKED_BY_LAYOUT = {"internlm2", "baichuan", "exaone", "telechat3"}                                 # round trip against the Llama form
@@ -1116,7 +1118,7 @@ def arch_catalog() -> dict:
             how = f"transformers logits (as {name}_text)"
         if name == "deepseek_v32":
             how = "transformers logits (as glm_moe_dsa)"
-        if name in ("pamasun", "govopel", "vavadra"):
+        if name in DESIGNS:
             how = "a plain PyTorch statement of the model (no library has it)"
         if name == "dbrx":
             how = "a plain PyTorch statement of the model (the transformers implementation is not usable)"
@@ -1166,19 +1168,9 @@ def cmd_random_init(a):
         save_hybrid_checkpoint(a.out, hybrid_config_dict(cfg), random_hybrid_weights(cfg, seed=a.seed), cfg)
         print("wrote", a.out)
         return
-    if cfg.model_type == "pamasun":
-        from .models.pamasun import random_pamasun_tensors, save_pamasun_checkpoint
-        save_pamasun_checkpoint(a.out, cfg, random_pamasun_tensors(cfg, seed=a.seed))
-        print("wrote", a.out)
-        return
-    if cfg.model_type == "govopel":
-        from .models.govopel import random_govopel_tensors, save_govopel_checkpoint
-        save_govopel_checkpoint(a.out, cfg, random_govopel_tensors(cfg, seed=a.seed))
-        print("wrote", a.out)
-        return
-    if cfg.model_type == "vavadra":
-        from .models.vavadra import random_vavadra_tensors, save_vavadra_checkpoint
-        save_vavadra_checkpoint(a.out, cfg, random_vavadra_tensors(cfg, seed=a.seed))
+    if cfg.model_type in DESIGNS:
+        tensors = design_fn(cfg.model_type, "random_{}_tensors")(cfg, seed=a.seed)
+        design_fn(cfg.model_type, "save_{}_checkpoint")(a.out, cfg, tensors)
         print("wrote", a.out)
         return
     w = random_weights(cfg, seed=a.seed, dtype=torch.bfloat16)

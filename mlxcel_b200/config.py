@@ -146,10 +146,16 @@ class ModelConfig:
         layers differ or whose keys and values have different widths; None = uniform."""
         return self.extra.get("kv_geometry")
 
+    def kv_means(self) -> list[int] | None:
+        """Tokens behind one row of block means of every KV-pool layer (0: none kept); None = no layer keeps any."""
+        return self.extra.get("kv_means")
+
     def kv_bytes_per_token(self, kv_bits: int = 16) -> int:
         geo = self.kv_geometry()
         if geo is not None:
-            return sum(h * (dk + dv) for h, dk, dv in geo) * kv_bits // 8
+            means = self.kv_means() or [0] * len(geo)
+            # (a page of 16 tokens holds the means of the blocks that end in it)
+            return sum(h * (dk + dv) * (16 + (-(-16 // m) if m else 0)) for (h, dk, dv), m in zip(geo, means)) * kv_bits // (8 * 16)
         per = self.num_key_value_heads * self.head_dim
         if kv_bits == 16:
             b = per * 2
@@ -1463,6 +1469,59 @@ def _vavadra(c: ModelConfig, raw: dict) -> None:
     c.intermediate_size = max([s["mlp"]["expert"]["ff"] for s in specs if s["mlp"]] or [1])
 
 
+def _clipped_or_routed(mlp: dict, what: str) -> dict:
+    """``mlp`` record of a feed-forward that is dense (clipped GLU) or a mixture of plain gated experts whose choice is
+    limited to the best groups of neighbouring experts."""
+    kind = mlp.get("kind", "dense")
+    if kind == "dense":
+        return dict(kind=kind, ff=int(mlp["ff"]), limit=float(mlp["limit"]))
+    if kind != "moe":
+        raise ValueError(f"{what}: unknown feed-forward kind {kind!r}")
+    r, g = mlp["router"], mlp["router"].get("groups") or {}
+    n, count, keep, top = int(r["experts"]), int(g.get("count", 1)), int(g.get("keep", 1)), int(r["top"])
+    if n < 1 or not 1 <= keep <= count or n % count or not 1 <= top <= n // count * keep:
+        raise ValueError(f"{what}: the router chooses {top} of {n} experts in {keep} of {count} groups")
+    return dict(kind=kind, expert=dict(ff=int(mlp["expert"]["ff"])), router=dict(experts=n, groups=dict(count=count, keep=keep), top=top))
+
+
+def _fusolix(c: ModelConfig, raw: dict) -> None:
+    """Fusolix: every layer runs windowed attention with block means and retention side by side, then a feed-forward (dense,
+    routed experts, or none); several residual streams are mixed by small matrices around each sub-layer, and a short
+    causal convolution is added to what a sub-layer reads. Each layer owns a KV-pool layer with rows of means and a state slab."""
+    c.vocab_size, c.hidden_size = int(raw["vocab"]), int(raw["width"])
+    c.embed_scale = float((raw.get("embedding") or {}).get("scale", 1.0))
+    c.rms_norm_eps = float(raw["norm"]["eps"])
+    c.extra["streams"], c.extra["taps"] = int(raw["streams"]), int(raw["canon"]["taps"])
+    if c.extra["streams"] < 1 or c.extra["taps"] < 1:
+        raise ValueError("a model needs a stream and its convolutions a tap")
+    specs = []
+    for i, spec in enumerate(raw["layers"]):
+        m, mlp, what = spec["mixer"], spec.get("mlp"), f"layer {i}"
+        if spec["type"] != "parallel":
+            raise ValueError(f"{what}: unknown mixer type {spec['type']!r}")
+        a, r = m["left"], m["right"]
+        a = dict(heads=int(a["heads"]), kv_heads=int(a["kv_heads"]), dim=int(a["dim"]), vdim=int(a["vdim"]), scale=float(a["scale"]),
+                 mask=dict(size=int(a["mask"]["size"]), pool=int(a["mask"]["pool"])))
+        r = dict(heads=int(r["heads"]), dim=int(r["dim"]), vdim=int(r["vdim"]), rot=_rotation(r["rot"], what), decay=[float(d) for d in r["decay"]])
+        if a["heads"] % a["kv_heads"]:
+            raise ValueError(f"{what}: heads must be a multiple of kv_heads")
+        if min(a["mask"].values()) < 1:
+            raise ValueError(f"{what}: an empty window or block")
+        if r["rot"]["dims"] > r["dim"] or len(r["decay"]) != r["heads"] or not all(0 <= d <= 1 for d in r["decay"]):
+            raise ValueError(f"{what}: rot.dims above dim, or not one decay between 0 and 1 per head")
+        specs.append(dict(type="parallel", mlp=None if mlp is None else _clipped_or_routed(mlp, what),
+                          mixer=dict(left=a, right=r, left_scale=float(m["left_scale"]), right_scale=float(m["right_scale"]))))
+    c.num_hidden_layers = len(specs)
+    c.extra["layer_specs"], c.extra["layer_runs"] = specs, list(range(len(specs)))
+    left = [s["mixer"]["left"] for s in specs]
+    c.extra["kv_geometry"] = [(m["kv_heads"], m["dim"], m["vdim"]) for m in left]
+    c.extra["kv_means"] = [m["mask"]["pool"] for m in left]
+    # (uniform fields other parts read: the first layer's)
+    c.num_attention_heads, c.num_key_value_heads, c.head_dim = (left[0]["heads"], left[0]["kv_heads"], left[0]["dim"]) if left else (1, 1, 16)
+    c.partial_rotary_factor = 0.0
+    c.intermediate_size = max([s["mlp"].get("ff") or s["mlp"]["expert"]["ff"] for s in specs if s["mlp"]] or [1])
+
+
 def _baichuan(c: ModelConfig, raw: dict) -> None:
     """Baichuan (7B layout): Llama block with q, k, v fused in ``W_pack`` (reference src/models/baichuan.rs).
     The 13B models replace RoPE by ALiBi, which no attention kernel here implements."""
@@ -1486,7 +1545,7 @@ FAMILIES = {
     "gpt_neox": _gpt_neox, "gpt2": _gpt2, "gpt_bigcode": _gpt2, "phi": _phi, "olmo": _olmo1, "granitemoe": _granitemoe, "granitemoehybrid": _granitemoehybrid, "jamba": _jamba, "bitnet": _bitnet, "lfm2_moe": _lfm2, "exaone": _exaone, "telechat3": _telechat3, "deepseek": _deepseek_v1, "recurrent_gemma": _recurrent_gemma, "glm_moe_dsa": _glm_moe_dsa, "deepseek_v32": _glm_moe_dsa, "mistral4": _mistral4, "afmoe": _afmoe, "dbrx": _dbrx, "llama4": _llama4, "llama4_text": _llama4, "qwen3_next": _qwen3_next, "qwen3_5": _qwen3_next, "qwen3_5_text": _qwen3_next, "qwen3_5_moe": _qwen3_next, "qwen3_5_moe_text": _qwen3_next, "falcon_h1": _falcon_h1, "cohere2": _cohere2, "arcee": _arcee, "glm": _glm, "glm4": _glm4, "glm4v": _glm4v, "glm4v_text": _glm4v, "glm4v_moe": _glm4v_moe, "glm4v_moe_text": _glm4v_moe, "cohere2_vision": _cohere2, "paddleocr_vl": _paddleocr_vl, "glm_ocr": _glm_ocr, "glm_ocr_text": _glm_ocr, "paddleocr_vl_text": _paddleocr_vl, "nemotron": _nemotron,
     "ministral3": _ministral3, "granitemoeshared": _granitemoeshared, "nanochat": _nanochat, "code_llama": _plain, "cwm": _plain, "glm4_moe_lite": _deepseek_v3,
     "vaultgemma": _vaultgemma, "solar_open": _solar_open, "minimax_m2": _minimax_m2, "exaone_moe": _exaone_moe, "lfm2": _lfm2, "internlm2": _plain, "baichuan": _baichuan,
-    "pamasun": _pamasun, "govopel": _govopel, "vavadra": _vavadra,
+    "pamasun": _pamasun, "govopel": _govopel, "vavadra": _vavadra, "fusolix": _fusolix,
 }
 
 
@@ -1569,6 +1628,13 @@ def preset(name: str) -> ModelConfig:
         delta = dict(type="delta", mlp=mlp, mixer=dict(heads=4, kv_heads=2, dim=32, vdim=24, conv=3))
         return ModelConfig.from_dict(dict(architecture="Vavadra", vocab=512, width=144, layers=[delta, lat, att, delta], norm=dict(eps=1e-5),
                                           embedding=dict(scale=4.0), logit_scale=1.5, loop=dict(start=1, stop=3, times=2)))
+    if name == "tiny-fusolix":
+        left = dict(heads=6, kv_heads=2, dim=32, vdim=24, scale=0.2, mask=dict(size=36, pool=4))
+        right = dict(heads=3, dim=24, vdim=40, rot=dict(dims=16, base=50000.0), decay=[0.75, 0.96875, 0.99609375])
+        dense = dict(type="parallel", mixer=dict(left=left, right=right, left_scale=0.8, right_scale=1.1), mlp=dict(kind="dense", ff=176, limit=2.0))
+        routed = dict(dense, mlp=dict(kind="moe", expert=dict(ff=48), router=dict(experts=8, groups=dict(count=4, keep=2), top=3)))
+        return ModelConfig.from_dict(dict(architecture="Fusolix", vocab=512, width=144, layers=[dense, routed, dict(dense, mlp=None), routed],
+                                          norm=dict(eps=1e-5), embedding=dict(scale=4.0), streams=3, canon=dict(taps=4)))
     if name == "mamba2-2.7b":
         return ModelConfig.from_dict(dict(
             model_type="mamba2", num_hidden_layers=64, hidden_size=2560, num_heads=80, head_dim=64,

@@ -78,6 +78,41 @@ typedef struct MxStreamExtras {
   float emb_scale;
 } MxStreamExtras;
 
+// One step between two sub-layers of a model with several residual streams (mx_streams_step). What a step does not have is NULL:
+//   ids, table           the streams start as emb_scale * table[ids[row]] (no branch then)
+//   y / moe_y, moe_inv, moe_w, moe_k, bias   what the last sub-layer returned: a row, or its token's moe_k expert rows (row
+//                        moe_inv[row * moe_k + k] of moe_y, weight moe_w[.]), plus a vector
+//   mix, w_out           x_t <- sum_s mix[s * streams + t] x_s + w_out[t] result
+//   w_in, norm_w, norm_b the next sub-layer's input: layer norm of sum_s w_in[s] x_s
+//   taps_w, taps, tail, slots, n_short   its convolution: taps_w [taps, dim] (last row: current token). Rows below n_short are pieces of
+//                        one token and are convolved here with the state tail[slots[row]] [taps - 1, dim], which advances
+//   x                    the input, activation type;  normed: the norm's result of the rows from n_short on (fp32, for
+//                        mx_streams_conv; unused with one tap)
+//   sum                  instead of the next input: the sum of the new streams (fp32), which are not written
+typedef struct MxStreamsStep {
+  float* xs;
+  const int* ids;
+  const void* table;
+  const void* y;
+  const void* moe_y;
+  const int* moe_inv;
+  const float* moe_w;
+  const float* bias;
+  const float* mix;
+  const float* w_out;
+  const float* w_in;
+  const float* norm_w;
+  const float* norm_b;
+  const float* taps_w;
+  float* tail;
+  const int* slots;
+  void* x;
+  float* normed;
+  float* sum;
+  int rows, dim, streams, vocab, moe_k, taps, n_short;
+  float emb_scale, eps;
+} MxStreamsStep;
+
 // out[M, N] = epilogue(x[M, K] @ w[N(+N), K]^T). bf16 operands, fp32 accumulation on the
 // 5th-generation tensor cores (tcgen05.mma, accumulators in TMEM, operand tiles brought by TMA).
 // For the gated epilogues `w` holds gate rows at [0, N) and up rows at [glu_offset, glu_offset + N).

@@ -58,8 +58,16 @@ struct DecodeParams {
   // maps == 2: differential heads. A query and key head of dk elements holds two maps of dk / 2, attentions of their own
   // over the same values; the result is (a1 - lambda a2) / rms(.) * gain. The maps are rows of the same tile (row 2 g +
   // map of head g, zero in the other map's columns), so keys and values are still read once per key head. Hq counts heads.
+  // With one map, gain is a plain factor of the result.
   int maps;
   float lambda, gain, eps;
+  long long out_stride;      // extended form: elements between output rows
+  // Block means (template parameter MEANS, with a window): beside the window's tokens, the mean key and value of every block of
+  // mean_of tokens that lies wholly before the window. The mean of block b is at place b - page * block_size / mean_of
+  // (integer division) of the page that holds the block's last token, mean_rows places per page. No distance bias then.
+  const __nv_bfloat16* k_mean;
+  const __nv_bfloat16* v_mean;
+  int mean_of, mean_rows;
 };
 
 // Loads 8 consecutive elements of a K/V row as floats.
@@ -610,7 +618,7 @@ constexpr int kDmThreads = kDmWarps * 32;
 constexpr int kDmStages = 3;
 constexpr int kDmKeys = 16;  // keys per group (one MMA k-step of P V)
 
-template <int DK, int DV, int KV_BITS, bool BS16, bool EXT>
+template <int DK, int DV, int KV_BITS, bool BS16, bool EXT, bool MEANS>
 __global__ void __launch_bounds__(kDmThreads)
 paged_decode_mma_kernel(const DecodeParams p, const int heads_per_key) {
   // DK / DV: tile widths of keys and values; the plain form has rows of exactly D = DK = DV elements,
@@ -618,6 +626,7 @@ paged_decode_mma_kernel(const DecodeParams p, const int heads_per_key) {
   constexpr int D = DK;
   static_assert(EXT || DK == DV, "plain form: one head width");
   static_assert(!EXT || KV_BITS == 16, "the extended form reads bf16 pools");
+  static_assert(EXT || !MEANS, "block means: extended form");
   constexpr int CH = DK / 8, CHV = DV / 8;
   constexpr int TILE_BYTES = kDmKeys * DK * 2;           // one K group in bf16
   constexpr int VTILE_BYTES = kDmKeys * DV * 2;          // one V group
@@ -653,7 +662,10 @@ paged_decode_mma_kernel(const DecodeParams p, const int heads_per_key) {
   if constexpr (EXT) {
     if (p.chunk > 0 && len > 0) begin = max(begin, (len - 1) / p.chunk * p.chunk);
   }
-  const int g_begin = begin / kDmKeys;                          // first key group
+  // Key groups: with MEANS the groups of 16 block means come first, numbered below the first group of tokens.
+  const int n_means = MEANS ? begin / p.mean_of : 0;            // blocks wholly before the window
+  const int t_begin = begin / kDmKeys;                          // first key group of tokens
+  const int g_begin = t_begin - (n_means + kDmKeys - 1) / kDmKeys;
   const int g_end = (len + kDmKeys - 1) / kDmKeys;              // one past the last key group
   const int n_groups = max(0, g_end - g_begin);
   int per = (n_groups + p.num_splits - 1) / p.num_splits;
@@ -670,7 +682,7 @@ paged_decode_mma_kernel(const DecodeParams p, const int heads_per_key) {
   if constexpr (BS16 && KV_BITS == 16) {
     constexpr int kPrefetchGroups = 8;
     const int grp = s_begin + static_cast<int>(threadIdx.x);
-    if (threadIdx.x < kPrefetchGroups && grp < s_end) {
+    if (threadIdx.x < kPrefetchGroups && grp < s_end && (!MEANS || grp >= t_begin)) {
       const size_t row16 = (static_cast<size_t>(table[grp]) * p.Hkv + h) * kDmKeys;
       bulk_prefetch_l2(static_cast<const __nv_bfloat16*>(p.k_pool) + row16 * dk, kDmKeys * dk * 2);
       bulk_prefetch_l2(static_cast<const __nv_bfloat16*>(p.v_pool) + row16 * dv, kDmKeys * dv * 2);
@@ -710,7 +722,14 @@ paged_decode_mma_kernel(const DecodeParams p, const int heads_per_key) {
     uint8_t* vs = ks + TILE_BYTES;
     if (grp < s_end) {
       const size_t row16 = (static_cast<size_t>(blk16) * p.Hkv + h) * kDmKeys;
-      const int rows_ok = len - grp * kDmKeys;  // rows below this index hold real keys
+      const bool mean = MEANS && grp < t_begin;
+      const int m0 = (grp - g_begin) * kDmKeys;                       // (first block of a group of means)
+      const int rows_ok = mean ? n_means - m0 : len - grp * kDmKeys;  // rows below this index hold real keys
+      int mean_row = 0;                                               // row of the group's mean `lane & 15` in the pools of means
+      if (MEANS && mean) {
+        const int b2 = min(m0 + (lane & 15), n_means - 1), page = ((b2 + 1) * p.mean_of - 1) / p.block_size;
+        mean_row = (table[page] * p.Hkv + h) * p.mean_rows + b2 - page * p.block_size / p.mean_of;
+      }
       if constexpr (!kQuant) {
         constexpr int CM = CH > CHV ? CH : CHV;
 #pragma unroll
@@ -719,7 +738,11 @@ paged_decode_mma_kernel(const DecodeParams p, const int heads_per_key) {
           const int r = i / CM, c = i - r * CM;
           const bool ok = r < rows_ok;
           size_t row;
-          if (BS16) {
+          const void *k_src = p.k_pool, *v_src = p.v_pool;
+          if (MEANS && mean) {                           // (the same for the whole warp)
+            row = __shfl_sync(0xffffffffu, mean_row, r);
+            k_src = p.k_mean, v_src = p.v_mean;
+          } else if (BS16) {
             row = row16 + r;
           } else {
             const int key = grp * kDmKeys + r;
@@ -736,10 +759,10 @@ paged_decode_mma_kernel(const DecodeParams p, const int heads_per_key) {
             const bool kok = ok && c * 8 < dk, vok = ok && c * 8 < dv;
             if (c < CH)
               cp_async16(smem_u32(ks) + swz<DK>(r, c),
-                         static_cast<const __nv_bfloat16*>(p.k_pool) + row * dk + (kok ? c * 8 : 0), kok);
+                         static_cast<const __nv_bfloat16*>(k_src) + row * dk + (kok ? c * 8 : 0), kok);
             if (c < CHV)
               cp_async16(smem_u32(vs) + swz<DV>(r, c),
-                         static_cast<const __nv_bfloat16*>(p.v_pool) + row * dv + (vok ? c * 8 : 0), vok);
+                         static_cast<const __nv_bfloat16*>(v_src) + row * dv + (vok ? c * 8 : 0), vok);
           }
         }
       }
@@ -787,7 +810,7 @@ paged_decode_mma_kernel(const DecodeParams p, const int heads_per_key) {
     cp_async_commit();
   };
   // Block-table entries are fetched one ring slot ahead of the loads that need them.
-  auto table_at = [&](int grp) -> int { return (BS16 && grp < s_end) ? table[grp] : 0; };
+  auto table_at = [&](int grp) -> int { return (BS16 && grp < s_end && (!MEANS || grp >= t_begin)) ? table[grp] : 0; };
 
   float m_lo = -INFINITY, m_hi = -INFINITY, l_lo = 0.f, l_hi = 0.f;
   float o_acc[DV / 8][4];
@@ -867,7 +890,9 @@ paged_decode_mma_kernel(const DecodeParams p, const int heads_per_key) {
       mma_bf16_16816(sacc[0], qf[kk], bfr[0], bfr[1]);
       mma_bf16_16816(sacc[1], qf[kk], bfr[2], bfr[3]);
     }
-    const int key0 = grp * kDmKeys;
+    const bool mean = MEANS && grp < t_begin;
+    const int key0 = mean ? (grp - g_begin) * kDmKeys : grp * kDmKeys;
+    const int key_lo = mean ? 0 : begin, key_hi = mean ? n_means : len;
     float tmax_lo = -INFINITY, tmax_hi = -INFINITY;
 #pragma unroll
     for (int nt = 0; nt < 2; ++nt) {
@@ -881,7 +906,7 @@ paged_decode_mma_kernel(const DecodeParams p, const int heads_per_key) {
           const float dist = static_cast<float>(max(len - 1 - key, 0));
           v -= (e < 2 ? b1_lo : b1_hi) * log2f(fmaf(e < 2 ? b2_lo : b2_hi, dist, 1.f));
         }
-        v = (key >= begin && key < len) ? v : -INFINITY;
+        v = (key >= key_lo && key < key_hi) ? v : -INFINITY;
         sacc[nt][e] = v;
         if (e < 2) tmax_lo = fmaxf(tmax_lo, v);
         else tmax_hi = fmaxf(tmax_hi, v);
@@ -984,8 +1009,9 @@ paged_decode_mma_kernel(const DecodeParams p, const int heads_per_key) {
     if constexpr (EXT) {
       if (p.gate != nullptr)
         r *= 1.f / (1.f + __expf(-__bfloat162float(p.gate[static_cast<size_t>(b) * p.gate_stride + col])));
+      r *= p.gain;
     }
-    p.out[static_cast<size_t>(b) * p.Hq * dv + col] = __float2bfloat16(r);
+    p.out[static_cast<size_t>(b) * (EXT ? p.out_stride : static_cast<long long>(p.Hq) * dv) + col] = __float2bfloat16(r);
   };
   float* part_ml = p.scratch_ml + part_idx * (static_cast<size_t>(G) * 2);
   // differential heads: row 2 g of the first warp's part holds a1 - lambda a2 of head g (each column is written by the one
@@ -997,7 +1023,7 @@ paged_decode_mma_kernel(const DecodeParams p, const int heads_per_key) {
       float ss = 0.f;
       for (int d = lane; d < dv; d += 32) ss += o[d] * o[d];
       const float r = p.gain / sqrtf(warp_sum(ss) / dv + p.eps);
-      __nv_bfloat16* dst = p.out + static_cast<size_t>(b) * p.Hq * dv + static_cast<size_t>(h * heads_per_key + g) * dv;
+      __nv_bfloat16* dst = p.out + static_cast<size_t>(b) * p.out_stride + static_cast<size_t>(h * heads_per_key + g) * dv;
       for (int d = lane; d < dv; d += 32) dst[d] = __float2bfloat16(o[d] * r);
     }
   };
@@ -1097,12 +1123,12 @@ paged_decode_mma_kernel(const DecodeParams p, const int heads_per_key) {
   for (int i = threadIdx.x; i < G * dv; i += kDmThreads) finish(i / dv, i % dv, merged(i / dv, i % dv));
 }
 
-template <int DK, int DV, int KV_BITS, bool BS16, bool EXT>
+template <int DK, int DV, int KV_BITS, bool BS16, bool EXT, bool MEANS = false>
 static int launch_decode_mma_bs(const DecodeParams& p, int G, int grid, cudaStream_t st) {
   constexpr int ring = kDmWarps * kDmStages * kDmKeys * (DK + DV) * 2;
   constexpr int smem = 16 * DK * 2 + ring;
   static_assert(ring >= kDmWarps * 16 * DV * 4, "merge buffer");
-  auto kern = paged_decode_mma_kernel<DK, DV, KV_BITS, BS16, EXT>;
+  auto kern = paged_decode_mma_kernel<DK, DV, KV_BITS, BS16, EXT, MEANS>;
   static bool configured = false;
   if (!configured) {
     cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
@@ -1122,6 +1148,9 @@ static int launch_decode_mma(const DecodeParams& p, int G, int grid, cudaStream_
 
 template <int DK, int DV>
 static int launch_decode_ext(const DecodeParams& p, int G, int grid, cudaStream_t st) {
+  if (p.mean_of > 0)
+    return p.block_size == kDmKeys ? launch_decode_mma_bs<DK, DV, 16, true, true, true>(p, G, grid, st)
+                                   : launch_decode_mma_bs<DK, DV, 16, false, true, true>(p, G, grid, st);
   if (p.block_size == kDmKeys) return launch_decode_mma_bs<DK, DV, 16, true, true>(p, G, grid, st);
   return launch_decode_mma_bs<DK, DV, 16, false, true>(p, G, grid, st);
 }
@@ -1238,21 +1267,24 @@ extern "C" int mx_paged_decode(const void* q, long long q_stride, const void* k_
 
 // Extended decode form over bf16 pools: key / value rows of Dk / Dv elements (multiples of 8, at most
 // 128), soft cap, chunked visibility, distance bias and output gate optional (0 / NULL). maps == 2: differential heads (Hq
-// heads whose Dk columns are both maps; scratch for 2 Hq heads; no sinks, bias or gate). -10 = not covered (use mx_paged_attention_any).
+// heads whose Dk columns are both maps; scratch for 2 Hq heads; no sinks, bias or gate), else gain multiplies the result. Output rows
+// are out_stride elements apart. mean_of > 0 (with a window; one map, no chunks, no bias): block means, see DecodeParams. -10 = not covered (use mx_paged_attention_any).
 extern "C" int mx_paged_decode_ext(const void* q, long long q_stride, const void* k_pool, const void* v_pool,
                                    const int* block_tables, const int* context_lens, const float* sinks,
                                    const float* bias_r1, const float* bias_r2, const void* gate, long long gate_stride,
-                                   void* out, float* scratch, int B, int Hq, int Hkv, int Dk, int Dv, int block_size,
-                                   int max_blocks, int window, int chunk, float scale, float softcap, int maps, float lambda,
-                                   float gain, float eps, int num_splits, void* stream_) {
+                                   void* out, long long out_stride, float* scratch, int B, int Hq, int Hkv, int Dk, int Dv,
+                                   int block_size, int max_blocks, int window, int chunk, float scale, float softcap, int maps,
+                                   float lambda, float gain, float eps, const void* k_mean, const void* v_mean, int mean_of,
+                                   int num_splits, void* stream_) {
   if (B <= 0) return 0;
   if (Hkv <= 0 || Hq % Hkv || (bias_r1 == nullptr) != (bias_r2 == nullptr)) return -1;
   if ((maps != 1 && maps != 2) || (maps == 2 && (sinks != nullptr || bias_r1 != nullptr || gate != nullptr))) return -1;
+  if (mean_of > 0 && (window <= 0 || chunk > 0 || maps != 1 || bias_r1 != nullptr || k_mean == nullptr || v_mean == nullptr)) return -1;
   const int G = Hq / Hkv;
   if (maps == 2 && (G > 8 || Dk % 16)) return -10;
   const auto al16 = [](const void* a) { return (reinterpret_cast<uintptr_t>(a) & 15) == 0; };
   if (G > 16 || Dk % 8 || Dv % 8 || Dk > 128 || Dv > 128 || block_size % 16 || q_stride % 8 || !al16(q) || !al16(k_pool) ||
-      !al16(v_pool))
+      !al16(v_pool) || !al16(k_mean) || !al16(v_mean))
     return -10;
   if (num_splits < 1) num_splits = 1;
   DecodeParams p{};
@@ -1280,6 +1312,11 @@ extern "C" int mx_paged_decode_ext(const void* q, long long q_stride, const void
   p.scale_log2 = scale * kLog2e;
   p.dk = Dk;
   p.dv = Dv;
+  p.out_stride = out_stride;
+  p.k_mean = static_cast<const __nv_bfloat16*>(k_mean);
+  p.v_mean = static_cast<const __nv_bfloat16*>(v_mean);
+  p.mean_of = mean_of;
+  p.mean_rows = mean_of > 0 ? (block_size + mean_of - 1) / mean_of : 0;
   p.chunk = chunk;
   p.softcap = softcap;
   p.bias_r1 = bias_r1;

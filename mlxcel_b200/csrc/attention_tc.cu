@@ -63,8 +63,13 @@ struct TcPrefillParams {
   const int* kv_starts;
   int kv_split;
   long long out_stride;      // elements between output rows
-  // Differential heads (MAPS == 2): the result is (a1 - lambda a2) / rms(.) * gain.
+  // Differential heads (MAPS == 2): the result is (a1 - lambda a2) / rms(.) * gain. With one map, gain is a plain factor
+  // of the extended form's result.
   float lambda, gain, eps;
+  // Block means (MEANS, with a window): beside the window's tokens, one key and value for every block of mean_of tokens
+  // wholly before the window, gathered to dense rows: block b of sequence s is row mean_starts[s] + b.
+  const int* mean_starts;
+  int mean_of;
 };
 
 // The extended form runs eight softmax warps instead of four, two per 32 query rows: each takes one half of
@@ -83,17 +88,21 @@ constexpr int kExtSmem = 8 * kBiasTab * 4 + 2 * 2 * kTcRows * 4 + 2 * kTcRows * 
 // maxima and sums per map and an accumulator each in TMEM; the epilogue combines the two in registers. Scores of map
 // 2's first tile run under the softmax of map 1's last one, as between any two tiles.
 //
+// Block means (MEANS): the walk begins with the tiles of 128 means that some query of the CTA sees, then the window's tokens. Rows of
+// a means' tile past a query's last visible block are masked (they belong to later blocks, the next sequence, or are zero).
+//
 // The second weight term takes the room of one V stage where both heads are 128 wide: a V tile is only
 // needed once its softmax is through, so its load still has most of a tile's time.
 __host__ __device__ constexpr int tc_v_stages(int dk, int dv, bool ext) { return (ext && dk >= 128 && dv == 128) ? 1 : kTcStages; }
 // Keys of 192 columns (and two maps of queries of 128) leave room for one K stage (free again as soon as its score MMA has run).
 __host__ __device__ constexpr int tc_k_stages(int dk, int maps) { return dk > 128 || (dk == 128 && maps == 2) ? 1 : kTcStages; }
 
-template <int DK, int DV, bool EXT, int MAPS>
+template <int DK, int DV, bool EXT, int MAPS, bool MEANS>
 __global__ void __launch_bounds__(tc_threads(EXT), 1)
 paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
                         const __grid_constant__ CUtensorMap map_v, const __grid_constant__ CUtensorMap map_kr,
-                        const TcPrefillParams p) {
+                        const __grid_constant__ CUtensorMap map_vm, const TcPrefillParams p) {
+  // (map_kr: the shared key part of dense rows, or the means' keys; map_vm: the means' values)
   constexpr int DC = DK / 64, DCV = DV / 64;          // 64-column (128-byte) sub-tiles per row
   constexpr int SUB_BYTES = 128 * 128;                // one [128 rows][64 cols] sub-tile
   constexpr int Q_BYTES = DC * SUB_BYTES;
@@ -112,6 +121,7 @@ paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
   static_assert((DK == 64 || DK == 128 || (EXT && DK == 192)) && (DV == 64 || DV == 128), "head dims");
   static_assert(EXT || DK == DV, "plain form: one head width");
   static_assert(MAPS == 1 || EXT, "differential heads: extended form");
+  static_assert(!MEANS || (EXT && MAPS == 1), "block means: extended form, one map");
   const int dk = EXT ? p.dk : DK, dv = EXT ? p.dv : DV;
 
   extern __shared__ uint8_t smem_raw[];
@@ -160,8 +170,10 @@ paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
   }
   kv_begin = (kv_begin / kTcKeys) * kTcKeys;
   const int key_tiles = (kv_end - kv_begin + kTcKeys - 1) / kTcKeys;
-  const int n_tiles = MAPS * key_tiles;               // tiles of the walk
-  const auto key_tile = [&](int j) { return MAPS == 2 && j >= key_tiles ? j - key_tiles : j; };
+  // (the last query of the tile sees the most means)
+  const int mean_tiles = MEANS ? (max(0, kv_end - p.window) / p.mean_of + kTcKeys - 1) / kTcKeys : 0;
+  const int n_tiles = MAPS * key_tiles + mean_tiles;  // tiles of the walk
+  const auto key_tile = [&](int j) { return MAPS == 2 && j >= key_tiles ? j - key_tiles : j - mean_tiles; };
   const auto map_of = [&](int j) { return MAPS == 2 && j >= key_tiles ? 1 : 0; };
   const int last_block = (ctx - 1) / kTcBlock;   // last pool block the sequence owns
 
@@ -240,6 +252,28 @@ paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
       // P V MMA of the same key tile: K of tile j + stages is requested a whole softmax earlier.
       // one pool block per lane; blocks past the sequence's last one repeat it (masked keys, but
       // the values multiplied by P = 0 must be finite)
+      if (MEANS && j < mean_tiles) {
+        // a tile of means: one box per 64-column sub-tile
+        if (lane == 0) {
+          const int m0 = p.mean_starts[s] + j * kTcKeys;
+          ok = mbar_wait(&k_empty[stage], phase ^ 1u, p.status, kErrAttnProducer);
+          if (ok) {
+            mbar_expect_tx(&k_full[stage], K_BYTES);
+            for (int c = 0; c < DC; ++c) tma_load_3d(k_sm + stage * K_BYTES + c * SUB_BYTES, &map_kr, &k_full[stage], c * 64, hkv, m0, pol_kv);
+            ok = mbar_wait(&kv_empty[vstage], vphase ^ 1u, p.status, kErrAttnProducer);
+          }
+          if (ok) {
+            mbar_expect_tx(&v_full[vstage], V_BYTES);
+            for (int c = 0; c < DCV; ++c) tma_load_3d(v_sm + vstage * V_BYTES + c * SUB_BYTES, &map_vm, &v_full[vstage], c * 64, hkv, m0, pol_kv);
+          }
+        }
+        ok = __shfl_sync(0xffffffffu, ok ? 1 : 0, 0) != 0;
+        if (++stage == KST) {
+          stage = 0;
+          phase ^= 1u;
+        }
+        continue;
+      }
       int row0 = 0;
       if (lane < kTcKeys / kTcBlock) {
         const int b = min((kv_begin + key_tile(j) * kTcKeys) / kTcBlock + lane, last_block);
@@ -315,7 +349,7 @@ paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
 #pragma unroll
           for (int term = 0; term < PTERMS; ++term) {
             const uint64_t da = umma_desc_k_sw128(pa + term * PHALF_BYTES + (kk >> 2) * SUB_BYTES + (kk & 3) * 32);
-            umma_bf16(tmem_base + O_COL + map_of(j) * DV, da, db, idesc_pv, (key_tile(j) > 0 || kk > 0 || term > 0) ? 1u : 0u);
+            umma_bf16(tmem_base + O_COL + map_of(j) * DV, da, db, idesc_pv, ((MEANS ? j : key_tile(j)) > 0 || kk > 0 || term > 0) ? 1u : 0u);
           }
         }
         umma_commit(&kv_empty[stage]);   // the V tile of this stage is consumed
@@ -355,14 +389,17 @@ paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
       if (!ok) break;
       tc_fence_after_sync();
       const int o_col = O_COL + map_of(j) * DV;
-      const int key0 = kv_begin + key_tile(j) * kTcKeys;
+      const bool mean = MEANS && j < mean_tiles;
+      const int key0 = mean ? j * kTcKeys : kv_begin + key_tile(j) * kTcKeys;      // (of a tile of means: its first block)
       // Only tiles that cross the diagonal, the window edge or the end need the mask.
       const bool need_mask = (key0 + kTcKeys - 1 > pos_base + tok0) ||
                              (p.window > 0 && key0 < pos_base + tok0 + kTcRows - p.window) ||
                              (EXT && p.chunk > 0 && key0 < (pos_base + tok0 + rows_valid - 1) / p.chunk * p.chunk);
       const int hkey0 = key0 + half * HC;   // first key of this thread's columns
       int lo = 0, hi = HC;   // valid key columns of this row: [lo, hi)
-      if (need_mask) {
+      if (mean) {
+        hi = min(HC, max(0, qpos + 1 - p.window) / p.mean_of - hkey0);
+      } else if (need_mask) {
         hi = min(HC, qpos - hkey0 + 1);
         if (p.window > 0) lo = max(0, qpos - p.window + 1 - hkey0);
         if (EXT && p.chunk > 0) lo = max(lo, qpos / p.chunk * p.chunk - hkey0);
@@ -404,7 +441,7 @@ paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
       __syncwarp();
       if (lane == 0) mbar_arrive(&s_empty[sb]);   // the score buffer may be overwritten
       float mx = -INFINITY;
-      if (need_mask) {
+      if (need_mask || mean) {
 #pragma unroll
         for (int i = 0; i < HC; ++i) {
           if (i < lo || i >= hi) sv[i] = -INFINITY;
@@ -559,7 +596,7 @@ paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
         osc = (m_used > -INFINITY) ? exp2f(m_used - m2) : 0.f;
         l = l * osc + exp2f(sk - m2);
       }
-      const float inv = l > 0.f ? osc / l : 0.f;
+      const float inv = l > 0.f ? (EXT ? osc * p.gain : osc) / l : 0.f;
       __nv_bfloat16* dst = p.out + static_cast<size_t>(q0 + tok0 + row) * p.out_stride + hq * dv;
 #pragma unroll
       for (int cc = 0; cc < DV / 32 / HALVES; ++cc) {
@@ -611,14 +648,14 @@ paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
   }
 }
 
-template <int DK, int DV, bool EXT, int MAPS = 1>
-static int launch_prefill_tc(const CUtensorMap& mq, const CUtensorMap& mk, const CUtensorMap& mv, const CUtensorMap& mkr,
+template <int DK, int DV, bool EXT, int MAPS = 1, bool MEANS = false>
+static int launch_prefill_tc(const CUtensorMap& mq, const CUtensorMap& mk, const CUtensorMap& mv, const CUtensorMap& mkr, const CUtensorMap& mvm,
                              const TcPrefillParams& p, int grid, cudaStream_t stream) {
   constexpr int SUB = 128 * 128;
   constexpr int smem = (DK / 64) * SUB * (MAPS + tc_k_stages(DK, MAPS)) + (DV / 64) * SUB * tc_v_stages(DK, DV, EXT) +
                        (EXT ? 4 : 2) * SUB + 1024 + 256 + (EXT ? kExtSmem : 0);
   static_assert(smem <= 227 * 1024, "shared memory");
-  auto kern = paged_prefill_tc_kernel<DK, DV, EXT, MAPS>;
+  auto kern = paged_prefill_tc_kernel<DK, DV, EXT, MAPS, MEANS>;
   static bool configured = false;
   if (!configured) {
     cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
@@ -626,7 +663,7 @@ static int launch_prefill_tc(const CUtensorMap& mq, const CUtensorMap& mk, const
     prefer_max_shared(kern);
     configured = true;
   }
-  return static_cast<int>(launch_kernel(kern, dim3(grid), dim3(tc_threads(EXT)), smem, stream, mq, mk, mv, mkr, p));
+  return static_cast<int>(launch_kernel(kern, dim3(grid), dim3(tc_threads(EXT)), smem, stream, mq, mk, mv, mkr, mvm, p));
 }
 
 }  // namespace mx
@@ -673,28 +710,35 @@ extern "C" int mx_paged_prefill_tc(const void* q, long long q_stride, const void
   const uint64_t pool_rows = static_cast<uint64_t>(pool_blocks) * Hkv * kTcBlock;
   if (!make_tensor_map_bf16(&mk, k_pool, pool_rows, D, D, kTcBlock, 64)) return -4;
   if (!make_tensor_map_bf16(&mv, v_pool, pool_rows, D, D, kTcBlock, 64)) return -4;
-  if (D == 64) return launch_prefill_tc<64, 64, false>(mq, mk, mv, mv, p, static_cast<int>(grid), stream);
-  return launch_prefill_tc<128, 128, false>(mq, mk, mv, mv, p, static_cast<int>(grid), stream);
+  if (D == 64) return launch_prefill_tc<64, 64, false>(mq, mk, mv, mv, mv, p, static_cast<int>(grid), stream);
+  return launch_prefill_tc<128, 128, false>(mq, mk, mv, mv, mv, p, static_cast<int>(grid), stream);
 }
 
 // Extended form: key / value rows of Dk / Dv elements (multiples of 8, at most 128); distance bias, output gate,
-// chunked visibility and soft cap optional (NULL / 0). maps == 2: differential heads, Dk columns hold both maps. Returns -10 when not covered (use mx_paged_attention_any).
+// chunked visibility and soft cap optional (NULL / 0). maps == 2: differential heads, Dk columns hold both maps, else gain multiplies
+// the result. Output rows are out_stride elements apart. mean_rows > 0 (with a window; one map, no chunks, no bias): block means,
+// k_means [mean_rows, Hkv, Dk] and v_means [mean_rows, Hkv, Dv] of blocks of mean_of tokens, sequence s from row mean_starts[s] on
+// (as many as its last query sees). Returns -10 when not covered (use mx_paged_attention_any).
 extern "C" int mx_paged_prefill_ext(const void* q, long long q_stride, const void* k_pool, const void* v_pool,
                                     long long pool_blocks, const int* block_tables, const int* cu_q,
                                     const int* context_lens, const float* sinks, const float* bias_r1,
                                     const float* bias_r2, const void* gate, long long gate_stride, void* out,
-                                    int num_seqs, int total_q, int max_q_len, int Hq, int Hkv, int Dk, int Dv,
+                                    long long out_stride, int num_seqs, int total_q, int max_q_len, int Hq, int Hkv, int Dk, int Dv,
                                     int block_size, int max_blocks, int window, int chunk, float scale, float softcap,
-                                    int maps, float lambda, float gain, float eps, void* status, void* stream_) {
+                                    int maps, float lambda, float gain, float eps, const void* k_means, const void* v_means,
+                                    const int* mean_starts, int mean_rows, int mean_of, void* status, void* stream_) {
   cudaStream_t stream = static_cast<cudaStream_t>(stream_);
   if (num_seqs <= 0 || total_q <= 0) return 0;
   if (Hkv <= 0 || Hq % Hkv || (bias_r1 == nullptr) != (bias_r2 == nullptr)) return -1;
   if ((maps != 1 && maps != 2) || (maps == 2 && (sinks != nullptr || bias_r1 != nullptr || gate != nullptr))) return -1;
+  if (mean_rows > 0 && (window <= 0 || chunk > 0 || maps != 1 || bias_r1 != nullptr || mean_of < 1 || k_means == nullptr || v_means == nullptr ||
+                        mean_starts == nullptr))
+    return -1;
   const auto al16 = [](const void* a) { return (reinterpret_cast<uintptr_t>(a) & 15) == 0; };
   if (Dk % maps) return -10;
   Dk /= maps;                          // columns of one map
-  if (block_size != kTcBlock || Dk % 8 || Dv % 8 || Dk > 128 || Dv > 128 || q_stride % 8 || gate_stride % 8 || !al16(q) ||
-      !al16(out) || !al16(gate) || !al16(k_pool) || !al16(v_pool))
+  if (block_size != kTcBlock || Dk % 8 || Dv % 8 || Dk > 128 || Dv > 128 || q_stride % 8 || gate_stride % 8 || out_stride % 8 || !al16(q) ||
+      !al16(out) || !al16(k_means) || !al16(v_means) || !al16(gate) || !al16(k_pool) || !al16(v_pool))
     return -10;
   TcPrefillParams p{};
   p.block_tables = block_tables;
@@ -708,7 +752,8 @@ extern "C" int mx_paged_prefill_ext(const void* q, long long q_stride, const voi
   p.Hkv = Hkv;
   p.max_blocks = max_blocks;
   p.window = window;
-  p.out_stride = static_cast<long long>(Hq) * Dv;
+  p.out_stride = out_stride;
+  p.gain = gain;
   p.tiles_per_seq = (max_q_len + kTcRows - 1) / kTcRows;
   p.scale_log2 = scale * 1.4426950408889634f;
   p.dk = Dk;
@@ -724,7 +769,7 @@ extern "C" int mx_paged_prefill_ext(const void* q, long long q_stride, const voi
   CUtensorMap mq, mk, mv;
   if (maps == 2) {
     // maps as groups of their own: a box that is wider than a map ends in zeros
-    p.lambda = lambda, p.gain = gain, p.eps = eps;
+    p.lambda = lambda, p.eps = eps;
     const uint64_t rows = static_cast<uint64_t>(pool_blocks) * Hkv * kTcBlock;
     if (!make_tensor_map_bf16_3d(&mq, q, total_q, 2ull * Hq, Dk, q_stride, Dk, kTcRows, 64) ||
         !make_tensor_map_bf16_3d(&mk, k_pool, rows, 2, Dk, 2ull * Dk, Dk, kTcBlock, 64) ||
@@ -732,10 +777,10 @@ extern "C" int mx_paged_prefill_ext(const void* q, long long q_stride, const voi
       return -4;
     const int g2 = static_cast<int>(grid);
     if (Dk <= 64)
-      return Dv <= 64 ? launch_prefill_tc<64, 64, true, 2>(mq, mk, mv, mv, p, g2, stream)
-                      : launch_prefill_tc<64, 128, true, 2>(mq, mk, mv, mv, p, g2, stream);
-    return Dv <= 64 ? launch_prefill_tc<128, 64, true, 2>(mq, mk, mv, mv, p, g2, stream)
-                    : launch_prefill_tc<128, 128, true, 2>(mq, mk, mv, mv, p, g2, stream);
+      return Dv <= 64 ? launch_prefill_tc<64, 64, true, 2>(mq, mk, mv, mv, mv, p, g2, stream)
+                      : launch_prefill_tc<64, 128, true, 2>(mq, mk, mv, mv, mv, p, g2, stream);
+    return Dv <= 64 ? launch_prefill_tc<128, 64, true, 2>(mq, mk, mv, mv, mv, p, g2, stream)
+                    : launch_prefill_tc<128, 128, true, 2>(mq, mk, mv, mv, mv, p, g2, stream);
   }
   // a query box may run into the next head's columns: the keys' columns there are zero
   if (!make_tensor_map_bf16(&mq, q, static_cast<uint64_t>(total_q), static_cast<uint64_t>(Hq) * Dk,
@@ -745,11 +790,25 @@ extern "C" int mx_paged_prefill_ext(const void* q, long long q_stride, const voi
   if (!make_tensor_map_bf16(&mk, k_pool, pool_rows, Dk, Dk, kTcBlock, 64)) return -4;
   if (!make_tensor_map_bf16(&mv, v_pool, pool_rows, Dv, Dv, kTcBlock, 64)) return -4;
   const int g = static_cast<int>(grid);
+  if (mean_rows > 0) {
+    p.mean_starts = mean_starts;
+    p.mean_of = mean_of;
+    CUtensorMap mkm, mvm;
+    const uint64_t rows = static_cast<uint64_t>(mean_rows);
+    if (!make_tensor_map_bf16_3d(&mkm, k_means, rows, Hkv, Dk, static_cast<uint64_t>(Hkv) * Dk, Dk, kTcKeys, 64) ||
+        !make_tensor_map_bf16_3d(&mvm, v_means, rows, Hkv, Dv, static_cast<uint64_t>(Hkv) * Dv, Dv, kTcKeys, 64))
+      return -4;
+    if (Dk <= 64)
+      return Dv <= 64 ? launch_prefill_tc<64, 64, true, 1, true>(mq, mk, mv, mkm, mvm, p, g, stream)
+                      : launch_prefill_tc<64, 128, true, 1, true>(mq, mk, mv, mkm, mvm, p, g, stream);
+    return Dv <= 64 ? launch_prefill_tc<128, 64, true, 1, true>(mq, mk, mv, mkm, mvm, p, g, stream)
+                    : launch_prefill_tc<128, 128, true, 1, true>(mq, mk, mv, mkm, mvm, p, g, stream);
+  }
   if (Dk <= 64)
-    return Dv <= 64 ? launch_prefill_tc<64, 64, true>(mq, mk, mv, mv, p, g, stream)
-                    : launch_prefill_tc<64, 128, true>(mq, mk, mv, mv, p, g, stream);
-  return Dv <= 64 ? launch_prefill_tc<128, 64, true>(mq, mk, mv, mv, p, g, stream)
-                  : launch_prefill_tc<128, 128, true>(mq, mk, mv, mv, p, g, stream);
+    return Dv <= 64 ? launch_prefill_tc<64, 64, true>(mq, mk, mv, mv, mv, p, g, stream)
+                    : launch_prefill_tc<64, 128, true>(mq, mk, mv, mv, mv, p, g, stream);
+  return Dv <= 64 ? launch_prefill_tc<128, 64, true>(mq, mk, mv, mv, mv, p, g, stream)
+                  : launch_prefill_tc<128, 128, true>(mq, mk, mv, mv, mv, p, g, stream);
 }
 
 // Latent attention over expanded rows: keys [k_nope (Dn) | shared rotated part (R)], values Dv wide. Sequence s owns query
@@ -781,6 +840,7 @@ extern "C" int mx_latent_prefill(const void* q, long long q_stride, const void* 
   p.dv = Dv;
   p.kv_starts = kv_starts;
   p.sinks = sinks;
+  p.gain = 1.f;
   p.window = window;
   p.kv_split = Dn;
   p.out_stride = out_stride;
@@ -795,8 +855,8 @@ extern "C" int mx_latent_prefill(const void* q, long long q_stride, const void* 
     return -4;
   const int g = static_cast<int>(grid);
   if (Dn <= 64)
-    return Dv <= 64 ? launch_prefill_tc<128, 64, true>(mq, mk, mv, mkr, p, g, stream)
-                    : launch_prefill_tc<128, 128, true>(mq, mk, mv, mkr, p, g, stream);
-  return Dv <= 64 ? launch_prefill_tc<192, 64, true>(mq, mk, mv, mkr, p, g, stream)
-                  : launch_prefill_tc<192, 128, true>(mq, mk, mv, mkr, p, g, stream);
+    return Dv <= 64 ? launch_prefill_tc<128, 64, true>(mq, mk, mv, mkr, mv, p, g, stream)
+                    : launch_prefill_tc<128, 128, true>(mq, mk, mv, mkr, mv, p, g, stream);
+  return Dv <= 64 ? launch_prefill_tc<192, 64, true>(mq, mk, mv, mkr, mv, p, g, stream)
+                  : launch_prefill_tc<192, 128, true>(mq, mk, mv, mkr, mv, p, g, stream);
 }

@@ -4,7 +4,8 @@
 //                       all experts, then top-k (optionally renormalised; Qwen-MoE). mode 1: top-k
 //                       on the logits, then softmax over the k selected logits (Mixtral, GPT-OSS:
 //                       src/models/gpt_oss.rs:402-446 of the reference).
-//   mx_moe_route_choice fp32 logits: chosen by softmax score + correction, weighted by the score * scale.
+//   mx_moe_route_choice fp32 logits: chosen by softmax score + correction (within the best groups of experts), weighted by the
+//                       score * scale, optionally over the sum of the chosen scores.
 //   mx_moe_align        counts the (token, slot) pairs routed to each LOCAL expert
 //                       [e_begin, e_end), builds exclusive offsets and the permutation that sorts
 //                       pairs by expert (stable in token order, so results are deterministic).
@@ -98,10 +99,12 @@ __global__ void moe_route_kernel(const __nv_bfloat16* __restrict__ logits, int* 
 }
 
 // One warp per token, fp32 logits: softmax over all experts (identity experts included), the k largest score + correction
-// (ties: lowest id), weight = score * scale.
+// (ties: lowest id), weight = score * scale. count > keep: the experts form `count` groups of neighbours, and only those of the
+// `keep` groups with the largest best member can be chosen. norm_eps >= 0: the chosen scores are divided by their sum + norm_eps.
 __global__ void __launch_bounds__(128)
 moe_route_choice_kernel(const float* __restrict__ logits, long long ld, const float* __restrict__ correction, int* __restrict__ ids,
-                        float* __restrict__ wts, int T, int E, int k, float scale) {
+                        float* __restrict__ wts, int T, int E, int k, float scale, int count, int keep, float norm_eps) {
+  __shared__ float best_of[4][512];                          // per warp: the experts' scores, then which groups are kept
   pdl_trigger();
   pdl_wait();
   const int t = (blockIdx.x * blockDim.x + threadIdx.x) >> 5, lane = threadIdx.x & 31;
@@ -128,6 +131,49 @@ moe_route_choice_kernel(const float* __restrict__ logits, long long ld, const fl
     p[i] *= inv;
     c[i] = e < E ? p[i] + (correction != nullptr ? correction[e] : 0.f) : -INFINITY;
   }
+  if (count > keep) {
+    float* top = best_of[threadIdx.x >> 5];
+    const int per = E / count;
+    // scores go through shared memory: a group's members are spread over the lanes
+#pragma unroll
+    for (int i = 0; i < 16; ++i)
+      if (lane + 32 * i < E) top[lane + 32 * i] = c[i];
+    __syncwarp();
+    float g[16];
+#pragma unroll
+    for (int i = 0; i < 16; ++i) {
+      g[i] = -INFINITY;
+      const int at = (lane + 32 * i) * per;
+      if (lane + 32 * i < count)
+        for (int e = 0; e < per; ++e) g[i] = fmaxf(g[i], top[at + e]);
+    }
+    unsigned kept = 0u;                                      // bit i: group lane + 32 i
+    for (int s = 0; s < keep; ++s) {
+      float best = -INFINITY;
+      int best_g = 0x7fffffff;
+#pragma unroll
+      for (int i = 0; i < 16; ++i)
+        if (!(kept >> i & 1u) && lane + 32 * i < count && (best_g == 0x7fffffff || g[i] > best)) best = g[i], best_g = lane + 32 * i;
+#pragma unroll
+      for (int o = 16; o > 0; o >>= 1) {
+        const float ob = __shfl_xor_sync(0xffffffffu, best, o);
+        const int og = __shfl_xor_sync(0xffffffffu, best_g, o);
+        if (og != 0x7fffffff && (best_g == 0x7fffffff || ob > best || (ob == best && og < best_g))) best = ob, best_g = og;
+      }
+      if (best_g != 0x7fffffff && (best_g & 31) == lane) kept |= 1u << (best_g >> 5);
+    }
+    __syncwarp();
+#pragma unroll
+    for (int i = 0; i < 16; ++i)
+      if (lane + 32 * i < count) top[lane + 32 * i] = kept >> i & 1u ? 1.f : 0.f;
+    __syncwarp();
+#pragma unroll
+    for (int i = 0; i < 16; ++i) {
+      const int e = lane + 32 * i;
+      if (e < E && top[e / per] == 0.f) c[i] = -INFINITY;
+    }
+  }
+  float chosen[kMaxTopK], total = 0.f;
   for (int s = 0; s < k; ++s) {
     float best = -INFINITY, score = 0.f;
     int best_e = 0x7fffffff;
@@ -144,11 +190,13 @@ moe_route_choice_kernel(const float* __restrict__ logits, long long ld, const fl
 #pragma unroll
     for (int i = 0; i < 16; ++i)
       if (lane + 32 * i == best_e) c[i] = -INFINITY;
-    if (lane == 0) {
-      ids[static_cast<size_t>(t) * k + s] = best_e;
-      wts[static_cast<size_t>(t) * k + s] = score * scale;
-    }
+    if (lane == 0) ids[static_cast<size_t>(t) * k + s] = best_e;
+    chosen[s] = score;
+    total += score;
   }
+  const float f = norm_eps >= 0.f ? scale / (total + norm_eps) : scale;
+  if (lane == 0)
+    for (int s = 0; s < k; ++s) wts[static_cast<size_t>(t) * k + s] = chosen[s] * f;
 }
 
 // Single CTA: histogram -> exclusive scan -> stable scatter. T * k pairs are at most a few
@@ -431,14 +479,15 @@ extern "C" int mx_moe_align(const int* topk_ids, int* expert_offsets, int* sorte
   return static_cast<int>(cudaGetLastError());
 }
 
-// logits fp32 [T, E], rows ld apart; correction fp32 [E] or NULL. E at most 512, k at most 16.
+// logits fp32 [T, E], rows ld apart; correction fp32 [E] or NULL. E at most 512, k at most 16. count / keep: groups of experts and
+// how many of them can be chosen from (1, 1: all); norm_eps < 0: the chosen scores are not divided by their sum.
 extern "C" int mx_moe_route_choice(const void* logits, long long ld, const void* correction, int* ids, float* wts, int T, int E, int k,
-                                   float scale, void* stream) {
+                                   float scale, int count, int keep, float norm_eps, void* stream) {
   if (T <= 0) return 0;
-  if (E > 512 || k > kMaxTopK || k > E || k < 1) return -1;
+  if (E > 512 || k > kMaxTopK || k > E || k < 1 || keep < 1 || count < keep || E % count || k > E / count * keep) return -1;
   return static_cast<int>(launch_kernel(moe_route_choice_kernel, dim3((T + 3) / 4), dim3(128), 0, static_cast<cudaStream_t>(stream),
                                         static_cast<const float*>(logits), ld, static_cast<const float*>(correction), ids, wts, T, E, k,
-                                        scale));
+                                        scale, count, keep, norm_eps));
 }
 
 // As mx_moe_align, and the inverse: inv_row[pair] = sorted row of the pair, -1 when its expert is not local.

@@ -6,7 +6,7 @@
 //   grouped_gemm_any  rows offsets[e] .. of a permuted row list times expert e's matrix
 //   attention_any  causal paged attention of any query rows (decode rows are pieces of one token):
 //                  sliding window, chunks, soft cap, sinks, logarithmic distance bias, output gate, key and value heads
-//                  of different width (which may lie in rows wider than they are), differential heads of two maps
+//                  of different width (which may lie in rows wider than they are), differential heads of two maps, block means
 #include "api.h"
 #include "typed.cuh"
 
@@ -120,8 +120,15 @@ struct AnyAttnParams {
   float scale, softcap;
   // maps == 2: differential heads. Query and key rows of a head hold two maps of Dk columns each (attentions of their own
   // over the same values); the result is (a1 - lambda a2) / rms(.) * gain.
+  // With one map, gain is a plain factor of the result.
   int maps;
   float lambda, gain, eps;
+  long long out_stride;
+  // mean_of > 0 (with a window): the mean key and value of every block of mean_of tokens wholly before the window are keys too;
+  // that of block b is at place b - page * block_size / mean_of of the page that holds the block's last token.
+  const void* k_mean;
+  const void* v_mean;
+  int mean_of, mean_rows;
 };
 
 // One CTA per (query row, query head). The warps take the 32-key chunks in turn: scores with one key
@@ -155,7 +162,8 @@ attention_any_kernel(const AnyAttnParams p) {
   const T* kp = static_cast<const T*>(p.k_pool);
   const T* vp = static_cast<const T*>(p.v_pool);
   const bool vec = p.Dk % 4 == 0 && p.ldk % 4 == 0;
-  T* out = static_cast<T*>(p.out) + (static_cast<size_t>(row) * p.Hq + h) * p.Dv;
+  T* out = static_cast<T*>(p.out) + static_cast<size_t>(row) * p.out_stride + static_cast<size_t>(h) * p.Dv;
+  const int n_means = p.mean_of > 0 ? first / p.mean_of : 0, n_keys = n_means + pos + 1 - first;   // the means come first
   for (int map = 0; map < p.maps; ++map) {
   const T* q = static_cast<const T*>(p.q) + static_cast<size_t>(row) * p.q_stride + (static_cast<size_t>(h) * p.maps + map) * p.Dk;
   __syncthreads();                                       // (the previous map's results have been read)
@@ -164,15 +172,22 @@ attention_any_kernel(const AnyAttnParams p) {
   float m = -INFINITY, l = 0.f, acc[NV];
 #pragma unroll
   for (int i = 0; i < NV; ++i) acc[i] = 0.f;
-  for (int c0 = first + warp * 32; c0 <= pos; c0 += kAaWarps * 32) {
-    const int key = c0 + lane;
-    const bool ok = key <= pos;
+  for (int c0 = warp * 32; c0 < n_keys; c0 += kAaWarps * 32) {
+    const int i0 = c0 + lane, key = first + i0 - n_means;
+    const bool ok = i0 < n_keys;
     float sc = -INFINITY;
-    long long prow = 0;
+    long long prow = 0;                                  // pool row; ~row of the means
     if (ok) {
-      const int blk = table[key / p.block_size];
-      prow = (static_cast<long long>(blk) * p.Hkv + hk) * p.block_size + key % p.block_size;
-      const T* kr = kp + prow * p.ldk + map * p.Dk;
+      const T* kr;
+      if (i0 < n_means) {
+        const int page = ((i0 + 1) * p.mean_of - 1) / p.block_size;
+        const long long m = (static_cast<long long>(table[page]) * p.Hkv + hk) * p.mean_rows + i0 - page * p.block_size / p.mean_of;
+        kr = static_cast<const T*>(p.k_mean) + m * p.ldk;
+        prow = ~m;
+      } else {
+        prow = (static_cast<long long>(table[key / p.block_size]) * p.Hkv + hk) * p.block_size + key % p.block_size;
+        kr = kp + prow * p.ldk + map * p.Dk;
+      }
       float d = 0.f;
       if (vec) {
         float e[4] = {0.f, 0.f, 0.f, 0.f};
@@ -197,10 +212,11 @@ attention_any_kernel(const AnyAttnParams p) {
     m = mn;
 #pragma unroll
     for (int i = 0; i < NV; ++i) acc[i] *= corr;
-    const int nk = min(32, pos + 1 - c0);
+    const int nk = min(32, n_keys - c0);
     for (int t = 0; t < nk; ++t) {
       const float pt = __shfl_sync(0xffffffffu, pr, t);
-      const T* vr = vp + __shfl_sync(0xffffffffu, prow, t) * p.ldv;
+      const long long vrow = __shfl_sync(0xffffffffu, prow, t);
+      const T* vr = vrow >= 0 ? vp + vrow * p.ldv : static_cast<const T*>(p.v_mean) + ~vrow * p.ldv;
 #pragma unroll
       for (int i = 0; i < NV; ++i) {
         const int d = lane + 32 * i;
@@ -236,7 +252,7 @@ attention_any_kernel(const AnyAttnParams p) {
       continue;
     }
     if (gate != nullptr) o *= sigmoid_f(to_f(gate[d]));
-    out[d] = from_f<T>(o);
+    out[d] = from_f<T>(o * p.gain);
   }
   }
   if (p.maps != 2) return;
@@ -313,15 +329,17 @@ extern "C" int mx_grouped_gemm_any(const void* x, const void* w, void* out, cons
 
 // Query row r of sequence s (cu_q[s] <= r < cu_q[s + 1]) is token context_lens[s] - (cu_q[s + 1] - r) of
 // its sequence. r1 / r2, sinks, gate may be NULL. Pools hold the activation type. maps == 2: differential heads (Dk columns of
-// a query and key head are both maps; no sinks, bias or gate).
+// a query and key head are both maps; no sinks, bias or gate), else gain multiplies the result. Output rows are out_stride
+// elements apart. mean_of > 0 (with a window; one map, no chunks, no bias): block means.
 extern "C" int mx_paged_attention_any(const void* q, long long q_stride, const void* k_pool, const void* v_pool,
                                       const void* block_tables, const void* cu_q, const void* context_lens,
                                       const void* sinks, const void* r1, const void* r2, const void* gate,
-                                      long long gate_stride, void* out, int num_seqs, int rows, int Hq, int Hkv, int Dk,
-                                      int Dv, int ldk, int ldv, int block_size, int max_blocks, int window, int chunk,
-                                      float scale, float softcap, int maps, float lambda, float gain, float eps, int fp32,
-                                      void* stream) {
+                                      long long gate_stride, void* out, long long out_stride, int num_seqs, int rows, int Hq,
+                                      int Hkv, int Dk, int Dv, int ldk, int ldv, int block_size, int max_blocks, int window,
+                                      int chunk, float scale, float softcap, int maps, float lambda, float gain, float eps,
+                                      const void* k_mean, const void* v_mean, int mean_of, int fp32, void* stream) {
   if (num_seqs <= 0 || rows <= 0) return 0;
+  if (mean_of > 0 && (window <= 0 || chunk > 0 || maps != 1 || r1 != nullptr || k_mean == nullptr || v_mean == nullptr)) return -1;
   if ((maps != 1 && maps != 2) || (maps == 2 && (Dk % 2 || sinks != nullptr || r1 != nullptr || gate != nullptr))) return -1;
   if (Hkv <= 0 || Hq % Hkv || Hq > 65535 || Dk <= 0 || Dv <= 0 || ldk < Dk || ldv < Dv ||
       (r1 == nullptr) != (r2 == nullptr))
@@ -329,7 +347,8 @@ extern "C" int mx_paged_attention_any(const void* q, long long q_stride, const v
   AnyAttnParams p{q, q_stride, k_pool, v_pool, static_cast<const int*>(block_tables), static_cast<const int*>(cu_q),
                   static_cast<const int*>(context_lens), static_cast<const float*>(sinks), static_cast<const float*>(r1),
                   static_cast<const float*>(r2), gate, gate_stride, out, num_seqs, Hq, Hkv, Dk / maps, Dv, ldk, ldv,
-                  block_size, max_blocks, window, chunk, scale, softcap, maps, lambda, gain, eps};
+                  block_size, max_blocks, window, chunk, scale, softcap, maps, lambda, gain, eps, out_stride, k_mean, v_mean,
+                  mean_of, mean_of > 0 ? (block_size + mean_of - 1) / mean_of : 0};
   auto st = static_cast<cudaStream_t>(stream);
   return fp32 ? launch_attention_any<float>(p, rows, st) : launch_attention_any<__nv_bfloat16>(p, rows, st);
 }

@@ -183,6 +183,8 @@ class Engine:
                                  "(their window layers already drop old blocks)")
             if getattr(self, "pipeline", None):
                 raise ValueError("context shift is not available under pipeline parallelism")
+            if cfg.kv_means():
+                raise ValueError("context shift is not available for models with block means (their blocks are counted from the start)")
             cap = e.max_model_len - e.block_size
             e.max_kv_size = min(e.max_kv_size, cap) if e.max_kv_size > 0 else cap
             if e.max_kv_size < 4 * e.block_size + e.n_keep:

@@ -13,6 +13,7 @@ import torch
 from .config import ModelConfig, preset
 from .engine import Engine, EngineConfig, SamplingParams, Sequence
 from .models.decoder import DecoderModel
+from .models.designs import DESIGNS, design_fn
 from .models.weights import ModelWeights, random_weights
 
 
@@ -28,14 +29,13 @@ class LLM:
         if model is not None:
             self.model = model
         elif cfg.model_type in ("mamba", "mamba2", "nemotron_h", "granitemoehybrid", "jamba", "qwen3_next", "qwen3_5", "qwen3_5_text",
-                                "qwen3_5_moe", "qwen3_5_moe_text", "falcon_h1", "lfm2", "lfm2_moe", "recurrent_gemma", "pamasun", "govopel",
-                                "vavadra"):
+                                "qwen3_5_moe", "qwen3_5_moe_text", "falcon_h1", "lfm2", "lfm2_moe", "recurrent_gemma", *DESIGNS):
             from .models.hybrid import HybridModel
             from .models.mamba1 import Mamba1Model
             from .models.mamba2 import Mamba2Model
             cls = {"mamba": Mamba1Model, "mamba2": Mamba2Model}.get(cfg.model_type, HybridModel)
             ec = engine_config or EngineConfig()
-            kw = dict(kv_bits=ec.kv_bits) if cfg.model_type in ("pamasun", "govopel", "vavadra") else {}
+            kw = dict(kv_bits=ec.kv_bits) if cfg.model_type in DESIGNS else {}
             self.model = cls(cfg, weights, comm=comm, max_seqs=ec.state_slots or 2 * ec.max_batch, **kw)
         else:
             self.model = DecoderModel(cfg, weights, comm=comm,
@@ -60,15 +60,9 @@ class LLM:
         if cfg.model_type == "nemotron_h":
             from .models.hybrid import random_hybrid_weights
             return LLM(cfg, random_hybrid_weights(cfg, seed=seed, dtype=dtype, device=device), engine_config, comm=comm)
-        if cfg.model_type == "pamasun":
-            from .models.pamasun import random_pamasun_weights
-            return LLM(cfg, random_pamasun_weights(cfg, seed=seed, dtype=dtype, device=device), engine_config, comm=comm)
-        if cfg.model_type == "govopel":
-            from .models.govopel import random_govopel_weights
-            return LLM(cfg, random_govopel_weights(cfg, seed=seed, dtype=dtype, device=device), engine_config, comm=comm)
-        if cfg.model_type == "vavadra":
-            from .models.vavadra import random_vavadra_weights
-            return LLM(cfg, random_vavadra_weights(cfg, seed=seed, dtype=dtype, device=device), engine_config, comm=comm)
+        if cfg.model_type in DESIGNS:
+            weights = design_fn(cfg.model_type, "random_{}_weights")(cfg, seed=seed, dtype=dtype, device=device)
+            return LLM(cfg, weights, engine_config, comm=comm)
         tp = comm.tp_size if comm is not None else 1
         rank = comm.tp_rank if comm is not None else 0
         hook = None
@@ -98,18 +92,9 @@ class LLM:
         from .tokenizer import load_tokenizer
 
         cfg = ModelConfig.from_path(path, config_overrides)
-        if cfg.model_type == "pamasun":
-            from .models.pamasun import load_pamasun_weights
-            return LLM(cfg, load_pamasun_weights(path, cfg, dtype=dtype or torch.bfloat16, device=device), engine_config,
-                       comm=comm, tokenizer=load_tokenizer(path))
-        if cfg.model_type == "govopel":
-            from .models.govopel import load_govopel_weights
-            return LLM(cfg, load_govopel_weights(path, cfg, dtype=dtype or torch.bfloat16, device=device), engine_config,
-                       comm=comm, tokenizer=load_tokenizer(path))
-        if cfg.model_type == "vavadra":
-            from .models.vavadra import load_vavadra_weights
-            return LLM(cfg, load_vavadra_weights(path, cfg, dtype=dtype or torch.bfloat16, device=device), engine_config,
-                       comm=comm, tokenizer=load_tokenizer(path))
+        if cfg.model_type in DESIGNS:
+            weights = design_fn(cfg.model_type, "load_{}_weights")(path, cfg, dtype=dtype or torch.bfloat16, device=device)
+            return LLM(cfg, weights, engine_config, comm=comm, tokenizer=load_tokenizer(path))
         if dtype not in (None, torch.bfloat16):
             raise ValueError(f"{cfg.model_type} models are served in bf16")
         if cfg.model_type == "mamba2":

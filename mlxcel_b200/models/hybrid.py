@@ -18,10 +18,12 @@ A second layout ("stream") serves designs that keep the residual in fp32 and nor
 both sides, behind it or in front of it only: ``h <- h + layer_scale * norm(branch(norm(h)))``, the inner norm left out
 where a block's ``norm`` is None, the outer one where its ``post_norm`` is. Its mixers are ``attention_mixer``
 (``models/attention_mixer.py``), ``latent_mixer`` (``models/latent_mixer.py``), ``general_delta``
-(``models/general_delta.py``) and ``gated_delta`` (``models/gated_delta.py``), its feed-forwards ``mlp`` and ``moe_stream``
-(``models/moe.py``), and ``HybridWeights.runs`` lists the layers in execution order: a layer may run several times
+(``models/general_delta.py``), ``gated_delta`` (``models/gated_delta.py``) and ``parallel_mixer`` (attention and retention side by
+side, ``models/parallel_mixer.py``), its feed-forwards ``mlp`` and ``moe_stream`` (``models/moe.py``), and ``HybridWeights.runs`` lists the layers in execution order: a layer may run several times
 with the same weights, each run with a KV-pool layer or state slab of its own; ``run_entries`` adds a vector, and the
-embedding once more, in front of a run (Pamasun, Govopel, Vavadra).
+embedding once more, in front of a run (Pamasun, Govopel, Vavadra). With ``HybridWeights.streams`` there are several residual
+streams instead of one, mixed around every sub-layer as its block's ``around`` says, with layer norms and a short convolution
+in front (``ops/streams.py``; Fusolix).
 
 Nemotron-H gives one block per layer through ``hybrid_override_pattern`` (``"M-M-M*-..."``); the other
 families have a mixer block and an MLP / MoE block per layer. Reference: src/models/nemotron_h.rs,
@@ -67,6 +69,8 @@ class HybridBlock:
     act_coef: torch.Tensor | None = None        # polynomial-norm activation (a, b, c, e)
     act_alpha: float = 1.702                    # clipped gated activation: slope of the gate's sigmoid, clip
     act_limit: float = 7.0
+    parallel: object | None = None              # ParallelMixerWeights
+    around: object | None = None                # several streams: ops.streams.Sublayer (norm is None then)
 
 
 @dataclass
@@ -79,6 +83,8 @@ class HybridWeights:
     runs: list | None = None                    # stream layout: the layers (lists of blocks) in execution order
     embed_norm: torch.Tensor | None = None      # stream layout: norm of the embedding itself
     run_entries: dict = field(default_factory=dict)   # stream layout: run index -> (add the embedding, fp32 vector to add) ahead of it
+    streams: int = 0                            # stream layout: residual streams (0: one, without ``around``)
+    final_norm_b: torch.Tensor | None = None    # several streams: bias of the final layer norm
 
 
 _KINDS = {"M": "mamba2", "m": "mamba1", "L": "gdn", "C": "shortconv", "R": "rglru", "P": "parallel", "*": "attention", "A": "attention", "-": "mlp", "G": "mlp",
@@ -687,20 +693,26 @@ class HybridModel:
     def _init_stream(self, max_seqs: int, kv_bits: int) -> None:
         from .gated_delta import GatedDeltaModel
         from .general_delta import GeneralDeltaModel
+        from .retention import RetentionModel
         cfg, w = self.cfg, self.w
         if kv_bits != 16:
             raise ValueError("this model keeps its KV unquantized (kv_bits must be 16)")
         self.dtype = w.embed.dtype
         # (block, index of its KV layer or state slab, run index behind its last block or -1)
         self.order: list = []
-        # KV splits of decode depend on (key heads, tokens a query sees at most or 0)
+        # KV splits of decode depend on (key heads, tokens a query sees at most or 0, tokens of a block mean or 0)
         delta, n_kv, self._kv_spans, self._latent_spans = [], 0, set(), set()
         for r, blocks in enumerate(w.runs):
             for blk in blocks:
                 idx = -1
                 if blk.kind == "attention_mixer":
                     idx, n_kv = n_kv, n_kv + 1
-                    self._kv_spans.add((blk.attn.kv_heads, blk.attn.window or blk.attn.chunk))
+                    self._kv_spans.add((blk.attn.kv_heads, blk.attn.window or blk.attn.chunk, blk.attn.means))
+                elif blk.kind == "parallel_mixer":
+                    a = blk.parallel.attn
+                    idx, n_kv = (n_kv, len(delta)), n_kv + 1
+                    self._kv_spans.add((a.kv_heads, a.window or a.chunk, a.means))
+                    delta.append(blk)
                 elif blk.kind == "latent_mixer":
                     idx, n_kv = n_kv, n_kv + 1
                     self._latent_spans.add((blk.attn.heads, blk.attn.window))
@@ -714,8 +726,15 @@ class HybridModel:
         self.num_kv_layers = n_kv
         self.Hq, self.Hkv, self.D = cfg.num_attention_heads, cfg.num_key_value_heads, cfg.head_dim
         # only the delta mixers carry state: a stack without them is served like any attention model
-        cls = GatedDeltaModel if kinds == {"gated_delta"} else GeneralDeltaModel
-        self.ssm = cls([blk.mamba for blk in delta], cfg.rms_norm_eps, self.device, max_seqs, self.comm) if delta else None
+        if w.streams:
+            # (the convolutions in front of the sub-layers keep their state in the same slots)
+            if kinds - {"parallel_mixer"}:
+                raise ValueError(f"no recurrent mixer with several streams but retention, not {sorted(kinds)}")
+            convs = [(blk.around.taps.shape[0], cfg.hidden_size) for blk, _, _ in self.order]
+            self.ssm = RetentionModel([blk.parallel.ret for blk in delta], convs, cfg.rms_norm_eps, self.device, max_seqs, self.comm)
+        else:
+            cls = GatedDeltaModel if kinds == {"gated_delta"} else GeneralDeltaModel
+            self.ssm = cls([blk.mamba for blk in delta], cfg.rms_norm_eps, self.device, max_seqs, self.comm) if delta else None
         self.recurrent = self.ssm is not None
         self.state_slots_on_device = self.recurrent
 
@@ -725,7 +744,7 @@ class HybridModel:
             return (ops.decode_splits(rows, self.Hkv, max_len),)
         from ..ops.latent import latent_splits
         from ..ops.stream import visible
-        return tuple(ops.decode_splits(rows, h, visible(max_len, n)) for h, n in sorted(self._kv_spans)) + \
+        return tuple(ops.decode_splits(rows, h, visible(max_len, n, m)) for h, n, m in sorted(self._kv_spans)) + \
             tuple(latent_splits(rows, h, visible(max_len, n)) for h, n in sorted(self._latent_spans))
 
     def state_slot(self, seq_id: int) -> int:
@@ -735,17 +754,39 @@ class HybridModel:
         if self.ssm is not None:
             self.ssm.release_seq(seq_id)
 
-    def _forward_stream(self, b: StepBatch, kv_layers) -> torch.Tensor:
-        """Layer runs of the stream layout. Returns the fp32 residual stream [T, H] (before the final norm)."""
+    def _branch(self, blk: HybridBlock, idx, x: torch.Tensor, b: StepBatch, kv_layers, pieces):
+        """One sub-layer of the stream layout: (its result, None) or (None, the rows of a token's experts)."""
         from ..ops import stream
         from .attention_mixer import attention_mixer
         from .latent_mixer import latent_mixer
         from .moe import moe_stream
+        from .parallel_mixer import parallel_mixer
+        eps = self.cfg.rms_norm_eps
+        if blk.kind == "attention_mixer":
+            return ops.linear(attention_mixer(blk.attn, x, b, kv_layers[idx], eps), blk.attn.out_proj), None
+        if blk.kind == "latent_mixer":
+            return ops.linear(latent_mixer(blk.attn, x, b, kv_layers[idx], eps), blk.attn.out_proj), None
+        if blk.kind in ("general_delta", "gated_delta"):
+            return ops.linear(self.ssm.mixer(idx, blk.mamba, x, pieces), blk.mamba.out_proj), None
+        if blk.kind == "parallel_mixer":
+            return parallel_mixer(blk.parallel, self.ssm, idx[1], x, b, kv_layers[idx[0]], pieces, eps), None
+        if blk.kind == "moe_stream":
+            return None, moe_stream(blk.moe, x)
+        if blk.act == "polynorm":
+            return ops.linear(stream.polynorm(ops.linear(x, blk.up), blk.act_coef, eps), blk.down), None
+        a = ops.glu_linear(x, blk.up, blk.up.shape[0] // 2, blk.act, alpha=blk.act_alpha, limit=blk.act_limit)
+        return ops.linear(a, blk.down), None
+
+    def _forward_stream(self, b: StepBatch, kv_layers) -> torch.Tensor:
+        """Layer runs of the stream layout. Returns the fp32 residual stream [T, H] (before the final norm)."""
+        from ..ops import stream
         cfg, eps, wb = self.cfg, self.cfg.rms_norm_eps, self.cfg.norm_weight_bias
         if b.embeds is not None:
             raise NotImplementedError("media embeddings with an fp32 residual stream")
         pieces = self.ssm.pieces(b) if self.ssm is not None else None
         self.captured = []
+        if self.w.streams:
+            return self._forward_streams(b, kv_layers, pieces)
         entries = {r: stream.Entry(vec, b.token_ids if again else None, self.w.embed, cfg.embed_scale)
                    for r, (again, vec) in self.w.run_entries.items()}
         first = entries.get(0)
@@ -753,19 +794,7 @@ class HybridModel:
                                    self.order[0][0].norm if self.order else self.w.final_norm, eps, wb, self.w.embed_norm,
                                    vec=None if first is None else first.vec)
         for n, (blk, idx, run) in enumerate(self.order):
-            rows = None
-            if blk.kind == "attention_mixer":
-                y = ops.linear(attention_mixer(blk.attn, x, b, kv_layers[idx], eps), blk.attn.out_proj)
-            elif blk.kind == "latent_mixer":
-                y = ops.linear(latent_mixer(blk.attn, x, b, kv_layers[idx], eps), blk.attn.out_proj)
-            elif blk.kind in ("general_delta", "gated_delta"):
-                y = ops.linear(self.ssm.mixer(idx, blk.mamba, x, pieces), blk.mamba.out_proj)
-            elif blk.kind == "moe_stream":
-                y, rows = None, moe_stream(blk.moe, x)
-            elif blk.act == "polynorm":
-                y = ops.linear(stream.polynorm(ops.linear(x, blk.up), blk.act_coef, eps), blk.down)
-            else:
-                y = ops.linear(ops.glu_linear(x, blk.up, blk.up.shape[0] // 2, blk.act, alpha=blk.act_alpha, limit=blk.act_limit), blk.down)
+            y, rows = self._branch(blk, idx, x, b, kv_layers, pieces)
             last = n + 1 == len(self.order)
             nxt = None if last else self.order[n + 1][0].norm
             entry = entries.get(run + 1) if run >= 0 and not last else None
@@ -775,6 +804,23 @@ class HybridModel:
                 y = rows = None
             x = stream.stream_norm(h, y, blk.post_norm, blk.layer_scale, nxt, eps, wb, dtype=self.dtype, plain=not last, moe=rows,
                                    entry=entry)
+        return h
+
+    def _forward_streams(self, b: StepBatch, kv_layers, pieces) -> torch.Tensor:
+        """The same with several residual streams. Returns their sum behind the last layer."""
+        from ..ops import streams
+        eps, order, tail = self.cfg.rms_norm_eps, self.order, self.ssm.tail
+        if not order:
+            raise ValueError("several residual streams need a layer")
+        xs, x = streams.embed_streams(b.token_ids, self.w.embed, self.cfg.embed_scale, self.w.streams, order[0][0].around, eps, tail[0], pieces)
+        for n, (blk, idx, run) in enumerate(order):
+            y, rows = self._branch(blk, idx, x, b, kv_layers, pieces)
+            if n + 1 == len(order):
+                h = streams.sum_streams(xs, blk.around, y, rows, self.dtype)
+            else:
+                x = streams.mix_streams(xs, blk.around, y, rows, order[n + 1][0].around, eps, self.dtype, tail[n + 1], pieces)
+            if run in self.capture_layers:
+                self.captured.append(h.clone() if n + 1 == len(order) else xs.sum(1))
         return h
 
     @torch.inference_mode()
@@ -839,9 +885,13 @@ class HybridModel:
 
     def logits(self, h: torch.Tensor, rows: torch.Tensor | None) -> torch.Tensor:
         if self.w.runs is not None:
-            from ..ops import stream
-            x = stream.stream_norm(h, None, None, None, self.w.final_norm, self.cfg.rms_norm_eps, self.cfg.norm_weight_bias,
-                                   dtype=self.dtype, rows=None if rows is None else rows.to(torch.int32))
+            from ..ops import stream, streams
+            rows = None if rows is None else rows.to(torch.int32)
+            if self.w.streams:
+                x = streams.layer_norm(h, self.w.final_norm, self.w.final_norm_b, self.cfg.rms_norm_eps, self.dtype, rows)
+            else:
+                x = stream.stream_norm(h, None, None, None, self.w.final_norm, self.cfg.rms_norm_eps, self.cfg.norm_weight_bias,
+                                       dtype=self.dtype, rows=rows)
             lg = ops.linear(x, self.w.lm_head, out_fp32=True)
             cap = self.cfg.final_logit_softcap
             return lg if cap <= 0 else stream.softcap_(lg, cap)

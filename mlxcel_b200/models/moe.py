@@ -100,11 +100,12 @@ def moe_forward(cfg, lw: LayerWeights, x: torch.Tensor, h: torch.Tensor, comm) -
 # ----------------------------------------------------------------------------- stream layout
 @dataclass
 class MoeBlockWeights:
-    """Mixture of clipped-GLU experts of the stream layout: softmax scores over all experts, chosen by score + correction,
-    weighted by score * scale. Experts from ``len(gate_up)`` on are identity experts; the shared expert is optional."""
+    """Mixture of gated experts of the stream layout: softmax scores over all experts, chosen by score + correction (in the
+    best groups of experts only, where there are groups), weighted by score * scale, the scores optionally divided by their
+    sum. Experts from ``len(gate_up)`` on are identity experts; the shared expert is optional."""
 
     router: torch.Tensor                      # [experts + identity experts, H]
-    correction: torch.Tensor                  # fp32, per expert
+    correction: torch.Tensor | None           # fp32, per expert
     gate_up: torch.Tensor                     # [experts, 2 * ff, H], gate rows first
     down: torch.Tensor                        # [experts, H, ff]
     top: int
@@ -114,13 +115,16 @@ class MoeBlockWeights:
     shared_gate_up: torch.Tensor | None = None
     shared_down: torch.Tensor | None = None
     shared_limit: float = 0.0
+    act: str = "clipped_swiglu"
+    groups: tuple = (1, 1)                    # (groups of neighbouring experts, how many of them can be chosen from)
+    normalise: bool = False
 
 
 def moe_stream(w: MoeBlockWeights, x: torch.Tensor) -> moe_ops.MoeRows:
     """x [T, H] normalised input. Returns the chosen experts' rows for the step of the stream that sums them up."""
-    ids, wts = moe_ops.route_choice(ops.linear(x, w.router, out_fp32=True), w.correction, w.top, w.scale)
-    rows = moe_ops.expert_rows(x, ids, wts, w.gate_up, w.down, w.alpha, w.limit)
+    ids, wts = moe_ops.route_choice(ops.linear(x, w.router, out_fp32=True), w.correction, w.top, w.scale, w.groups, w.normalise)
+    rows = moe_ops.expert_rows(x, ids, wts, w.gate_up, w.down, w.alpha, w.limit, act=w.act)
     if w.shared_gate_up is not None:
-        a = ops.glu_linear(x, w.shared_gate_up, w.shared_gate_up.shape[0] // 2, "clipped_swiglu", alpha=w.alpha, limit=w.shared_limit)
+        a = ops.glu_linear(x, w.shared_gate_up, w.shared_gate_up.shape[0] // 2, w.act, alpha=w.alpha, limit=w.shared_limit)
         rows.shared = ops.linear(a, w.shared_down)
     return rows

@@ -21,7 +21,9 @@ _ACT_TO_EPI = {"silu": EPI_SWIGLU, "gelu_tanh": EPI_GEGLU, "clipped_swiglu": EPI
 
 @dataclass
 class KVLayer:
-    """One layer's slice of the paged KV pool: ``[num_blocks, Hkv, block_size, D]``."""
+    """One layer's slice of the paged KV pool: ``[num_blocks, Hkv, block_size, D]``. Layers with block means also keep the
+    mean key and value of every full run of ``mean_of`` tokens, ``[num_blocks, Hkv, ceil(block_size / mean_of), D]``: a page holds
+    the means of the runs that end in it, so it can be shared and copied like its tokens."""
 
     k: torch.Tensor
     v: torch.Tensor
@@ -29,6 +31,9 @@ class KVLayer:
     v_meta: torch.Tensor | None
     block_size: int
     kv_bits: int = 16
+    k_mean: torch.Tensor | None = None
+    v_mean: torch.Tensor | None = None
+    mean_of: int = 0
 
 
 def _lib_call(name: str, *args) -> None:

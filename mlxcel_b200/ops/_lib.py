@@ -108,7 +108,7 @@ def _declare(lib) -> None:
         "mx_dequantize": [_vp, _vp, _vp, _vp, _ll, _i, _i, _i, _i, _vp],
         "mx_moe_route": [_vp, _vp, _vp, _i, _i, _i, _i, _i, _vp],
         "mx_moe_align": [_vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _vp],
-        "mx_moe_route_choice": [_vp, _ll, _vp, _vp, _vp, _i, _i, _i, _f, _vp],
+        "mx_moe_route_choice": [_vp, _ll, _vp, _vp, _vp, _i, _i, _i, _f, _i, _i, _f, _vp],
         "mx_moe_align_inv": [_vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _vp],
         "mx_grouped_gemm_any": [_vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _ll, _i, _vp],
         "mx_moe_gather_rows_n": [_vp, _vp, _vp, _vp, _i, _i, _vp],

@@ -119,8 +119,8 @@ def latent_attention(q, kv, tables, lens, cu, out, *, H: int, C: int, scale: flo
     if cu is None:
         cu = torch.arange(rows + 1, dtype=torch.int32, device=q.device)
     _call("mx_paged_attention_any", q.data_ptr(), q.stride(0), kv.k.data_ptr(), kv.k.data_ptr(), tables.data_ptr(), cu.data_ptr(),
-          lens.data_ptr(), _lib.ptr(sinks), None, None, None, 0, out.data_ptr(), lens.shape[0], rows, H, 1, W, C, W, W, kv.block_size,
-          tables.shape[1], window, 0, float(scale), 0.0, 1, 0.0, 1.0, 0.0, _fp32(q), _lib.stream())
+          lens.data_ptr(), _lib.ptr(sinks), None, None, None, 0, out.data_ptr(), out.stride(0), lens.shape[0], rows, H, 1, W, C, W, W,
+          kv.block_size, tables.shape[1], window, 0, float(scale), 0.0, 1, 0.0, 1.0, 0.0, None, None, 0, _fp32(q), _lib.stream())
 
 
 def latent_gather(kv, tables, bounds, rows: int, zero=None):

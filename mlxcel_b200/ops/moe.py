@@ -287,6 +287,9 @@ def moe_experts_rows(x: torch.Tensor, ids_c: torch.Tensor, row_map: torch.Tensor
 
 
 # ----------------------------------------------------------------------------- stream layout
+NORM_EPS = 1e-20                          # added to the sum of the chosen scores before they are divided by it
+
+
 @dataclass
 class MoeRows:
     """What a token's chosen experts returned, before they are summed: pair (t, s) went to expert ``ids[t, s]`` with weight
@@ -310,31 +313,41 @@ class MoeRows:
         return out if self.shared is None else out + self.shared.float()
 
 
-def route_choice_ref(logits, correction, k: int, scale: float):
+def route_choice_ref(logits, correction, k: int, scale: float, groups=(1, 1), normalise: bool = False):
     p = torch.softmax(logits.float(), -1)
-    ids = (p if correction is None else p + correction).topk(k, -1)[1]
-    return ids.to(torch.int32).contiguous(), (p.gather(1, ids) * scale).contiguous()
+    c, (count, keep) = p if correction is None else p + correction, groups
+    if count > keep:
+        best = c.view(c.shape[0], count, -1).amax(-1).topk(keep, -1)[1]
+        kept = torch.zeros(c.shape[0], count, dtype=torch.bool, device=c.device).scatter_(1, best, True)
+        c = c.masked_fill(~kept.repeat_interleave(c.shape[1] // count, 1), float("-inf"))
+    ids = c.topk(k, -1)[1]
+    w = p.gather(1, ids)
+    w = w / (w.sum(-1, keepdim=True) + NORM_EPS) if normalise else w
+    return ids.to(torch.int32).contiguous(), (w * scale).contiguous()
 
 
-def route_choice(logits: torch.Tensor, correction: torch.Tensor | None, k: int, scale: float):
+def route_choice(logits: torch.Tensor, correction: torch.Tensor | None, k: int, scale: float, groups: tuple[int, int] = (1, 1),
+                 normalise: bool = False):
     """Router logits [T, E] fp32 -> (ids [T, k] int32, weights [T, k] fp32): the k experts with the largest softmax score plus
-    ``correction`` (fp32 [E]), weighted by the score itself times ``scale``, not renormalised."""
+    ``correction`` (fp32 [E]), weighted by the score itself times ``scale``. ``groups = (count, keep)``: the experts form ``count``
+    groups of neighbours, and only those of the ``keep`` groups with the largest best member can be chosen. ``normalise``: the
+    chosen scores are divided by their sum first."""
     T, E = logits.shape
     if not logits.is_cuda or E > 512 or k > 16:
-        return route_choice_ref(logits, correction, k, scale)
-    assert logits.dtype == torch.float32 and logits.stride(1) == 1
+        return route_choice_ref(logits, correction, k, scale, groups, normalise)
+    assert logits.dtype == torch.float32 and logits.stride(1) == 1 and E % groups[0] == 0
     ids = torch.empty(T, k, dtype=torch.int32, device=logits.device)
     wts = torch.empty(T, k, dtype=torch.float32, device=logits.device)
     rc = _lib.load().mx_moe_route_choice(logits.data_ptr(), logits.stride(0), _lib.ptr(correction), ids.data_ptr(), wts.data_ptr(), T, E,
-                                         k, float(scale), _lib.stream())
+                                         k, float(scale), *groups, NORM_EPS if normalise else -1.0, _lib.stream())
     _lib.count_launch()
     _lib.check(rc, "mx_moe_route_choice")
     return ids, wts
 
 
 def expert_rows(x: torch.Tensor, ids: torch.Tensor, wts: torch.Tensor, w_gate_up: torch.Tensor, w_down: torch.Tensor, alpha: float,
-                limit: float, force_any: bool = False) -> MoeRows:
-    """The chosen experts' clipped-GLU rows of every token, unsummed. ``w_gate_up`` [E, 2 I, H] (gate rows first), ``w_down``
+                limit: float, force_any: bool = False, act: str = "clipped_swiglu") -> MoeRows:
+    """The chosen experts' gated rows (clipped GLU, or ``act``) of every token, unsummed. ``w_gate_up`` [E, 2 I, H] (gate rows first), ``w_down``
     [E, H, I]; ids from E on are identity experts and cost nothing here. bf16 rows of widths TMA can address run the
     grouped tcgen05 GEMMs, the rest the SIMT ones."""
     T, k = ids.shape
@@ -344,7 +357,7 @@ def expert_rows(x: torch.Tensor, ids: torch.Tensor, wts: torch.Tensor, w_gate_up
         for e in range(E):
             tok, slot = torch.nonzero(ids == e, as_tuple=True)
             inv[tok * k + slot] = torch.arange(tok.numel(), dtype=torch.int32) + sum(r.shape[0] for r in y)
-            a = ref.glu_linear(x[tok], w_gate_up[e], I, ref.EPI_CLIPPED_SWIGLU, None, alpha, limit)
+            a = ref.glu_linear(x[tok], w_gate_up[e], I, _ACT_TO_EPI[act], None, alpha, limit)
             y.append(ref.linear(a, w_down[e]))
         return MoeRows(torch.cat(y), x, ids, inv, wts, E)
     lib, st, dev, pairs = _lib.load(), _lib.stream(), x.device, T * k
@@ -361,7 +374,7 @@ def expert_rows(x: torch.Tensor, ids: torch.Tensor, wts: torch.Tensor, w_gate_up
         _lib.check(lib.mx_moe_gather_rows_n(x.data_ptr(), token.data_ptr(), offsets[E:].data_ptr(), xs.data_ptr(), pairs, H, st),
                    "mx_moe_gather_rows_n")
         _lib.count_launch()
-        a = grouped_linear(xs, w_gate_up, offsets, I, None, "clipped_swiglu", alpha, limit)
+        a = grouped_linear(xs, w_gate_up, offsets, I, None, act, alpha, limit)
         return MoeRows(grouped_linear(a, w_down, offsets, H), x, ids, inv, wts, E)
 
     def grouped(rows, w, row_map):
@@ -373,7 +386,7 @@ def expert_rows(x: torch.Tensor, ids: torch.Tensor, wts: torch.Tensor, w_gate_up
         return out
     z = grouped(x, w_gate_up, token)
     a = torch.empty(pairs, I, dtype=x.dtype, device=dev)
-    _lib.check(lib.mx_glu_rows(z.data_ptr(), z.stride(0), a.data_ptr(), pairs, I, ref.EPI_CLIPPED_SWIGLU, float(alpha), float(limit),
+    _lib.check(lib.mx_glu_rows(z.data_ptr(), z.stride(0), a.data_ptr(), pairs, I, _ACT_TO_EPI[act], float(alpha), float(limit),
                                1 if x.dtype == torch.float32 else 0, st), "mx_glu_rows")
     _lib.count_launch()
     return MoeRows(grouped(a, w_down, None), x, ids, inv, wts, E)

@@ -25,9 +25,10 @@ _SIG = {
     "mx_softcap_rows": [_vp, _ll, _f, _vp],
     "mx_rope_norm_append": [_vp, _ll, _vp, _vp, _vp, _f] + [_vp] * 4 + [_i] * 9 + [_f, _i, _vp],
     "mx_qk_norm_append": [_vp, _ll, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _f, _i, _vp],
-    "mx_paged_attention_any": [_vp, _ll] + [_vp] * 9 + [_ll, _vp] + [_i] * 12 + [_f, _f, _i, _f, _f, _f, _i, _vp],
-    "mx_paged_decode_ext": [_vp, _ll] + [_vp] * 8 + [_ll, _vp, _vp] + [_i] * 9 + [_f, _f, _i, _f, _f, _f, _i, _vp],
-    "mx_paged_prefill_ext": [_vp, _ll, _vp, _vp, _ll] + [_vp] * 7 + [_ll, _vp] + [_i] * 11 + [_f, _f, _i, _f, _f, _f, _vp, _vp],
+    "mx_paged_attention_any": [_vp, _ll] + [_vp] * 9 + [_ll, _vp, _ll] + [_i] * 12 + [_f, _f, _i, _f, _f, _f, _vp, _vp, _i, _i, _vp],
+    "mx_paged_decode_ext": [_vp, _ll] + [_vp] * 8 + [_ll, _vp, _ll, _vp] + [_i] * 9 + [_f, _f, _i, _f, _f, _f, _vp, _vp, _i, _i, _vp],
+    "mx_paged_prefill_ext": [_vp, _ll, _vp, _vp, _ll] + [_vp] * 7 + [_ll, _vp, _ll] + [_i] * 11 + [_f, _f, _i, _f, _f, _f, _vp, _vp, _vp, _i, _i,
+                                                                                                    _vp, _vp],
     "mx_delta_rule": [_vp, _ll] + [_vp] * 11 + [_i] * 6 + [_f, _f, _f, _i, _i, _vp],
 }
 NOT_COVERED = -10        # a tensor-core kernel refuses the geometry: the shape-agnostic one takes it
@@ -52,9 +53,12 @@ def _fp32(t: torch.Tensor) -> int:
     return 1 if t.dtype == torch.float32 else 0
 
 
-def visible(max_len: int, span: int) -> int:
-    """Tokens a query sees at most: a window or chunk of ``span`` (0: all) of ``max_len``."""
-    return min(max_len, span) if span > 0 else max_len
+def visible(max_len: int, span: int, means: int = 0) -> int:
+    """Keys a query sees at most: a window or chunk of ``span`` tokens (0: all) of ``max_len`` and, with ``means``, one for every
+    block of so many tokens before the window."""
+    if span <= 0:
+        return max_len
+    return min(max_len, span) + (max(0, max_len - span) // means if means else 0)
 
 
 def _rms(x: torch.Tensor, eps: float) -> torch.Tensor:
@@ -245,7 +249,7 @@ def qk_norm_append(qkv, slots, kv, *, Hq: int, Hkv: int, Dk: int, Dv: int, q_nor
 
 
 def paged_attention_ref(q, kv, tables, lens, cu, *, Hq, Hkv, Dk, Dv, scale, window=0, sinks=None, dist_bias=None, gate=None,
-                        softcap=0.0, chunk=0, diff=None):
+                        softcap=0.0, chunk=0, diff=None, means=False, gain=1.0):
     if diff is not None:
         # the maps as two attentions whose queries are zero in the other map's columns
         factor, gain, eps = diff
@@ -275,10 +279,18 @@ def paged_attention_ref(q, kv, tables, lens, cu, *, Hq, Hkv, Dk, Dv, scale, wind
         vis = (d >= 0) & (d < window) if window > 0 else d >= 0
         vis = vis & (kp // chunk == qp // chunk) if chunk > 0 else vis
         sc = sc.masked_fill(~vis, float("-inf"))
+        if means:
+            # blocks of tokens that lie wholly before a query's window, as one key and value each
+            from .block_means import mean_rows_ref
+            nb = max(0, n - window) // kv.mean_of
+            km, vm = mean_rows_ref(kv, tables[s], nb)
+            old = (torch.arange(nb, device=q.device)[None] + 1) * kv.mean_of <= qp - window + 1
+            ms = torch.einsum("hgqd,hkd->hgqk", qs, km) * scale
+            sc, v = torch.cat([sc, ms.masked_fill(~old, float("-inf"))], -1), torch.cat([v, vm], 1)
         if sinks is not None:
             sc = torch.cat([sc, sinks.float().reshape(Hkv, G, 1, 1).expand(Hkv, G, ql, 1)], -1)
-        p = torch.softmax(sc, -1)[..., :n]
-        o = torch.einsum("hgqk,hkd->hgqd", p, v).permute(2, 0, 1, 3).reshape(ql, Hq * Dv)
+        p = torch.softmax(sc, -1)[..., :v.shape[1]]
+        o = gain * torch.einsum("hgqk,hkd->hgqd", p, v).permute(2, 0, 1, 3).reshape(ql, Hq * Dv)
         if gate is not None:
             o = o * torch.sigmoid(gate[q0:q1].float())
         out[q0:q1] = o.to(q.dtype)
@@ -287,7 +299,7 @@ def paged_attention_ref(q, kv, tables, lens, cu, *, Hq, Hkv, Dk, Dv, scale, wind
 
 def paged_attention(q, kv, tables, lens, cu, out, *, Hq: int, Hkv: int, Dk: int, Dv: int, scale: float, max_q_len: int,
                     max_len: int = 0, window: int = 0, sinks=None, dist_bias=None, gate=None, softcap: float = 0.0, chunk: int = 0,
-                    diff: tuple | None = None, force_any: bool = False) -> None:
+                    diff: tuple | None = None, means: tuple | None = None, gain: float = 1.0, force_any: bool = False) -> None:
     """Causal paged attention of the query rows of every sequence (the last ``cu[s+1] - cu[s]`` of its ``lens[s]``
     tokens) into ``out`` [rows, Hq * Dv]. ``cu=None`` says one row per sequence (decode).
 
@@ -296,7 +308,9 @@ def paged_attention(q, kv, tables, lens, cu, out, *, Hq: int, Hkv: int, Dk: int,
     (counted from the sequence's start); ``sinks`` adds ``exp(sink)`` to the denominator; ``gate`` ([rows, Hq * Dv], may be a column slice) multiplies the result by
     its sigmoid; ``diff = (factor, gain, eps)``: differential heads, the Dk columns of a query and key head are two maps of
     Dk / 2 (scores and softmax of their own, the same values) and the result is ``a1 - factor a2`` over its root mean square,
-    times ``gain``. bf16 pools with row widths that are multiples of 8 up to 128 take the tensor-core kernels
+    times ``gain``; ``means`` (with a window): the blocks of ``kv.mean_of`` tokens wholly before a query's window are keys too, by
+    their means; for prompt portions ``(bounds, rows)`` of :func:`block_means.portion_means`, for decode rows any tuple;
+    ``gain`` multiplies the heads. ``out`` may be a column slice. bf16 pools with row widths that are multiples of 8 up to 128 take the tensor-core kernels
     (flash decoding with split KV; tcgen05 prefill); the rest the SIMT one."""
     rows = q.shape[0]
     if rows == 0:
@@ -304,30 +318,39 @@ def paged_attention(q, kv, tables, lens, cu, out, *, Hq: int, Hkv: int, Dk: int,
     if not q.is_cuda:
         c = torch.arange(rows + 1) if cu is None else cu
         out.copy_(paged_attention_ref(q, kv, tables, lens, c, Hq=Hq, Hkv=Hkv, Dk=Dk, Dv=Dv, scale=scale, window=window,
-                                      sinks=sinks, dist_bias=dist_bias, gate=gate, softcap=softcap, chunk=chunk, diff=diff))
+                                      sinks=sinks, dist_bias=dist_bias, gate=gate, softcap=softcap, chunk=chunk, diff=diff,
+                                      means=means is not None, gain=gain))
         return
+    assert gain == 1.0 or diff is None
+    assert means is None or (window > 0 and kv.mean_of > 0 and chunk == 0 and dist_bias is None and diff is None), "block means stand beside a window"
     assert diff is None or (Dk % 2 == 0 and sinks is None and dist_bias is None and gate is None), "differential heads: plain scores"
-    maps, (lam, gain, eps) = (1, (0.0, 1.0, 0.0)) if diff is None else (2, diff)
+    maps, (lam, gain, eps) = (1, (0.0, gain, 0.0)) if diff is None else (2, diff)
     dargs = (maps, float(lam), float(gain), float(eps))
     r1, r2 = dist_bias if dist_bias is not None else (None, None)
-    assert kv.k.dtype == q.dtype and q.stride(1) == 1 and out.is_contiguous() and out.dtype == q.dtype
+    assert kv.k.dtype == q.dtype and q.stride(1) == 1 and out.stride(1) == 1 and out.dtype == q.dtype
+    km, vm, P = (kv.k_mean.data_ptr(), kv.v_mean.data_ptr(), kv.mean_of) if means is not None else (None, None, 0)
     assert gate is None or (gate.stride(1) == 1 and gate.dtype == q.dtype)
     gs = gate.stride(0) if gate is not None else 0
     head = (q.data_ptr(), q.stride(0), kv.k.data_ptr(), kv.v.data_ptr())
-    tail = (_lib.ptr(sinks), _lib.ptr(r1), _lib.ptr(r2), _lib.ptr(gate), gs, out.data_ptr())
-    if q.dtype == torch.bfloat16 and not force_any:
+    tail = (_lib.ptr(sinks), _lib.ptr(r1), _lib.ptr(r2), _lib.ptr(gate), gs, out.data_ptr(), out.stride(0))
+    if q.dtype == torch.bfloat16 and not force_any and Dk % 8 == Dv % 8 == 0:
         from . import _decode_scratch, decode_splits
         if cu is None:
-            splits = decode_splits(rows, Hkv, visible(max_len or tables.shape[1] * kv.block_size, window or chunk))
+            splits = decode_splits(rows, Hkv, visible(max_len or tables.shape[1] * kv.block_size, window or chunk, P))
             scratch = _decode_scratch(q.device, int(_lib.load().mx_paged_decode_scratch_floats(rows, maps * Hq, Dv, splits)))
             rc = _fn("mx_paged_decode_ext")(*head, tables.data_ptr(), lens.data_ptr(), *tail, scratch.data_ptr(), rows, Hq,
                                             Hkv, Dk, Dv, kv.block_size, tables.shape[1], window, chunk, float(scale),
-                                            float(softcap), *dargs, splits, _lib.stream())
+                                            float(softcap), *dargs, km, vm, P, splits, _lib.stream())
         else:
+            gathered = (None, None, None, 0)
+            if means is not None and means[1]:
+                from .block_means import gather
+                gk, gv = gather(kv, tables, *means)
+                gathered = (gk.data_ptr(), gv.data_ptr(), means[0].data_ptr(), means[1])
             rc = _fn("mx_paged_prefill_ext")(*head, kv.k.shape[0], tables.data_ptr(), cu.data_ptr(), lens.data_ptr(), *tail,
                                              lens.shape[0], rows, max_q_len, Hq, Hkv, Dk, Dv, kv.block_size, tables.shape[1],
-                                             window, chunk, float(scale), float(softcap), *dargs, _lib.workspace(q.device).data_ptr(),
-                                             _lib.stream())
+                                             window, chunk, float(scale), float(softcap), *dargs, *gathered, P,
+                                             _lib.workspace(q.device).data_ptr(), _lib.stream())
         if rc != NOT_COVERED:
             _lib.count_launch()
             _lib.check(rc, "paged attention")
@@ -335,7 +358,8 @@ def paged_attention(q, kv, tables, lens, cu, out, *, Hq: int, Hkv: int, Dk: int,
     if cu is None:
         cu = torch.arange(rows + 1, dtype=torch.int32, device=q.device)
     _call("mx_paged_attention_any", *head, tables.data_ptr(), cu.data_ptr(), lens.data_ptr(), *tail, lens.shape[0], rows, Hq,
-          Hkv, Dk, Dv, Dk, Dv, kv.block_size, tables.shape[1], window, chunk, float(scale), float(softcap), *dargs, _fp32(q), _lib.stream())
+          Hkv, Dk, Dv, Dk, Dv, kv.block_size, tables.shape[1], window, chunk, float(scale), float(softcap), *dargs, km, vm, P,
+          _fp32(q), _lib.stream())
 
 
 # ----------------------------------------------------------------------------- generalized delta rule

@@ -18,7 +18,6 @@ import os
 import sys
 
 LIVE_REQUESTS = 4
-FP32_MODELS = ("govopel", "pamasun", "vavadra")
 
 
 def build_engine(model_dir: str, dtype: str, max_tokens: int, device: str):
@@ -28,10 +27,11 @@ def build_engine(model_dir: str, dtype: str, max_tokens: int, device: str):
     from .config import ModelConfig
     from .engine import EngineConfig
     from .llm import LLM
+    from .models.designs import DESIGNS
     from .ops import _lib
 
     cfg = ModelConfig.from_path(model_dir)
-    if dtype == "float32" and cfg.model_type not in FP32_MODELS:
+    if dtype == "float32" and cfg.model_type not in DESIGNS:
         raise SystemExit(3)
     _lib.prefer_units(_build.MODEL_UNITS.get(cfg.model_type))
     torch.backends.cuda.matmul.allow_tf32 = False

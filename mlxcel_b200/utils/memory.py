@@ -23,6 +23,16 @@ def _recurrent_block(cfg: ModelConfig, kind: str) -> tuple[int, int]:
     if x.get("layer_specs"):
         # (a repeated layer's weights count once, its state for every run)
         spec = x["layer_specs"][kind]
+        if cfg.model_type == "fusolix":
+            a, r, mlp, S, K = spec["mixer"]["left"], spec["mixer"]["right"], spec["mlp"], x["streams"], x["taps"]
+            par = (h + 1) * (a["heads"] * a["dim"] + a["kv_heads"] * (a["dim"] + a["vdim"])) + h * (a["heads"] * a["vdim"] + 1)
+            par += h * r["heads"] * (2 * r["dim"] + 3 * r["vdim"])
+            around, st = h * (2 + K) + S * (S + 2), 4 * ((K - 1) * h * (2 if mlp else 1) + r["heads"] * r["dim"] * r["vdim"])
+            if mlp and mlp["kind"] == "dense":
+                par += 3 * h * mlp["ff"]
+            elif mlp:
+                par += mlp["router"]["experts"] * h * (1 + 3 * mlp["expert"]["ff"])
+            return par + around * (2 if mlp else 1), st
         m, ff = spec["mixer"], (spec["mlp"] or {}).get("ff", 0)
         if cfg.model_type == "vavadra":
             st, mlp, d, v, n = 0, spec["mlp"], m["dim"], m["vdim"], m["heads"]

@@ -5,11 +5,7 @@ import torch
 from mlxcel_b200.config import ModelConfig
 from mlxcel_b200.engine import EngineConfig
 from mlxcel_b200.llm import LLM
-from mlxcel_b200.models.govopel import build_govopel_weights
-from mlxcel_b200.models.pamasun import build_pamasun_weights
-from mlxcel_b200.models.vavadra import build_vavadra_weights
-
-BUILDERS = {"pamasun": build_pamasun_weights, "govopel": build_govopel_weights, "vavadra": build_vavadra_weights}
+from mlxcel_b200.models.designs import design_fn
 
 
 def llm_for(raw, tensors, device, dtype, **ecfg):
@@ -17,7 +13,7 @@ def llm_for(raw, tensors, device, dtype, **ecfg):
     kw = dict(max_batch=4, max_prefill_seqs=4, state_slots=4, block_size=16, num_blocks=48, max_num_batched_tokens=768,
               max_model_len=768, prefix_cache=False, watermark=0.0)
     kw.update(ecfg)
-    return LLM(cfg, BUILDERS[cfg.model_type](tensors.__getitem__, cfg, dtype, device), EngineConfig(**kw))
+    return LLM(cfg, design_fn(cfg.model_type, "build_{}_weights")(tensors.__getitem__, cfg, dtype, device), EngineConfig(**kw))
 
 
 def tokens_for(raw, n, seed):
