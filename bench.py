@@ -139,7 +139,7 @@ def main() -> None:
     ap.add_argument("--watchdog", type=int, default=1500,
                     help="seconds without finishing a round before every thread's stack is dumped and the "
                          "process exits (a stuck multi-rank run then ends by itself)")
-    ap.add_argument("--design", default=None, choices=["pamasun", "govopel", "vavadra"],
+    ap.add_argument("--design", default=None, choices=["fusolix", "govopel", "pamasun", "vavadra"],
                     help="instead of the serving benchmark: prefill / decode throughput and kernel times of this design "
                          "beside the closest existing model at equal size (one GPU, random weights)")
     args = ap.parse_args()

@@ -36,7 +36,8 @@ NVCC_FLAGS = [
 # Sources a model family needs, for processes that serve one model from a tree without a built library:
 # they compile these alone, into a library of their own (the full one is used where it exists).
 MODEL_UNITS = {
-    "fusolix": ("attention", "attention_tc", "block_means", "gemm", "misc", "moe", "retention", "sampling", "simt", "stream_norm", "streams"),
+    "fusolix": ("attention", "attention_tc", "block_means", "gemm", "misc", "moe", "retention", "retention_tc", "sampling", "simt",
+                "stream_norm", "streams"),
     "govopel": ("attention", "attention_tc", "gemm", "latent", "latent_tc", "misc", "rope_norm", "sampling", "simt", "stream_norm"),
     "pamasun": ("attention", "attention_tc", "delta_rule", "gemm", "misc", "sampling", "simt", "stream_norm"),
     "vavadra": ("attention", "attention_tc", "gated_delta", "gemm", "latent", "latent_tc", "misc", "moe", "sampling", "simt", "stream_norm"),

@@ -6,28 +6,14 @@
 // Kernels:
 //   retention_step   pieces of one token (decode): one CTA per (head, row); rotation, recurrence, norm and gate fused, the state
 //                    streams through registers once
-//   retention_prep / retention_scan / retention_post   longer pieces: rotation of all tokens at once into zero-padded fp32
-//                    rows; the recurrence with the state in registers, two channels per packed fp32 instruction; norm and gate
+//   retention_chunks (retention_tc.cu)   longer pieces, bf16: chunks of 128 tokens on the tensor cores
+//   retention_prep / retention_scan / retention_post   the same for fp32 and other sizes: rotation of all tokens at once into
+//                    zero-padded fp32 rows; the recurrence with the state in registers, two channels per packed fp32
+//                    instruction; norm and gate
 #include "api.h"
-#include "typed.cuh"
+#include "retention.cuh"
 
 namespace mx {
-
-struct RetentionParams {
-  const void* proj;          // rows q [H D] | k [H D] | v [H V] | gate [H V], ld elements apart
-  long long ld;
-  const int* positions;
-  const float* inv_freq;     // [rot / 2]
-  const float* decay;        // [H]
-  float* memory;
-  const int* slots;          // per piece; a negative slot marks a padding row (its output is zero)
-  const int* cu;
-  const int* reset;
-  void* out;                 // rows of H V, ldo elements apart
-  long long ldo;
-  int H, D, V, rot, pieces;
-  float norm_eps, gain;
-};
 
 __device__ __forceinline__ float ret_silu(float x) { return x * sigmoid_f(x); }
 
@@ -117,22 +103,6 @@ __global__ void __launch_bounds__(kRsThreads) retention_step_kernel(const Retent
 }
 
 // ----------------------------------------------------------------------------- longer pieces
-// Scratch of one call over N tokens (rows row0 .. row0 + N - 1), fp32, widths padded with zeros:
-//   q [N, H, DP] | k [N, H, DP] | v [N, H, VP] | o [N, H, VP]
-struct RetentionScratch {
-  float *q, *k, *v, *o;
-};
-__host__ __device__ inline int ret_dp(int D) { return D <= 32 ? 32 : D <= 64 ? 64 : D <= 128 ? 128 : D <= 256 ? 256 : 512; }
-__host__ __device__ inline int ret_vp(int V) { return (V + 31) / 32 * 32; }
-__host__ __device__ inline RetentionScratch ret_scratch(float* s, long long N, int H, int D, int V) {
-  RetentionScratch r;
-  r.q = s;
-  r.k = r.q + N * H * ret_dp(D);
-  r.v = r.k + N * H * ret_dp(D);
-  r.o = r.v + N * H * ret_vp(V);
-  return r;
-}
-
 // One CTA per token: the angles once, then all heads.
 template <typename T>
 __global__ void __launch_bounds__(256) retention_prep_kernel(const RetentionParams p, float* __restrict__ scratch, int row0, int N) {
@@ -299,16 +269,16 @@ __global__ void __launch_bounds__(kRcThreads) retention_scan_kernel(const Retent
     }
 }
 
-// One warp per (token, head): o / rms(o) * silu(gate) * gain.
+// One warp per (token, head): o / rms(o) * silu(gate) * gain. Rows of o are ret_vp(V) wide, zero from V on.
 template <typename T>
-__global__ void __launch_bounds__(256) retention_post_kernel(const RetentionParams p, float* __restrict__ scratch, int row0, int N) {
+__global__ void __launch_bounds__(256) retention_post_kernel(const RetentionParams p, const float* __restrict__ rows_o, int row0, int N) {
   pdl_trigger();
   pdl_wait();
   const int lane = threadIdx.x & 31, V = p.V, VP = ret_vp(V);
   const unsigned gw = blockIdx.x * (blockDim.x / 32) + (threadIdx.x >> 5);
   if (gw >= static_cast<unsigned>(N) * p.H) return;
   const int n = static_cast<int>(gw / p.H), h = static_cast<int>(gw - static_cast<unsigned>(n) * p.H);
-  const float* o = ret_scratch(scratch, N, p.H, p.D, V).o + (static_cast<size_t>(n) * p.H + h) * VP;
+  const float* o = rows_o + (static_cast<size_t>(n) * p.H + h) * VP;
   const T* z = static_cast<const T*>(p.proj) + static_cast<size_t>(row0 + n) * p.ld + 2 * p.H * p.D + p.H * V + h * V;
   T* out = static_cast<T*>(p.out) + static_cast<size_t>(row0 + n) * p.ldo + static_cast<size_t>(h) * V;
   float s = 0.f;
@@ -343,8 +313,14 @@ static int launch_retention_scan(const RetentionParams& p, float* scratch, int p
 }
 
 template <typename T>
-static int retention_typed(RetentionParams p, int pieces, int n_short, int rows, float* scratch, int form, cudaStream_t st) {
-  (void)form;
+static int launch_retention_post(const RetentionParams& p, const float* o, int row0, int N, cudaStream_t st) {
+  const long long warps = static_cast<long long>(N) * p.H;
+  if (warps > 0x7fffffffll) return -1;
+  return static_cast<int>(launch_kernel(retention_post_kernel<T>, dim3(static_cast<unsigned>((warps + 7) / 8)), dim3(256), 0, st, p, o, row0, N));
+}
+
+template <typename T>
+static int retention_typed(RetentionParams p, int pieces, int n_short, int rows, float* scratch, int form, int* status, cudaStream_t st) {
   if (n_short > 0) {
     const bool vec = p.V % 4 == 0 && p.ld % 4 == 0 && 2 * p.H * p.D % 4 == 0 && aligned_to(p.proj, sizeof(T) * 4) && aligned_to(p.memory, 16);
     const int groups = p.V / (vec ? 4 : 1), cols = groups < kRsThreads ? groups : kRsThreads;
@@ -359,6 +335,12 @@ static int retention_typed(RetentionParams p, int pieces, int n_short, int rows,
   if (np <= 0 || N <= 0) return 0;
   if (scratch == nullptr || !aligned_to(scratch, 16)) return -1;
   p.slots += n_short, p.cu += n_short, p.reset += n_short, p.pieces = np;
+  if (sizeof(T) == 2 && form == 0 && ret_chunk_covered(p.D, p.V, p.rot)) {
+    if (!aligned_to(p.proj, 16) || p.ld % 8 || !aligned_to(p.out, 16) || p.ldo % 8) return -1;
+    float* o = p.V > kRetTile ? scratch + static_cast<long long>(N) * p.rot : nullptr;
+    const int rc = launch_retention_chunks(p, scratch, o, np, n_short, N, status, st);
+    return rc || o == nullptr ? rc : launch_retention_post<T>(p, o, n_short, N, st);
+  }
   int rc = static_cast<int>(launch_kernel(retention_prep_kernel<T>, dim3(N), dim3(256), static_cast<size_t>(p.rot) * 4, st, p, scratch, n_short, N));
   if (rc) return rc;
   const int dp = ret_dp(p.D);
@@ -370,26 +352,29 @@ static int retention_typed(RetentionParams p, int pieces, int n_short, int rows,
   else if (dp == 256) rc = launch_retention_scan<32, 2>(p, scratch, np, n_short, N, st);
   else rc = launch_retention_scan<64, 2>(p, scratch, np, n_short, N, st);
   if (rc) return rc;
-  const long long warps = static_cast<long long>(N) * p.H;
-  if (warps > 0x7fffffffll) return -1;
-  return static_cast<int>(launch_kernel(retention_post_kernel<T>, dim3(static_cast<unsigned>((warps + 7) / 8)), dim3(256), 0, st, p, scratch, n_short, N));
+  return launch_retention_post<T>(p, ret_scratch(scratch, N, p.H, p.D, p.V).o, n_short, N, st);
 }
 
 }  // namespace mx
 
 using namespace mx;
 
-extern "C" long long mx_retention_scratch_floats(int tokens, int H, int D, int V, int bf16, int form) {
-  (void)bf16, (void)form;
+extern "C" int mx_retention_chunk_covered(int D, int V, int rot) { return ret_chunk_covered(D, V, rot) ? 1 : 0; }
+
+// form 0: bf16 pieces of covered sizes (mx_retention_chunk_covered) run in chunks; 1: token by token.
+extern "C" long long mx_retention_scratch_floats(int tokens, int H, int D, int V, int rot, int bf16, int form) {
+  if (bf16 && form == 0 && ret_chunk_covered(D, V, rot)) return ret_chunk_floats(tokens, H, V, rot) + 4;
   return static_cast<long long>(tokens) * H * (2ll * ret_dp(D) + 2ll * ret_vp(V));
 }
 
 // A ragged batch of pieces (token rows cu[j] .. cu[j + 1] - 1 of proj, positions and out, state slot slots[j], reset[j] starts from
 // zero). The first n_short pieces hold exactly one token each; rows is the total number of token rows. D at most 512.
-// scratch: mx_retention_scratch_floats(rows - n_short, ...) floats, or NULL when every piece is short.
+// scratch: mx_retention_scratch_floats(rows - n_short, ...) floats, or NULL when every piece is short. The chunked form needs proj and out
+// aligned to 16 bytes with row strides of whole 16-byte groups.
 extern "C" int mx_retention(const void* proj, long long ld, const void* positions, const void* inv_freq, const void* decay, void* memory,
                             const void* slots, const void* cu, const void* reset, void* out, long long ldo, void* scratch, int pieces,
-                            int n_short, int rows, int H, int D, int V, int rot, float norm_eps, float gain, int fp32, int form, void* stream) {
+                            int n_short, int rows, int H, int D, int V, int rot, float norm_eps, float gain, int fp32, int form, void* status,
+                            void* stream) {
   if (pieces <= 0 || rows <= 0) return 0;
   if (H <= 0 || D <= 0 || D > 512 || V <= 0 || rot < 0 || rot > D || rot % 2 || pieces > 65535 || n_short < 0 || n_short > pieces) return -1;
   RetentionParams p{proj, ld, static_cast<const int*>(positions), static_cast<const float*>(inv_freq), static_cast<const float*>(decay),
@@ -397,6 +382,7 @@ extern "C" int mx_retention(const void* proj, long long ld, const void* position
                     H, D, V, rot, pieces, norm_eps, gain};
   auto st = static_cast<cudaStream_t>(stream);
   auto* sc = static_cast<float*>(scratch);
-  return fp32 ? retention_typed<float>(p, pieces, n_short, rows, sc, form, st)
-              : retention_typed<__nv_bfloat16>(p, pieces, n_short, rows, sc, form, st);
+  auto* sw = static_cast<int*>(status);
+  return fp32 ? retention_typed<float>(p, pieces, n_short, rows, sc, form, sw, st)
+              : retention_typed<__nv_bfloat16>(p, pieces, n_short, rows, sc, form, sw, st);
 }

@@ -7,7 +7,7 @@ import torch
 from . import _lib
 from .stream import _call, _f, _fp32, _i, _ll, _rms, _SIG, _vp, rotate_half
 
-_SIG["mx_retention"] = [_vp, _ll] + [_vp] * 8 + [_ll, _vp] + [_i] * 7 + [_f, _f, _i, _i, _vp]
+_SIG["mx_retention"] = [_vp, _ll] + [_vp] * 8 + [_ll, _vp] + [_i] * 7 + [_f, _f, _i, _i, _vp, _vp]
 
 
 def retention_ref(proj, positions, inv_freq, decay, memory, slots, cu, reset, out, norm_eps: float, gain: float):
@@ -37,7 +37,8 @@ def retention(proj, positions, inv_freq, decay, memory, slots, cu, reset, out, *
     dimensions / 2] (dimension i turns with i + dims / 2); ``decay`` fp32 [H]; ``memory`` [slots, H, D, V] fp32 is advanced in
     place; ``slots`` / ``reset`` [pieces], ``cu`` [pieces + 1] int32 (the first ``n_short`` pieces are decode rows of one token; a
     negative slot marks a padding row). The result is the read-out over its root mean square per head, times silu(gate),
-    times ``gain``. ``form`` 1 keeps longer pieces on the token-by-token kernel."""
+    times ``gain``. Longer pieces of bf16 rows with key heads of up to 128 run in chunks on the tensor cores; ``form`` 1 keeps
+    them on the token-by-token kernel, which takes the rest."""
     if proj.shape[0] == 0:
         return
     if not proj.is_cuda:
@@ -48,10 +49,13 @@ def retention(proj, positions, inv_freq, decay, memory, slots, cu, reset, out, *
     lib = _lib.load()
     floats = lib.mx_retention_scratch_floats
     if not floats.argtypes:
-        floats.argtypes, floats.restype = [_i] * 6, _ll
-    bf = 0 if proj.dtype == torch.float32 else 1
-    scratch = torch.empty(int(floats(rows - n_short, H, D, V, bf, form)), dtype=torch.float32, device=proj.device) if pieces > n_short else None
+        floats.argtypes, floats.restype = [_i] * 7, _ll
+    bf, rot = (0 if proj.dtype == torch.float32 else 1), 2 * inv_freq.shape[0]
+    if (proj.data_ptr() | out.data_ptr()) % 16 or proj.stride(0) % 8 or out.stride(0) % 8:
+        form = 1
+    scratch = torch.empty(int(floats(rows - n_short, H, D, V, rot, bf, form)), dtype=torch.float32, device=proj.device) if pieces > n_short else None
     _call("mx_retention", proj.data_ptr(), proj.stride(0), positions.data_ptr(), inv_freq.data_ptr(), decay.data_ptr(), memory.data_ptr(),
           slots.data_ptr(), cu.data_ptr(), reset.data_ptr(), out.data_ptr(), out.stride(0), _lib.ptr(scratch), pieces, n_short, rows, H, D, V,
-          2 * inv_freq.shape[0], float(norm_eps), float(gain), _fp32(proj), form, _lib.stream())
-    _lib.count_launch((1 if n_short and pieces > n_short else 0) + (2 if pieces > n_short else 0))
+          rot, float(norm_eps), float(gain), _fp32(proj), form, _lib.workspace(proj.device).data_ptr(), _lib.stream())
+    chunks = bf and form == 0 and lib.mx_retention_chunk_covered(D, V, rot)
+    _lib.count_launch((1 if n_short and pieces > n_short else 0) + ((1 if chunks and V <= 128 else 2) if pieces > n_short else 0))

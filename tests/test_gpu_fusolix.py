@@ -241,7 +241,7 @@ def _oracle_retention(p, H, D, V, rot, decay, eps, gain):
 
 RETENTION = [  # heads, key width, value width, rotated
     (4, 64, 32, 64), (2, 128, 128, 128), (3, 10, 7, 6), (1, 34, 13, 2), (5, 40, 24, 20), (2, 16, 64, 8), (8, 8, 8, 8), (1, 256, 64, 128), (2, 200, 40, 100),
-    (1, 300, 20, 10), (2, 96, 160, 48), (3, 32, 128, 16), (20, 64, 64, 32), (2, 24, 300, 4)]
+    (1, 300, 20, 10), (2, 96, 160, 48), (3, 32, 128, 16), (20, 64, 64, 32), (2, 24, 300, 4), (2, 72, 264, 32), (2, 40, 48, 0), (1, 128, 72, 112)]
 
 
 @pytest.mark.parametrize("form", [0, 1])
@@ -271,7 +271,7 @@ def test_retention(H, D, V, rot, dtype, form):
             pos.append(torch.arange(at[s], at[s] + c))
             at[s] += c
         proj = torch.cat(proj).to(DEV)
-        wide = torch.full((proj.shape[0], H * V + 11), 9.0, dtype=dtype, device=DEV)
+        wide = torch.full((proj.shape[0], H * V + 16 + -(H * V) % 8), 9.0, dtype=dtype, device=DEV)
         retention.retention(proj, torch.cat(pos).int().to(DEV), inv, decay.to(DEV), memory, _i32([-1 if s is None else s for s, _ in st]),
                             _i32(bounds([c for _, c in st])), _i32(reset), wide[:, 8:8 + H * V], norm_eps=1e-5, gain=0.7, n_short=nd, form=form)
         for got, ref in zip(wide[:, 8:8 + H * V].cpu().split([c for _, c in st]), exp):
@@ -281,6 +281,27 @@ def test_retention(H, D, V, rot, dtype, form):
                 assert not got.any()
         assert (wide[:, :8] == 9).all() and (wide[:, 8 + H * V:] == 9).all()
     assert (memory[4] == 7).all() and _status_ok()
+    for s, p in seq.items():                              # the state is fp32 whatever the rows are
+        m = p.shape[0]
+        k = O.rotate(p.double()[:, H * D:2 * H * D].view(m, H, D), rot) * D ** -0.5
+        fade = decay.double()[None] ** torch.arange(m - 1, -1, -1)[:, None].double()
+        assert_close(memory[s], torch.einsum("nhd,nhv->hdv", k * fade[..., None], p.double()[:, 2 * H * D:2 * H * D + H * V].view(m, H, V)), F32, f32=1e-4)
+
+
+def test_retention_over_long_portions():
+    """Chunks follow chunks: 700 tokens at once, from a state, and again in portions that end inside chunks; far positions."""
+    g, H, D, V, rot, n = _gen(1), 3, 64, 96, dict(dims=32, base=1e4), 1500
+    proj = torch.randn(n, 2 * H * (D + V), generator=g).to(BF16)
+    decay, inv = torch.tensor([0.9, 0.999, 1.0]), rope_inv_freq(32, 1e4, None)[0].to(DEV)
+    want = _oracle_retention(proj.double(), H, D, V, rot, decay.double(), 1e-5, 1.0)
+    for sizes in ([1500], [700, 800], [130, 127, 1, 128, 129, 600, 385]):
+        memory, at, out = torch.full((2, H, D, V), 5.0, device=DEV), 0, torch.empty(n, H * V, dtype=BF16, device=DEV)
+        for c in sizes:
+            retention.retention(proj[at:at + c].to(DEV), torch.arange(at, at + c, dtype=torch.int32, device=DEV), inv, decay.to(DEV), memory, _i32([1]),
+                                _i32([0, c]), _i32([int(at == 0)]), out[at:at + c], norm_eps=1e-5)
+            at += c
+        assert_close(out, want, BF16)
+    assert _status_ok()
 
 
 # ----------------------------------------------------------------------------- whole models
