@@ -19,26 +19,40 @@ struct MeansParams {
   int n, num_seqs, k0, Hkv, Dk, Dv, block_size, max_blocks, P, places;
 };
 
+// V consecutive elements as they lie in memory (V = 1, or 16 bytes).
+template <typename T, int V>
+struct Group {
+  alignas(V * sizeof(T)) T v[V];
+  __device__ __forceinline__ void load(const T* p) {
+    if constexpr (V == 1) v[0] = *p;
+    else *reinterpret_cast<uint4*>(v) = *reinterpret_cast<const uint4*>(p);
+  }
+  __device__ __forceinline__ void store(T* p) const {
+    if constexpr (V == 1) *p = v[0];
+    else *reinterpret_cast<uint4*>(p) = *reinterpret_cast<const uint4*>(v);
+  }
+};
+
 // One thread per V elements of a token's key and value heads. A token that ends a block also sums the block up: rows of this
 // call from the source (they are being appended now), earlier ones from the pool, oldest first.
 template <typename T, int V>
 __global__ void __launch_bounds__(256) kv_append_means_kernel(const MeansParams p) {
+  constexpr int B = 4;                                    // rows of a block requested at a time
   pdl_trigger();
   pdl_wait();
   const int kg = p.Hkv * (p.Dk / V), per = kg + p.Hkv * (p.Dv / V);
   const unsigned i = blockIdx.x * 256u + threadIdx.x, tt = i / per;
   if (tt >= static_cast<unsigned>(p.n)) return;
-  const int t = static_cast<int>(tt), g = static_cast<int>(i - tt * per), slot = p.slots[t];
+  const int t = static_cast<int>(tt), g = static_cast<int>(i - tt * per), slot = p.slots[t], pos = p.positions[t];
   if (slot < 0) return;
   const bool key = g < kg;
   const int D = key ? p.Dk : p.Dv, j = key ? g : g - kg, head = j / (D / V), col = (j - head * (D / V)) * V;
   const T* src = static_cast<const T*>(p.src) + p.k0 + (key ? 0 : p.Hkv * p.Dk) + head * D + col;
   T* pool = static_cast<T*>(key ? p.k : p.v);
   const int blk = slot / p.block_size, off = slot - blk * p.block_size;
-  float f[V];
-  load_v<V>(src + static_cast<size_t>(t) * p.ld, f);
-  store_v<V>(pool + ((static_cast<size_t>(blk) * p.Hkv + head) * p.block_size + off) * D + col, f);
-  const int pos = p.positions[t];
+  Group<T, V> own;
+  own.load(src + static_cast<size_t>(t) * p.ld);
+  own.store(pool + ((static_cast<size_t>(blk) * p.Hkv + head) * p.block_size + off) * D + col);
   if ((pos + 1) % p.P != 0) return;
   int lo = 0, first = t;                                  // the token's sequence and its first row
   if (p.cu == nullptr) {
@@ -56,22 +70,30 @@ __global__ void __launch_bounds__(256) kv_append_means_kernel(const MeansParams 
   float sum[V];
 #pragma unroll
   for (int e = 0; e < V; ++e) sum[e] = 0.f;
-  for (int back = p.P - 1; back >= 0; --back) {
-    float a[V];
-    if (t - back >= first) {
-      load_v<V>(src + static_cast<size_t>(t - back) * p.ld, a);
-    } else {
-      const int q = pos - back, page = q / p.block_size;
-      load_v<V>(pool + ((static_cast<size_t>(table[page]) * p.Hkv + head) * p.block_size + (q - page * p.block_size)) * D + col, a);
+  for (int back = p.P - 1; back > 0; back -= B) {
+    Group<T, V> a[B];
+#pragma unroll
+    for (int b = 0; b < B; ++b) {
+      const int k = max(back - b, 1);
+      if (t - k >= first) {
+        a[b].load(src + static_cast<size_t>(t - k) * p.ld);
+      } else {
+        const int q = pos - k, page = q / p.block_size;
+        a[b].load(pool + ((static_cast<size_t>(table[page]) * p.Hkv + head) * p.block_size + (q - page * p.block_size)) * D + col);
+      }
     }
 #pragma unroll
-    for (int e = 0; e < V; ++e) sum[e] += a[e];
-  }
+    for (int b = 0; b < B; ++b)
+      if (back - b > 0) {
 #pragma unroll
-  for (int e = 0; e < V; ++e) sum[e] /= static_cast<float>(p.P);
+        for (int e = 0; e < V; ++e) sum[e] += to_f(a[b].v[e]);
+      }
+  }
+  Group<T, V> mean;
+#pragma unroll
+  for (int e = 0; e < V; ++e) mean.v[e] = from_f<T>((sum[e] + to_f(own.v[e])) / static_cast<float>(p.P));
   const int page = pos / p.block_size, at = (pos + 1) / p.P - 1 - page * p.block_size / p.P;
-  T* mean = static_cast<T*>(key ? p.k_mean : p.v_mean);
-  store_v<V>(mean + ((static_cast<size_t>(table[page]) * p.Hkv + head) * p.places + at) * D + col, sum);
+  mean.store(static_cast<T*>(key ? p.k_mean : p.v_mean) + ((static_cast<size_t>(table[page]) * p.Hkv + head) * p.places + at) * D + col);
 }
 
 // Row r of the result is block r - bounds[s] of sequence s (bounds[s] <= r < bounds[s + 1]); BYTES of it per thread.
@@ -115,15 +137,15 @@ extern "C" int mx_kv_append_means(const void* src, long long ld, const void* pos
   const MeansParams p{src, ld, static_cast<const int*>(positions), static_cast<const int*>(slots), static_cast<const int*>(tables),
                       static_cast<const int*>(cu), k, v, k_mean, v_mean, n, num_seqs, Hq * Dk, Hkv, Dk, Dv, block_size, max_blocks, P,
                       (block_size + P - 1) / P};
-  const size_t ab = fp32 ? 16 : 8;
-  const bool vec = Dk % 4 == 0 && Dv % 4 == 0 && ld % 4 == 0 && aligned_to(src, ab) && aligned_to(k, ab) && aligned_to(v, ab) &&
-                   aligned_to(k_mean, ab) && aligned_to(v_mean, ab);
-  const long long threads = static_cast<long long>(n) * Hkv * (Dk + Dv) / (vec ? 4 : 1);
+  const int V = fp32 ? 4 : 8;                             // elements of 16 bytes
+  const bool vec = Dk % V == 0 && Dv % V == 0 && ld % V == 0 && aligned_to(src, 16) && aligned_to(k, 16) && aligned_to(v, 16) &&
+                   aligned_to(k_mean, 16) && aligned_to(v_mean, 16);
+  const long long threads = static_cast<long long>(n) * Hkv * (Dk + Dv) / (vec ? V : 1);
   if (threads > 0x7fffffffll) return -1;
   const dim3 grid(static_cast<unsigned>((threads + 255) / 256)), block(256);
   auto st = static_cast<cudaStream_t>(stream);
   if (fp32) return static_cast<int>(launch_kernel(vec ? kv_append_means_kernel<float, 4> : kv_append_means_kernel<float, 1>, grid, block, 0, st, p));
-  return static_cast<int>(launch_kernel(vec ? kv_append_means_kernel<__nv_bfloat16, 4> : kv_append_means_kernel<__nv_bfloat16, 1>, grid, block, 0, st, p));
+  return static_cast<int>(launch_kernel(vec ? kv_append_means_kernel<__nv_bfloat16, 8> : kv_append_means_kernel<__nv_bfloat16, 1>, grid, block, 0, st, p));
 }
 
 // kb / vb: bytes of a key and value row.

@@ -35,6 +35,12 @@ __global__ void __launch_bounds__(512) streams_step_kernel(const MxStreamsStep p
     known = id >= 0 && id < p.vocab;
     er = static_cast<const T*>(p.table) + static_cast<size_t>(known ? id : 0) * dim;
   }
+  const int K = p.taps;
+  const bool single = row < p.n_short;                     // a piece of one token
+  const int slot = single ? p.slots[row] : 0;
+  float* tail = single && slot >= 0 ? p.tail + static_cast<size_t>(slot) * (K - 1) * dim : nullptr;
+  if (tail != nullptr)                                     // (its state is needed behind the norm)
+    for (int c = threadIdx.x * 32; c < (K - 1) * dim; c += blockDim.x * 32) asm volatile("prefetch.global.L2 [%0];" ::"l"(tail + c));
   float u[VPT][V], s[1] = {0.f};
 #pragma unroll
   for (int i = 0; i < VPT; ++i) {
@@ -116,10 +122,6 @@ __global__ void __launch_bounds__(512) streams_step_kernel(const MxStreamsStep p
   }
   block_sums<1>(s, red);
   const float r = 1.f / sqrtf(s[0] / dim + p.eps);
-  const int K = p.taps;
-  const bool single = row < p.n_short;                     // a piece of one token
-  const int slot = single ? p.slots[row] : 0;
-  float* tail = single && slot >= 0 ? p.tail + static_cast<size_t>(slot) * (K - 1) * dim : nullptr;
 #pragma unroll
   for (int i = 0; i < VPT; ++i) {
     const int c = (threadIdx.x + i * blockDim.x) * V;
@@ -273,7 +275,9 @@ template <typename T, int V, int S>
 static int launch_step(const MxStreamsStep& p, cudaStream_t st) {
   const int groups = (p.dim + V - 1) / V;
   int threads = (groups + 31) / 32 * 32;
-  threads = threads < 64 ? 64 : threads <= 256 ? threads : groups > 256 * 8 ? 512 : 256;
+  // (few rows: all of a row's accesses at once; many: more rows per SM)
+  const int most = p.rows <= 296 || groups > 256 * 8 ? 512 : 256;
+  threads = threads < 64 ? 64 : threads <= most ? threads : most;
   const int need = (groups + threads - 1) / threads;
   const dim3 grid(p.rows), block(threads);
   if (need <= 1) return static_cast<int>(launch_kernel(streams_step_kernel<T, V, 1, S>, grid, block, 0, st, p));
