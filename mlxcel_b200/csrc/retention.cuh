@@ -23,7 +23,7 @@ struct RetentionParams {
 
 // Scratch of the token-by-token kernels over N tokens (rows row0 .. row0 + N - 1), fp32, widths padded with zeros:
 //   q [N, H, DP] | k [N, H, DP] | v [N, H, VP] | o [N, H, VP]
-// and of the chunked form: angles [N, rot / 2] (cosine, sine) | o [N, H, VP] where the heads are wider than a tile.
+// and of the chunked form: cosines [N, rot / 2] | sines [N, rot / 2] | o [N, H, VP] where the heads are wider than a tile.
 struct RetentionScratch {
   float *q, *k, *v, *o;
 };
